@@ -24,6 +24,7 @@ typedef enum vb200_epilogue {
     VB200_EPI_BF16 = 0,     /* out_bf16[m, n]  = acc                                            */
     VB200_EPI_F32 = 1,      /* out_f32[m, n]   = acc            (logits)                        */
     VB200_EPI_ADD_F32 = 2,  /* out_f32[m, n]  += acc            (residual: h = h + proj(x))     */
+    VB200_EPI_RELU2 = 4,    /* out_bf16[m, n]  = max(acc, 0)^2                                  */
     VB200_EPI_SWIGLU = 3    /* out_bf16[m, n/2] = silu(acc[m, n]) * acc[m, n+1], n even:
                                W holds gate and up rows interleaved (row 2j = gate_j,
                                row 2j+1 = up_j), see vb200_interleave_rows                      */
@@ -83,6 +84,7 @@ typedef struct vb200_linear_args {
     int32_t rms_dim;
     float rms_eps;
     const float* row_scale;             /* [M] or NULL */
+    const float* addend;                /* [M, N] fp32, row stride ldo, or NULL (VB200_EPI_ADD_F32 only): out += acc + addend */
 } vb200_linear_args;
 int vb200_linear_ex(const vb200_linear_args* a);
 /* inv_rms[m] = 1 / sqrt(mean(h[m, :]^2) + eps), h fp32 [M, dim] with row stride ld elements. */

@@ -86,6 +86,7 @@ class LinearArgs(C.Structure):
         ("M", C.c_int32), ("N", C.c_int32), ("K", C.c_int32), ("epilogue", C.c_int32), ("splits", C.c_int32),
         ("bias", C.c_void_p), ("scaled_copy", C.c_void_p), ("copy_scale", C.c_void_p),
         ("rms_rows", C.c_void_p), ("rms_ld", C.c_int64), ("rms_dim", C.c_int32), ("rms_eps", C.c_float), ("row_scale", C.c_void_p),
+        ("addend", C.c_void_p),
     ]
 
 
@@ -99,7 +100,7 @@ class GreedyArgs(C.Structure):
     ]
 
 
-EPI_BF16, EPI_F32, EPI_ADD_F32, EPI_SWIGLU = 0, 1, 2, 3
+EPI_BF16, EPI_F32, EPI_ADD_F32, EPI_SWIGLU, EPI_RELU2 = 0, 1, 2, 3, 4
 
 _lib = None
 

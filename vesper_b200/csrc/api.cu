@@ -600,7 +600,7 @@ int vb200_linear_bias(int device, void* stream, const void* x, int64_t ldx, cons
                       const float* bias, void* out, int64_t ldo, int32_t M, int32_t N, int32_t K,
                       int32_t epilogue, int32_t splits) {
     if (!x || !w || !out || M <= 0 || N <= 0 || K <= 0) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: null pointer or non-positive size");
-    if (epilogue < VB200_EPI_BF16 || epilogue > VB200_EPI_SWIGLU) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: unknown epilogue");
+    if (epilogue < VB200_EPI_BF16 || epilogue > VB200_EPI_RELU2) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: unknown epilogue");
     if (ldx < K || ldw < K) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: ldx and ldw must be >= K");
     const int64_t out_cols = epilogue == VB200_EPI_SWIGLU ? N / 2 : N;
     if (ldo < out_cols) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: ldo smaller than the output row");
@@ -636,7 +636,7 @@ int vb200_linear_f32(int device, void* stream, const float* x, int64_t ldx, cons
 int vb200_linear_ex(const vb200_linear_args* a) {
     if (!a || a->struct_size != sizeof(vb200_linear_args)) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_args: null or struct_size mismatch");
     if (!a->x || !a->w || !a->out || a->M <= 0 || a->N <= 0 || a->K <= 0) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: null pointer or non-positive size");
-    if (a->epilogue < VB200_EPI_BF16 || a->epilogue > VB200_EPI_SWIGLU) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: unknown epilogue");
+    if (a->epilogue < VB200_EPI_BF16 || a->epilogue > VB200_EPI_RELU2) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: unknown epilogue");
     if (a->ldx < a->K || a->ldw < a->K) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: ldx and ldw must be >= K");
     const int64_t out_cols = a->epilogue == VB200_EPI_SWIGLU ? a->N / 2 : a->N;
     if (a->ldo < out_cols) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: ldo smaller than the output row");
@@ -646,6 +646,7 @@ int vb200_linear_ex(const vb200_linear_args* a) {
         return set_detail(VB200_ERR_ALIGNMENT, "vb200_linear_ex: K % 8, and 16-byte aligned bases and row strides, are required");
     if (a->scaled_copy && (a->epilogue != VB200_EPI_ADD_F32 || !a->copy_scale))
         return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: scaled_copy needs the += epilogue and copy_scale");
+    if (a->addend && a->epilogue != VB200_EPI_ADD_F32) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: addend needs the += epilogue");
     if (a->rms_rows && (a->rms_dim <= 0 || a->rms_dim % 4 != 0 || a->rms_ld % 4 != 0 || (a->rms_ld != 0 && a->rms_ld < a->rms_dim) || !aligned16(a->rms_rows)))
         return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: rms_dim must be a positive multiple of 4 and rms_rows 16-byte aligned");
     if (a->rms_rows && a->M > 64 && !a->row_scale)
@@ -657,6 +658,7 @@ int vb200_linear_ex(const vb200_linear_args* a) {
     p.M = a->M; p.N = a->N; p.K = a->K; p.epilogue = a->epilogue; p.splits = a->splits;
     p.bias = a->bias;
     p.scaled_copy = a->scaled_copy; p.copy_scale = a->copy_scale;
+    p.addend = a->addend;
     if (a->row_scale) p.row_scale = a->row_scale;              // a precomputed factor wins over the in-kernel one
     else if (a->rms_rows && a->M <= 64) {
         p.rms_rows = a->rms_rows; p.rms_dim = a->rms_dim; p.rms_eps = a->rms_eps;

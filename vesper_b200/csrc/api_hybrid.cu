@@ -1,0 +1,170 @@
+// extern "C" entry points of vesper_b200_hybrid.h: argument validation and orchestration.
+#include "hybrid.cuh"
+
+namespace vb200 {
+
+namespace {
+thread_local const char* t_latent_kernel = "";
+thread_local const char* t_ssd_kernel = "";
+bool aligned16(const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; }
+bool dtype_ok(int d) { return d == VB200_F32 || d == VB200_BF16; }
+}  // namespace
+
+void note_latent_kernel(const char* name) { t_latent_kernel = name; }
+void note_ssd_kernel(const char* name) { t_ssd_kernel = name; }
+
+// Streaming multiprocessors of the current device (148 where no device answers: workspace sizes on a machine without a GPU).
+int device_sm_count() {
+    static int cache[64] = {0};
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) { (void)cudaGetLastError(); return 148; }
+    if (cache[dev] == 0) {
+        int n = 0;
+        if (cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev) != cudaSuccess || n <= 0) { (void)cudaGetLastError(); n = 148; }
+        cache[dev] = n;
+    }
+    return cache[dev];
+}
+
+namespace {
+
+int validate_latent(const vb200_latent_args* a, const char* who) {
+    if (!a || a->struct_size != sizeof(vb200_latent_args)) return set_detail(VB200_ERR_INVALID_ARG, "vb200_latent_args: null or struct_size mismatch");
+    if (!dtype_ok(a->dtype)) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_latent: dtype must be bf16 or fp32");
+    if (a->B <= 0 || a->T <= 0 || a->H <= 0 || a->dim <= 0 || a->rot_dim < 0 || a->rot_dim % 2 != 0 || a->vdim <= 0 || a->rank <= 0 || a->window <= 0 || a->ring <= 0)
+        return set_detail(VB200_ERR_INVALID_ARG, "vb200_latent: sizes must be positive and rot_dim even");
+    if (a->rank > 2048 || a->rot_dim > 1024 || a->dim > 1024 || a->vdim > 1024) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_latent: rank above 2048 or a head size above 1024");
+    if (a->H > 65535 || a->B > 65535) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_latent: more than 65535 heads or rows");
+    if (a->start_pos < 0 || !a->pos || !a->proj || !a->c_norm || !a->cache || (a->rot_dim > 0 && !a->inv_freq)) return set_detail(VB200_ERR_INVALID_ARG, who);
+    const int64_t width = static_cast<int64_t>(a->H) * (a->dim + a->rot_dim) + a->rank + a->rot_dim;
+    if (a->ldp < width || a->ldc != vb200_latent_row(a->rank, a->rot_dim)) return set_detail(VB200_ERR_INVALID_ARG, "vb200_latent: a row stride does not hold its row");
+    if (!aligned16(a->proj) || !aligned16(a->cache)) return set_detail(VB200_ERR_ALIGNMENT, "vb200_latent: 16-byte alignment required");
+    return VB200_OK;
+}
+
+}  // namespace
+}  // namespace vb200
+
+using namespace vb200;
+
+extern "C" {
+
+int vb200_embed_sequence(const vb200_embed_args* a) {
+    if (!a || a->struct_size != sizeof(vb200_embed_args)) return set_detail(VB200_ERR_INVALID_ARG, "vb200_embed_args: null or struct_size mismatch");
+    if (!dtype_ok(a->dtype)) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_embed_sequence: dtype must be bf16 or fp32");
+    if (!a->ids || !a->table || !a->lens || !a->step_pos || !a->prev || !a->h || a->B <= 0 || a->T <= 0 || a->dim <= 0 || a->vocab <= 0)
+        return set_detail(VB200_ERR_INVALID_ARG, "vb200_embed_sequence: null pointer or non-positive size");
+    if (a->bigram && a->buckets <= 0) return set_detail(VB200_ERR_INVALID_ARG, "vb200_embed_sequence: a bigram table needs buckets > 0");
+    if (a->scaled_out && !a->scale) return set_detail(VB200_ERR_INVALID_ARG, "vb200_embed_sequence: scaled_out without scale");
+    DeviceGuard g;
+    if (int rc = g.init(a->device)) return rc;
+    int* status = kernel_status_word();
+    if (!status) return VB200_ERR_CUDA;
+    return launch_embed_sequence(static_cast<cudaStream_t>(a->stream), *a, status);
+}
+
+int vb200_residual_add(int device, void* stream, float* h, const float* addend, const float* vec, int32_t M, int32_t dim,
+                       const float* scale, void* scaled_out) {
+    if (!h || M <= 0 || dim <= 0 || (scaled_out && !scale)) return set_detail(VB200_ERR_INVALID_ARG, "vb200_residual_add: bad arguments");
+    DeviceGuard g;
+    if (int rc = g.init(device)) return rc;
+    return launch_residual_add(static_cast<cudaStream_t>(stream), h, addend, vec, M, dim, scale, scaled_out);
+}
+
+int vb200_rms_norm_f32(int device, void* stream, const float* x, const float* w, float* out, int32_t M, int32_t dim, int32_t count, float eps) {
+    if (!x || !w || !out || M <= 0 || dim <= 0 || count <= 0 || count > dim) return set_detail(VB200_ERR_INVALID_ARG, "vb200_rms_norm_f32: bad arguments");
+    DeviceGuard g;
+    if (int rc = g.init(device)) return rc;
+    return launch_rms_norm_f32(static_cast<cudaStream_t>(stream), x, w, out, M, dim, count, eps);
+}
+
+int vb200_linear_f32_ex(int device, void* stream, const float* x, int64_t ldx, const float* w, int64_t ldw, const float* bias,
+                        const float* addend, float* out, int64_t ldo, int32_t M, int32_t N, int32_t K, int32_t epilogue) {
+    if (!x || !w || !out || M <= 0 || N <= 0 || K <= 0) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_f32_ex: null pointer or non-positive size");
+    if (ldx < K || ldw < K || ldo < N) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_f32_ex: a row stride is smaller than its row");
+    if (epilogue != VB200_EPI_F32 && epilogue != VB200_EPI_ADD_F32 && epilogue != VB200_EPI_RELU2)
+        return set_detail(VB200_ERR_UNSUPPORTED, "vb200_linear_f32_ex: epilogue not available in fp32");
+    DeviceGuard g;
+    if (int rc = g.init(device)) return rc;
+    return launch_linear_f32(static_cast<cudaStream_t>(stream), x, ldx, w, ldw, bias, out, ldo, M, N, K, epilogue, addend);
+}
+
+size_t vb200_latent_workspace_bytes(const vb200_latent_args* a) {
+    if (!a || a->struct_size != sizeof(vb200_latent_args) || a->B <= 0 || a->H <= 0 || a->rank <= 0 || a->ring <= 0) return 0;
+    const LatentPlan pl = plan_latent(*a);
+    return ((pl.q_floats + 63) / 64 * 64 + pl.part_floats) * sizeof(float);
+}
+
+int vb200_latent_append(const vb200_latent_args* a) {
+    if (int rc = validate_latent(a, "vb200_latent_append: null pointer or negative start_pos")) return rc;
+    if (!a->ctx_latent || !aligned16(a->ctx_latent)) return set_detail(VB200_ERR_INVALID_ARG, "vb200_latent_append: ctx_latent must be given and 16-byte aligned");
+    DeviceGuard g;
+    if (int rc = g.init(a->device)) return rc;
+    return launch_latent_append(static_cast<cudaStream_t>(a->stream), *a);
+}
+
+int vb200_latent_prefill(const vb200_latent_args* a) {
+    if (int rc = validate_latent(a, "vb200_latent_prefill: null pointer or negative start_pos")) return rc;
+    if (!a->ctx_latent || !a->ctx_kv || !a->out) return set_detail(VB200_ERR_INVALID_ARG, "vb200_latent_prefill: null pointer");
+    if (a->ldkv < static_cast<int64_t>(a->H) * (a->dim + a->vdim) || a->ldo < static_cast<int64_t>(a->H) * a->vdim)
+        return set_detail(VB200_ERR_INVALID_ARG, "vb200_latent_prefill: a row stride does not hold its row");
+    DeviceGuard g;
+    if (int rc = g.init(a->device)) return rc;
+    int* status = kernel_status_word();
+    if (!status) return VB200_ERR_CUDA;
+    cudaStream_t s = static_cast<cudaStream_t>(a->stream);
+    profile_mark_begin(s);
+    const bool tuned = latent_sm100_supported(*a);
+    const int rc = tuned ? launch_latent_prefill_sm100(s, *a, status) : launch_latent_prefill_generic(s, *a);
+    note_latent_kernel(tuned ? "latent_prefill_sm100_kernel" : "latent_prefill_generic_kernel");
+    profile_mark_end(s);
+    return rc;
+}
+
+int vb200_latent_decode(const vb200_latent_args* a) {
+    if (int rc = validate_latent(a, "vb200_latent_decode: null pointer or negative start_pos")) return rc;
+    if (a->T != 1) return set_detail(VB200_ERR_INVALID_ARG, "vb200_latent_decode: one token per row");
+    if (!a->w_uk || !a->w_uv || !a->out) return set_detail(VB200_ERR_INVALID_ARG, "vb200_latent_decode: null pointer");
+    if (a->ldu % 8 != 0 || a->ldu < a->rank || !aligned16(a->w_uk) || !aligned16(a->w_uv))
+        return set_detail(VB200_ERR_ALIGNMENT, "vb200_latent_decode: ldu must be a multiple of 8 that holds a latent, the weights 16-byte aligned");
+    if (a->ldo < static_cast<int64_t>(a->H) * a->vdim) return set_detail(VB200_ERR_INVALID_ARG, "vb200_latent_decode: ldo smaller than the output row");
+    if (!a->workspace || a->workspace_bytes < vb200_latent_workspace_bytes(a)) return set_detail(VB200_ERR_WORKSPACE, "vb200_latent_decode: workspace too small");
+    if (!aligned16(a->workspace)) return set_detail(VB200_ERR_ALIGNMENT, "vb200_latent_decode: workspace must be 16-byte aligned");
+    DeviceGuard g;
+    if (int rc = g.init(a->device)) return rc;
+    int* status = kernel_status_word();
+    if (!status) return VB200_ERR_CUDA;
+    return launch_latent_decode(static_cast<cudaStream_t>(a->stream), *a, status);
+}
+
+const char* vb200_last_latent_kernel(void) { return t_latent_kernel; }
+
+static bool ssd_sizes_ok(const vb200_ssd_args* a) {
+    return a && a->struct_size == sizeof(vb200_ssd_args) && a->B > 0 && a->T > 0 && a->H > 0 && a->P > 0 && a->N > 0 && a->G > 0 && a->taps > 0 && a->norm_groups > 0;
+}
+
+size_t vb200_ssd_workspace_bytes(const vb200_ssd_args* a) { return ssd_sizes_ok(a) ? plan_ssd(*a).total : 0; }
+
+int vb200_ssd_forward(const vb200_ssd_args* a) {
+    if (!ssd_sizes_ok(a)) return set_detail(VB200_ERR_INVALID_ARG, "vb200_ssd_args: null, struct_size mismatch or non-positive size");
+    if (!dtype_ok(a->dtype)) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_ssd_forward: dtype must be bf16 or fp32");
+    if (a->H % a->G != 0 || (static_cast<int64_t>(a->H) * a->P) % a->norm_groups != 0)
+        return set_detail(VB200_ERR_INVALID_ARG, "vb200_ssd_forward: heads must divide into the groups, inner into the norm groups");
+    if (a->taps > 32) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_ssd_forward: more than 32 convolution taps");
+    if (a->B > 65535 || static_cast<int64_t>(a->B) * a->T > 65535LL * 1024) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_ssd_forward: batch too large");
+    if (!a->proj || !a->conv_w || !a->conv_b || !a->dt_bias || !a->A_log || !a->D || !a->norm_w || !a->pos || !a->conv_state || !a->state || !a->out)
+        return set_detail(VB200_ERR_INVALID_ARG, "vb200_ssd_forward: null pointer");
+    const int64_t inner = static_cast<int64_t>(a->H) * a->P;
+    if (a->ldp < 2 * inner + 2LL * a->G * a->N + a->H || a->ldo < inner) return set_detail(VB200_ERR_INVALID_ARG, "vb200_ssd_forward: a row stride does not hold its row");
+    if (!aligned16(a->proj) || !aligned16(a->conv_state) || !aligned16(a->state) || !aligned16(a->workspace))
+        return set_detail(VB200_ERR_ALIGNMENT, "vb200_ssd_forward: 16-byte alignment required");
+    const SsdPlan pl = plan_ssd(*a);
+    if (!a->workspace || a->workspace_bytes < pl.total) return set_detail(VB200_ERR_WORKSPACE, "vb200_ssd_forward: workspace too small");
+    DeviceGuard g;
+    if (int rc = g.init(a->device)) return rc;
+    return launch_ssd(static_cast<cudaStream_t>(a->stream), *a, pl);
+}
+
+const char* vb200_last_ssd_kernel(void) { return t_ssd_kernel; }
+
+}  // extern "C"

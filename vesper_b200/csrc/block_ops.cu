@@ -240,7 +240,8 @@ int launch_row_inv_rms(cudaStream_t s, const float* h, long long ld, float* inv_
 // fp32 y = x W^T + bias on CUDA cores: 64 x 64 output tiles, 16 x 16 threads with a 4 x 4 register block each, K in
 // steps of 16 through shared memory.  For the reference's fp32 modules (parity at 1e-4); bf16 goes to linear_sm100.cu.
 __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict__ x, long long ldx, const float* __restrict__ w, long long ldw,
-                                                         const float* __restrict__ bias, float* __restrict__ out, long long ldo, int M, int N, int K) {
+                                                         const float* __restrict__ bias, float* __restrict__ out, long long ldo, int M, int N, int K,
+                                                         int epilogue, const float* __restrict__ addend) {
     __shared__ float xs[16][64 + 1], ws[16][64 + 1];
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
@@ -269,14 +270,20 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
-            if (m < M && n < N) out[static_cast<long long>(m) * ldo + n] = acc[i][j] + (bias ? bias[n] : 0.f);
+            if (m >= M || n >= N) continue;
+            const long long idx = static_cast<long long>(m) * ldo + n;
+            float v = acc[i][j] + (bias ? bias[n] : 0.f);
+            if (addend) v += addend[idx];
+            if (epilogue == VB200_EPI_ADD_F32) v += out[idx];
+            else if (epilogue == VB200_EPI_RELU2) { v = fmaxf(v, 0.f); v *= v; }
+            out[idx] = v;
         }
 }
 
 int launch_linear_f32(cudaStream_t s, const float* x, long long ldx, const float* w, long long ldw, const float* bias, float* out,
-                      long long ldo, int M, int N, int K) {
+                      long long ldo, int M, int N, int K, int epilogue, const float* addend) {
     dim3 grid(static_cast<unsigned>((N + 63) / 64), static_cast<unsigned>((M + 63) / 64));
-    linear_f32_kernel<<<grid, 256, 0, s>>>(x, ldx, w, ldw, bias, out, ldo, M, N, K);
+    linear_f32_kernel<<<grid, 256, 0, s>>>(x, ldx, w, ldw, bias, out, ldo, M, N, K, epilogue, addend);
     note_launch();
     VB200_CUDA_TRY(cudaPeekAtLastError());
     return VB200_OK;

@@ -1,0 +1,146 @@
+// Shared pieces of the hybrid-decoder kernels (latent attention, Mamba-2, sequence operators).
+#pragma once
+
+#include "kernels.h"
+#include "../../include/vesper_b200_hybrid.h"
+
+namespace vb200 {
+
+constexpr float kLog2e = 1.4426950408889634f;
+
+// Launch with the programmatic-dependent-launch attribute; the kernel starts with pdl_begin().
+template <typename... KArgs, typename... Args>
+int launch_pdl(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s, Args... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid;
+    cfg.blockDim = block;
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = s;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    VB200_CUDA_TRY(cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...));
+    note_launch();
+    return VB200_OK;
+}
+
+// Raises a kernel's dynamic shared memory limit (a no-op below the 48 KB default).
+template <typename Kernel>
+int allow_smem(Kernel kernel, size_t bytes) {
+    if (bytes <= 48 * 1024) return VB200_OK;
+    VB200_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(bytes)));
+    return VB200_OK;
+}
+
+int device_sm_count();                           // api_hybrid.cu
+void note_latent_kernel(const char* name);
+void note_ssd_kernel(const char* name);
+
+// ---- sequence_ops.cu ----
+int launch_embed_sequence(cudaStream_t s, const vb200_embed_args& a, int* status);
+int launch_residual_add(cudaStream_t s, float* h, const float* addend, const float* vec, int M, int dim, const float* scale, void* scaled_out);
+int launch_rms_norm_f32(cudaStream_t s, const float* x, const float* w, float* out, int M, int dim, int count, float eps);
+
+// ---- latent attention ----
+inline int pad_to(int x, int m) { return (x + m - 1) / m * m; }
+// Split plan and workspace of a decode step: absorbed queries [B, H, qld] fp32, then per (row, head, split) the
+// unnormalised latent sum [rank16], the reference maximum (log2 units) and the sum of weights.
+struct LatentPlan {
+    int n_max;          // keys a row can have
+    int splits;
+    int rank16, rot16, qld, part_ld;
+    size_t q_floats, part_floats;
+};
+LatentPlan plan_latent(const vb200_latent_args& a);
+bool latent_mma_supported(const vb200_latent_args& a);
+bool latent_sm100_supported(const vb200_latent_args& a);
+int launch_latent_append(cudaStream_t s, const vb200_latent_args& a);
+int launch_latent_prefill_generic(cudaStream_t s, const vb200_latent_args& a);
+int launch_latent_prefill_sm100(cudaStream_t s, const vb200_latent_args& a, int* status);       // latent_prefill_sm100.cu
+int launch_latent_decode(cudaStream_t s, const vb200_latent_args& a, int* status);
+int launch_latent_split_mma(cudaStream_t s, const vb200_latent_args& a, const LatentPlan& pl, const float* q, float* part, int* status);   // latent_decode_mma.cu
+
+// ---- Mamba-2 ----
+struct SsdPlan {
+    int channels, Pp;
+    bool chunked;
+    int chunk, n_chunks;
+    size_t conv_bytes, gated_bytes, chunk_bytes, total;     // conv output | gated y | chunk states
+};
+SsdPlan plan_ssd(const vb200_ssd_args& a);
+bool ssd_chunk_supported(const vb200_ssd_args& a);
+int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl);
+int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, const void* xbc, void* gated, float* states);   // ssd_chunk.cu
+
+#ifdef __CUDACC__
+// Programmatic dependent launch: let the next kernel be scheduled, then wait for the previous one's results.
+__device__ __forceinline__ void pdl_begin() {
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+}
+__device__ __forceinline__ float warp_sum_f(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
+    return v;
+}
+__device__ __forceinline__ float warp_max_f(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xFFFFFFFFu, v, o));
+    return v;
+}
+// Sum over a CTA of W warps; `part` holds W floats and may be reused after the next barrier.
+template <int W>
+__device__ __forceinline__ float block_sum(float v, float* part) {
+    v = warp_sum_f(v);
+    if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.f;
+#pragma unroll
+    for (int i = 0; i < W; ++i) t += part[i];
+    return t;
+}
+__device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
+__device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+// cos / sin of position * f: the product and the reduction to one turn in fp64, the functions in fp32.
+__device__ __forceinline__ float2 rope_cs(int position, double f) {
+    const double turns = static_cast<double>(position) * f * 0.15915494309189533577;
+    const float r = static_cast<float>((turns - rint(turns)) * 6.283185307179586476925);
+    float s, c;
+    sincosf(r, &s, &c);
+    return make_float2(c, s);
+}
+// eight consecutive elements (16-byte aligned for bf16, 32 for fp32)
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const float2 f = Elem<__nv_bfloat16>::unpack2(w[i]);
+        v[2 * i] = f.x; v[2 * i + 1] = f.y;
+    }
+}
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
+    uint4 u;
+    u.x = Elem<__nv_bfloat16>::pack2(v[0], v[1]); u.y = Elem<__nv_bfloat16>::pack2(v[2], v[3]);
+    u.z = Elem<__nv_bfloat16>::pack2(v[4], v[5]); u.w = Elem<__nv_bfloat16>::pack2(v[6], v[7]);
+    *reinterpret_cast<uint4*>(p) = u;
+}
+__device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+// x = hi + lo with both halves bf16 (16 of fp32's 24 significand bits): an fp32 operand of a bf16 tensor-core product
+__device__ __forceinline__ void split_hi_lo(float x, float y, uint32_t& hi, uint32_t& lo) {
+    hi = Elem<__nv_bfloat16>::pack2(x, y);
+    const float2 h = Elem<__nv_bfloat16>::unpack2(hi);
+    lo = Elem<__nv_bfloat16>::pack2(x - h.x, y - h.y);
+}
+#endif
+
+}  // namespace vb200

@@ -175,6 +175,7 @@ struct LinearParams {
     int rms_dim;
     float rms_eps;
     const float* row_scale;          // [M] or null
+    const float* addend;             // += epilogue: a second fp32 matrix [M, N] (row stride ldo) added with it, or null
 };
 int launch_linear(cudaStream_t s, const LinearParams& p);
 // inv_rms[m] = 1 / sqrt(mean(h[m,:]^2) + eps)
@@ -184,8 +185,9 @@ int launch_row_inv_rms(cudaStream_t s, const float* h, long long ld, float* inv_
 int launch_interleave_rows(cudaStream_t s, const void* a, const void* b, void* out, long long rows, long long cols);
 int launch_rms_norm(cudaStream_t s, const float* x, const float* weight, void* out_bf16, int M, int dim, float eps);
 int launch_silu_mul(cudaStream_t s, const void* gate, const void* up, void* out, long long n);
+// epilogue: VB200_EPI_F32, VB200_EPI_ADD_F32 or VB200_EPI_RELU2 (all fp32 here); addend as in LinearParams
 int launch_linear_f32(cudaStream_t s, const float* x, long long ldx, const float* w, long long ldw, const float* bias, float* out,
-                      long long ldo, int M, int N, int K);
+                      long long ldo, int M, int N, int K, int epilogue = VB200_EPI_F32, const float* addend = nullptr);
 // norm_w / norm_out (nullable): also out_norm[m,:] = rmsnorm(out[m,:]) * norm_w as bf16
 int launch_embedding(cudaStream_t s, const void* ids, int ids64, const void* table, float* out, int M, int dim,
                      int vocab, int* status, const float* norm_w = nullptr, void* norm_out = nullptr, float norm_eps = 0.f,

@@ -12,7 +12,7 @@
 //                         cluster, which reduce their partial tiles through distributed shared
 //                         memory in a fixed order (deterministic) before the leader's epilogue.
 // Epilogues (fused, per output element): store bf16 | store fp32 | fp32 accumulate into the residual
-// stream | SwiGLU over interleaved (gate, up) weight rows -> bf16 (src/nn/swiglu.cpp:36-48,
+// stream (optionally plus a second fp32 addend) | squared ReLU -> bf16 | SwiGLU over interleaved (gate, up) weight rows -> bf16 (src/nn/swiglu.cpp:36-48,
 // ops::silu_mul src/ops/elementwise.cpp:1297-1328).
 #include "kernels.h"
 
@@ -115,7 +115,17 @@ __device__ __forceinline__ void store_row32(const LinearParams& p, int row, int 
         return;
     }
     const int n_valid = min(32, p.N - col0);
-    if (EPI == VB200_EPI_BF16) {
+    if (EPI == VB200_EPI_RELU2) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) { const float r = fmaxf(__uint_as_float(acc[j]), 0.f); acc[j] = __float_as_uint(r * r); }
+    }
+    if (EPI == VB200_EPI_ADD_F32 && p.addend != nullptr) {
+        const float* ad = p.addend + static_cast<long long>(row) * p.ldo + col0;
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+            if (j < n_valid) acc[j] = __float_as_uint(__uint_as_float(acc[j]) + ad[j]);
+    }
+    if (EPI == VB200_EPI_BF16 || EPI == VB200_EPI_RELU2) {
         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + static_cast<long long>(row) * p.ldo + col0;
         if (n_valid == 32) {
 #pragma unroll
@@ -507,10 +517,13 @@ linear_skinny_kernel(const __grid_constant__ LinearMaps maps, LinearParams p, in
             for (int j = 0; j < MT; ++j) {
                 if (j >= m_count) break;
                 const long long idx = static_cast<long long>(j) * p.ldo + n;
-                if (EPI == VB200_EPI_BF16) static_cast<__nv_bfloat16*>(p.out)[idx] = __float2bfloat16_rn(acc[j]);
+                if (EPI == VB200_EPI_RELU2) {
+                    const float r = fmaxf(acc[j], 0.f);
+                    static_cast<__nv_bfloat16*>(p.out)[idx] = __float2bfloat16_rn(r * r);
+                } else if (EPI == VB200_EPI_BF16) static_cast<__nv_bfloat16*>(p.out)[idx] = __float2bfloat16_rn(acc[j]);
                 else if (EPI == VB200_EPI_F32) static_cast<float*>(p.out)[idx] = acc[j];
                 else {
-                    const float hv = static_cast<float*>(p.out)[idx] + acc[j];
+                    const float hv = static_cast<float*>(p.out)[idx] + (p.addend != nullptr ? acc[j] + p.addend[idx] : acc[j]);
                     static_cast<float*>(p.out)[idx] = hv;
                     if (p.scaled_copy != nullptr)
                         static_cast<__nv_bfloat16*>(p.scaled_copy)[static_cast<long long>(j) * p.N + n] = __float2bfloat16_rn(hv * __ldg(p.copy_scale + n));
@@ -680,6 +693,7 @@ int launch_linear(cudaStream_t s, const LinearParams& p) {
             return VB200_OK;
         }
         case VB200_EPI_SWIGLU: return launch_epi<VB200_EPI_SWIGLU>(s, p);
+        case VB200_EPI_RELU2: return launch_epi<VB200_EPI_RELU2>(s, p);
         default: return set_detail(VB200_ERR_INVALID_ARG, "unknown linear epilogue");
     }
 }

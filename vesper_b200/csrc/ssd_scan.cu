@@ -1,0 +1,290 @@
+// The Mamba-2 mixer around its projections: causal convolution, the recurrence token by token (any sizes, fp32 or bf16;
+// one launch per decode step with the convolution inside), and the gated group RMSNorm.  The chunked form of the
+// recurrence for prompts is in ssd_chunk.cu.
+#include "hybrid.cuh"
+
+namespace vb200 {
+namespace {
+
+struct SsdParams {
+    int B, T, H, P, N, G, taps, channels, Pp;
+    long long ldp;
+    const float *conv_w, *conv_b, *dt_bias, *A_log, *D;
+    const int *slots, *pos;
+    int slices, p4s, rows;      // scan kernel: slices of a head's columns, float4 columns per slice, state rows per pass
+};
+
+constexpr int kConvTile = 32;   // tokens per CTA
+
+// grid (channel blocks, token tiles, B); a thread owns VEC channels.  Only the first tile's CTA reads the state (the
+// inputs ahead of the portion) and it alone writes it, after its own reads.
+template <typename T, int VEC, int TAPS>
+__global__ void __launch_bounds__(128)
+ssd_conv_kernel(SsdParams p, const T* __restrict__ proj, T* __restrict__ state, T* __restrict__ out) {
+    pdl_begin();
+    const int c0 = (blockIdx.x * 128 + threadIdx.x) * VEC;
+    if (c0 >= p.channels) return;
+    const int b = blockIdx.z, t0 = blockIdx.y * kConvTile, t1 = min(p.T, t0 + kConvTile);
+    const int taps = TAPS > 0 ? TAPS : p.taps;
+    const int pos = p.pos[b], slot = p.slots ? p.slots[b] : b;
+    const T* in = proj + static_cast<long long>(b) * p.T * p.ldp + static_cast<long long>(p.H) * p.P + c0;
+    T* st = state + static_cast<long long>(slot) * taps * p.channels + c0;
+    T* o = out + static_cast<long long>(b) * p.T * p.channels + c0;
+    auto fetch = [&](int t, float (&v)[VEC]) {           // the input of portion token t, which may lie ahead of the portion
+        const T* src = t >= 0 ? in + static_cast<long long>(t) * p.ldp
+                              : (pos + t >= 0 ? st + static_cast<long long>((pos + t) % taps) * p.channels : nullptr);
+        if (src == nullptr) {
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) v[j] = 0.f;
+        } else if constexpr (VEC == 8) {
+            load8(src, v);
+        } else {
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) v[j] = Elem<T>::to_f(src[j]);
+        }
+    };
+    auto emit = [&](int t, float (&a)[VEC]) {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) a[j] = silu_exact(a[j]);
+        T* dst = o + static_cast<long long>(t) * p.channels;
+        if constexpr (VEC == 8) store8(dst, a);
+        else {
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) dst[j] = Elem<T>::from_f(a[j]);
+        }
+    };
+    float bias[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) bias[j] = p.conv_b[c0 + j];
+    if constexpr (TAPS > 0) {
+        float w[TAPS][VEC], x[TAPS][VEC];
+#pragma unroll
+        for (int j = 0; j < VEC; ++j)
+#pragma unroll
+            for (int k = 0; k < TAPS; ++k) w[k][j] = p.conv_w[static_cast<long long>(c0 + j) * TAPS + k];
+#pragma unroll
+        for (int k = 0; k < TAPS - 1; ++k) fetch(t0 - (TAPS - 1) + k, x[k]);
+        for (int t = t0; t < t1; ++t) {
+            fetch(t, x[TAPS - 1]);
+            float a[VEC];
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) {
+                a[j] = bias[j];
+#pragma unroll
+                for (int k = 0; k < TAPS; ++k) a[j] = fmaf(w[k][j], x[k][j], a[j]);
+            }
+            emit(t, a);
+#pragma unroll
+            for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) x[k][j] = x[k + 1][j];
+        }
+    } else {
+        for (int t = t0; t < t1; ++t) {
+            float a[VEC];
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) a[j] = bias[j];
+            for (int k = 0; k < taps; ++k) {
+                float v[VEC];
+                fetch(t - (taps - 1) + k, v);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) a[j] = fmaf(p.conv_w[static_cast<long long>(c0 + j) * taps + k], v[j], a[j]);
+            }
+            emit(t, a);
+        }
+    }
+    if (t0 == 0) {
+        for (int t = max(0, p.T - (taps - 1)); t < p.T; ++t) {
+            T* dst = st + static_cast<long long>((pos + t) % taps) * p.channels;
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) dst[j] = in[static_cast<long long>(t) * p.ldp + j];
+        }
+    }
+}
+
+// grid (H * slices, B), 256 threads: thread = one float4 column of the slice x every `rows`-th state row, the state in
+// registers over the whole portion.  STEP: one token, its convolution computed here and its input stored in the ring
+// (nobody reads that ring row in this step).
+template <typename T, int NI, bool STEP>
+__global__ void __launch_bounds__(256)
+ssd_scan_kernel(SsdParams p, const T* __restrict__ proj, const T* __restrict__ xbc, T* __restrict__ conv_state, float* __restrict__ state, float* __restrict__ gated) {
+    pdl_begin();
+    extern __shared__ float sm[];
+    const int h = blockIdx.x / p.slices, sl = blockIdx.x - h * p.slices, b = blockIdx.y;
+    const int g = h / (p.H / p.G), inner = p.H * p.P;
+    const int pos = p.pos[b], slot = p.slots ? p.slots[b] : b;
+    const int pc0 = sl * p.p4s * 4, pcn = min(p.P - pc0, p.p4s * 4);          // this slice's columns
+    const int width = p.p4s * 4, buf_floats = width + 2 * p.N;
+    float* red = sm + 2 * buf_floats;                                          // [rows][width]
+    const int c4 = threadIdx.x % p.p4s, r = threadIdx.x / p.p4s;
+    const bool active = r < p.rows && pc0 + c4 * 4 < p.Pp;
+    float* sp = state + (static_cast<long long>(slot) * p.H + h) * p.N * p.Pp + pc0 + c4 * 4;
+    float4 S[NI];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        const int n = r + i * p.rows;
+        S[i] = active && n < p.N && pos > 0 ? *reinterpret_cast<const float4*>(sp + static_cast<long long>(n) * p.Pp) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const float nA = -expf(p.A_log[h]), dtb = p.dt_bias[h], Dh = p.D[h];
+    for (int t = 0; t < p.T; ++t) {
+        const long long m = static_cast<long long>(b) * p.T + t;
+        const T* prow = proj + m * p.ldp;
+        float* buf = sm + (t & 1) * buf_floats;
+        float *xs = buf, *Bs = buf + width, *Cs = Bs + p.N;
+        for (int i = threadIdx.x; i < width + 2 * p.N; i += 256) {
+            int ch;
+            if (i < width) {
+                if (i >= pcn) { buf[i] = 0.f; continue; }
+                ch = h * p.P + pc0 + i;
+            } else {
+                const int k = i - width;
+                ch = inner + (k < p.N ? g * p.N + k : p.G * p.N + g * p.N + k - p.N);
+            }
+            float v;
+            if constexpr (STEP) {
+                const T cur = prow[inner + ch];
+                T* st = conv_state + static_cast<long long>(slot) * p.taps * p.channels + ch;
+                const float* w = p.conv_w + static_cast<long long>(ch) * p.taps;
+                float a = p.conv_b[ch];
+                for (int k = 0; k < p.taps - 1; ++k) {
+                    const int q = pos - (p.taps - 1) + k;
+                    if (q >= 0) a = fmaf(w[k], Elem<T>::to_f(st[static_cast<long long>(q % p.taps) * p.channels]), a);
+                }
+                a = fmaf(w[p.taps - 1], Elem<T>::to_f(cur), a);
+                v = Elem<T>::to_f(Elem<T>::from_f(silu_exact(a)));
+                if (i < width || (sl == 0 && h % (p.H / p.G) == 0)) st[static_cast<long long>(pos % p.taps) * p.channels] = cur;
+            } else {
+                v = Elem<T>::to_f(xbc[m * p.channels + ch]);
+            }
+            buf[i] = v;
+        }
+        const float dt = softplus_f(Elem<T>::to_f(prow[2 * inner + 2 * p.G * p.N + h]) + dtb), decay = expf(nA * dt);
+        __syncthreads();
+        if (active) {
+            const float4 x4 = *reinterpret_cast<const float4*>(xs + c4 * 4);
+            const float4 dx = make_float4(dt * x4.x, dt * x4.y, dt * x4.z, dt * x4.w);
+            float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int n = r + i * p.rows;
+                if (n < p.N) {
+                    const float bn = Bs[n], cn = Cs[n];
+                    S[i].x = fmaf(decay, S[i].x, bn * dx.x); S[i].y = fmaf(decay, S[i].y, bn * dx.y);
+                    S[i].z = fmaf(decay, S[i].z, bn * dx.z); S[i].w = fmaf(decay, S[i].w, bn * dx.w);
+                    y.x = fmaf(cn, S[i].x, y.x); y.y = fmaf(cn, S[i].y, y.y);
+                    y.z = fmaf(cn, S[i].z, y.z); y.w = fmaf(cn, S[i].w, y.w);
+                }
+            }
+            *reinterpret_cast<float4*>(red + r * width + c4 * 4) = y;
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < pcn; i += 256) {
+            float y = 0.f;
+            for (int k = 0; k < p.rows; ++k) y += red[k * width + i];
+            y = fmaf(Dh, xs[i], y);
+            const int col = h * p.P + pc0 + i;
+            gated[m * inner + col] = y * silu_exact(Elem<T>::to_f(prow[col]));
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        const int n = r + i * p.rows;
+        if (active && n < p.N) *reinterpret_cast<float4*>(sp + static_cast<long long>(n) * p.Pp) = S[i];
+    }
+}
+
+// grid (norm groups, rows), 128 threads.
+template <typename GT, typename T>
+__global__ void __launch_bounds__(128)
+gated_group_norm_kernel(const GT* __restrict__ gated, int inner, int part_len, const float* __restrict__ w, float eps, T* __restrict__ out, long long ldo) {
+    pdl_begin();
+    const long long m = blockIdx.y;
+    const int c0 = blockIdx.x * part_len;
+    const GT* src = gated + m * inner + c0;
+    __shared__ float part[4];
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < part_len; i += 128) { const float v = Elem<GT>::to_f(src[i]); ss += v * v; }
+    const float inv = 1.0f / sqrtf(block_sum<4>(ss, part) / static_cast<float>(part_len) + eps);
+    for (int i = threadIdx.x; i < part_len; i += 128) out[m * ldo + c0 + i] = Elem<T>::from_f(Elem<GT>::to_f(src[i]) * inv * w[c0 + i]);
+}
+
+}  // namespace
+
+SsdPlan plan_ssd(const vb200_ssd_args& a) {
+    SsdPlan pl{};
+    pl.channels = a.H * a.P + 2 * a.G * a.N;
+    pl.Pp = pad_to(a.P, 4);
+    pl.chunked = a.form != 1 && ssd_chunk_supported(a) && (a.form == 2 || a.T >= 16);
+    pl.chunk = 64;
+    pl.n_chunks = (a.T + pl.chunk - 1) / pl.chunk;
+    const size_t esz = a.dtype == VB200_F32 ? 4 : 2, M = static_cast<size_t>(a.B) * a.T;
+    auto up = [](size_t x) { return (x + 255) / 256 * 256; };
+    pl.conv_bytes = a.T > 1 ? up(M * pl.channels * esz) : 0;
+    pl.gated_bytes = up(M * a.H * a.P * (pl.chunked ? 2 : 4));
+    pl.chunk_bytes = pl.chunked ? up(sizeof(float) * (static_cast<size_t>(a.B) * pl.n_chunks * a.H * (static_cast<size_t>(a.N) * pl.Pp + 1))) : 0;
+    pl.total = pl.conv_bytes + pl.gated_bytes + pl.chunk_bytes;
+    return pl;
+}
+
+int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl) {
+    SsdParams p{};
+    p.B = a.B; p.T = a.T; p.H = a.H; p.P = a.P; p.N = a.N; p.G = a.G; p.taps = a.taps; p.channels = pl.channels; p.Pp = pl.Pp;
+    p.ldp = a.ldp; p.conv_w = a.conv_w; p.conv_b = a.conv_b; p.dt_bias = a.dt_bias; p.A_log = a.A_log; p.D = a.D; p.slots = a.slots; p.pos = a.pos;
+    // slices: few enough state rows per thread for registers, and enough CTAs for the machine
+    const int P4 = pl.Pp / 4;
+    int slices = (P4 + 255) / 256;
+    auto per_thread = [&](int sl) { const int w = (P4 + sl - 1) / sl; return (a.N + 256 / w - 1) / (256 / w); };
+    while (slices < P4 && per_thread(slices) > 16) ++slices;
+    if (per_thread(slices) > 16) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_ssd_forward: state size above 4096");
+    while (2 * slices <= P4 && static_cast<long long>(a.B) * a.H * slices * 2 <= device_sm_count()) slices *= 2;
+    p.slices = slices;
+    p.p4s = (P4 + slices - 1) / slices;
+    p.rows = 256 / p.p4s;
+    const int ni = (a.N + p.rows - 1) / p.rows;
+    uint8_t* ws = static_cast<uint8_t*>(a.workspace);
+    void* xbc = ws;
+    void* gated = ws + pl.conv_bytes;
+    float* states = reinterpret_cast<float*>(ws + pl.conv_bytes + pl.gated_bytes);
+    const unsigned M = static_cast<unsigned>(a.B * a.T);
+    const int part_len = a.H * a.P / a.norm_groups;
+
+    auto go = [&](auto tag) -> int {
+        using T = decltype(tag);
+        const T* proj = static_cast<const T*>(a.proj);
+        if (a.T > 1) {
+            const bool vec = (a.H * a.P) % 8 == 0 && p.channels % 8 == 0 && a.ldp % 8 == 0;
+            auto conv = [&](auto kernel, int v) {
+                const dim3 grid(static_cast<unsigned>((p.channels + 128 * v - 1) / (128 * v)), static_cast<unsigned>((a.T + kConvTile - 1) / kConvTile), static_cast<unsigned>(a.B));
+                return launch_pdl(kernel, grid, dim3(128), 0, s, p, proj, static_cast<T*>(a.conv_state), static_cast<T*>(xbc));
+            };
+            const int rc = vec ? (a.taps == 4 ? conv(ssd_conv_kernel<T, 8, 4>, 8) : conv(ssd_conv_kernel<T, 8, 0>, 8))
+                               : (a.taps == 4 ? conv(ssd_conv_kernel<T, 1, 4>, 1) : conv(ssd_conv_kernel<T, 1, 0>, 1));
+            if (rc) return rc;
+        }
+        if constexpr (sizeof(T) == 2) {
+            if (pl.chunked) {
+                if (int rc = launch_ssd_chunks(s, a, pl, xbc, gated, states)) return rc;
+                return launch_pdl(gated_group_norm_kernel<__nv_bfloat16, T>, dim3(static_cast<unsigned>(a.norm_groups), M), dim3(128), 0, s,
+                                  static_cast<const __nv_bfloat16*>(gated), a.H * a.P, part_len, a.norm_w, a.eps, static_cast<T*>(a.out), static_cast<long long>(a.ldo));
+            }
+        }
+        const size_t smem = sizeof(float) * (2 * (p.p4s * 4 + 2 * a.N) + p.rows * p.p4s * 4);
+        const dim3 grid(static_cast<unsigned>(a.H * p.slices), static_cast<unsigned>(a.B));
+        auto scan = [&](auto kernel) -> int {
+            if (int rc = allow_smem(kernel, smem)) return rc;
+            return launch_pdl(kernel, grid, dim3(256), smem, s, p, proj, static_cast<const T*>(xbc), static_cast<T*>(a.conv_state), a.state, static_cast<float*>(gated));
+        };
+        int rc;
+        profile_mark_begin(s);
+        if (a.T == 1) rc = ni <= 4 ? scan(ssd_scan_kernel<T, 4, true>) : ni <= 8 ? scan(ssd_scan_kernel<T, 8, true>) : scan(ssd_scan_kernel<T, 16, true>);
+        else rc = ni <= 4 ? scan(ssd_scan_kernel<T, 4, false>) : ni <= 8 ? scan(ssd_scan_kernel<T, 8, false>) : scan(ssd_scan_kernel<T, 16, false>);
+        profile_mark_end(s);
+        if (rc) return rc;
+        note_ssd_kernel(a.T == 1 ? "ssd_scan_kernel (step)" : "ssd_scan_kernel");
+        return launch_pdl(gated_group_norm_kernel<float, T>, dim3(static_cast<unsigned>(a.norm_groups), M), dim3(128), 0, s, static_cast<const float*>(gated),
+                          a.H * a.P, part_len, a.norm_w, a.eps, static_cast<T*>(a.out), static_cast<long long>(a.ldo));
+    };
+    return a.dtype == VB200_F32 ? go(float{}) : go(__nv_bfloat16{});
+}
+
+}  // namespace vb200

@@ -37,6 +37,7 @@ struct GenerationTimings {
 class Generator {
 public:
     explicit Generator(models::TransformerLM* model) : model_(model) {}
+    explicit Generator(models::LanguageModel* model) : model_(model) {}        // any registered architecture
 
     // prompt_ids [Batch, PromptLen] Int32 / Int64; returns [Batch, PromptLen + generated] Int32 on
     // the prompt's device.
@@ -45,10 +46,10 @@ public:
     void set_use_graph(bool on) { use_graph_ = on; }
     void set_poll_every(int n) { poll_every_ = n > 0 ? n : 1; }
     const GenerationTimings& last_timings() const { return timings_; }
-    models::TransformerLM* model() { return model_; }
+    models::LanguageModel* model() { return model_; }
 
 private:
-    models::TransformerLM* model_;
+    models::LanguageModel* model_;
     bool use_graph_ = true;
     int poll_every_ = 16;
     GenerationTimings timings_;

@@ -13,6 +13,7 @@
 #pragma once
 #include <vesper/core/tensor.h>
 #include <vesper/models/config.h>
+#include <vesper/models/language_model.h>
 #include <vesper/nn/transformer.h>
 
 #include <map>
@@ -22,7 +23,7 @@
 
 namespace vesper::models {
 
-class TransformerLM {
+class TransformerLM : public LanguageModel {
 public:
     explicit TransformerLM(const TransformerConfig& config);
     ~TransformerLM();
@@ -31,40 +32,27 @@ public:
     // tok_embeddings.weight, layers.N.attention_norm.weight, layers.N.attention.wqkv.weight,
     // layers.N.attention.wo.weight, layers.N.ffn_norm.weight, layers.N.feed_forward.{gate,up,down}_proj.weight,
     // norm.weight, output.weight.
-    std::map<std::string, std::vector<int64_t>> parameter_shapes() const;
+    std::map<std::string, std::vector<int64_t>> parameter_shapes() const override;
     // Loads one parameter from host fp32 values (rounded to bf16 for matrices; norm weights stay fp32).
-    void load_parameter(const std::string& name, const float* host_values, int64_t numel);
+    void load_parameter(const std::string& name, const float* host_values, int64_t numel) override;
 
     // tokens [Batch, NewTokens] Int32 or Int64 (CPU or CUDA); returns fp32 logits
     // [Batch, NewTokens, Vocab], or [Batch, 1, Vocab] for the last position when last_only.
-    Tensor forward_with_cache(const Tensor& tokens, int64_t start_pos, bool last_only = false);
+    Tensor forward_with_cache(const Tensor& tokens, int64_t start_pos, bool last_only = false) override;
 
-    void init_cache(int64_t batch_size, Device device);
-    void clear_cache();
+    void init_cache(int64_t batch_size, Device device) override;
+    void clear_cache() override;
     bool has_cache() const { return !kv_caches_.empty(); }
     const TransformerConfig& config() const { return config_; }
     int64_t num_parameters() const;
 
-    // ---- device-resident decode step, used by generation::Generator ----
-    // One greedy decode step for the whole batch with no host round trip: embeds ids_dev
-    // [Batch] int32, runs every block at the per-sequence positions in the device length array
-    // (advanced by one inside), writes logits and the arg-max ids back into ids_dev; appends the new
-    // id to history_dev [Batch, history_ld] at column = the new length and updates done_dev.
-    // All launches go to the current stream and are CUDA-graph capturable after one eager call.
-    struct DecodeState {
-        Tensor ids;        // [B] int32: in = token to process, out = next token
-        Tensor lens;       // [B] int32: cached length per sequence
-        Tensor history;    // [B, history_ld] int32
-        Tensor done;       // [B] int32
-        Tensor stop_ids;   // [n_stop] int32 (may be undefined)
-        int64_t prompt_len = 0;
-        int64_t min_new_tokens = 0;
-        int64_t max_len = 0;          // upper bound of any sequence length during the loop (plans the split-KV launch)
-    };
-    void decode_step(DecodeState& st);
-    // Greedy pick on the logits of the last forward_with_cache(..., last_only=true) call: writes
-    // st.ids, st.history[:, lens], st.done.
-    void pick_from_last_logits(DecodeState& st);
+    int64_t vocab_size() const override { return config_.vocab_size; }
+    int64_t max_seq_len() const override { return config_.max_seq_len; }
+    bool device_decode() const override { return config_.head_dim() == 128; }
+    void decode_step(DecodeState& st) override;
+
+protected:
+    const Tensor& last_logits() const override;
 
 private:
     struct Layer;

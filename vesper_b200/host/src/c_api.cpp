@@ -1,7 +1,9 @@
-// extern "C" facade over models::TransformerLM and generation::Generator for harnesses that
+// extern "C" facade over models::LanguageModel (any registered architecture) and generation::Generator for harnesses that
 // cannot include C++ headers (the Python tests and the benchmark bind it with ctypes).  Host
 // arrays in, host arrays out; errors come back as -1 with the text in vbh_last_error().
 #include <vesper/generation/generator.h>
+#include <vesper/models/hybrid.h>
+#include <vesper/models/language_model.h>
 #include <vesper/models/transformer.h>
 #include <vesper/nn/gqa_attention.h>
 
@@ -11,6 +13,9 @@
 using vesper::Device;
 using vesper::DType;
 using vesper::Tensor;
+using vesper::models::HybridLM;
+using vesper::models::LanguageModel;
+using vesper::models::LoadOptions;
 using vesper::models::TransformerConfig;
 using vesper::models::TransformerLM;
 
@@ -100,24 +105,91 @@ void* vbh_model_new(int64_t vocab, int64_t dim, int64_t n_layers, int64_t n_head
         TransformerConfig c;
         c.vocab_size = vocab; c.dim = dim; c.n_layers = n_layers; c.n_heads = n_heads; c.n_kv_heads = n_kv_heads;
         c.ffn_hidden_dim = ffn_hidden; c.max_seq_len = max_seq_len; c.norm_eps = norm_eps; c.rope_base = rope_base;
-        return new TransformerLM(c);
+        return static_cast<LanguageModel*>(new TransformerLM(c));
     } catch (const std::exception& e) { g_err = e.what(); return nullptr; }
 }
-void vbh_model_free(void* m) { delete static_cast<TransformerLM*>(m); }
+// Any registered architecture: from a folder with config.json and model.safetensors, or from the text of a configuration
+// (weights then come through vbh_model_set_param).  f32: Float32 instead of BFloat16.
+static LoadOptions load_options(int f32, int64_t max_seq_len, int64_t max_sequences) {
+    LoadOptions o;
+    o.dtype = f32 ? DType::Float32 : DType::BFloat16;
+    o.max_seq_len = max_seq_len;
+    if (max_sequences > 0) o.max_sequences = max_sequences;
+    return o;
+}
+void* vbh_model_load(const char* folder, int f32, int64_t max_seq_len, int64_t max_sequences) {
+    try { return vesper::models::load_model(folder, load_options(f32, max_seq_len, max_sequences)).release(); }
+    catch (const std::exception& e) { g_err = e.what(); return nullptr; }
+}
+void* vbh_model_from_config(const char* text, int f32, int64_t max_seq_len, int64_t max_sequences) {
+    try { return vesper::models::make_model(vesper::Json::parse(text), load_options(f32, max_seq_len, max_sequences)).release(); }
+    catch (const std::exception& e) { g_err = e.what(); return nullptr; }
+}
+int64_t vbh_model_vocab(void* m) { return static_cast<LanguageModel*>(m)->vocab_size(); }
+// "name d0 d1 ...\n" per parameter; returns the length, writes at most `room` bytes.
+int64_t vbh_model_parameters(void* m, char* out, int64_t room) {
+    std::string s;
+    for (const auto& kv : static_cast<LanguageModel*>(m)->parameter_shapes()) {
+        s += kv.first;
+        for (int64_t d : kv.second) s += " " + std::to_string(d);
+        s += "\n";
+    }
+    if (out && room > static_cast<int64_t>(s.size())) std::memcpy(out, s.c_str(), s.size() + 1);
+    return static_cast<int64_t>(s.size());
+}
+int64_t vbh_sequence_open(void* m) {
+    try { return static_cast<LanguageModel*>(m)->open_sequence(); }
+    catch (const std::exception& e) { g_err = e.what(); return -1; }
+}
+int vbh_sequence_close(void* m, int64_t seq) {
+    try { static_cast<LanguageModel*>(m)->close_sequence(seq); return 0; }
+    catch (const std::exception& e) { g_err = e.what(); return -1; }
+}
+// logits_host: [n_rows, vocab] fp32, the rows of this call's tokens that `rows` lists (none wanted: n_rows = 0)
+int vbh_sequence_extend(void* m, int64_t seq, const int32_t* ids_host, int64_t T, const int64_t* rows, int64_t n_rows, float* logits_host) {
+    try {
+        auto* lm = static_cast<LanguageModel*>(m);
+        Tensor y = lm->extend(seq, ids_to_device(ids_host, 1, T)).view({T, lm->vocab_size()});
+        for (int64_t i = 0; i < n_rows; ++i) {
+            if (rows[i] < 0 || rows[i] >= T) throw std::runtime_error("vbh_sequence_extend: row out of range");
+            y.narrow(0, rows[i], 1).copy_to_host(logits_host + i * lm->vocab_size());
+        }
+        if (n_rows == 0) vesper::Stream::current(Device::CUDA).synchronize();
+        return 0;
+    } catch (const std::exception& e) { g_err = e.what(); return -1; }
+}
+// Hybrid decoders: the residual stream after every layer execution of one forward call, [executions, B * T, width].
+int64_t vbh_model_layer_executions(void* m) {
+    auto* h = dynamic_cast<HybridLM*>(static_cast<LanguageModel*>(m));
+    return h ? h->layer_executions() : 0;
+}
+int vbh_model_forward_tapped(void* m, const int32_t* ids_host, int64_t B, int64_t T, int64_t start_pos, float* logits_host, float* tap_host) {
+    try {
+        auto* h = dynamic_cast<HybridLM*>(static_cast<LanguageModel*>(m));
+        if (!h) throw std::runtime_error("layer taps are available for hybrid decoders");
+        Tensor tap = vesper::empty({h->layer_executions(), B * T, h->config().width}, DType::Float32, Device::CUDA);
+        struct Off { HybridLM* h; ~Off() { h->set_layer_tap(Tensor()); } } off{h};
+        h->set_layer_tap(tap);
+        h->forward_with_cache(ids_to_device(ids_host, B, T), start_pos).copy_to_host(logits_host);
+        tap.copy_to_host(tap_host);
+        return 0;
+    } catch (const std::exception& e) { g_err = e.what(); return -1; }
+}
+void vbh_model_free(void* m) { delete static_cast<LanguageModel*>(m); }
 
 int vbh_model_set_param(void* m, const char* name, const float* data, int64_t numel) {
-    try { static_cast<TransformerLM*>(m)->load_parameter(name, data, numel); return 0; }
+    try { static_cast<LanguageModel*>(m)->load_parameter(name, data, numel); return 0; }
     catch (const std::exception& e) { g_err = e.what(); return -1; }
 }
 int vbh_model_init_cache(void* m, int64_t B) {
-    try { static_cast<TransformerLM*>(m)->init_cache(B, Device::CUDA); return 0; }
+    try { static_cast<LanguageModel*>(m)->init_cache(B, Device::CUDA); return 0; }
     catch (const std::exception& e) { g_err = e.what(); return -1; }
 }
 // logits_host: [B, T, vocab] fp32, or [B, 1, vocab] when last_only
 int vbh_model_forward_with_cache(void* m, const int32_t* ids_host, int64_t B, int64_t T, int64_t start_pos,
                                  int last_only, float* logits_host) {
     try {
-        Tensor y = static_cast<TransformerLM*>(m)->forward_with_cache(ids_to_device(ids_host, B, T), start_pos, last_only != 0);
+        Tensor y = static_cast<LanguageModel*>(m)->forward_with_cache(ids_to_device(ids_host, B, T), start_pos, last_only != 0);
         y.copy_to_host(logits_host);
         return 0;
     } catch (const std::exception& e) { g_err = e.what(); return -1; }
@@ -128,7 +200,7 @@ int64_t vbh_generate_greedy(void* m, const int32_t* prompt_host, int64_t B, int6
                             const int64_t* stop_ids, int64_t n_stop, int64_t min_new, int use_graph,
                             int32_t* out_host, double* timings) {
     try {
-        vesper::generation::Generator gen(static_cast<TransformerLM*>(m));
+        vesper::generation::Generator gen(static_cast<LanguageModel*>(m));
         gen.set_use_graph(use_graph != 0);
         vesper::generation::SamplingParams sp;
         sp.do_sample = false;

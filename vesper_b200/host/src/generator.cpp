@@ -26,8 +26,8 @@ Tensor Generator::generate(const Tensor& prompt_ids, const SamplingParams& param
     if (params.do_sample) throw std::runtime_error("Generator: only greedy decoding (do_sample = false) is built on this path");
     if (params.repetition_penalty != 1.0f) throw std::runtime_error("Generator: repetition_penalty is not part of this path");
     const int64_t B = prompt_ids.shape()[0], P = prompt_ids.shape()[1], max_new = params.max_new_tokens;
-    const auto& cfg = model_->config();
-    if (P + max_new > cfg.max_seq_len) throw std::runtime_error("Total sequence length would exceed model's max_seq_len");
+    const bool device_decode = model_->device_decode();
+    if (P + max_new > model_->max_seq_len()) throw std::runtime_error("Total sequence length would exceed model's max_seq_len");
     const Device out_device = prompt_ids.device();
     // the loop runs on a stream of its own (the legacy default stream cannot be captured into a graph);
     // work already queued on the caller's stream is waited for first, and the caller's stream is current
@@ -43,7 +43,7 @@ Tensor Generator::generate(const Tensor& prompt_ids, const SamplingParams& param
     model_->init_cache(B, Device::CUDA);
 
     // device-resident loop state
-    models::TransformerLM::DecodeState st;
+    models::LanguageModel::DecodeState st;
     st.ids = zeros({B}, DType::Int32, Device::CUDA);
     st.done = zeros({B}, DType::Int32, Device::CUDA);
     st.history = zeros({B, P + max_new}, DType::Int32, Device::CUDA);
@@ -87,7 +87,7 @@ Tensor Generator::generate(const Tensor& prompt_ids, const SamplingParams& param
     cuda_check(cudaEventRecord(pre.b, stream), "cudaEventRecord");
 
     // decode: step i feeds the token picked at step i-1 (position P + i - 1) and picks the next
-    const bool graph_ok = use_graph_ && cfg.head_dim() == 128 && max_new > 2;
+    const bool graph_ok = use_graph_ && device_decode && max_new > 2;
     cudaGraph_t graph = nullptr;
     cudaGraphExec_t exec = nullptr;
     std::vector<int32_t> done_host(static_cast<size_t>(B));
@@ -100,8 +100,8 @@ Tensor Generator::generate(const Tensor& prompt_ids, const SamplingParams& param
     bool stopped = max_new > 0 && !params.stop_token_ids.empty() && all_done();
     int64_t steps = 0;
     while (!stopped && generated < max_new) {
-        if (cfg.head_dim() != 128) {
-            // host-positioned fallback for head sizes without the device-position decode kernel
+        if (!device_decode) {
+            // host-positioned steps for models without a device-position decode step
             Tensor tok = st.ids.view({B, 1});
             model_->forward_with_cache(tok, P + generated - 1, true);
             std::vector<int32_t> lens(static_cast<size_t>(B), static_cast<int32_t>(P + generated));

@@ -340,30 +340,7 @@ Tensor TransformerLM::forward_with_cache(const Tensor& tokens, int64_t start_pos
     return out;
 }
 
-void TransformerLM::pick_from_last_logits(DecodeState& st) {
-    Buffers& b = *buf_;
-    const int64_t B = st.ids.shape()[0];
-    vb200_greedy_args g{};
-    g.struct_size = sizeof(g);
-    g.device = b.h.device_index();
-    g.stream = current_stream();
-    g.logits = b.logits.data_ptr<float>();
-    g.ld_logits = config_.vocab_size;
-    g.B = static_cast<int>(B);
-    g.vocab = static_cast<int>(config_.vocab_size);
-    g.out_ids = st.ids.data_ptr<int32_t>();
-    g.history = st.history.data_ptr<int32_t>();
-    g.history_ld = st.history.strides()[0];
-    g.pos_dev = st.lens.data_ptr<int32_t>();
-    g.pos_base = static_cast<int>(st.prompt_len);
-    if (st.stop_ids.defined() && st.stop_ids.numel() > 0) {
-        g.stop_ids = st.stop_ids.data_ptr<int32_t>();
-        g.n_stop = static_cast<int>(st.stop_ids.numel());
-    }
-    g.min_new_tokens = static_cast<int>(st.min_new_tokens);
-    g.done = st.done.data_ptr<int32_t>();
-    check(vb200_greedy_step(&g), "greedy_step");
-}
+const Tensor& TransformerLM::last_logits() const { return buf_->logits; }
 
 void TransformerLM::decode_step(DecodeState& st) {
     if (kv_caches_.empty()) throw std::runtime_error("KV cache not initialized. Call init_cache first.");

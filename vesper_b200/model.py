@@ -1,9 +1,10 @@
-"""ctypes binding of the C facade of the host layer (libvesper_b200_host.so: models::TransformerLM
+"""ctypes binding of the C facade of the host layer (libvesper_b200_host.so: models::LanguageModel
 and generation::Generator, vesper_b200/host/src/c_api.cpp) for the Python tests and the benchmark.
 Every computation happens in the CUDA library underneath; there is no fallback."""
 from __future__ import annotations
 
 import ctypes as C
+import json
 import os
 
 import numpy as np
@@ -13,7 +14,9 @@ HOST_LIB_PATH = os.path.join(PKG, "lib", "libvesper_b200_host.so")
 
 HOST_EXPORTS = ["vbh_last_error", "vbh_model_new", "vbh_model_free", "vbh_model_set_param", "vbh_model_init_cache",
                 "vbh_model_forward_with_cache", "vbh_generate_greedy", "vbh_attn_new", "vbh_attn_free", "vbh_attn_load",
-                "vbh_kvcache_new", "vbh_kvcache_free", "vbh_kvcache_len", "vbh_attn_forward"]
+                "vbh_kvcache_new", "vbh_kvcache_free", "vbh_kvcache_len", "vbh_attn_forward",
+                "vbh_model_load", "vbh_model_from_config", "vbh_model_vocab", "vbh_model_parameters", "vbh_sequence_open", "vbh_sequence_close",
+                "vbh_sequence_extend", "vbh_model_layer_executions", "vbh_model_forward_tapped"]
 
 _host = None
 _i64 = C.c_int64
@@ -48,6 +51,17 @@ def load_host():
     L.vbh_kvcache_free.argtypes = [C.c_void_p]
     L.vbh_kvcache_len.argtypes = [C.c_void_p]
     L.vbh_attn_forward.argtypes = [C.c_void_p, _f32p, _i64, _i64, _i64, C.c_int, C.c_int, C.c_void_p, _i64, _f32p]
+    for name in ("vbh_model_load", "vbh_model_from_config"):
+        getattr(L, name).argtypes = [C.c_char_p, C.c_int, _i64, _i64]
+        getattr(L, name).restype = C.c_void_p
+    for name in ("vbh_model_vocab", "vbh_sequence_open", "vbh_model_layer_executions"):
+        getattr(L, name).argtypes = [C.c_void_p]
+        getattr(L, name).restype = _i64
+    L.vbh_model_parameters.argtypes = [C.c_void_p, C.c_char_p, _i64]
+    L.vbh_model_parameters.restype = _i64
+    L.vbh_sequence_close.argtypes = [C.c_void_p, _i64]
+    L.vbh_sequence_extend.argtypes = [C.c_void_p, _i64, _i32p, _i64, C.POINTER(_i64), _i64, _f32p]
+    L.vbh_model_forward_tapped.argtypes = [C.c_void_p, _i32p, _i64, _i64, _i64, _f32p, _f32p]
     _host = L
     return L
 
@@ -68,14 +82,15 @@ def param_shapes(vocab, dim, n_layers, n_heads, n_kv_heads, ffn_hidden):
     return out
 
 
-class TransformerLM:
-    def __init__(self, vocab, dim, n_layers, n_heads, n_kv_heads, ffn_hidden, max_seq_len, norm_eps=1e-6, rope_base=10000.0):
+class LanguageModel:
+    """A decoder of the host layer (models::LanguageModel), whatever its architecture: see load_model / model_from_config."""
+
+    def __init__(self, handle):
         self.L = load_host()
-        self.vocab = vocab
-        self.cfg = dict(vocab=vocab, dim=dim, n_layers=n_layers, n_heads=n_heads, n_kv_heads=n_kv_heads, ffn_hidden=ffn_hidden)
-        self.h = self.L.vbh_model_new(vocab, dim, n_layers, n_heads, n_kv_heads, ffn_hidden, max_seq_len, norm_eps, rope_base)
+        self.h = handle
         if not self.h:
             raise RuntimeError(self.L.vbh_last_error().decode())
+        self.vocab = self.L.vbh_model_vocab(self.h)
 
     def _chk(self, rc):
         if rc < 0:
@@ -83,7 +98,10 @@ class TransformerLM:
         return rc
 
     def param_shapes(self):
-        return param_shapes(**self.cfg)
+        n = self.L.vbh_model_parameters(self.h, None, 0)
+        buf = C.create_string_buffer(n + 1)
+        self.L.vbh_model_parameters(self.h, buf, n + 1)
+        return {f[0]: tuple(int(d) for d in f[1:]) for f in (line.split() for line in buf.value.decode().splitlines())}
 
     def set_param(self, name, value):
         value = np.ascontiguousarray(value, dtype=np.float32)
@@ -98,6 +116,31 @@ class TransformerLM:
         y = np.empty((B, 1 if last_only else T, self.vocab), np.float32)
         self._chk(self.L.vbh_model_forward_with_cache(self.h, ids.ctypes.data_as(_i32p), B, T, start_pos, int(last_only), y.ctypes.data_as(_f32p)))
         return y
+
+    # sequences one at a time, each with cache / state of its own
+    def open_sequence(self):
+        return self._chk(self.L.vbh_sequence_open(self.h))
+
+    def extend(self, seq, ids, rows=None):
+        """Feeds the sequence's next tokens; fp32 logits [len(rows), vocab] of the listed ones (default: all)."""
+        ids = np.ascontiguousarray(ids, dtype=np.int32)
+        rows = np.ascontiguousarray(range(len(ids)) if rows is None else rows, dtype=np.int64)
+        y = np.empty((len(rows), self.vocab), np.float32)
+        self._chk(self.L.vbh_sequence_extend(self.h, seq, ids.ctypes.data_as(_i32p), len(ids), rows.ctypes.data_as(C.POINTER(_i64)), len(rows),
+                                              y.ctypes.data_as(_f32p)))
+        return y
+
+    def close_sequence(self, seq):
+        self._chk(self.L.vbh_sequence_close(self.h, seq))
+
+    def forward_tapped(self, ids, start_pos, width):
+        """forward_with_cache plus the residual stream after every layer execution [executions, B, T, width] (hybrid decoders)."""
+        ids = np.ascontiguousarray(ids, dtype=np.int32)
+        B, T = ids.shape
+        y = np.empty((B, T, self.vocab), np.float32)
+        tap = np.empty((self.L.vbh_model_layer_executions(self.h), B, T, width), np.float32)
+        self._chk(self.L.vbh_model_forward_tapped(self.h, ids.ctypes.data_as(_i32p), B, T, start_pos, y.ctypes.data_as(_f32p), tap.ctypes.data_as(_f32p)))
+        return y, tap
 
     def generate_greedy(self, prompt, max_new, stop_ids=(), min_new=0, use_graph=True):
         """Returns (tokens [B, P + generated] int32, timings dict)."""
@@ -118,6 +161,25 @@ class TransformerLM:
 
     def __del__(self):
         self.close()
+
+
+class TransformerLM(LanguageModel):
+    def __init__(self, vocab, dim, n_layers, n_heads, n_kv_heads, ffn_hidden, max_seq_len, norm_eps=1e-6, rope_base=10000.0):
+        cfg = dict(vocab=vocab, dim=dim, n_layers=n_layers, n_heads=n_heads, n_kv_heads=n_kv_heads, ffn_hidden=ffn_hidden)
+        self.cfg = cfg
+        super().__init__(load_host().vbh_model_new(vocab, dim, n_layers, n_heads, n_kv_heads, ffn_hidden, max_seq_len, norm_eps, rope_base))
+
+
+def load_model(folder, dtype="bfloat16", max_seq_len=0, max_sequences=0):
+    """A model folder (config.json, model.safetensors); the class comes from the configuration's "architecture"."""
+    L = load_host()
+    return LanguageModel(L.vbh_model_load(os.fsencode(folder), int(dtype == "float32"), max_seq_len, max_sequences))
+
+
+def model_from_config(config, dtype="bfloat16", max_seq_len=0, max_sequences=0):
+    """A model of a registered architecture from a configuration dict, weights to be set with set_param."""
+    L = load_host()
+    return LanguageModel(L.vbh_model_from_config(json.dumps(config).encode(), int(dtype == "float32"), max_seq_len, max_sequences))
 
 
 def _fp(a):
