@@ -1,6 +1,8 @@
 // extern "C" entry points of vesper_b200_hybrid.h: argument validation and orchestration.
 #include "hybrid.cuh"
 
+#include <cstdio>
+
 namespace vb200 {
 
 namespace {
@@ -24,6 +26,31 @@ int device_sm_count() {
         cache[dev] = n;
     }
     return cache[dev];
+}
+
+int make_map_4d(CUtensorMap* m, const void* ptr, int c, int heads, long long rows, int batch, long long head_stride, long long row_stride, long long batch_stride,
+                int box_rows) {
+    using Encode = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*, const cuuint32_t*,
+                                CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+    static Encode encode = []() -> Encode {
+        void* fn = nullptr;
+        cudaDriverEntryPointQueryResult q;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &q) != cudaSuccess || q != cudaDriverEntryPointSuccess) return nullptr;
+        return reinterpret_cast<Encode>(fn);
+    }();
+    if (!encode) return set_detail(VB200_ERR_CUDA, "cuTensorMapEncodeTiled is not available from the driver");
+    const cuuint64_t dims[4] = {static_cast<cuuint64_t>(c), static_cast<cuuint64_t>(heads), static_cast<cuuint64_t>(rows), static_cast<cuuint64_t>(batch)};
+    const cuuint64_t strides[3] = {static_cast<cuuint64_t>(head_stride) * 2, static_cast<cuuint64_t>(row_stride) * 2, static_cast<cuuint64_t>(batch_stride) * 2};
+    const cuuint32_t box[4] = {64, 1, static_cast<cuuint32_t>(box_rows), 1};
+    const cuuint32_t es[4] = {1, 1, 1, 1};
+    const CUresult r = encode(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(ptr), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                              CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) {
+        static thread_local char buf[96];
+        snprintf(buf, sizeof(buf), "cuTensorMapEncodeTiled failed with CUresult %d", static_cast<int>(r));
+        return set_detail(VB200_ERR_CUDA, buf);
+    }
+    return VB200_OK;
 }
 
 namespace {

@@ -177,6 +177,16 @@ __device__ __forceinline__ bool mbar_wait_warp(uint64_t* bar, uint32_t parity, c
     return __all_sync(0xFFFFFFFFu, ok);
 }
 
+// After an expired wait the CTA leaves early while bulk copies it issued may still be landing in
+// its shared memory: stay resident for a bounded time (far longer than a copy takes) before exiting.
+__device__ __forceinline__ void abort_linger(volatile int* abort_flag) {
+    if (*abort_flag && threadIdx.x == 0) {
+        const long long t0 = clock64();
+        while (clock64() - t0 < 2000000LL) {}
+    }
+    __syncthreads();
+}
+
 // ---- proxy / tcgen05 fences ----
 __device__ __forceinline__ void fence_proxy_async_smem() {
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");

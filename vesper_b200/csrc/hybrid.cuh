@@ -34,6 +34,10 @@ int allow_smem(Kernel kernel, size_t bytes) {
     return VB200_OK;
 }
 
+// bf16 4-D tensor map (c, h, row, batch) over strided memory (strides in elements), box [64 c][1][box_rows][1], 128-byte
+// swizzle; reads past an extent return zeros.  Base and strides must be multiples of 16 bytes.
+int make_map_4d(CUtensorMap* m, const void* ptr, int c, int heads, long long rows, int batch, long long head_stride, long long row_stride, long long batch_stride,
+                int box_rows);                   // api_hybrid.cu
 int device_sm_count();                           // api_hybrid.cu
 void note_latent_kernel(const char* name);
 void note_ssd_kernel(const char* name);
@@ -66,11 +70,11 @@ int launch_latent_split_mma(cudaStream_t s, const vb200_latent_args& a, const La
 struct SsdPlan {
     int channels, Pp;
     bool chunked;
-    int chunk, n_chunks;
     size_t conv_bytes, gated_bytes, chunk_bytes, total;     // conv output | gated y | chunk states
 };
 SsdPlan plan_ssd(const vb200_ssd_args& a);
 bool ssd_chunk_supported(const vb200_ssd_args& a);
+void plan_ssd_chunks(const vb200_ssd_args& a, int* slices, int* n_seg, int* seg_chunks);          // ssd_chunk.cu
 int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl);
 int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, const void* xbc, void* gated, float* states);   // ssd_chunk.cu
 

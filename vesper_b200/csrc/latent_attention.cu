@@ -41,6 +41,10 @@ __device__ void latent_row(const LatentParams& p, const T* __restrict__ src, con
         if (ring_row != nullptr) ring_row[i] = v;
         if (ctx_row != nullptr) ctx_row[i] = v;
     }
+    for (int i = p.rank + threadIdx.x; i < p.rot_off; i += W * 32) {      // context rows feed a product over the padded width
+        if (old_copy != nullptr) old_copy[i] = Elem<T>::from_f(0.f);
+        if (ctx_row != nullptr) ctx_row[i] = Elem<T>::from_f(0.f);
+    }
     const int half = p.rot / 2;
     for (int i = threadIdx.x; i < half; i += W * 32) {
         const float u = Elem<T>::to_f(src[p.rank + i]), v = Elem<T>::to_f(src[p.rank + half + i]);

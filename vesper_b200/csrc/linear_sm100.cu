@@ -47,15 +47,6 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
           "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
         : "r"(taddr) : "memory");
 }
-// After an expired wait the CTA leaves early while bulk copies it issued may still be landing in
-// its shared memory: stay resident for a bounded time (far longer than a copy takes) before exiting.
-__device__ __forceinline__ void abort_linger(volatile int* abort_flag) {
-    if (*abort_flag && threadIdx.x == 0) {
-        const long long t0 = clock64();
-        while (clock64() - t0 < 2000000LL) {}
-    }
-    __syncthreads();
-}
 // 32-byte global accesses (sm_100): half as many store instructions per row segment as 16-byte ones.  The
 // interface promises 16-byte alignment only, so a segment that is not 32-byte aligned goes as two halves.
 __device__ __forceinline__ void st_global_v8(void* ptr, const uint32_t (&w)[8]) {

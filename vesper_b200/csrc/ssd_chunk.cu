@@ -1,5 +1,316 @@
+// The Mamba-2 recurrence over a prompt in chunks of 64 tokens, as matrix products (bf16 inputs):
+//
+//   la_i = log2 of the decay from the chunk's start through token i        (fp32 running sum of -exp(A) dt)
+//   y_i  = 2^la_i C_i S  +  sum_{j <= i} (C_i . B_j) 2^(la_i - la_j) dt_j x_j  +  D x_i
+//   S   <- 2^la_last S   +  sum_j 2^(la_last - la_j) dt_j B_j x_j^T
+//
+// One CTA of four warps walks the chunks of one (batch, head, column slice) with S in its MMA accumulators: warp-level
+// m16n8k16 products, fp32 accumulation.  C, B and x are bf16 values as they come from the convolution; everything the
+// decays touch (the weights of the second sum, the weighted B of the state update, S itself as a right operand) enters
+// as hi + lo bf16 halves, so the recurrence keeps fp32-class accuracy.
+// When batch x heads does not fill the machine the portion is cut into segments: a first pass computes what each
+// segment adds to the state, a small kernel chains them, and the walk starts every segment from its own state.
 #include "hybrid.cuh"
+
 namespace vb200 {
-bool ssd_chunk_supported(const vb200_ssd_args&) { return false; }
-int launch_ssd_chunks(cudaStream_t, const vb200_ssd_args&, const SsdPlan&, const void*, void*, float*) { return VB200_ERR_UNSUPPORTED; }
+namespace {
+
+constexpr int kChunk = 64;
+constexpr int kPad = 8;                  // bf16 of row padding: ldmatrix rows fall into distinct banks
+
+struct ChunkParams {
+    int T, H, P, N, G, channels, Pp, N16, slices, pw;       // pw: columns per slice
+    int n_seg, seg_chunks;
+    long long ldp;
+    const __nv_bfloat16 *proj, *xbc;
+    const float *dt_bias, *A_log, *D;
+    const int *slots, *pos;
+    float* state;                        // [slots, H, N, Pp]
+    float *seg_state, *seg_decay;        // [B, n_seg, H, N, Pp], [B, n_seg, H] (n_seg > 1)
+    __nv_bfloat16* gated;                // [B*T, H * P]
+};
+
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+__device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], const __nv_bfloat16* ptr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(ptr)) : "memory");
+}
+__device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], const __nv_bfloat16* ptr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(ptr)) : "memory");
+}
+
+// MT: 16-row tiles of S per warp (rows dealt to the four warps in turn); PT: 8-column tiles of the slice.
+// OUT: the walk (outputs and, in the last segment, the final state); else the first pass (what a segment adds to S).
+template <int MT, int PT, bool OUT>
+__global__ void __launch_bounds__(128)
+ssd_chunk_kernel(ChunkParams p) {
+    pdl_begin();
+    extern __shared__ __align__(16) uint8_t smem[];
+    const int ldn = p.N16 + kPad;
+    constexpr int kPw = PT * 8, ldp_s = kPw + kPad;
+    __nv_bfloat16* Bs = reinterpret_cast<__nv_bfloat16*>(smem);        // [64][ldn]
+    __nv_bfloat16* xs = Bs + kChunk * ldn;                             // [64][ldp_s]
+    __nv_bfloat16* Cs = xs + kChunk * ldp_s;                           // [64][ldn]
+    __nv_bfloat16* Sh = Cs + kChunk * ldn;                             // [N16][ldp_s] high halves, then low halves
+    __nv_bfloat16* Sl = Sh + p.N16 * ldp_s;
+    __shared__ float la[kChunk], dtv[kChunk], wv[kChunk];
+
+    const int seg = blockIdx.x, h = blockIdx.y / p.slices, sl = blockIdx.y % p.slices, b = blockIdx.z;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3, mi = lane >> 3, mr = lane & 7;
+    const int grp = h / (p.H / p.G), inner = p.H * p.P, p0 = sl * kPw, pn = min(p.P - p0, kPw);
+    const int slot = p.slots ? p.slots[b] : b;
+    const float nA2 = -expf(p.A_log[h]) * kLog2e, dtb = p.dt_bias[h], Dh = OUT ? p.D[h] : 0.f;
+    const long long seg_row = (static_cast<long long>(b) * p.n_seg + seg) * p.H + h;
+
+    // rows mt*16 + g, +8 and columns p0 + pt*8 + 2*t4 of the state
+    float S[MT][PT][4];
+    float* sp = p.state + (static_cast<long long>(slot) * p.H + h) * p.N * p.Pp + p0;
+    {
+        const float* src = nullptr;
+        if (OUT) src = p.n_seg > 1 ? p.seg_state + seg_row * p.N * p.Pp + p0 : (p.pos[b] > 0 ? sp : nullptr);
+#pragma unroll
+        for (int i = 0; i < MT; ++i)
+#pragma unroll
+            for (int x = 0; x < PT; ++x)
+#pragma unroll
+                for (int hf = 0; hf < 2; ++hf) {
+                    const int n = (warp + 4 * i) * 16 + g + hf * 8, c = x * 8 + t4 * 2;
+                    float2 v = make_float2(0.f, 0.f);
+                    if (src != nullptr && n < p.N && c < pn) v = *reinterpret_cast<const float2*>(src + static_cast<long long>(n) * p.Pp + c);
+                    S[i][x][hf * 2] = v.x; S[i][x][hf * 2 + 1] = v.y;
+                }
+    }
+    float log_decay = 0.f;
+    const int c_begin = seg * p.seg_chunks, c_end = min((p.T + kChunk - 1) / kChunk, c_begin + p.seg_chunks);
+    for (int ch = c_begin; ch < c_end; ++ch) {
+        const int t0 = ch * kChunk, tn = min(kChunk, p.T - t0);
+        const long long m0 = static_cast<long long>(b) * p.T + t0;
+        const __nv_bfloat16* src = p.xbc + m0 * p.channels;
+        // ---- tiles: 16-byte pieces, zero past the portion and past a matrix's width ----
+        const int nv = p.N16 / 8, pv = kPw / 8;
+        for (int i = threadIdx.x; i < kChunk * nv; i += 128) {
+            const int r = i / nv, c = (i - r * nv) * 8;
+            const bool ok = r < tn && c < p.N;
+            const __nv_bfloat16* q = src + static_cast<long long>(r) * p.channels + inner + grp * p.N + c;
+            *reinterpret_cast<uint4*>(Bs + r * ldn + c) = ok ? *reinterpret_cast<const uint4*>(q) : make_uint4(0, 0, 0, 0);
+            if (OUT) *reinterpret_cast<uint4*>(Cs + r * ldn + c) = ok ? *reinterpret_cast<const uint4*>(q + p.G * p.N) : make_uint4(0, 0, 0, 0);
+        }
+        for (int i = threadIdx.x; i < kChunk * pv; i += 128) {
+            const int r = i / pv, c = (i - r * pv) * 8;
+            *reinterpret_cast<uint4*>(xs + r * ldp_s + c) =
+                r < tn && c < pn ? *reinterpret_cast<const uint4*>(src + static_cast<long long>(r) * p.channels + h * p.P + p0 + c) : make_uint4(0, 0, 0, 0);
+        }
+        if (warp == 0) {                        // dt and the running log-decay: two tokens per lane
+            float d[2], a[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int r = lane * 2 + e;
+                d[e] = r < tn ? softplus_f(__bfloat162float(p.proj[(m0 + r) * p.ldp + 2 * inner + 2 * p.G * p.N + h]) + dtb) : 0.f;
+                a[e] = nA2 * d[e];
+            }
+            float s = a[0] + a[1];
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float v = __shfl_up_sync(0xFFFFFFFFu, s, o);
+                if (lane >= o) s += v;
+            }
+            const float excl = s - (a[0] + a[1]), l0 = excl + a[0], l1 = l0 + a[1], last = __shfl_sync(0xFFFFFFFFu, l1, 31);
+            la[lane * 2] = l0; la[lane * 2 + 1] = l1;
+            dtv[lane * 2] = d[0]; dtv[lane * 2 + 1] = d[1];
+            wv[lane * 2] = d[0] * exp2f(last - l0); wv[lane * 2 + 1] = d[1] * exp2f(last - l1);
+        }
+        if (OUT) {
+#pragma unroll
+            for (int i = 0; i < MT; ++i) {
+                const int n = (warp + 4 * i) * 16 + g;
+                if ((warp + 4 * i) * 16 >= p.N16) break;
+#pragma unroll
+                for (int x = 0; x < PT; ++x)
+#pragma unroll
+                    for (int hf = 0; hf < 2; ++hf) {
+                        uint32_t hi, lo;
+                        split_hi_lo(S[i][x][hf * 2], S[i][x][hf * 2 + 1], hi, lo);
+                        const int at = (n + hf * 8) * ldp_s + x * 8 + t4 * 2;
+                        *reinterpret_cast<uint32_t*>(Sh + at) = hi;
+                        *reinterpret_cast<uint32_t*>(Sl + at) = lo;
+                    }
+            }
+        }
+        __syncthreads();
+        const float last = la[kChunk - 1];
+        if (OUT) {
+            const int rt = warp;                // this warp's 16 tokens
+            const int ra = rt * 16 + g, rb = ra + 8;
+            float y[PT][4] = {};
+            for (int ks = 0; ks < p.N16 / 16; ++ks) {
+                uint32_t a[4];
+                ldmatrix4(a, Cs + (rt * 16 + (mi & 1) * 8 + mr) * ldn + ks * 16 + (mi >> 1) * 8);
+#pragma unroll
+                for (int x = 0; x < PT; x += 2) {
+                    uint32_t bh[4], bl[4];
+                    const int at = (ks * 16 + (mi & 1) * 8 + mr) * ldp_s + x * 8 + (mi >> 1) * 8;
+                    ldmatrix4_trans(bh, Sh + at);
+                    ldmatrix4_trans(bl, Sl + at);
+                    mma_bf16(y[x], a, bh[0], bh[1]);
+                    mma_bf16(y[x + 1], a, bh[2], bh[3]);
+                    mma_bf16(y[x], a, bl[0], bl[1]);
+                    mma_bf16(y[x + 1], a, bl[2], bl[3]);
+                }
+            }
+            const float laa = la[ra], lab = la[rb], ea = exp2f(laa), eb = exp2f(lab);
+#pragma unroll
+            for (int x = 0; x < PT; ++x) { y[x][0] *= ea; y[x][1] *= ea; y[x][2] *= eb; y[x][3] *= eb; }
+            for (int jb = 0; jb <= rt; ++jb) {
+                float gm[2][4] = {};
+                for (int ks = 0; ks < p.N16 / 16; ++ks) {
+                    uint32_t a[4], bq[4];
+                    ldmatrix4(a, Cs + (rt * 16 + (mi & 1) * 8 + mr) * ldn + ks * 16 + (mi >> 1) * 8);
+                    ldmatrix4(bq, Bs + (jb * 16 + (mi >> 1) * 8 + mr) * ldn + ks * 16 + (mi & 1) * 8);
+                    mma_bf16(gm[0], a, bq[0], bq[1]);
+                    mma_bf16(gm[1], a, bq[2], bq[3]);
+                }
+                uint32_t ah[4], al[4];
+#pragma unroll
+                for (int x = 0; x < 2; ++x) {
+                    const int j = jb * 16 + x * 8 + t4 * 2;
+                    const float l0 = la[j], l1 = la[j + 1], d0 = dtv[j], d1 = dtv[j + 1];
+                    const float w00 = j <= ra ? gm[x][0] * exp2f(laa - l0) * d0 : 0.f, w01 = j + 1 <= ra ? gm[x][1] * exp2f(laa - l1) * d1 : 0.f;
+                    const float w10 = j <= rb ? gm[x][2] * exp2f(lab - l0) * d0 : 0.f, w11 = j + 1 <= rb ? gm[x][3] * exp2f(lab - l1) * d1 : 0.f;
+                    split_hi_lo(w00, w01, ah[x * 2], al[x * 2]);
+                    split_hi_lo(w10, w11, ah[x * 2 + 1], al[x * 2 + 1]);
+                }
+#pragma unroll
+                for (int x = 0; x < PT; x += 2) {
+                    uint32_t bx[4];
+                    ldmatrix4_trans(bx, xs + (jb * 16 + (mi & 1) * 8 + mr) * ldp_s + x * 8 + (mi >> 1) * 8);
+                    mma_bf16(y[x], ah, bx[0], bx[1]);
+                    mma_bf16(y[x + 1], ah, bx[2], bx[3]);
+                    mma_bf16(y[x], al, bx[0], bx[1]);
+                    mma_bf16(y[x + 1], al, bx[2], bx[3]);
+                }
+            }
+#pragma unroll
+            for (int x = 0; x < PT; ++x)
+#pragma unroll
+                for (int hf = 0; hf < 2; ++hf) {
+                    const int r = hf ? rb : ra, c = x * 8 + t4 * 2;
+                    if (r >= tn || c >= pn) continue;
+                    const float2 xv = Elem<__nv_bfloat16>::unpack2(*reinterpret_cast<const uint32_t*>(xs + r * ldp_s + c));
+                    const float2 zv = Elem<__nv_bfloat16>::unpack2(*reinterpret_cast<const uint32_t*>(p.proj + (m0 + r) * p.ldp + h * p.P + p0 + c));
+                    *reinterpret_cast<uint32_t*>(p.gated + (m0 + r) * inner + h * p.P + p0 + c) =
+                        Elem<__nv_bfloat16>::pack2(fmaf(Dh, xv.x, y[x][hf * 2]) * silu_exact(zv.x), fmaf(Dh, xv.y, y[x][hf * 2 + 1]) * silu_exact(zv.y));
+                }
+        }
+        // ---- state update ----
+        const float decay = exp2f(last);
+        log_decay += last;
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+            const int n0 = (warp + 4 * i) * 16;
+            if (n0 >= p.N16) break;
+#pragma unroll
+            for (int x = 0; x < PT; ++x)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) S[i][x][e] *= decay;
+#pragma unroll
+            for (int ks = 0; ks < kChunk / 16; ++ks) {
+                uint32_t a[4], ah[4], al[4];
+                ldmatrix4_trans(a, Bs + (ks * 16 + (mi >> 1) * 8 + mr) * ldn + n0 + (mi & 1) * 8);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int j = ks * 16 + (e >> 1) * 8 + t4 * 2;
+                    const float2 v = Elem<__nv_bfloat16>::unpack2(a[e]);
+                    split_hi_lo(v.x * wv[j], v.y * wv[j + 1], ah[e], al[e]);
+                }
+#pragma unroll
+                for (int x = 0; x < PT; x += 2) {
+                    uint32_t bx[4];
+                    ldmatrix4_trans(bx, xs + (ks * 16 + (mi & 1) * 8 + mr) * ldp_s + x * 8 + (mi >> 1) * 8);
+                    mma_bf16(S[i][x], ah, bx[0], bx[1]);
+                    mma_bf16(S[i][x + 1], ah, bx[2], bx[3]);
+                    mma_bf16(S[i][x], al, bx[0], bx[1]);
+                    mma_bf16(S[i][x + 1], al, bx[2], bx[3]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    if (OUT && seg + 1 < p.n_seg) return;
+    float* dst = OUT ? sp : p.seg_state + seg_row * p.N * p.Pp + p0;
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int x = 0; x < PT; ++x)
+#pragma unroll
+            for (int hf = 0; hf < 2; ++hf) {
+                const int n = (warp + 4 * i) * 16 + g + hf * 8, c = x * 8 + t4 * 2;
+                if (n < p.N && c < pn) *reinterpret_cast<float2*>(dst + static_cast<long long>(n) * p.Pp + c) = make_float2(S[i][x][hf * 2], S[i][x][hf * 2 + 1]);
+            }
+    if (!OUT && sl == 0 && threadIdx.x == 0) p.seg_decay[seg_row] = log_decay;
+}
+
+// seg_state[seg] <- the state every segment starts from.  grid (blocks of a head's state, H, B).
+__global__ void __launch_bounds__(256)
+ssd_segment_scan_kernel(ChunkParams p) {
+    pdl_begin();
+    const int i = blockIdx.x * 256 + threadIdx.x, h = blockIdx.y, b = blockIdx.z, size = p.N * p.Pp;
+    if (i >= size) return;
+    float run = p.pos[b] > 0 ? p.state[(static_cast<long long>(p.slots ? p.slots[b] : b) * p.H + h) * size + i] : 0.f;
+    for (int s = 0; s < p.n_seg; ++s) {
+        const long long row = (static_cast<long long>(b) * p.n_seg + s) * p.H + h;
+        const float add = s + 1 < p.n_seg ? p.seg_state[row * size + i] : 0.f;
+        p.seg_state[row * size + i] = run;
+        if (s + 1 < p.n_seg) run = fmaf(exp2f(p.seg_decay[row]), run, add);
+    }
+}
+
+}  // namespace
+
+bool ssd_chunk_supported(const vb200_ssd_args& a) {
+    return a.dtype == VB200_BF16 && a.P % 8 == 0 && a.N % 8 == 0 && a.N <= 256 && a.ldp % 8 == 0 && a.H * ((a.P + 31) / 32) <= 65535;
+}
+
+// Column slices of a head and segments of a portion.
+void plan_ssd_chunks(const vb200_ssd_args& a, int* slices, int* n_seg, int* seg_chunks) {
+    const int pw = a.N <= 128 ? 64 : 32, chunks = (a.T + kChunk - 1) / kChunk;
+    *slices = (a.P + pw - 1) / pw;
+    const long long ctas = static_cast<long long>(a.B) * a.H * *slices;
+    long long want = (2LL * device_sm_count() + ctas - 1) / ctas;
+    if (want > chunks / 2) want = chunks / 2;
+    if (want < 1) want = 1;
+    *seg_chunks = static_cast<int>((chunks + want - 1) / want);
+    *n_seg = (chunks + *seg_chunks - 1) / *seg_chunks;
+}
+
+int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, const void* xbc, void* gated, float* states) {
+    ChunkParams p{};
+    p.T = a.T; p.H = a.H; p.P = a.P; p.N = a.N; p.G = a.G; p.channels = pl.channels; p.Pp = pl.Pp; p.N16 = pad_to(a.N, 16);
+    plan_ssd_chunks(a, &p.slices, &p.n_seg, &p.seg_chunks);
+    p.ldp = a.ldp;
+    p.proj = static_cast<const __nv_bfloat16*>(a.proj); p.xbc = static_cast<const __nv_bfloat16*>(xbc);
+    p.dt_bias = a.dt_bias; p.A_log = a.A_log; p.D = a.D; p.slots = a.slots; p.pos = a.pos; p.state = a.state;
+    p.seg_decay = states;
+    p.seg_state = states + (static_cast<long long>(a.B) * p.n_seg * a.H + 63) / 64 * 64;
+    p.gated = static_cast<__nv_bfloat16*>(gated);
+    auto go = [&](auto first, auto walk, int pt) -> int {
+        const size_t tiles = 2 * (static_cast<size_t>(kChunk) * (p.N16 + kPad) + kChunk * (pt * 8 + kPad));
+        const size_t all = tiles + 2 * (static_cast<size_t>(kChunk) * (p.N16 + kPad) + 2 * static_cast<size_t>(p.N16) * (pt * 8 + kPad));
+        const unsigned hs = static_cast<unsigned>(a.H * p.slices), bs = static_cast<unsigned>(a.B);
+        if (int rc = allow_smem(first, tiles)) return rc;
+        if (int rc = allow_smem(walk, all)) return rc;
+        if (p.n_seg > 1) {
+            if (int rc = launch_pdl(first, dim3(static_cast<unsigned>(p.n_seg - 1), hs, bs), dim3(128), tiles, s, p)) return rc;
+            if (int rc = launch_pdl(ssd_segment_scan_kernel, dim3(static_cast<unsigned>((a.N * p.Pp + 255) / 256), static_cast<unsigned>(a.H), bs), dim3(256), 0, s, p)) return rc;
+        }
+        profile_mark_begin(s);
+        const int rc = launch_pdl(walk, dim3(static_cast<unsigned>(p.n_seg), hs, bs), dim3(128), all, s, p);
+        profile_mark_end(s);
+        return rc;
+    };
+    note_ssd_kernel("ssd_chunk_kernel");
+    return a.N <= 128 ? go(ssd_chunk_kernel<2, 8, false>, ssd_chunk_kernel<2, 8, true>, 8) : go(ssd_chunk_kernel<4, 4, false>, ssd_chunk_kernel<4, 4, true>, 4);
+}
+
+}  // namespace vb200

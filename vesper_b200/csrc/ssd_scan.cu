@@ -214,14 +214,16 @@ SsdPlan plan_ssd(const vb200_ssd_args& a) {
     SsdPlan pl{};
     pl.channels = a.H * a.P + 2 * a.G * a.N;
     pl.Pp = pad_to(a.P, 4);
-    pl.chunked = a.form != 1 && ssd_chunk_supported(a) && (a.form == 2 || a.T >= 16);
-    pl.chunk = 64;
-    pl.n_chunks = (a.T + pl.chunk - 1) / pl.chunk;
+    pl.chunked = a.T > 1 && a.form != 1 && ssd_chunk_supported(a) && (a.form == 2 || a.T >= 16);
     const size_t esz = a.dtype == VB200_F32 ? 4 : 2, M = static_cast<size_t>(a.B) * a.T;
     auto up = [](size_t x) { return (x + 255) / 256 * 256; };
     pl.conv_bytes = a.T > 1 ? up(M * pl.channels * esz) : 0;
     pl.gated_bytes = up(M * a.H * a.P * (pl.chunked ? 2 : 4));
-    pl.chunk_bytes = pl.chunked ? up(sizeof(float) * (static_cast<size_t>(a.B) * pl.n_chunks * a.H * (static_cast<size_t>(a.N) * pl.Pp + 1))) : 0;
+    if (pl.chunked) {
+        int slices, n_seg, seg_chunks;
+        plan_ssd_chunks(a, &slices, &n_seg, &seg_chunks);
+        if (n_seg > 1) pl.chunk_bytes = up(sizeof(float) * (static_cast<size_t>(a.B) * n_seg * a.H * (static_cast<size_t>(a.N) * pl.Pp + 1) + 64));
+    }
     pl.total = pl.conv_bytes + pl.gated_bytes + pl.chunk_bytes;
     return pl;
 }
