@@ -774,6 +774,10 @@ def run_ours(args):
     dec = bench_decode(cx, args.decode_steps, W) if only in ("all", "decode") else None
     shd = bench_sharded(cx) if only in ("all", "sharded") else None
     mdl = bench_model(cx, layers=args.model_layers, new=args.model_new) if only in ("all", "model") else None
+    hyb = None
+    if only == "hybrid":
+        from vesper_b200.hybrid_bench import bench_hybrid
+        hyb = bench_hybrid(cx, K, W, layers=args.model_layers, part=args.hybrid_part)
     cpu_baseline = None
     if cx.rank == 0 and cx.world == 1 and not args.no_cpu_baseline and only == "all":
         cpu_baseline, _ = cpu_prefill_sample(target_seconds=12.0)
@@ -795,6 +799,8 @@ def run_ours(args):
             "decode_sharded": shd,
             "model": mdl,
         }
+        if hyb is not None:
+            line["hybrid"] = hyb
         if cpu_baseline is not None:
             line["cpu_baseline"] = cpu_baseline
         emit(line)
@@ -826,7 +832,9 @@ def main():
     ap.add_argument("--decode-steps", type=int, default=C3["steps"], help="consecutive decode steps (default: the workload's 256)")
     ap.add_argument("--model-layers", type=int, default=0, help="profiling runs: depth of the model section's decoder (default: the workload's 24)")
     ap.add_argument("--model-new", type=int, default=0, help="profiling runs: tokens to generate in the model section (default: 128)")
-    ap.add_argument("--only", default="all", choices=["all", "prefill", "decode", "sharded", "model"], help="run one section (profiling runs)")
+    ap.add_argument("--only", default="all", choices=["all", "prefill", "decode", "sharded", "model", "hybrid"],
+                    help="run one section (profiling runs); hybrid: the hybrid decoder's mixers and model beside the Llama-style decoder (not part of the default run)")
+    ap.add_argument("--hybrid-part", default="all", choices=["all", "kernels", "models"])
     args = ap.parse_args()
     if args.impl == "reference":
         run_reference(args)

@@ -86,7 +86,7 @@ typedef struct vb200_latent_args {
     const double* inv_freq;      /* device [rot_dim / 2] */
     void* proj;  int64_t ldp;    /* [B*T, ldp]: q [H * (dim + rot_dim)] | c before its norm [rank] | key part before rotation [rot_dim];
                                     a prompt pass rotates q in place */
-    const void* c_norm;          /* [rank] fp32 */
+    const float* c_norm;         /* [rank] */
     const void* w_uk;            /* [H * dim, ldu] */
     const void* w_uv;            /* [H * vdim, ldu] */
     int64_t ldu;                 /* >= rank, multiple of 8, columns past rank zero */

@@ -26,6 +26,11 @@ def test_header_symbols_are_exported(lib):
     for n in block:
         assert hasattr(lib, n), f"{n} declared in include/vesper_b200_block.h but not exported"
     assert sorted(capi.BLOCK_EXPORTS) == block
+    from vesper_b200 import hybrid_capi
+    hybrid = [n for n in declared_symbols("vesper_b200_hybrid.h") if n not in ("vb200_latent_row", "vb200_latent_rot_offset", "vb200_latent_context")]   # inline
+    for n in hybrid:
+        assert hasattr(lib, n), f"{n} declared in include/vesper_b200_hybrid.h but not exported"
+    assert sorted(hybrid_capi.HYBRID_EXPORTS) == hybrid
 
 
 def test_struct_layout_and_host_helpers(lib):

@@ -396,7 +396,7 @@ def linear(x, w, out, epilogue=EPI_BF16, splits=0, stream=None, bias=None):
 
 
 def linear_ex(x, w, out, *, epilogue=EPI_BF16, splits=0, bias=None, scaled_copy=None, copy_scale=None, rms_rows=None, rms_eps=0.0,
-              row_scale=None, stream=None):
+              row_scale=None, addend=None, stream=None):
     """vb200_linear_ex: the GEMM with bias and the two halves of a deferred RMSNorm."""
     a = LinearArgs()
     a.struct_size = C.sizeof(LinearArgs)
@@ -407,6 +407,7 @@ def linear_ex(x, w, out, *, epilogue=EPI_BF16, splits=0, bias=None, scaled_copy=
     a.N = w.shape[0]
     a.epilogue, a.splits = epilogue, splits
     a.bias, a.scaled_copy, a.copy_scale, a.row_scale = _ptr(bias), _ptr(scaled_copy), _ptr(copy_scale), _ptr(row_scale)
+    a.addend = _ptr(addend)
     if rms_rows is not None:
         a.rms_rows, a.rms_ld, a.rms_dim, a.rms_eps = _ptr(rms_rows), rms_rows.stride(0), rms_rows.shape[1], rms_eps
     check(load().vb200_linear_ex(C.byref(a)))

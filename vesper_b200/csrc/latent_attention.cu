@@ -91,14 +91,33 @@ latent_append_kernel(LatentParams p, T* __restrict__ proj, T* __restrict__ cache
         }
     }
     const int hq = p.dim + p.rot;
-    latent_row<T, 4>(p, row + static_cast<long long>(p.H) * hq, cs, ring_row, old_copy, crow + static_cast<long long>(n_old + t) * p.ldc, part);
-    for (int i = threadIdx.x; i < p.H * half; i += blockDim.x) {
-        const int h = i / half, j = i - h * half;
-        T* q = row + static_cast<long long>(h) * hq + p.dim;
-        const float u = Elem<T>::to_f(q[j]), v = Elem<T>::to_f(q[j + half]);
-        q[j] = Elem<T>::from_f(u * cs[j].x - v * cs[j].y);
-        q[j + half] = Elem<T>::from_f(v * cs[j].x + u * cs[j].y);
+    if (half % 8 == 0 && p.dim % 8 == 0 && p.ldp % 8 == 0) {        // eight pairs per thread
+        const int groups = half / 8;
+        for (int i = threadIdx.x; i < p.H * groups; i += blockDim.x) {
+            const int h = i / groups, j = (i - h * groups) * 8;
+            T* q = row + static_cast<long long>(h) * hq + p.dim + j;
+            float u[8], v[8], a[8], c[8];
+            load8(q, u);
+            load8(q + half, v);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                const float2 w = cs[j + e];
+                a[e] = u[e] * w.x - v[e] * w.y;
+                c[e] = v[e] * w.x + u[e] * w.y;
+            }
+            store8(q, a);
+            store8(q + half, c);
+        }
+    } else {
+        for (int i = threadIdx.x; i < p.H * half; i += blockDim.x) {
+            const int h = i / half, j = i - h * half;
+            T* q = row + static_cast<long long>(h) * hq + p.dim;
+            const float u = Elem<T>::to_f(q[j]), v = Elem<T>::to_f(q[j + half]);
+            q[j] = Elem<T>::from_f(u * cs[j].x - v * cs[j].y);
+            q[j + half] = Elem<T>::from_f(v * cs[j].x + u * cs[j].y);
+        }
     }
+    latent_row<T, 4>(p, row + static_cast<long long>(p.H) * hq, cs, ring_row, old_copy, crow + static_cast<long long>(n_old + t) * p.ldc, part);
 }
 
 constexpr int kBT = 4;           // batch rows per CTA of the two per-head products (their weights are read once per CTA)
@@ -228,7 +247,7 @@ latent_split_generic_kernel(LatentParams p, const float* __restrict__ qa, const 
     }
     __syncthreads();
     float* out = part + ((static_cast<long long>(b) * p.H + h) * p.splits + split) * p.part_ld;
-    for (int i = threadIdx.x; i < p.rank; i += 128) out[i] = acc[i];
+    for (int i = threadIdx.x; i < p.rank16; i += 128) out[i] = i < p.rank ? acc[i] : 0.f;
     if (threadIdx.x == 0) { out[p.rank16] = m; out[p.rank16 + 1] = l; }
 }
 
@@ -262,14 +281,19 @@ latent_value_kernel(LatentParams p, const float* __restrict__ part, const T* __r
         for (int s = lane; s < p.splits; s += 32) coef[warp * p.splits + s] *= inv;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < kBT * p.rank16; i += 256) {
-        const int b = i / p.rank16, c = i - b * p.rank16;
-        float v = 0.f;
-        if (b < nb && c < p.rank) {
+    for (int i = threadIdx.x; i < kBT * p.rank16 / 4; i += 256) {        // four columns of one sequence, all slices' loads in flight
+        const int b = i / (p.rank16 / 4), c = (i - b * (p.rank16 / 4)) * 4;
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (b < nb) {
             const float* rec = part + (static_cast<long long>(b0 + b) * p.H + h) * p.splits * p.part_ld + c;
-            for (int s = 0; s < p.splits; ++s) v = fmaf(coef[b * p.splits + s], rec[static_cast<long long>(s) * p.part_ld], v);
+#pragma unroll 8
+            for (int s = 0; s < p.splits; ++s) {
+                const float4 r = *reinterpret_cast<const float4*>(rec + static_cast<long long>(s) * p.part_ld);
+                const float w = coef[b * p.splits + s];
+                v.x = fmaf(w, r.x, v.x); v.y = fmaf(w, r.y, v.y); v.z = fmaf(w, r.z, v.z); v.w = fmaf(w, r.w, v.w);
+            }
         }
-        o[i] = v;
+        *reinterpret_cast<float4*>(o + b * p.rank16 + c) = v;
     }
     __syncthreads();
     const int rank8 = (p.rank + 7) / 8 * 8;
@@ -346,7 +370,7 @@ LatentParams params_of(const vb200_latent_args& a) {
     p.B = a.B; p.T = a.T; p.H = a.H; p.dim = a.dim; p.rot = a.rot_dim; p.vdim = a.vdim; p.rank = a.rank;
     p.window = a.window; p.ring = a.ring; p.scale = a.scale; p.eps = a.eps; p.inv_freq = a.inv_freq;
     p.ldp = a.ldp; p.ldu = a.ldu; p.ldc = a.ldc; p.ldo = a.ldo; p.ldkv = a.ldkv;
-    p.c_norm = static_cast<const float*>(a.c_norm); p.sink = a.sink; p.slots = a.slots; p.pos = a.pos;
+    p.c_norm = a.c_norm; p.sink = a.sink; p.slots = a.slots; p.pos = a.pos;
     p.start_pos = a.start_pos;
     p.n_ctx = vb200_latent_context(a.start_pos, a.T, a.window);
     p.rot_off = vb200_latent_rot_offset(a.rank);
@@ -368,7 +392,7 @@ LatentPlan plan_latent(const vb200_latent_args& a) {
     // two CTAs per SM, at least 64 keys each
     const bool mma = latent_mma_supported(a);
     const long long units = static_cast<long long>(a.B) * (mma ? (a.H + 15) / 16 : a.H);
-    long long want = (2LL * device_sm_count() + units - 1) / units;
+    long long want = 2LL * device_sm_count() / units;           // rounded down: a few CTAs more would be a second wave
     const long long most = (pl.n_max + 63) / 64;
     if (want > most) want = most;
     if (want > 128) want = 128;

@@ -8,7 +8,8 @@
 //                                                B = rows by ldmatrix) and add their partial S through shared memory
 //   O[head, c]  += P[head, key] row[key, c]      each warp owns 16-column blocks of the latent (B by ldmatrix.trans)
 // A 32-key tile arrives as TMA boxes of [32 keys x 64 columns] with the 128-byte swizzle (4-D maps over the ring, zero
-// fill past the latent's and the rotated part's width), in a ring of stages filled by one producer warp.
+// fill past the latent's and the rotated part's width), in a ring of stages that thread 0 refills: the barrier after
+// the scores of a tile tells it that every warp is done with the tile before.
 #include "hybrid.cuh"
 
 namespace vb200 {
@@ -34,7 +35,7 @@ struct LatentSplitParams {
 };
 
 __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], uint32_t addr) {
@@ -56,13 +57,13 @@ struct __align__(16) LatentSplitSmem {
     float red[kWarps][16][kRedLd];
     __nv_bfloat16 p_hi[16][kPLd], p_lo[16][kPLd];
     float alpha[16];
-    uint64_t full[kStagesMax], empty[kStagesMax];
+    uint64_t full[kStagesMax];
     int abort_flag;
 };
 
 // KS: 16-column steps per warp; NP: 16-column output blocks per warp.
 template <int KS, int NP>
-__global__ void __launch_bounds__((kWarps + 1) * 32, 2)
+__global__ void __launch_bounds__(kWarps * 32, 2)
 latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSplitParams p) {
     extern __shared__ uint8_t raw[];
     uint8_t* tiles = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~static_cast<uintptr_t>(1023));
@@ -71,7 +72,7 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int split = blockIdx.x, h0 = blockIdx.y * 16, b = blockIdx.z;
     if (tid == 0) {
-        for (int i = 0; i < p.stages; ++i) { mbar_init(&sm.full[i], 1); mbar_init(&sm.empty[i], kWarps); }
+        for (int i = 0; i < p.stages; ++i) mbar_init(&sm.full[i], 1);
         sm.abort_flag = 0;
         mbar_fence_init();
     }
@@ -81,22 +82,20 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
     const int n = min(p.pos[b] + 1, p.ring), chunk = (n + p.splits - 1) / p.splits;
     const int k0 = split * chunk, k1 = min(n, k0 + chunk);
     const int n_tiles = k1 > k0 ? (k1 - k0 + kTile - 1) / kTile : 0;
-
-    if (warp == kWarps) {
-        if (lane == 0) {
-            const int slot = p.slots ? p.slots[b] : b;
-            for (int i = 0; i < n_tiles; ++i) {
-                const int s = i % p.stages;
-                if (i >= p.stages && !mbar_wait(&sm.empty[s], (i / p.stages - 1) & 1, ctx, 0xC1)) break;
-                uint8_t* st = tiles + s * stage_bytes;
-                mbar_arrive_expect_tx(&sm.full[s], stage_bytes);
-                for (int x = 0; x < p.nbox; ++x) {
-                    const bool rot = x >= p.nbc;
-                    tma_load_4d(st + x * kBox, rot ? &maps.r : &maps.c, &sm.full[s], (rot ? x - p.nbc : x) * 64, 0, k0 + i * kTile, slot);
-                }
-            }
+    const int slot = p.slots ? p.slots[b] : b;
+    auto load_tile = [&](int i) {
+        const int s = i % p.stages;
+        uint8_t* st = tiles + s * stage_bytes;
+        mbar_arrive_expect_tx(&sm.full[s], stage_bytes);
+        for (int x = 0; x < p.nbox; ++x) {
+            const bool rot = x >= p.nbc;
+            tma_load_4d(st + x * kBox, rot ? &maps.r : &maps.c, &sm.full[s], (rot ? x - p.nbc : x) * 64, 0, k0 + i * kTile, slot);
         }
-    } else {
+    };
+    if (tid == 0)
+        for (int i = 0; i < min(p.stages, n_tiles); ++i) load_tile(i);
+
+    {
         const int g = lane >> 2, t = lane & 3;
         // A fragments of this warp's steps: rows = heads h0 + g, h0 + g + 8
         uint32_t qh[KS][4], ql[KS][4];
@@ -126,23 +125,23 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
             const bool ok = mbar_wait_warp(&sm.full[s], (it / p.stages) & 1, ctx, 0xC2);
             uint8_t* tile = tiles + s * stage_bytes;
             const uint32_t tile_a = smem_u32(tile);
-            float c[4][4] = {};
+            float c[4][4] = {}, cl[4][4] = {};
             if (ok) {
 #pragma unroll
                 for (int i = 0; i < KS; ++i) {
                     const int kk = warp + i * kWarps;
                     if (kk >= p.ks) break;
                     const int kc = kk < p.ksc ? kk : kk - p.ksc, box = (kk < p.ksc ? 0 : p.nbc) + (kc >> 2), ch = (kc & 3) * 2 + (mi & 1);
+                    uint32_t bq[2][4];
 #pragma unroll
                     for (int half = 0; half < 2; ++half) {
                         const int key = half * 16 + (mi >> 1) * 8 + mr;
-                        uint32_t bq[4];
-                        ldmatrix4(bq, tile_a + box * kBox + key * 128 + ((ch ^ (key & 7)) << 4));
-                        mma_bf16(c[half * 2], qh[i], bq[0], bq[1]);
-                        mma_bf16(c[half * 2 + 1], qh[i], bq[2], bq[3]);
-                        mma_bf16(c[half * 2], ql[i], bq[0], bq[1]);
-                        mma_bf16(c[half * 2 + 1], ql[i], bq[2], bq[3]);
+                        ldmatrix4(bq[half], tile_a + box * kBox + key * 128 + ((ch ^ (key & 7)) << 4));
                     }
+#pragma unroll
+                    for (int x = 0; x < 4; ++x) mma_bf16(c[x], qh[i], bq[x >> 1][(x & 1) * 2], bq[x >> 1][(x & 1) * 2 + 1]);
+#pragma unroll
+                    for (int x = 0; x < 4; ++x) mma_bf16(cl[x], ql[i], bq[x >> 1][(x & 1) * 2], bq[x >> 1][(x & 1) * 2 + 1]);
                 }
                 if (valid < kTile) {
                     // rows past the slice hold other tokens (or another sequence's): their weight is zero, and so must their
@@ -160,10 +159,11 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
             }
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
-                *reinterpret_cast<float2*>(&sm.red[warp][g][x * 8 + t * 2]) = make_float2(c[x][0], c[x][1]);
-                *reinterpret_cast<float2*>(&sm.red[warp][g + 8][x * 8 + t * 2]) = make_float2(c[x][2], c[x][3]);
+                *reinterpret_cast<float2*>(&sm.red[warp][g][x * 8 + t * 2]) = make_float2(c[x][0] + cl[x][0], c[x][1] + cl[x][1]);
+                *reinterpret_cast<float2*>(&sm.red[warp][g + 8][x * 8 + t * 2]) = make_float2(c[x][2] + cl[x][2], c[x][3] + cl[x][3]);
             }
             if (consumers_sync_any(!ok)) break;                  // a wait ran out: all consumers leave together
+            if (tid == 0 && it > 0 && it - 1 + p.stages < n_tiles) load_tile(it - 1 + p.stages);
             float2 sv = make_float2(0.f, 0.f);
 #pragma unroll
             for (int w = 0; w < kWarps; ++w) {
@@ -196,25 +196,23 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
                 ldmatrix4(pl[ks], smem_u32(&sm.p_lo[(mi & 1) * 8 + mr][ks * 16 + (mi >> 1) * 8]));
             }
 #pragma unroll
-            for (int i = 0; i < NP; ++i) {
-                const int blk = warp + i * kWarps;
-                if (blk >= p.ksc) break;
+            for (int i = 0; i < NP; ++i)
 #pragma unroll
                 for (int x = 0; x < 2; ++x) { o[i][x][0] *= a0; o[i][x][1] *= a0; o[i][x][2] *= a1; o[i][x][3] *= a1; }
 #pragma unroll
-                for (int ks = 0; ks < 2; ++ks) {
-                    const int key = ks * 16 + (mi & 1) * 8 + mr, ch = (blk & 3) * 2 + (mi >> 1);
-                    uint32_t bv[4];
-                    ldmatrix4_trans(bv, tile_a + (blk >> 2) * kBox + key * 128 + ((ch ^ (key & 7)) << 4));
-                    mma_bf16(o[i][0], ph[ks], bv[0], bv[1]);
-                    mma_bf16(o[i][1], ph[ks], bv[2], bv[3]);
-                    mma_bf16(o[i][0], pl[ks], bv[0], bv[1]);
-                    mma_bf16(o[i][1], pl[ks], bv[2], bv[3]);
+            for (int ks = 0; ks < 2; ++ks) {
+                const int key = ks * 16 + (mi & 1) * 8 + mr;
+                uint32_t bv[NP][4];
+#pragma unroll
+                for (int i = 0; i < NP; ++i) {
+                    const int blk = min(warp + i * kWarps, p.ksc - 1), ch = (blk & 3) * 2 + (mi >> 1);      // a block too many is computed and dropped
+                    ldmatrix4_trans(bv[i], tile_a + (blk >> 2) * kBox + key * 128 + ((ch ^ (key & 7)) << 4));
                 }
+#pragma unroll
+                for (int i = 0; i < NP; ++i) { mma_bf16(o[i][0], ph[ks], bv[i][0], bv[i][1]); mma_bf16(o[i][1], ph[ks], bv[i][2], bv[i][3]); }
+#pragma unroll
+                for (int i = 0; i < NP; ++i) { mma_bf16(o[i][0], pl[ks], bv[i][0], bv[i][1]); mma_bf16(o[i][1], pl[ks], bv[i][2], bv[i][3]); }
             }
-            if (valid < kTile) fence_proxy_async_smem();         // the clearing stores come before any later bulk copy
-            __syncwarp();
-            if (lane == 0) mbar_arrive(&sm.empty[s]);
         }
         float* out = p.part + ((static_cast<long long>(b) * p.H) * p.splits + split) * p.part_ld;
         const long long head_ld = static_cast<long long>(p.splits) * p.part_ld;
@@ -260,7 +258,7 @@ int launch_latent_split_mma(cudaStream_t s, const vb200_latent_args& a, const La
     const size_t smem = 1024 + static_cast<size_t>(p.stages) * stage + sizeof(LatentSplitSmem);
     auto go = [&](auto kernel) -> int {
         if (int rc = allow_smem(kernel, smem)) return rc;
-        return launch_pdl(kernel, dim3(static_cast<unsigned>(pl.splits), static_cast<unsigned>((a.H + 15) / 16), static_cast<unsigned>(a.B)), dim3((kWarps + 1) * 32), smem, s, maps, p);
+        return launch_pdl(kernel, dim3(static_cast<unsigned>(pl.splits), static_cast<unsigned>((a.H + 15) / 16), static_cast<unsigned>(a.B)), dim3(kWarps * 32), smem, s, maps, p);
     };
     note_latent_kernel("latent_split_mma_kernel");
     if (p.ks <= 16 && p.ksc <= 8) return go(latent_split_mma_kernel<2, 1>);

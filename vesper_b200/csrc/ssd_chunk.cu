@@ -4,7 +4,7 @@
 //   y_i  = 2^la_i C_i S  +  sum_{j <= i} (C_i . B_j) 2^(la_i - la_j) dt_j x_j  +  D x_i
 //   S   <- 2^la_last S   +  sum_j 2^(la_last - la_j) dt_j B_j x_j^T
 //
-// One CTA of four warps walks the chunks of one (batch, head, column slice) with S in its MMA accumulators: warp-level
+// One CTA of eight warps walks the chunks of one (batch, head, column slice) with S in its MMA accumulators: warp-level
 // m16n8k16 products, fp32 accumulation.  C, B and x are bf16 values as they come from the convolution; everything the
 // decays touch (the weights of the second sum, the weighted B of the state update, S itself as a right operand) enters
 // as hi + lo bf16 halves, so the recurrence keeps fp32-class accuracy.
@@ -16,6 +16,7 @@ namespace vb200 {
 namespace {
 
 constexpr int kChunk = 64;
+constexpr int kThreads = 256;
 constexpr int kPad = 8;                  // bf16 of row padding: ldmatrix rows fall into distinct banks
 
 struct ChunkParams {
@@ -31,7 +32,7 @@ struct ChunkParams {
 };
 
 __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 __device__ __forceinline__ void ldmatrix4(uint32_t (&r)[4], const __nv_bfloat16* ptr) {
@@ -41,15 +42,19 @@ __device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], const __nv_bfl
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(ptr)) : "memory");
 }
 
-// MT: 16-row tiles of S per warp (rows dealt to the four warps in turn); PT: 8-column tiles of the slice.
+// Brings a line closer while the current chunk computes.
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
+// MT: 16-row tiles of S per warp (rows dealt to the eight warps in turn); PT: 8-column tiles of the slice.  In the
+// output products warp w has token rows 16 (w & 3) .. and column half w >> 2.
 // OUT: the walk (outputs and, in the last segment, the final state); else the first pass (what a segment adds to S).
 template <int MT, int PT, bool OUT>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(kThreads, 2)
 ssd_chunk_kernel(ChunkParams p) {
     pdl_begin();
     extern __shared__ __align__(16) uint8_t smem[];
     const int ldn = p.N16 + kPad;
-    constexpr int kPw = PT * 8, ldp_s = kPw + kPad;
+    constexpr int kPw = PT * 8, ldp_s = kPw + kPad, HT = PT / 2;
     __nv_bfloat16* Bs = reinterpret_cast<__nv_bfloat16*>(smem);        // [64][ldn]
     __nv_bfloat16* xs = Bs + kChunk * ldn;                             // [64][ldp_s]
     __nv_bfloat16* Cs = xs + kChunk * ldp_s;                           // [64][ldn]
@@ -76,7 +81,7 @@ ssd_chunk_kernel(ChunkParams p) {
             for (int x = 0; x < PT; ++x)
 #pragma unroll
                 for (int hf = 0; hf < 2; ++hf) {
-                    const int n = (warp + 4 * i) * 16 + g + hf * 8, c = x * 8 + t4 * 2;
+                    const int n = (warp + 8 * i) * 16 + g + hf * 8, c = x * 8 + t4 * 2;
                     float2 v = make_float2(0.f, 0.f);
                     if (src != nullptr && n < p.N && c < pn) v = *reinterpret_cast<const float2*>(src + static_cast<long long>(n) * p.Pp + c);
                     S[i][x][hf * 2] = v.x; S[i][x][hf * 2 + 1] = v.y;
@@ -89,20 +94,26 @@ ssd_chunk_kernel(ChunkParams p) {
         const long long m0 = static_cast<long long>(b) * p.T + t0;
         const __nv_bfloat16* src = p.xbc + m0 * p.channels;
         // ---- tiles: 16-byte pieces, zero past the portion and past a matrix's width ----
-        const int nv = p.N16 / 8, pv = kPw / 8;
-        for (int i = threadIdx.x; i < kChunk * nv; i += 128) {
+        const int nv = p.N16 / 8;
+        constexpr int pv = kPw / 8;
+        for (int i = threadIdx.x; i < kChunk * nv; i += kThreads) {
             const int r = i / nv, c = (i - r * nv) * 8;
             const bool ok = r < tn && c < p.N;
             const __nv_bfloat16* q = src + static_cast<long long>(r) * p.channels + inner + grp * p.N + c;
-            *reinterpret_cast<uint4*>(Bs + r * ldn + c) = ok ? *reinterpret_cast<const uint4*>(q) : make_uint4(0, 0, 0, 0);
-            if (OUT) *reinterpret_cast<uint4*>(Cs + r * ldn + c) = ok ? *reinterpret_cast<const uint4*>(q + p.G * p.N) : make_uint4(0, 0, 0, 0);
+            uint4 vb = make_uint4(0, 0, 0, 0), vc = vb;
+            if (ok) {
+                vb = *reinterpret_cast<const uint4*>(q);
+                if (OUT) vc = *reinterpret_cast<const uint4*>(q + p.G * p.N);
+            }
+            *reinterpret_cast<uint4*>(Bs + r * ldn + c) = vb;
+            if (OUT) *reinterpret_cast<uint4*>(Cs + r * ldn + c) = vc;
         }
-        for (int i = threadIdx.x; i < kChunk * pv; i += 128) {
+        for (int i = threadIdx.x; i < kChunk * pv; i += kThreads) {
             const int r = i / pv, c = (i - r * pv) * 8;
             *reinterpret_cast<uint4*>(xs + r * ldp_s + c) =
                 r < tn && c < pn ? *reinterpret_cast<const uint4*>(src + static_cast<long long>(r) * p.channels + h * p.P + p0 + c) : make_uint4(0, 0, 0, 0);
         }
-        if (warp == 0) {                        // dt and the running log-decay: two tokens per lane
+        if (warp == 7) {                        // dt and the running log-decay: two tokens per lane
             float d[2], a[2];
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
@@ -124,8 +135,8 @@ ssd_chunk_kernel(ChunkParams p) {
         if (OUT) {
 #pragma unroll
             for (int i = 0; i < MT; ++i) {
-                const int n = (warp + 4 * i) * 16 + g;
-                if ((warp + 4 * i) * 16 >= p.N16) break;
+                const int n = (warp + 8 * i) * 16 + g;
+                if ((warp + 8 * i) * 16 >= p.N16) break;
 #pragma unroll
                 for (int x = 0; x < PT; ++x)
 #pragma unroll
@@ -139,63 +150,80 @@ ssd_chunk_kernel(ChunkParams p) {
             }
         }
         __syncthreads();
+        if (ch + 1 < c_end) {                   // the next chunk's own lines (B and C are shared by the heads of a group)
+            const int r = threadIdx.x & 63, what = threadIdx.x >> 6;
+            if (t0 + kChunk + r < p.T) {
+                if (what == 0) prefetch_l2(src + static_cast<long long>(kChunk + r) * p.channels + h * p.P + p0);
+                else if (what == 1 && OUT) prefetch_l2(p.proj + (m0 + kChunk + r) * p.ldp + h * p.P + p0);
+                else if (what == 2) prefetch_l2(p.proj + (m0 + kChunk + r) * p.ldp + 2 * inner + 2 * p.G * p.N + h);
+            }
+        }
         const float last = la[kChunk - 1];
         if (OUT) {
-            const int rt = warp;                // this warp's 16 tokens
+            const int rt = warp & 3, x0 = (warp >> 2) * HT;        // this warp's 16 tokens and column tiles
             const int ra = rt * 16 + g, rb = ra + 8;
-            float y[PT][4] = {};
+            float y[HT][4] = {}, yl[HT][4] = {};
+            const __nv_bfloat16* crow = Cs + (rt * 16 + (mi & 1) * 8 + mr) * ldn + (mi >> 1) * 8;
+#pragma unroll 2
             for (int ks = 0; ks < p.N16 / 16; ++ks) {
-                uint32_t a[4];
-                ldmatrix4(a, Cs + (rt * 16 + (mi & 1) * 8 + mr) * ldn + ks * 16 + (mi >> 1) * 8);
+                uint32_t a[4], bh[HT / 2][4], bl[HT / 2][4];
+                ldmatrix4(a, crow + ks * 16);
 #pragma unroll
-                for (int x = 0; x < PT; x += 2) {
-                    uint32_t bh[4], bl[4];
-                    const int at = (ks * 16 + (mi & 1) * 8 + mr) * ldp_s + x * 8 + (mi >> 1) * 8;
-                    ldmatrix4_trans(bh, Sh + at);
-                    ldmatrix4_trans(bl, Sl + at);
-                    mma_bf16(y[x], a, bh[0], bh[1]);
-                    mma_bf16(y[x + 1], a, bh[2], bh[3]);
-                    mma_bf16(y[x], a, bl[0], bl[1]);
-                    mma_bf16(y[x + 1], a, bl[2], bl[3]);
+                for (int x = 0; x < HT / 2; ++x) {
+                    const int at = (ks * 16 + (mi & 1) * 8 + mr) * ldp_s + (x0 + 2 * x) * 8 + (mi >> 1) * 8;
+                    ldmatrix4_trans(bh[x], Sh + at);
+                    ldmatrix4_trans(bl[x], Sl + at);
                 }
+#pragma unroll
+                for (int x = 0; x < HT; ++x) mma_bf16(y[x], a, bh[x / 2][(x & 1) * 2], bh[x / 2][(x & 1) * 2 + 1]);
+#pragma unroll
+                for (int x = 0; x < HT; ++x) mma_bf16(yl[x], a, bl[x / 2][(x & 1) * 2], bl[x / 2][(x & 1) * 2 + 1]);
             }
             const float laa = la[ra], lab = la[rb], ea = exp2f(laa), eb = exp2f(lab);
 #pragma unroll
-            for (int x = 0; x < PT; ++x) { y[x][0] *= ea; y[x][1] *= ea; y[x][2] *= eb; y[x][3] *= eb; }
+            for (int x = 0; x < HT; ++x) {
+                y[x][0] = (y[x][0] + yl[x][0]) * ea; y[x][1] = (y[x][1] + yl[x][1]) * ea;
+                y[x][2] = (y[x][2] + yl[x][2]) * eb; y[x][3] = (y[x][3] + yl[x][3]) * eb;
+            }
             for (int jb = 0; jb <= rt; ++jb) {
-                float gm[2][4] = {};
-                for (int ks = 0; ks < p.N16 / 16; ++ks) {
+                float gm[2][2][4] = {};                            // even and odd steps of the inner dimension
+                const __nv_bfloat16* brow = Bs + (jb * 16 + (mi >> 1) * 8 + mr) * ldn + (mi & 1) * 8;
+                auto step = [&](int ks, float (&acc)[2][4]) {
                     uint32_t a[4], bq[4];
-                    ldmatrix4(a, Cs + (rt * 16 + (mi & 1) * 8 + mr) * ldn + ks * 16 + (mi >> 1) * 8);
-                    ldmatrix4(bq, Bs + (jb * 16 + (mi >> 1) * 8 + mr) * ldn + ks * 16 + (mi & 1) * 8);
-                    mma_bf16(gm[0], a, bq[0], bq[1]);
-                    mma_bf16(gm[1], a, bq[2], bq[3]);
-                }
+                    ldmatrix4(a, crow + ks * 16);
+                    ldmatrix4(bq, brow + ks * 16);
+                    mma_bf16(acc[0], a, bq[0], bq[1]);
+                    mma_bf16(acc[1], a, bq[2], bq[3]);
+                };
+                const int nk = p.N16 / 16;
+#pragma unroll 2
+                for (int ks = 0; ks + 1 < nk; ks += 2) { step(ks, gm[0]); step(ks + 1, gm[1]); }
+                if (nk & 1) step(nk - 1, gm[0]);
                 uint32_t ah[4], al[4];
 #pragma unroll
                 for (int x = 0; x < 2; ++x) {
                     const int j = jb * 16 + x * 8 + t4 * 2;
                     const float l0 = la[j], l1 = la[j + 1], d0 = dtv[j], d1 = dtv[j + 1];
-                    const float w00 = j <= ra ? gm[x][0] * exp2f(laa - l0) * d0 : 0.f, w01 = j + 1 <= ra ? gm[x][1] * exp2f(laa - l1) * d1 : 0.f;
-                    const float w10 = j <= rb ? gm[x][2] * exp2f(lab - l0) * d0 : 0.f, w11 = j + 1 <= rb ? gm[x][3] * exp2f(lab - l1) * d1 : 0.f;
+                    const float w00 = j <= ra ? (gm[0][x][0] + gm[1][x][0]) * exp2f(laa - l0) * d0 : 0.f;
+                    const float w01 = j + 1 <= ra ? (gm[0][x][1] + gm[1][x][1]) * exp2f(laa - l1) * d1 : 0.f;
+                    const float w10 = j <= rb ? (gm[0][x][2] + gm[1][x][2]) * exp2f(lab - l0) * d0 : 0.f;
+                    const float w11 = j + 1 <= rb ? (gm[0][x][3] + gm[1][x][3]) * exp2f(lab - l1) * d1 : 0.f;
                     split_hi_lo(w00, w01, ah[x * 2], al[x * 2]);
                     split_hi_lo(w10, w11, ah[x * 2 + 1], al[x * 2 + 1]);
                 }
+                uint32_t bx[HT / 2][4];
 #pragma unroll
-                for (int x = 0; x < PT; x += 2) {
-                    uint32_t bx[4];
-                    ldmatrix4_trans(bx, xs + (jb * 16 + (mi & 1) * 8 + mr) * ldp_s + x * 8 + (mi >> 1) * 8);
-                    mma_bf16(y[x], ah, bx[0], bx[1]);
-                    mma_bf16(y[x + 1], ah, bx[2], bx[3]);
-                    mma_bf16(y[x], al, bx[0], bx[1]);
-                    mma_bf16(y[x + 1], al, bx[2], bx[3]);
-                }
+                for (int x = 0; x < HT / 2; ++x) ldmatrix4_trans(bx[x], xs + (jb * 16 + (mi & 1) * 8 + mr) * ldp_s + (x0 + 2 * x) * 8 + (mi >> 1) * 8);
+#pragma unroll
+                for (int x = 0; x < HT; ++x) mma_bf16(y[x], ah, bx[x / 2][(x & 1) * 2], bx[x / 2][(x & 1) * 2 + 1]);
+#pragma unroll
+                for (int x = 0; x < HT; ++x) mma_bf16(y[x], al, bx[x / 2][(x & 1) * 2], bx[x / 2][(x & 1) * 2 + 1]);
             }
 #pragma unroll
-            for (int x = 0; x < PT; ++x)
+            for (int x = 0; x < HT; ++x)
 #pragma unroll
                 for (int hf = 0; hf < 2; ++hf) {
-                    const int r = hf ? rb : ra, c = x * 8 + t4 * 2;
+                    const int r = hf ? rb : ra, c = (x0 + x) * 8 + t4 * 2;
                     if (r >= tn || c >= pn) continue;
                     const float2 xv = Elem<__nv_bfloat16>::unpack2(*reinterpret_cast<const uint32_t*>(xs + r * ldp_s + c));
                     const float2 zv = Elem<__nv_bfloat16>::unpack2(*reinterpret_cast<const uint32_t*>(p.proj + (m0 + r) * p.ldp + h * p.P + p0 + c));
@@ -208,7 +236,7 @@ ssd_chunk_kernel(ChunkParams p) {
         log_decay += last;
 #pragma unroll
         for (int i = 0; i < MT; ++i) {
-            const int n0 = (warp + 4 * i) * 16;
+            const int n0 = (warp + 8 * i) * 16;
             if (n0 >= p.N16) break;
 #pragma unroll
             for (int x = 0; x < PT; ++x)
@@ -216,8 +244,10 @@ ssd_chunk_kernel(ChunkParams p) {
                 for (int e = 0; e < 4; ++e) S[i][x][e] *= decay;
 #pragma unroll
             for (int ks = 0; ks < kChunk / 16; ++ks) {
-                uint32_t a[4], ah[4], al[4];
+                uint32_t a[4], ah[4], al[4], bx[PT / 2][4];
                 ldmatrix4_trans(a, Bs + (ks * 16 + (mi >> 1) * 8 + mr) * ldn + n0 + (mi & 1) * 8);
+#pragma unroll
+                for (int x = 0; x < PT / 2; ++x) ldmatrix4_trans(bx[x], xs + (ks * 16 + (mi & 1) * 8 + mr) * ldp_s + x * 16 + (mi >> 1) * 8);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int j = ks * 16 + (e >> 1) * 8 + t4 * 2;
@@ -225,14 +255,9 @@ ssd_chunk_kernel(ChunkParams p) {
                     split_hi_lo(v.x * wv[j], v.y * wv[j + 1], ah[e], al[e]);
                 }
 #pragma unroll
-                for (int x = 0; x < PT; x += 2) {
-                    uint32_t bx[4];
-                    ldmatrix4_trans(bx, xs + (ks * 16 + (mi & 1) * 8 + mr) * ldp_s + x * 8 + (mi >> 1) * 8);
-                    mma_bf16(S[i][x], ah, bx[0], bx[1]);
-                    mma_bf16(S[i][x + 1], ah, bx[2], bx[3]);
-                    mma_bf16(S[i][x], al, bx[0], bx[1]);
-                    mma_bf16(S[i][x + 1], al, bx[2], bx[3]);
-                }
+                for (int x = 0; x < PT; ++x) mma_bf16(S[i][x], ah, bx[x / 2][(x & 1) * 2], bx[x / 2][(x & 1) * 2 + 1]);
+#pragma unroll
+                for (int x = 0; x < PT; ++x) mma_bf16(S[i][x], al, bx[x / 2][(x & 1) * 2], bx[x / 2][(x & 1) * 2 + 1]);
             }
         }
         __syncthreads();
@@ -245,7 +270,7 @@ ssd_chunk_kernel(ChunkParams p) {
         for (int x = 0; x < PT; ++x)
 #pragma unroll
             for (int hf = 0; hf < 2; ++hf) {
-                const int n = (warp + 4 * i) * 16 + g + hf * 8, c = x * 8 + t4 * 2;
+                const int n = (warp + 8 * i) * 16 + g + hf * 8, c = x * 8 + t4 * 2;
                 if (n < p.N && c < pn) *reinterpret_cast<float2*>(dst + static_cast<long long>(n) * p.Pp + c) = make_float2(S[i][x][hf * 2], S[i][x][hf * 2 + 1]);
             }
     if (!OUT && sl == 0 && threadIdx.x == 0) p.seg_decay[seg_row] = log_decay;
@@ -301,16 +326,16 @@ int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl
         if (int rc = allow_smem(first, tiles)) return rc;
         if (int rc = allow_smem(walk, all)) return rc;
         if (p.n_seg > 1) {
-            if (int rc = launch_pdl(first, dim3(static_cast<unsigned>(p.n_seg - 1), hs, bs), dim3(128), tiles, s, p)) return rc;
+            if (int rc = launch_pdl(first, dim3(static_cast<unsigned>(p.n_seg - 1), hs, bs), dim3(kThreads), tiles, s, p)) return rc;
             if (int rc = launch_pdl(ssd_segment_scan_kernel, dim3(static_cast<unsigned>((a.N * p.Pp + 255) / 256), static_cast<unsigned>(a.H), bs), dim3(256), 0, s, p)) return rc;
         }
         profile_mark_begin(s);
-        const int rc = launch_pdl(walk, dim3(static_cast<unsigned>(p.n_seg), hs, bs), dim3(128), all, s, p);
+        const int rc = launch_pdl(walk, dim3(static_cast<unsigned>(p.n_seg), hs, bs), dim3(kThreads), all, s, p);
         profile_mark_end(s);
         return rc;
     };
     note_ssd_kernel("ssd_chunk_kernel");
-    return a.N <= 128 ? go(ssd_chunk_kernel<2, 8, false>, ssd_chunk_kernel<2, 8, true>, 8) : go(ssd_chunk_kernel<4, 4, false>, ssd_chunk_kernel<4, 4, true>, 4);
+    return a.N <= 128 ? go(ssd_chunk_kernel<1, 8, false>, ssd_chunk_kernel<1, 8, true>, 8) : go(ssd_chunk_kernel<2, 4, false>, ssd_chunk_kernel<2, 4, true>, 4);
 }
 
 }  // namespace vb200

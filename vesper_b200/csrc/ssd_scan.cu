@@ -64,20 +64,25 @@ ssd_conv_kernel(SsdParams p, const T* __restrict__ proj, T* __restrict__ state, 
             for (int k = 0; k < TAPS; ++k) w[k][j] = p.conv_w[static_cast<long long>(c0 + j) * TAPS + k];
 #pragma unroll
         for (int k = 0; k < TAPS - 1; ++k) fetch(t0 - (TAPS - 1) + k, x[k]);
-        for (int t = t0; t < t1; ++t) {
-            fetch(t, x[TAPS - 1]);
-            float a[VEC];
+        for (int tb = t0; tb < t1; tb += 4) {              // four tokens' loads in flight
+            float nx[4][VEC];
 #pragma unroll
-            for (int j = 0; j < VEC; ++j) {
-                a[j] = bias[j];
+            for (int u = 0; u < 4; ++u) fetch(min(tb + u, t1 - 1), nx[u]);
 #pragma unroll
-                for (int k = 0; k < TAPS; ++k) a[j] = fmaf(w[k][j], x[k][j], a[j]);
+            for (int u = 0; u < 4; ++u) {
+                if (tb + u >= t1) break;
+                float a[VEC];
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) {
+                    x[TAPS - 1][j] = nx[u][j];
+                    a[j] = bias[j];
+#pragma unroll
+                    for (int k = 0; k < TAPS; ++k) a[j] = fmaf(w[k][j], x[k][j], a[j]);
+#pragma unroll
+                    for (int k = 0; k < TAPS - 1; ++k) x[k][j] = x[k + 1][j];
+                }
+                emit(tb + u, a);
             }
-            emit(t, a);
-#pragma unroll
-            for (int k = 0; k < TAPS - 1; ++k)
-#pragma unroll
-                for (int j = 0; j < VEC; ++j) x[k][j] = x[k + 1][j];
         }
     } else {
         for (int t = t0; t < t1; ++t) {
@@ -106,7 +111,7 @@ ssd_conv_kernel(SsdParams p, const T* __restrict__ proj, T* __restrict__ state, 
 // registers over the whole portion.  STEP: one token, its convolution computed here and its input stored in the ring
 // (nobody reads that ring row in this step).
 template <typename T, int NI, bool STEP>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, NI <= 4 ? 4 : NI <= 8 ? 3 : 2)
 ssd_scan_kernel(SsdParams p, const T* __restrict__ proj, const T* __restrict__ xbc, T* __restrict__ conv_state, float* __restrict__ state, float* __restrict__ gated) {
     pdl_begin();
     extern __shared__ float sm[];
@@ -126,6 +131,7 @@ ssd_scan_kernel(SsdParams p, const T* __restrict__ proj, const T* __restrict__ x
         S[i] = active && n < p.N && pos > 0 ? *reinterpret_cast<const float4*>(sp + static_cast<long long>(n) * p.Pp) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     const float nA = -expf(p.A_log[h]), dtb = p.dt_bias[h], Dh = p.D[h];
+    const int ring = STEP ? pos % p.taps : 0;              // this token's row of the convolution ring
     for (int t = 0; t < p.T; ++t) {
         const long long m = static_cast<long long>(b) * p.T + t;
         const T* prow = proj + m * p.ldp;
@@ -146,13 +152,14 @@ ssd_scan_kernel(SsdParams p, const T* __restrict__ proj, const T* __restrict__ x
                 T* st = conv_state + static_cast<long long>(slot) * p.taps * p.channels + ch;
                 const float* w = p.conv_w + static_cast<long long>(ch) * p.taps;
                 float a = p.conv_b[ch];
-                for (int k = 0; k < p.taps - 1; ++k) {
-                    const int q = pos - (p.taps - 1) + k;
-                    if (q >= 0) a = fmaf(w[k], Elem<T>::to_f(st[static_cast<long long>(q % p.taps) * p.channels]), a);
+#pragma unroll 4
+                for (int k = max(0, p.taps - 1 - pos); k < p.taps - 1; ++k) {       // the inputs of earlier tokens, oldest first
+                    const int row = ring + 1 + k < p.taps ? ring + 1 + k : ring + 1 + k - p.taps;
+                    a = fmaf(w[k], Elem<T>::to_f(st[static_cast<long long>(row) * p.channels]), a);
                 }
                 a = fmaf(w[p.taps - 1], Elem<T>::to_f(cur), a);
                 v = Elem<T>::to_f(Elem<T>::from_f(silu_exact(a)));
-                if (i < width || (sl == 0 && h % (p.H / p.G) == 0)) st[static_cast<long long>(pos % p.taps) * p.channels] = cur;
+                if (i < width || (sl == 0 && h % (p.H / p.G) == 0)) st[static_cast<long long>(ring) * p.channels] = cur;
             } else {
                 v = Elem<T>::to_f(xbc[m * p.channels + ch]);
             }
@@ -193,19 +200,57 @@ ssd_scan_kernel(SsdParams p, const T* __restrict__ proj, const T* __restrict__ x
     }
 }
 
-// grid (norm groups, rows), 128 threads.
-template <typename GT, typename T>
+// grid (norm groups, rows), 128 threads.  VEC: eight elements at a time, up to 64 per thread held in registers.
+template <typename GT, typename T, bool VEC>
 __global__ void __launch_bounds__(128)
 gated_group_norm_kernel(const GT* __restrict__ gated, int inner, int part_len, const float* __restrict__ w, float eps, T* __restrict__ out, long long ldo) {
     pdl_begin();
     const long long m = blockIdx.y;
     const int c0 = blockIdx.x * part_len;
     const GT* src = gated + m * inner + c0;
+    T* dst = out + m * ldo + c0;
     __shared__ float part[4];
     float ss = 0.f;
-    for (int i = threadIdx.x; i < part_len; i += 128) { const float v = Elem<GT>::to_f(src[i]); ss += v * v; }
-    const float inv = 1.0f / sqrtf(block_sum<4>(ss, part) / static_cast<float>(part_len) + eps);
-    for (int i = threadIdx.x; i < part_len; i += 128) out[m * ldo + c0 + i] = Elem<T>::from_f(Elem<GT>::to_f(src[i]) * inv * w[c0 + i]);
+    if constexpr (VEC) {
+        constexpr int kMax = 8;
+        float v[kMax][8];
+        const int n8 = part_len / 8;
+#pragma unroll
+        for (int i = 0; i < kMax; ++i) {
+            const int k = threadIdx.x + i * 128;
+            if (k < n8) load8(src + k * 8, v[i]);
+        }
+#pragma unroll
+        for (int i = 0; i < kMax; ++i)
+            if (threadIdx.x + i * 128 < n8) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) ss += v[i][e] * v[i][e];
+            }
+        const float inv = 1.0f / sqrtf(block_sum<4>(ss, part) / static_cast<float>(part_len) + eps);
+#pragma unroll
+        for (int i = 0; i < kMax; ++i) {
+            const int k = threadIdx.x + i * 128;
+            if (k >= n8) break;
+            float wv[8];
+            load8(w + c0 + k * 8, wv);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) wv[e] *= v[i][e] * inv;
+            store8(dst + k * 8, wv);
+        }
+    } else {
+        for (int i = threadIdx.x; i < part_len; i += 128) { const float v = Elem<GT>::to_f(src[i]); ss += v * v; }
+        const float inv = 1.0f / sqrtf(block_sum<4>(ss, part) / static_cast<float>(part_len) + eps);
+        for (int i = threadIdx.x; i < part_len; i += 128) dst[i] = Elem<T>::from_f(Elem<GT>::to_f(src[i]) * inv * w[c0 + i]);
+    }
+}
+
+template <typename GT, typename T>
+int launch_group_norm(cudaStream_t s, const vb200_ssd_args& a, const void* gated) {
+    const int inner = a.H * a.P, len = inner / a.norm_groups;
+    const bool vec = len % 8 == 0 && len <= 8192 && a.ldo % 8 == 0 && reinterpret_cast<uintptr_t>(a.norm_w) % 16 == 0 && reinterpret_cast<uintptr_t>(a.out) % 16 == 0;
+    const dim3 grid(static_cast<unsigned>(a.norm_groups), static_cast<unsigned>(a.B * a.T));
+    return launch_pdl(vec ? gated_group_norm_kernel<GT, T, true> : gated_group_norm_kernel<GT, T, false>, grid, dim3(128), 0, s, static_cast<const GT*>(gated), inner, len,
+                      a.norm_w, a.eps, static_cast<T*>(a.out), static_cast<long long>(a.ldo));
 }
 
 }  // namespace
@@ -247,8 +292,6 @@ int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl) {
     void* xbc = ws;
     void* gated = ws + pl.conv_bytes;
     float* states = reinterpret_cast<float*>(ws + pl.conv_bytes + pl.gated_bytes);
-    const unsigned M = static_cast<unsigned>(a.B * a.T);
-    const int part_len = a.H * a.P / a.norm_groups;
 
     auto go = [&](auto tag) -> int {
         using T = decltype(tag);
@@ -266,8 +309,7 @@ int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl) {
         if constexpr (sizeof(T) == 2) {
             if (pl.chunked) {
                 if (int rc = launch_ssd_chunks(s, a, pl, xbc, gated, states)) return rc;
-                return launch_pdl(gated_group_norm_kernel<__nv_bfloat16, T>, dim3(static_cast<unsigned>(a.norm_groups), M), dim3(128), 0, s,
-                                  static_cast<const __nv_bfloat16*>(gated), a.H * a.P, part_len, a.norm_w, a.eps, static_cast<T*>(a.out), static_cast<long long>(a.ldo));
+                return launch_group_norm<__nv_bfloat16, T>(s, a, gated);
             }
         }
         const size_t smem = sizeof(float) * (2 * (p.p4s * 4 + 2 * a.N) + p.rows * p.p4s * 4);
@@ -283,8 +325,7 @@ int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl) {
         profile_mark_end(s);
         if (rc) return rc;
         note_ssd_kernel(a.T == 1 ? "ssd_scan_kernel (step)" : "ssd_scan_kernel");
-        return launch_pdl(gated_group_norm_kernel<float, T>, dim3(static_cast<unsigned>(a.norm_groups), M), dim3(128), 0, s, static_cast<const float*>(gated),
-                          a.H * a.P, part_len, a.norm_w, a.eps, static_cast<T*>(a.out), static_cast<long long>(a.ldo));
+        return launch_group_norm<float, T>(s, a, gated);
     };
     return a.dtype == VB200_F32 ? go(float{}) : go(__nv_bfloat16{});
 }
