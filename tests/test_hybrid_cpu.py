@@ -82,7 +82,7 @@ def test_workspace_plans(lib):
     q = 2 * 16 * 576
     assert sizes[0] == 4 * (q + 2 * 16 * 516)              # one slice: queries and one record per head
     s = hc.SsdArgs(struct_size=C.sizeof(hc.SsdArgs), dtype=1, B=1, T=1, H=8, P=64, N=128, G=1, taps=4, norm_groups=1)
-    assert L.vb200_ssd_workspace_bytes(C.byref(s)) == 8 * 64 * 4
+    assert L.vb200_ssd_workspace_bytes(C.byref(s)) == (8 * 64 + 2 * 128) * 2 + 8 * 64 * 4       # convolution output, gated values
     s.struct_size = a.struct_size = 8
     assert L.vb200_ssd_workspace_bytes(C.byref(s)) == 0 and L.vb200_latent_workspace_bytes(C.byref(a)) == 0
     assert L.vb200_ssd_forward(C.byref(s)) == -1 and L.vb200_latent_decode(C.byref(a)) == -1 and L.vb200_embed_sequence(None) == -1

@@ -106,6 +106,11 @@ __device__ __forceinline__ float block_sum(float v, float* part) {
     return t;
 }
 __device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
+// fp32 all the way in the fp32 form; the approximate exponential and division (a few ulp) where the result becomes bf16
+template <typename T> __device__ __forceinline__ float silu_for(float x) {
+    if constexpr (sizeof(T) == 4) return silu_exact(x);
+    else return __fdividef(x, 1.0f + __expf(-x));
+}
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 // cos / sin of position * f: the product and the reduction to one turn in fp64, the functions in fp32.
 __device__ __forceinline__ float2 rope_cs(int position, double f) {

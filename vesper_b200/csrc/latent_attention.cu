@@ -26,6 +26,7 @@ struct LatentParams {
     int splits, rank16, rot16, qld, part_ld;
     int n_rc;                    // 128-column blocks of a latent
     int rot_off;
+    int src_aligned;             // latents start at 16-byte boundaries of a projection row
 };
 
 // One latent row: c = rmsnorm(src[0..rank)) * w, key part rotated.  ring_row receives it (nullable), after the row it
@@ -33,6 +34,24 @@ struct LatentParams {
 template <typename T, int W>
 __device__ void latent_row(const LatentParams& p, const T* __restrict__ src, const float2* cs, T* ring_row, T* old_copy, T* ctx_row, float* part) {
     float ss = 0.f;
+    if (p.rank % 8 == 0 && p.rank <= W * 256 && p.src_aligned) {          // eight columns per thread, one pass
+        const int i = threadIdx.x * 8;
+        const bool on = i < p.rank;
+        float v[8] = {}, w[8] = {};
+        if (on) {
+            load8(src + i, v);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) { w[e] = p.c_norm[i + e]; ss += v[e] * v[e]; }
+        }
+        const float inv = 1.0f / sqrtf(block_sum<W>(ss, part) / static_cast<float>(p.rank) + p.eps);
+        if (on) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = v[e] * inv * w[e];
+            if (old_copy != nullptr) { float o[8]; load8(ring_row + i, o); store8(old_copy + i, o); }
+            if (ring_row != nullptr) store8(ring_row + i, v);
+            if (ctx_row != nullptr) store8(ctx_row + i, v);
+        }
+    } else {
     for (int i = threadIdx.x; i < p.rank; i += W * 32) { const float v = Elem<T>::to_f(src[i]); ss += v * v; }
     const float inv = 1.0f / sqrtf(block_sum<W>(ss, part) / static_cast<float>(p.rank) + p.eps);
     for (int i = threadIdx.x; i < p.rank; i += W * 32) {
@@ -40,6 +59,7 @@ __device__ void latent_row(const LatentParams& p, const T* __restrict__ src, con
         if (old_copy != nullptr) old_copy[i] = ring_row[i];
         if (ring_row != nullptr) ring_row[i] = v;
         if (ctx_row != nullptr) ctx_row[i] = v;
+    }
     }
     for (int i = p.rank + threadIdx.x; i < p.rot_off; i += W * 32) {      // context rows feed a product over the padded width
         if (old_copy != nullptr) old_copy[i] = Elem<T>::from_f(0.f);
@@ -154,7 +174,7 @@ latent_query_kernel(LatentParams p, const T* __restrict__ proj, const T* __restr
     float acc[kBT][8] = {};
     if (c0 < (p.rank + 7) / 8 * 8) {
         const T* w = w_uk + static_cast<long long>(h) * p.dim * p.ldu + c0;
-#pragma unroll 4
+#pragma unroll 8
         for (int d = dg; d < p.dim; d += 16) {
             float wv[8];
             load8(w + static_cast<long long>(d) * p.ldu, wv);
@@ -304,9 +324,11 @@ latent_value_kernel(LatentParams p, const float* __restrict__ part, const T* __r
             float wv[8];
             load8(w + c, wv);
 #pragma unroll
-            for (int b = 0; b < kBT; ++b)
-#pragma unroll
-                for (int j = 0; j < 8; ++j) acc[b] = fmaf(wv[j], o[b * p.rank16 + c + j], acc[b]);
+            for (int b = 0; b < kBT; ++b) {
+                const float4 x = *reinterpret_cast<const float4*>(o + b * p.rank16 + c), y = *reinterpret_cast<const float4*>(o + b * p.rank16 + c + 4);
+                acc[b] = fmaf(wv[0], x.x, fmaf(wv[1], x.y, fmaf(wv[2], x.z, fmaf(wv[3], x.w, acc[b]))));
+                acc[b] = fmaf(wv[4], y.x, fmaf(wv[5], y.y, fmaf(wv[6], y.z, fmaf(wv[7], y.w, acc[b]))));
+            }
         }
 #pragma unroll
         for (int b = 0; b < kBT; ++b) {
@@ -377,6 +399,7 @@ LatentParams params_of(const vb200_latent_args& a) {
     const LatentPlan pl = plan_latent(a);
     p.splits = pl.splits; p.rank16 = pl.rank16; p.rot16 = pl.rot16; p.qld = pl.qld; p.part_ld = pl.part_ld;
     p.n_rc = (p.rank16 + 127) / 128;
+    p.src_aligned = a.ldp % 8 == 0 && (static_cast<long long>(a.H) * (a.dim + a.rot_dim)) % 8 == 0;
     return p;
 }
 

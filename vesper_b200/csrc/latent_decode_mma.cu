@@ -1,8 +1,8 @@
 // Decode attention over latents (one token per sequence, absorbed queries) with warp-level MMAs.
 //
 // Every head reads the same latent rows, so up to 16 heads of a sequence form the rows of m16n8k16 products and each row
-// of the ring is fetched once per 16 heads.  The queries arrive in fp32 with scale * log2 e folded in and enter the
-// products as hi + lo bf16 halves, the softmax weights likewise, so scores and weights keep fp32-class accuracy.
+// of the ring is fetched once per 16 heads.  The queries (fp32, scale * log2 e folded in) are rounded to bf16 like any
+// projection's output; scores and softmax stay fp32, and the weights enter the second product as hi + lo bf16 halves.
 //
 //   S[head, key] = q'[head, :] . row[key, :]     the 8 consumer warps take 16-column steps in turn (A in registers,
 //                                                B = rows by ldmatrix) and add their partial S through shared memory
@@ -20,6 +20,7 @@ constexpr int kBox = kTile * 128;
 constexpr int kWarps = 8;                // consumer warps
 constexpr int kStagesMax = 6;
 constexpr int kRedLd = 40;               // floats per row of a partial score tile: 8-row float2 accesses without conflicts
+constexpr float kGrow = 8.0f;
 constexpr int kPLd = 40;                 // bf16 per row of a weight tile: ldmatrix phases without conflicts
 
 struct LatentCacheMaps { CUtensorMap c, r; };
@@ -98,7 +99,7 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
     {
         const int g = lane >> 2, t = lane & 3;
         // A fragments of this warp's steps: rows = heads h0 + g, h0 + g + 8
-        uint32_t qh[KS][4], ql[KS][4];
+        uint32_t qh[KS][4];
 #pragma unroll
         for (int i = 0; i < KS; ++i) {
             const int kk = warp + i * kWarps;
@@ -107,7 +108,7 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
                 const int h = h0 + g + (e & 1) * 8;
                 float2 v = make_float2(0.f, 0.f);
                 if (kk < p.ks && h < p.H) v = *reinterpret_cast<const float2*>(p.q + (static_cast<long long>(b) * p.H + h) * p.qld + kk * 16 + (e >> 1) * 8 + t * 2);
-                split_hi_lo(v.x, v.y, qh[i][e], ql[i][e]);
+                qh[i][e] = Elem<__nv_bfloat16>::pack2(v.x, v.y);
             }
         }
         float o[NP][2][4];
@@ -119,29 +120,34 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
                 for (int e = 0; e < 4; ++e) o[i][x][e] = 0.f;
         const int row = tid >> 4, kp = (tid & 15) * 2;           // softmax: this thread's head and two keys
         float m = -1e30f, l = 0.f;
-        const int mi = lane >> 3, mr = lane & 7;                 // ldmatrix: matrix and row this lane addresses
+        // ldmatrix offsets inside a tile: this lane addresses row mr (mod 8) of matrix mi; 16 keys on = 2048 bytes
+        const int mi = lane >> 3, mr = lane & 7;
+        uint32_t s_off[KS], v_off[NP];
+#pragma unroll
+        for (int i = 0; i < KS; ++i) {
+            const int kk = min(warp + i * kWarps, p.ks - 1), kc = kk < p.ksc ? kk : kk - p.ksc, box = (kk < p.ksc ? 0 : p.nbc) + (kc >> 2), ch = (kc & 3) * 2 + (mi & 1);
+            s_off[i] = box * kBox + ((mi >> 1) * 8 + mr) * 128 + ((ch ^ mr) << 4);
+        }
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+            const int blk = min(warp + i * kWarps, p.ksc - 1), ch = (blk & 3) * 2 + (mi >> 1);      // a block too many is computed and dropped
+            v_off[i] = (blk >> 2) * kBox + ((mi & 1) * 8 + mr) * 128 + ((ch ^ mr) << 4);
+        }
+        const uint32_t p_hi_a = smem_u32(&sm.p_hi[(mi & 1) * 8 + mr][(mi >> 1) * 8]), p_lo_a = smem_u32(&sm.p_lo[(mi & 1) * 8 + mr][(mi >> 1) * 8]);
         for (int it = 0; it < n_tiles; ++it) {
             const int s = it % p.stages, valid = min(kTile, k1 - k0 - it * kTile);
             const bool ok = mbar_wait_warp(&sm.full[s], (it / p.stages) & 1, ctx, 0xC2);
             uint8_t* tile = tiles + s * stage_bytes;
             const uint32_t tile_a = smem_u32(tile);
-            float c[4][4] = {}, cl[4][4] = {};
+            float c[4][4] = {};
             if (ok) {
 #pragma unroll
-                for (int i = 0; i < KS; ++i) {
-                    const int kk = warp + i * kWarps;
-                    if (kk >= p.ks) break;
-                    const int kc = kk < p.ksc ? kk : kk - p.ksc, box = (kk < p.ksc ? 0 : p.nbc) + (kc >> 2), ch = (kc & 3) * 2 + (mi & 1);
+                for (int i = 0; i < KS; ++i) {                   // steps past the last one have zero queries
                     uint32_t bq[2][4];
-#pragma unroll
-                    for (int half = 0; half < 2; ++half) {
-                        const int key = half * 16 + (mi >> 1) * 8 + mr;
-                        ldmatrix4(bq[half], tile_a + box * kBox + key * 128 + ((ch ^ (key & 7)) << 4));
-                    }
+                    ldmatrix4(bq[0], tile_a + s_off[i]);
+                    ldmatrix4(bq[1], tile_a + s_off[i] + 2048);
 #pragma unroll
                     for (int x = 0; x < 4; ++x) mma_bf16(c[x], qh[i], bq[x >> 1][(x & 1) * 2], bq[x >> 1][(x & 1) * 2 + 1]);
-#pragma unroll
-                    for (int x = 0; x < 4; ++x) mma_bf16(cl[x], ql[i], bq[x >> 1][(x & 1) * 2], bq[x >> 1][(x & 1) * 2 + 1]);
                 }
                 if (valid < kTile) {
                     // rows past the slice hold other tokens (or another sequence's): their weight is zero, and so must their
@@ -159,8 +165,8 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
             }
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
-                *reinterpret_cast<float2*>(&sm.red[warp][g][x * 8 + t * 2]) = make_float2(c[x][0] + cl[x][0], c[x][1] + cl[x][1]);
-                *reinterpret_cast<float2*>(&sm.red[warp][g + 8][x * 8 + t * 2]) = make_float2(c[x][2] + cl[x][2], c[x][3] + cl[x][3]);
+                *reinterpret_cast<float2*>(&sm.red[warp][g][x * 8 + t * 2]) = make_float2(c[x][0], c[x][1]);
+                *reinterpret_cast<float2*>(&sm.red[warp][g + 8][x * 8 + t * 2]) = make_float2(c[x][2], c[x][3]);
             }
             if (consumers_sync_any(!ok)) break;                  // a wait ran out: all consumers leave together
             if (tid == 0 && it > 0 && it - 1 + p.stages < n_tiles) load_tile(it - 1 + p.stages);
@@ -175,8 +181,9 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
             float mt = fmaxf(sv.x, sv.y);
 #pragma unroll
             for (int x = 8; x > 0; x >>= 1) mt = fmaxf(mt, __shfl_xor_sync(0xFFFFFFFFu, mt, x));
-            const float m_new = fmaxf(m, mt), alpha = exp2f(m - m_new);
-            const float p0 = exp2f(sv.x - m_new), p1 = exp2f(sv.y - m_new);
+            // the reference maximum follows only when a row grows by more than 2^8 beyond it: most tiles rescale nothing
+            const float m_new = mt > m + kGrow ? mt : m, alpha = fast_exp2(m - m_new);
+            const float p0 = fast_exp2(sv.x - m_new), p1 = fast_exp2(sv.y - m_new);
             float ls = p0 + p1;
 #pragma unroll
             for (int x = 8; x > 0; x >>= 1) ls += __shfl_xor_sync(0xFFFFFFFFu, ls, x);
@@ -192,22 +199,20 @@ latent_split_mma_kernel(const __grid_constant__ LatentCacheMaps maps, LatentSpli
             uint32_t ph[2][4], pl[2][4];
 #pragma unroll
             for (int ks = 0; ks < 2; ++ks) {
-                ldmatrix4(ph[ks], smem_u32(&sm.p_hi[(mi & 1) * 8 + mr][ks * 16 + (mi >> 1) * 8]));
-                ldmatrix4(pl[ks], smem_u32(&sm.p_lo[(mi & 1) * 8 + mr][ks * 16 + (mi >> 1) * 8]));
+                ldmatrix4(ph[ks], p_hi_a + ks * 32);
+                ldmatrix4(pl[ks], p_lo_a + ks * 32);
+            }
+            if (__any_sync(0xFFFFFFFFu, a0 != 1.0f || a1 != 1.0f)) {
+#pragma unroll
+                for (int i = 0; i < NP; ++i)
+#pragma unroll
+                    for (int x = 0; x < 2; ++x) { o[i][x][0] *= a0; o[i][x][1] *= a0; o[i][x][2] *= a1; o[i][x][3] *= a1; }
             }
 #pragma unroll
-            for (int i = 0; i < NP; ++i)
-#pragma unroll
-                for (int x = 0; x < 2; ++x) { o[i][x][0] *= a0; o[i][x][1] *= a0; o[i][x][2] *= a1; o[i][x][3] *= a1; }
-#pragma unroll
             for (int ks = 0; ks < 2; ++ks) {
-                const int key = ks * 16 + (mi & 1) * 8 + mr;
                 uint32_t bv[NP][4];
 #pragma unroll
-                for (int i = 0; i < NP; ++i) {
-                    const int blk = min(warp + i * kWarps, p.ksc - 1), ch = (blk & 3) * 2 + (mi >> 1);      // a block too many is computed and dropped
-                    ldmatrix4_trans(bv[i], tile_a + (blk >> 2) * kBox + key * 128 + ((ch ^ (key & 7)) << 4));
-                }
+                for (int i = 0; i < NP; ++i) ldmatrix4_trans(bv[i], tile_a + v_off[i] + ks * 2048);
 #pragma unroll
                 for (int i = 0; i < NP; ++i) { mma_bf16(o[i][0], ph[ks], bv[i][0], bv[i][1]); mma_bf16(o[i][1], ph[ks], bv[i][2], bv[i][3]); }
 #pragma unroll

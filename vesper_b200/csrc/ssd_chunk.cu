@@ -42,12 +42,17 @@ __device__ __forceinline__ void ldmatrix4_trans(uint32_t (&r)[4], const __nv_bfl
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(ptr)) : "memory");
 }
 
-// Brings a line closer while the current chunk computes.
-__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+__device__ __forceinline__ void cp_async16(const __nv_bfloat16* dst, const void* src, bool ok) {       // zeros when !ok
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_wait_all() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
 // MT: 16-row tiles of S per warp (rows dealt to the eight warps in turn); PT: 8-column tiles of the slice.  In the
 // output products warp w has token rows 16 (w & 3) .. and column half w >> 2.
 // OUT: the walk (outputs and, in the last segment, the final state); else the first pass (what a segment adds to S).
+// B and x of the next chunk are copied (cp.async) into second buffers while this one computes, C once its last reader
+// is through; step sizes and gates are fetched ahead into registers.
 template <int MT, int PT, bool OUT>
 __global__ void __launch_bounds__(kThreads, 2)
 ssd_chunk_kernel(ChunkParams p) {
@@ -55,12 +60,14 @@ ssd_chunk_kernel(ChunkParams p) {
     extern __shared__ __align__(16) uint8_t smem[];
     const int ldn = p.N16 + kPad;
     constexpr int kPw = PT * 8, ldp_s = kPw + kPad, HT = PT / 2;
-    __nv_bfloat16* Bs = reinterpret_cast<__nv_bfloat16*>(smem);        // [64][ldn]
-    __nv_bfloat16* xs = Bs + kChunk * ldn;                             // [64][ldp_s]
-    __nv_bfloat16* Cs = xs + kChunk * ldp_s;                           // [64][ldn]
-    __nv_bfloat16* Sh = Cs + kChunk * ldn;                             // [N16][ldp_s] high halves, then low halves
+    const int b_size = kChunk * ldn;
+    constexpr int x_size = kChunk * ldp_s;
+    __nv_bfloat16* Bbuf = reinterpret_cast<__nv_bfloat16*>(smem);      // 2 x [64][ldn]
+    __nv_bfloat16* xbuf = Bbuf + 2 * b_size;                           // 2 x [64][ldp_s]
+    __nv_bfloat16* Cs = xbuf + 2 * x_size;                             // [64][ldn]
+    __nv_bfloat16* Sh = Cs + b_size;                                   // [N16][ldp_s] high halves, then low halves
     __nv_bfloat16* Sl = Sh + p.N16 * ldp_s;
-    __shared__ float la[kChunk], dtv[kChunk], wv[kChunk];
+    __shared__ float s_la[2][kChunk], s_dt[2][kChunk], s_w[2][kChunk];
 
     const int seg = blockIdx.x, h = blockIdx.y / p.slices, sl = blockIdx.y % p.slices, b = blockIdx.z;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3, mi = lane >> 3, mr = lane & 7;
@@ -68,6 +75,61 @@ ssd_chunk_kernel(ChunkParams p) {
     const int slot = p.slots ? p.slots[b] : b;
     const float nA2 = -expf(p.A_log[h]) * kLog2e, dtb = p.dt_bias[h], Dh = OUT ? p.D[h] : 0.f;
     const long long seg_row = (static_cast<long long>(b) * p.n_seg + seg) * p.H + h;
+    const int c_begin = seg * p.seg_chunks, c_end = min((p.T + kChunk - 1) / kChunk, c_begin + p.seg_chunks);
+    const __nv_bfloat16* xbc = p.xbc + static_cast<long long>(b) * p.T * p.channels;
+    const __nv_bfloat16* proj = p.proj + static_cast<long long>(b) * p.T * p.ldp;
+
+    // ---- tile copies: 16-byte pieces, zero past the portion and past a matrix's width ----
+    const int nv = p.N16 / 8;
+    auto copy_nb = [&](const __nv_bfloat16* dst, int ch, int col0) {
+        for (int i = threadIdx.x; i < kChunk * nv; i += kThreads) {
+            const int r = i / nv, c = (i - r * nv) * 8, t = ch * kChunk + r;
+            const bool ok = t < p.T && c < p.N;
+            cp_async16(dst + r * ldn + c, xbc + (ok ? static_cast<long long>(t) * p.channels + col0 + c : 0), ok);
+        }
+    };
+    auto copy_x = [&](const __nv_bfloat16* dst, int ch) {
+        constexpr int pv = kPw / 8;
+        for (int i = threadIdx.x; i < kChunk * pv; i += kThreads) {
+            const int r = i / pv, c = (i % pv) * 8, t = ch * kChunk + r;
+            const bool ok = t < p.T && c < pn;
+            cp_async16(dst + r * ldp_s + c, xbc + (ok ? static_cast<long long>(t) * p.channels + h * p.P + p0 + c : 0), ok);
+        }
+    };
+    const int col_b = inner + grp * p.N, col_c = col_b + p.G * p.N, col_dt = 2 * inner + 2 * p.G * p.N + h;
+    // step sizes and the running log-decay of a chunk: warp 7, two tokens per lane
+    auto fetch_dt = [&](int ch, float (&raw)[2]) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int t = ch * kChunk + lane * 2 + e;
+            raw[e] = t < p.T ? __bfloat162float(proj[static_cast<long long>(t) * p.ldp + col_dt]) : 0.f;
+        }
+    };
+    auto scan_dt = [&](int ch, const float (&raw)[2]) {
+        float d[2], a[2];
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            d[e] = ch * kChunk + lane * 2 + e < p.T ? softplus_f(raw[e] + dtb) : 0.f;
+            a[e] = nA2 * d[e];
+        }
+        float s = a[0] + a[1];
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float v = __shfl_up_sync(0xFFFFFFFFu, s, o);
+            if (lane >= o) s += v;
+        }
+        const float excl = s - (a[0] + a[1]), l0 = excl + a[0], l1 = l0 + a[1], last = __shfl_sync(0xFFFFFFFFu, l1, 31);
+        const int q = ch & 1;
+        s_la[q][lane * 2] = l0; s_la[q][lane * 2 + 1] = l1;
+        s_dt[q][lane * 2] = d[0]; s_dt[q][lane * 2 + 1] = d[1];
+        s_w[q][lane * 2] = d[0] * fast_exp2(last - l0); s_w[q][lane * 2 + 1] = d[1] * fast_exp2(last - l1);
+    };
+    float raw_dt[2] = {0.f, 0.f};
+    copy_nb(Bbuf + (c_begin & 1) * b_size, c_begin, col_b);
+    copy_x(xbuf + (c_begin & 1) * x_size, c_begin);
+    if (OUT) copy_nb(Cs, c_begin, col_c);
+    cp_commit();
+    if (warp == 7) { fetch_dt(c_begin, raw_dt); scan_dt(c_begin, raw_dt); }
 
     // rows mt*16 + g, +8 and columns p0 + pt*8 + 2*t4 of the state
     float S[MT][PT][4];
@@ -87,104 +149,72 @@ ssd_chunk_kernel(ChunkParams p) {
                     S[i][x][hf * 2] = v.x; S[i][x][hf * 2 + 1] = v.y;
                 }
     }
+    auto publish_state = [&] {                      // S as the right operand of the next chunk's C S
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+            if ((warp + 8 * i) * 16 >= p.N16) break;
+            const int at0 = ((warp + 8 * i) * 16 + g) * ldp_s + t4 * 2;
+#pragma unroll
+            for (int x = 0; x < PT; ++x)
+#pragma unroll
+                for (int hf = 0; hf < 2; ++hf) {
+                    uint32_t hi, lo;
+                    split_hi_lo(S[i][x][hf * 2], S[i][x][hf * 2 + 1], hi, lo);
+                    *reinterpret_cast<uint32_t*>(Sh + at0 + hf * 8 * ldp_s + x * 8) = hi;
+                    *reinterpret_cast<uint32_t*>(Sl + at0 + hf * 8 * ldp_s + x * 8) = lo;
+                }
+        }
+    };
+    if (OUT) publish_state();
     float log_decay = 0.f;
-    const int c_begin = seg * p.seg_chunks, c_end = min((p.T + kChunk - 1) / kChunk, c_begin + p.seg_chunks);
     for (int ch = c_begin; ch < c_end; ++ch) {
-        const int t0 = ch * kChunk, tn = min(kChunk, p.T - t0);
-        const long long m0 = static_cast<long long>(b) * p.T + t0;
-        const __nv_bfloat16* src = p.xbc + m0 * p.channels;
-        // ---- tiles: 16-byte pieces, zero past the portion and past a matrix's width ----
-        const int nv = p.N16 / 8;
-        constexpr int pv = kPw / 8;
-        for (int i = threadIdx.x; i < kChunk * nv; i += kThreads) {
-            const int r = i / nv, c = (i - r * nv) * 8;
-            const bool ok = r < tn && c < p.N;
-            const __nv_bfloat16* q = src + static_cast<long long>(r) * p.channels + inner + grp * p.N + c;
-            uint4 vb = make_uint4(0, 0, 0, 0), vc = vb;
-            if (ok) {
-                vb = *reinterpret_cast<const uint4*>(q);
-                if (OUT) vc = *reinterpret_cast<const uint4*>(q + p.G * p.N);
-            }
-            *reinterpret_cast<uint4*>(Bs + r * ldn + c) = vb;
-            if (OUT) *reinterpret_cast<uint4*>(Cs + r * ldn + c) = vc;
-        }
-        for (int i = threadIdx.x; i < kChunk * pv; i += kThreads) {
-            const int r = i / pv, c = (i - r * pv) * 8;
-            *reinterpret_cast<uint4*>(xs + r * ldp_s + c) =
-                r < tn && c < pn ? *reinterpret_cast<const uint4*>(src + static_cast<long long>(r) * p.channels + h * p.P + p0 + c) : make_uint4(0, 0, 0, 0);
-        }
-        if (warp == 7) {                        // dt and the running log-decay: two tokens per lane
-            float d[2], a[2];
-#pragma unroll
-            for (int e = 0; e < 2; ++e) {
-                const int r = lane * 2 + e;
-                d[e] = r < tn ? softplus_f(__bfloat162float(p.proj[(m0 + r) * p.ldp + 2 * inner + 2 * p.G * p.N + h]) + dtb) : 0.f;
-                a[e] = nA2 * d[e];
-            }
-            float s = a[0] + a[1];
-#pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float v = __shfl_up_sync(0xFFFFFFFFu, s, o);
-                if (lane >= o) s += v;
-            }
-            const float excl = s - (a[0] + a[1]), l0 = excl + a[0], l1 = l0 + a[1], last = __shfl_sync(0xFFFFFFFFu, l1, 31);
-            la[lane * 2] = l0; la[lane * 2 + 1] = l1;
-            dtv[lane * 2] = d[0]; dtv[lane * 2 + 1] = d[1];
-            wv[lane * 2] = d[0] * exp2f(last - l0); wv[lane * 2 + 1] = d[1] * exp2f(last - l1);
-        }
-        if (OUT) {
-#pragma unroll
-            for (int i = 0; i < MT; ++i) {
-                const int n = (warp + 8 * i) * 16 + g;
-                if ((warp + 8 * i) * 16 >= p.N16) break;
-#pragma unroll
-                for (int x = 0; x < PT; ++x)
-#pragma unroll
-                    for (int hf = 0; hf < 2; ++hf) {
-                        uint32_t hi, lo;
-                        split_hi_lo(S[i][x][hf * 2], S[i][x][hf * 2 + 1], hi, lo);
-                        const int at = (n + hf * 8) * ldp_s + x * 8 + t4 * 2;
-                        *reinterpret_cast<uint32_t*>(Sh + at) = hi;
-                        *reinterpret_cast<uint32_t*>(Sl + at) = lo;
-                    }
-            }
-        }
-        __syncthreads();
-        if (ch + 1 < c_end) {                   // the next chunk's own lines (B and C are shared by the heads of a group)
-            const int r = threadIdx.x & 63, what = threadIdx.x >> 6;
-            if (t0 + kChunk + r < p.T) {
-                if (what == 0) prefetch_l2(src + static_cast<long long>(kChunk + r) * p.channels + h * p.P + p0);
-                else if (what == 1 && OUT) prefetch_l2(p.proj + (m0 + kChunk + r) * p.ldp + h * p.P + p0);
-                else if (what == 2) prefetch_l2(p.proj + (m0 + kChunk + r) * p.ldp + 2 * inner + 2 * p.G * p.N + h);
-            }
+        const int tn = min(kChunk, p.T - ch * kChunk), q = ch & 1;
+        const long long m0 = static_cast<long long>(b) * p.T + ch * kChunk;
+        const __nv_bfloat16 *Bs = Bbuf + q * b_size, *xs = xbuf + q * x_size;
+        const float *la = s_la[q], *dtv = s_dt[q], *wv = s_w[q];
+        cp_wait_all();
+        __syncthreads();                            // tiles, step sizes and S of this chunk are in place; the other buffers are free
+        const bool more = ch + 1 < c_end;
+        if (more) {
+            copy_nb(Bbuf + (q ^ 1) * b_size, ch + 1, col_b);
+            copy_x(xbuf + (q ^ 1) * x_size, ch + 1);
+            cp_commit();
+            if (warp == 7) fetch_dt(ch + 1, raw_dt);
         }
         const float last = la[kChunk - 1];
         if (OUT) {
             const int rt = warp & 3, x0 = (warp >> 2) * HT;        // this warp's 16 tokens and column tiles
             const int ra = rt * 16 + g, rb = ra + 8;
-            float y[HT][4] = {}, yl[HT][4] = {};
+            uint32_t z[HT][2];
+            const __nv_bfloat16* zrow = p.proj + m0 * p.ldp + h * p.P + p0 + x0 * 8 + t4 * 2;
+#pragma unroll
+            for (int x = 0; x < HT; ++x)
+#pragma unroll
+                for (int hf = 0; hf < 2; ++hf) {
+                    const int r = hf ? rb : ra;
+                    z[x][hf] = r < tn && (x0 + x) * 8 < pn ? *reinterpret_cast<const uint32_t*>(zrow + static_cast<long long>(r) * p.ldp + x * 8) : 0u;
+                }
+            float y[HT][4] = {};
             const __nv_bfloat16* crow = Cs + (rt * 16 + (mi & 1) * 8 + mr) * ldn + (mi >> 1) * 8;
+            const int s_at = ((mi & 1) * 8 + mr) * ldp_s + x0 * 8 + (mi >> 1) * 8;
+            const int nk = p.N16 / 16;
 #pragma unroll 2
-            for (int ks = 0; ks < p.N16 / 16; ++ks) {
+            for (int ks = 0; ks < nk; ++ks) {
                 uint32_t a[4], bh[HT / 2][4], bl[HT / 2][4];
                 ldmatrix4(a, crow + ks * 16);
 #pragma unroll
                 for (int x = 0; x < HT / 2; ++x) {
-                    const int at = (ks * 16 + (mi & 1) * 8 + mr) * ldp_s + (x0 + 2 * x) * 8 + (mi >> 1) * 8;
-                    ldmatrix4_trans(bh[x], Sh + at);
-                    ldmatrix4_trans(bl[x], Sl + at);
+                    ldmatrix4_trans(bh[x], Sh + s_at + ks * 16 * ldp_s + x * 16);
+                    ldmatrix4_trans(bl[x], Sl + s_at + ks * 16 * ldp_s + x * 16);
                 }
 #pragma unroll
                 for (int x = 0; x < HT; ++x) mma_bf16(y[x], a, bh[x / 2][(x & 1) * 2], bh[x / 2][(x & 1) * 2 + 1]);
 #pragma unroll
-                for (int x = 0; x < HT; ++x) mma_bf16(yl[x], a, bl[x / 2][(x & 1) * 2], bl[x / 2][(x & 1) * 2 + 1]);
+                for (int x = 0; x < HT; ++x) mma_bf16(y[x], a, bl[x / 2][(x & 1) * 2], bl[x / 2][(x & 1) * 2 + 1]);
             }
-            const float laa = la[ra], lab = la[rb], ea = exp2f(laa), eb = exp2f(lab);
+            const float laa = la[ra], lab = la[rb], ea = fast_exp2(laa), eb = fast_exp2(lab);
 #pragma unroll
-            for (int x = 0; x < HT; ++x) {
-                y[x][0] = (y[x][0] + yl[x][0]) * ea; y[x][1] = (y[x][1] + yl[x][1]) * ea;
-                y[x][2] = (y[x][2] + yl[x][2]) * eb; y[x][3] = (y[x][3] + yl[x][3]) * eb;
-            }
+            for (int x = 0; x < HT; ++x) { y[x][0] *= ea; y[x][1] *= ea; y[x][2] *= eb; y[x][3] *= eb; }
             for (int jb = 0; jb <= rt; ++jb) {
                 float gm[2][2][4] = {};                            // even and odd steps of the inner dimension
                 const __nv_bfloat16* brow = Bs + (jb * 16 + (mi >> 1) * 8 + mr) * ldn + (mi & 1) * 8;
@@ -195,7 +225,6 @@ ssd_chunk_kernel(ChunkParams p) {
                     mma_bf16(acc[0], a, bq[0], bq[1]);
                     mma_bf16(acc[1], a, bq[2], bq[3]);
                 };
-                const int nk = p.N16 / 16;
 #pragma unroll 2
                 for (int ks = 0; ks + 1 < nk; ks += 2) { step(ks, gm[0]); step(ks + 1, gm[1]); }
                 if (nk & 1) step(nk - 1, gm[0]);
@@ -203,11 +232,15 @@ ssd_chunk_kernel(ChunkParams p) {
 #pragma unroll
                 for (int x = 0; x < 2; ++x) {
                     const int j = jb * 16 + x * 8 + t4 * 2;
-                    const float l0 = la[j], l1 = la[j + 1], d0 = dtv[j], d1 = dtv[j + 1];
-                    const float w00 = j <= ra ? (gm[0][x][0] + gm[1][x][0]) * exp2f(laa - l0) * d0 : 0.f;
-                    const float w01 = j + 1 <= ra ? (gm[0][x][1] + gm[1][x][1]) * exp2f(laa - l1) * d1 : 0.f;
-                    const float w10 = j <= rb ? (gm[0][x][2] + gm[1][x][2]) * exp2f(lab - l0) * d0 : 0.f;
-                    const float w11 = j + 1 <= rb ? (gm[0][x][3] + gm[1][x][3]) * exp2f(lab - l1) * d1 : 0.f;
+                    const float2 l = *reinterpret_cast<const float2*>(la + j), d = *reinterpret_cast<const float2*>(dtv + j);
+                    float w00 = (gm[0][x][0] + gm[1][x][0]) * (fast_exp2(laa - l.x) * d.x), w01 = (gm[0][x][1] + gm[1][x][1]) * (fast_exp2(laa - l.y) * d.y);
+                    float w10 = (gm[0][x][2] + gm[1][x][2]) * (fast_exp2(lab - l.x) * d.x), w11 = (gm[0][x][3] + gm[1][x][3]) * (fast_exp2(lab - l.y) * d.y);
+                    if (jb == rt) {                                // the diagonal block: later tokens have no weight
+                        if (j > ra) w00 = 0.f;
+                        if (j + 1 > ra) w01 = 0.f;
+                        if (j > rb) w10 = 0.f;
+                        if (j + 1 > rb) w11 = 0.f;
+                    }
                     split_hi_lo(w00, w01, ah[x * 2], al[x * 2]);
                     split_hi_lo(w10, w11, ah[x * 2 + 1], al[x * 2 + 1]);
                 }
@@ -219,20 +252,27 @@ ssd_chunk_kernel(ChunkParams p) {
 #pragma unroll
                 for (int x = 0; x < HT; ++x) mma_bf16(y[x], al, bx[x / 2][(x & 1) * 2], bx[x / 2][(x & 1) * 2 + 1]);
             }
+            __nv_bfloat16* grow = p.gated + m0 * inner + h * p.P + p0 + x0 * 8 + t4 * 2;
 #pragma unroll
             for (int x = 0; x < HT; ++x)
 #pragma unroll
                 for (int hf = 0; hf < 2; ++hf) {
-                    const int r = hf ? rb : ra, c = (x0 + x) * 8 + t4 * 2;
-                    if (r >= tn || c >= pn) continue;
-                    const float2 xv = Elem<__nv_bfloat16>::unpack2(*reinterpret_cast<const uint32_t*>(xs + r * ldp_s + c));
-                    const float2 zv = Elem<__nv_bfloat16>::unpack2(*reinterpret_cast<const uint32_t*>(p.proj + (m0 + r) * p.ldp + h * p.P + p0 + c));
-                    *reinterpret_cast<uint32_t*>(p.gated + (m0 + r) * inner + h * p.P + p0 + c) =
-                        Elem<__nv_bfloat16>::pack2(fmaf(Dh, xv.x, y[x][hf * 2]) * silu_exact(zv.x), fmaf(Dh, xv.y, y[x][hf * 2 + 1]) * silu_exact(zv.y));
+                    const int r = hf ? rb : ra;
+                    if (r >= tn || (x0 + x) * 8 >= pn) continue;
+                    const float2 xv = Elem<__nv_bfloat16>::unpack2(*reinterpret_cast<const uint32_t*>(xs + r * ldp_s + (x0 + x) * 8 + t4 * 2));
+                    const float2 zv = Elem<__nv_bfloat16>::unpack2(z[x][hf]);
+                    *reinterpret_cast<uint32_t*>(grow + static_cast<long long>(r) * inner + x * 8) =
+                        Elem<__nv_bfloat16>::pack2(fmaf(Dh, xv.x, y[x][hf * 2]) * silu_for<__nv_bfloat16>(zv.x), fmaf(Dh, xv.y, y[x][hf * 2 + 1]) * silu_for<__nv_bfloat16>(zv.y));
                 }
+            if (more) {
+                __syncthreads();                    // C and the published S have been read
+                copy_nb(Cs, ch + 1, col_c);
+                cp_commit();
+            }
         }
+        if (more && warp == 7) scan_dt(ch + 1, raw_dt);
         // ---- state update ----
-        const float decay = exp2f(last);
+        const float decay = fast_exp2(last);
         log_decay += last;
 #pragma unroll
         for (int i = 0; i < MT; ++i) {
@@ -248,11 +288,11 @@ ssd_chunk_kernel(ChunkParams p) {
                 ldmatrix4_trans(a, Bs + (ks * 16 + (mi >> 1) * 8 + mr) * ldn + n0 + (mi & 1) * 8);
 #pragma unroll
                 for (int x = 0; x < PT / 2; ++x) ldmatrix4_trans(bx[x], xs + (ks * 16 + (mi & 1) * 8 + mr) * ldp_s + x * 16 + (mi >> 1) * 8);
+                const float2 w0 = *reinterpret_cast<const float2*>(wv + ks * 16 + t4 * 2), w1 = *reinterpret_cast<const float2*>(wv + ks * 16 + 8 + t4 * 2);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const int j = ks * 16 + (e >> 1) * 8 + t4 * 2;
-                    const float2 v = Elem<__nv_bfloat16>::unpack2(a[e]);
-                    split_hi_lo(v.x * wv[j], v.y * wv[j + 1], ah[e], al[e]);
+                    const float2 v = Elem<__nv_bfloat16>::unpack2(a[e]), w = e < 2 ? w0 : w1;
+                    split_hi_lo(v.x * w.x, v.y * w.y, ah[e], al[e]);
                 }
 #pragma unroll
                 for (int x = 0; x < PT; ++x) mma_bf16(S[i][x], ah, bx[x / 2][(x & 1) * 2], bx[x / 2][(x & 1) * 2 + 1]);
@@ -260,7 +300,7 @@ ssd_chunk_kernel(ChunkParams p) {
                 for (int x = 0; x < PT; ++x) mma_bf16(S[i][x], al, bx[x / 2][(x & 1) * 2], bx[x / 2][(x & 1) * 2 + 1]);
             }
         }
-        __syncthreads();
+        if (OUT && more) publish_state();
     }
     if (OUT && seg + 1 < p.n_seg) return;
     float* dst = OUT ? sp : p.seg_state + seg_row * p.N * p.Pp + p0;
@@ -320,8 +360,8 @@ int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl
     p.seg_state = states + (static_cast<long long>(a.B) * p.n_seg * a.H + 63) / 64 * 64;
     p.gated = static_cast<__nv_bfloat16*>(gated);
     auto go = [&](auto first, auto walk, int pt) -> int {
-        const size_t tiles = 2 * (static_cast<size_t>(kChunk) * (p.N16 + kPad) + kChunk * (pt * 8 + kPad));
-        const size_t all = tiles + 2 * (static_cast<size_t>(kChunk) * (p.N16 + kPad) + 2 * static_cast<size_t>(p.N16) * (pt * 8 + kPad));
+        const size_t nb = static_cast<size_t>(kChunk) * (p.N16 + kPad), xb = static_cast<size_t>(kChunk) * (pt * 8 + kPad);
+        const size_t tiles = 2 * (2 * nb + 2 * xb), all = tiles + 2 * (nb + 2 * static_cast<size_t>(p.N16) * (pt * 8 + kPad));
         const unsigned hs = static_cast<unsigned>(a.H * p.slices), bs = static_cast<unsigned>(a.B);
         if (int rc = allow_smem(first, tiles)) return rc;
         if (int rc = allow_smem(walk, all)) return rc;

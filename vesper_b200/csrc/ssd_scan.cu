@@ -1,6 +1,7 @@
 // The Mamba-2 mixer around its projections: causal convolution, the recurrence token by token (any sizes, fp32 or bf16;
-// one launch per decode step with the convolution inside), and the gated group RMSNorm.  The chunked form of the
-// recurrence for prompts is in ssd_chunk.cu.
+// decode steps and short portions), and the gated group RMSNorm.  The chunked form of the recurrence for prompts is in
+// ssd_chunk.cu.  (The convolution of a decode step is a launch of its own: inside the recurrence every head of a group
+// would repeat it for B and C, and measured slower.)
 #include "hybrid.cuh"
 
 namespace vb200 {
@@ -15,6 +16,18 @@ struct SsdParams {
 };
 
 constexpr int kConvTile = 32;   // tokens per CTA
+constexpr int kAhead = 8;       // tokens whose loads are in flight
+
+__device__ __forceinline__ void load2(const __nv_bfloat16* p, float (&v)[2]) {
+    const float2 f = Elem<__nv_bfloat16>::unpack2(*reinterpret_cast<const uint32_t*>(p));
+    v[0] = f.x; v[1] = f.y;
+}
+__device__ __forceinline__ void load2(const float* p, float (&v)[2]) {
+    const float2 f = *reinterpret_cast<const float2*>(p);
+    v[0] = f.x; v[1] = f.y;
+}
+__device__ __forceinline__ void store2(__nv_bfloat16* p, const float (&v)[2]) { *reinterpret_cast<uint32_t*>(p) = Elem<__nv_bfloat16>::pack2(v[0], v[1]); }
+__device__ __forceinline__ void store2(float* p, const float (&v)[2]) { *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]); }
 
 // grid (channel blocks, token tiles, B); a thread owns VEC channels.  Only the first tile's CTA reads the state (the
 // inputs ahead of the portion) and it alone writes it, after its own reads.
@@ -36,8 +49,8 @@ ssd_conv_kernel(SsdParams p, const T* __restrict__ proj, T* __restrict__ state, 
         if (src == nullptr) {
 #pragma unroll
             for (int j = 0; j < VEC; ++j) v[j] = 0.f;
-        } else if constexpr (VEC == 8) {
-            load8(src, v);
+        } else if constexpr (VEC == 2) {
+            load2(src, v);
         } else {
 #pragma unroll
             for (int j = 0; j < VEC; ++j) v[j] = Elem<T>::to_f(src[j]);
@@ -45,9 +58,9 @@ ssd_conv_kernel(SsdParams p, const T* __restrict__ proj, T* __restrict__ state, 
     };
     auto emit = [&](int t, float (&a)[VEC]) {
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) a[j] = silu_exact(a[j]);
+        for (int j = 0; j < VEC; ++j) a[j] = silu_for<T>(a[j]);
         T* dst = o + static_cast<long long>(t) * p.channels;
-        if constexpr (VEC == 8) store8(dst, a);
+        if constexpr (VEC == 2) store2(dst, a);
         else {
 #pragma unroll
             for (int j = 0; j < VEC; ++j) dst[j] = Elem<T>::from_f(a[j]);
@@ -64,12 +77,12 @@ ssd_conv_kernel(SsdParams p, const T* __restrict__ proj, T* __restrict__ state, 
             for (int k = 0; k < TAPS; ++k) w[k][j] = p.conv_w[static_cast<long long>(c0 + j) * TAPS + k];
 #pragma unroll
         for (int k = 0; k < TAPS - 1; ++k) fetch(t0 - (TAPS - 1) + k, x[k]);
-        for (int tb = t0; tb < t1; tb += 4) {              // four tokens' loads in flight
-            float nx[4][VEC];
+        for (int tb = t0; tb < t1; tb += kAhead) {
+            float nx[kAhead][VEC];
 #pragma unroll
-            for (int u = 0; u < 4; ++u) fetch(min(tb + u, t1 - 1), nx[u]);
+            for (int u = 0; u < kAhead; ++u) fetch(min(tb + u, t1 - 1), nx[u]);
 #pragma unroll
-            for (int u = 0; u < 4; ++u) {
+            for (int u = 0; u < kAhead; ++u) {
                 if (tb + u >= t1) break;
                 float a[VEC];
 #pragma unroll
@@ -108,11 +121,10 @@ ssd_conv_kernel(SsdParams p, const T* __restrict__ proj, T* __restrict__ state, 
 }
 
 // grid (H * slices, B), 256 threads: thread = one float4 column of the slice x every `rows`-th state row, the state in
-// registers over the whole portion.  STEP: one token, its convolution computed here and its input stored in the ring
-// (nobody reads that ring row in this step).
-template <typename T, int NI, bool STEP>
+// registers over the whole portion (decode: one token).
+template <typename T, int NI>
 __global__ void __launch_bounds__(256, NI <= 4 ? 4 : NI <= 8 ? 3 : 2)
-ssd_scan_kernel(SsdParams p, const T* __restrict__ proj, const T* __restrict__ xbc, T* __restrict__ conv_state, float* __restrict__ state, float* __restrict__ gated) {
+ssd_scan_kernel(SsdParams p, const T* __restrict__ proj, const T* __restrict__ xbc, float* __restrict__ state, float* __restrict__ gated) {
     pdl_begin();
     extern __shared__ float sm[];
     const int h = blockIdx.x / p.slices, sl = blockIdx.x - h * p.slices, b = blockIdx.y;
@@ -131,7 +143,6 @@ ssd_scan_kernel(SsdParams p, const T* __restrict__ proj, const T* __restrict__ x
         S[i] = active && n < p.N && pos > 0 ? *reinterpret_cast<const float4*>(sp + static_cast<long long>(n) * p.Pp) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     const float nA = -expf(p.A_log[h]), dtb = p.dt_bias[h], Dh = p.D[h];
-    const int ring = STEP ? pos % p.taps : 0;              // this token's row of the convolution ring
     for (int t = 0; t < p.T; ++t) {
         const long long m = static_cast<long long>(b) * p.T + t;
         const T* prow = proj + m * p.ldp;
@@ -146,24 +157,7 @@ ssd_scan_kernel(SsdParams p, const T* __restrict__ proj, const T* __restrict__ x
                 const int k = i - width;
                 ch = inner + (k < p.N ? g * p.N + k : p.G * p.N + g * p.N + k - p.N);
             }
-            float v;
-            if constexpr (STEP) {
-                const T cur = prow[inner + ch];
-                T* st = conv_state + static_cast<long long>(slot) * p.taps * p.channels + ch;
-                const float* w = p.conv_w + static_cast<long long>(ch) * p.taps;
-                float a = p.conv_b[ch];
-#pragma unroll 4
-                for (int k = max(0, p.taps - 1 - pos); k < p.taps - 1; ++k) {       // the inputs of earlier tokens, oldest first
-                    const int row = ring + 1 + k < p.taps ? ring + 1 + k : ring + 1 + k - p.taps;
-                    a = fmaf(w[k], Elem<T>::to_f(st[static_cast<long long>(row) * p.channels]), a);
-                }
-                a = fmaf(w[p.taps - 1], Elem<T>::to_f(cur), a);
-                v = Elem<T>::to_f(Elem<T>::from_f(silu_exact(a)));
-                if (i < width || (sl == 0 && h % (p.H / p.G) == 0)) st[static_cast<long long>(ring) * p.channels] = cur;
-            } else {
-                v = Elem<T>::to_f(xbc[m * p.channels + ch]);
-            }
-            buf[i] = v;
+            buf[i] = Elem<T>::to_f(xbc[m * p.channels + ch]);
         }
         const float dt = softplus_f(Elem<T>::to_f(prow[2 * inner + 2 * p.G * p.N + h]) + dtb), decay = expf(nA * dt);
         __syncthreads();
@@ -190,7 +184,7 @@ ssd_scan_kernel(SsdParams p, const T* __restrict__ proj, const T* __restrict__ x
             for (int k = 0; k < p.rows; ++k) y += red[k * width + i];
             y = fmaf(Dh, xs[i], y);
             const int col = h * p.P + pc0 + i;
-            gated[m * inner + col] = y * silu_exact(Elem<T>::to_f(prow[col]));
+            gated[m * inner + col] = y * silu_for<T>(Elem<T>::to_f(prow[col]));
         }
     }
 #pragma unroll
@@ -262,7 +256,7 @@ SsdPlan plan_ssd(const vb200_ssd_args& a) {
     pl.chunked = a.T > 1 && a.form != 1 && ssd_chunk_supported(a) && (a.form == 2 || a.T >= 16);
     const size_t esz = a.dtype == VB200_F32 ? 4 : 2, M = static_cast<size_t>(a.B) * a.T;
     auto up = [](size_t x) { return (x + 255) / 256 * 256; };
-    pl.conv_bytes = a.T > 1 ? up(M * pl.channels * esz) : 0;
+    pl.conv_bytes = up(M * pl.channels * esz);
     pl.gated_bytes = up(M * a.H * a.P * (pl.chunked ? 2 : 4));
     if (pl.chunked) {
         int slices, n_seg, seg_chunks;
@@ -296,13 +290,13 @@ int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl) {
     auto go = [&](auto tag) -> int {
         using T = decltype(tag);
         const T* proj = static_cast<const T*>(a.proj);
-        if (a.T > 1) {
-            const bool vec = (a.H * a.P) % 8 == 0 && p.channels % 8 == 0 && a.ldp % 8 == 0;
+        {
+            const bool vec = (a.H * a.P) % 2 == 0 && p.channels % 2 == 0 && a.ldp % 2 == 0;
             auto conv = [&](auto kernel, int v) {
                 const dim3 grid(static_cast<unsigned>((p.channels + 128 * v - 1) / (128 * v)), static_cast<unsigned>((a.T + kConvTile - 1) / kConvTile), static_cast<unsigned>(a.B));
                 return launch_pdl(kernel, grid, dim3(128), 0, s, p, proj, static_cast<T*>(a.conv_state), static_cast<T*>(xbc));
             };
-            const int rc = vec ? (a.taps == 4 ? conv(ssd_conv_kernel<T, 8, 4>, 8) : conv(ssd_conv_kernel<T, 8, 0>, 8))
+            const int rc = vec ? (a.taps == 4 ? conv(ssd_conv_kernel<T, 2, 4>, 2) : conv(ssd_conv_kernel<T, 2, 0>, 2))
                                : (a.taps == 4 ? conv(ssd_conv_kernel<T, 1, 4>, 1) : conv(ssd_conv_kernel<T, 1, 0>, 1));
             if (rc) return rc;
         }
@@ -316,15 +310,14 @@ int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl) {
         const dim3 grid(static_cast<unsigned>(a.H * p.slices), static_cast<unsigned>(a.B));
         auto scan = [&](auto kernel) -> int {
             if (int rc = allow_smem(kernel, smem)) return rc;
-            return launch_pdl(kernel, grid, dim3(256), smem, s, p, proj, static_cast<const T*>(xbc), static_cast<T*>(a.conv_state), a.state, static_cast<float*>(gated));
+            return launch_pdl(kernel, grid, dim3(256), smem, s, p, proj, static_cast<const T*>(xbc), a.state, static_cast<float*>(gated));
         };
         int rc;
         profile_mark_begin(s);
-        if (a.T == 1) rc = ni <= 4 ? scan(ssd_scan_kernel<T, 4, true>) : ni <= 8 ? scan(ssd_scan_kernel<T, 8, true>) : scan(ssd_scan_kernel<T, 16, true>);
-        else rc = ni <= 4 ? scan(ssd_scan_kernel<T, 4, false>) : ni <= 8 ? scan(ssd_scan_kernel<T, 8, false>) : scan(ssd_scan_kernel<T, 16, false>);
+        rc = ni <= 4 ? scan(ssd_scan_kernel<T, 4>) : ni <= 8 ? scan(ssd_scan_kernel<T, 8>) : scan(ssd_scan_kernel<T, 16>);
         profile_mark_end(s);
         if (rc) return rc;
-        note_ssd_kernel(a.T == 1 ? "ssd_scan_kernel (step)" : "ssd_scan_kernel");
+        note_ssd_kernel("ssd_scan_kernel");
         return launch_group_norm<float, T>(s, a, gated);
     };
     return a.dtype == VB200_F32 ? go(float{}) : go(__nv_bfloat16{});
