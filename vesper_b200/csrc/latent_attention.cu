@@ -146,9 +146,18 @@ constexpr int kBT = 4;           // batch rows per CTA of the two per-head produ
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_query_kernel(LatentParams p, const T* __restrict__ proj, const T* __restrict__ w_uk, T* __restrict__ cache, float* __restrict__ qa) {
-    pdl_begin();
     extern __shared__ float sm[];
     __shared__ float part[8];
+    // weights do not depend on the previous kernel: the first eight rows of this thread stream while it finishes
+    constexpr int kAhead = 8;
+    Raw8<T> ahead[kAhead];
+    const int cg = threadIdx.x & 15, dg = threadIdx.x >> 4, c0 = (blockIdx.x % p.n_rc) * 128 + cg * 8;
+    const bool mine = static_cast<int>(blockIdx.x) < p.H * p.n_rc && c0 < (p.rank + 7) / 8 * 8;
+    const T* wrow = w_uk + static_cast<long long>(blockIdx.x / p.n_rc) * p.dim * p.ldu + c0;
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i)
+        if (mine && dg + 16 * i < p.dim) ahead[i].load(wrow + static_cast<long long>(dg + 16 * i) * p.ldu);
+    pdl_begin();
     const int b0 = blockIdx.y * kBT, hq = p.dim + p.rot, half = p.rot / 2;
     if (static_cast<int>(blockIdx.x) >= p.H * p.n_rc) {           // the new latent row of one sequence
         const int b = b0 + blockIdx.x - p.H * p.n_rc;
@@ -170,21 +179,21 @@ latent_query_kernel(LatentParams p, const T* __restrict__ proj, const T* __restr
         qs[i] = b < nb ? Elem<T>::to_f(proj[static_cast<long long>(b0 + b) * p.ldp + static_cast<long long>(h) * hq + d]) : 0.f;
     }
     __syncthreads();
-    const int cg = threadIdx.x & 15, dg = threadIdx.x >> 4, c0 = rc * 128 + cg * 8;
     float acc[kBT][8] = {};
-    if (c0 < (p.rank + 7) / 8 * 8) {
-        const T* w = w_uk + static_cast<long long>(h) * p.dim * p.ldu + c0;
-#pragma unroll 8
-        for (int d = dg; d < p.dim; d += 16) {
-            float wv[8];
-            load8(w + static_cast<long long>(d) * p.ldu, wv);
+    if (mine) {
+        auto add = [&](int d, const float (&wv)[8]) {
 #pragma unroll
             for (int b = 0; b < kBT; ++b) {
                 const float q = qs[b * p.dim + d];
 #pragma unroll
                 for (int j = 0; j < 8; ++j) acc[b][j] = fmaf(q, wv[j], acc[b][j]);
             }
-        }
+        };
+        float wv[8];
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i)
+            if (dg + 16 * i < p.dim) { ahead[i].get(wv); add(dg + 16 * i, wv); }
+        for (int d = dg + 16 * kAhead; d < p.dim; d += 16) { load8(wrow + static_cast<long long>(d) * p.ldu, wv); add(d, wv); }
     }
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 #pragma unroll
@@ -273,17 +282,28 @@ latent_split_generic_kernel(LatentParams p, const float* __restrict__ qa, const 
 
 constexpr int kValueRows = 32;           // rows of W_uv_h per CTA
 
-// grid (H * ceil(vdim / 32), ceil(B / kBT)), 256 threads.
+// grid (H * ceil(vdim / 32), ceil(B / kBT)), 256 threads: a warp has four rows of W_uv_h, fetched before the wait for
+// latents of up to 512 columns.
 template <typename T>
 __global__ void __launch_bounds__(256)
 latent_value_kernel(LatentParams p, const float* __restrict__ part, const T* __restrict__ w_uv, T* __restrict__ out) {
-    pdl_begin();
     extern __shared__ float sm[];
     float* o = sm;                               // [kBT][rank16]
     float* coef = o + kBT * p.rank16;            // [kBT][splits]
     const int n_vc = (p.vdim + kValueRows - 1) / kValueRows;
     const int h = blockIdx.x / n_vc, v0 = (blockIdx.x % n_vc) * kValueRows, b0 = blockIdx.y * kBT;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nb = min(kBT, p.B - b0);
+    const int rank8 = (p.rank + 7) / 8 * 8;
+    constexpr int kRowsPerWarp = kValueRows / 8, kPieces = 2;
+    Raw8<T> ahead[kRowsPerWarp][kPieces];
+#pragma unroll
+    for (int r = 0; r < kRowsPerWarp; ++r)
+#pragma unroll
+        for (int k = 0; k < kPieces; ++k) {
+            const int v = v0 + warp + 8 * r, c = lane * 8 + 256 * k;
+            if (v < p.vdim && c < rank8) ahead[r][k].load(w_uv + (static_cast<long long>(h) * p.vdim + v) * p.ldu + c);
+        }
+    pdl_begin();
     if (warp < nb) {
         const float* rec = part + (static_cast<long long>(b0 + warp) * p.H + h) * p.splits * p.part_ld + p.rank16;
         const float sink = p.sink ? p.sink[h] * kLog2e : -INFINITY;
@@ -292,48 +312,60 @@ latent_value_kernel(LatentParams p, const float* __restrict__ part, const T* __r
         m = warp_max_f(m);
         float l = 0.f;
         for (int s = lane; s < p.splits; s += 32) {
-            const float c = exp2f(rec[static_cast<long long>(s) * p.part_ld] - m);
+            const float2 ml = *reinterpret_cast<const float2*>(rec + static_cast<long long>(s) * p.part_ld);
+            const float c = exp2f(ml.x - m);
             coef[warp * p.splits + s] = c;
-            l += c * rec[static_cast<long long>(s) * p.part_ld + 1];
+            l += c * ml.y;
         }
         l = warp_sum_f(l) + (p.sink ? exp2f(sink - m) : 0.f);
         const float inv = 1.0f / l;
         for (int s = lane; s < p.splits; s += 32) coef[warp * p.splits + s] *= inv;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < kBT * p.rank16 / 4; i += 256) {        // four columns of one sequence, all slices' loads in flight
+    for (int i = threadIdx.x; i < kBT * p.rank16 / 4; i += 256) {        // four columns of one sequence, many slices' loads in flight
         const int b = i / (p.rank16 / 4), c = (i - b * (p.rank16 / 4)) * 4;
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
         if (b < nb) {
             const float* rec = part + (static_cast<long long>(b0 + b) * p.H + h) * p.splits * p.part_ld + c;
-#pragma unroll 8
-            for (int s = 0; s < p.splits; ++s) {
-                const float4 r = *reinterpret_cast<const float4*>(rec + static_cast<long long>(s) * p.part_ld);
-                const float w = coef[b * p.splits + s];
-                v.x = fmaf(w, r.x, v.x); v.y = fmaf(w, r.y, v.y); v.z = fmaf(w, r.z, v.z); v.w = fmaf(w, r.w, v.w);
+            constexpr int kBatch = 8;
+            for (int s0 = 0; s0 < p.splits; s0 += kBatch) {
+                float4 r[kBatch];
+#pragma unroll
+                for (int u = 0; u < kBatch; ++u) r[u] = *reinterpret_cast<const float4*>(rec + static_cast<long long>(min(s0 + u, p.splits - 1)) * p.part_ld);
+#pragma unroll
+                for (int u = 0; u < kBatch; ++u) {
+                    const float w = s0 + u < p.splits ? coef[b * p.splits + s0 + u] : 0.f;
+                    v.x = fmaf(w, r[u].x, v.x); v.y = fmaf(w, r[u].y, v.y); v.z = fmaf(w, r[u].z, v.z); v.w = fmaf(w, r[u].w, v.w);
+                }
             }
         }
         *reinterpret_cast<float4*>(o + b * p.rank16 + c) = v;
     }
     __syncthreads();
-    const int rank8 = (p.rank + 7) / 8 * 8;
-    for (int v = v0 + warp; v < min(p.vdim, v0 + kValueRows); v += 8) {
-        const T* w = w_uv + (static_cast<long long>(h) * p.vdim + v) * p.ldu;
+#pragma unroll
+    for (int r = 0; r < kRowsPerWarp; ++r) {
+        const int v = v0 + warp + 8 * r;
+        if (v >= p.vdim) break;
         float acc[kBT] = {};
-        for (int c = lane * 8; c < rank8; c += 256) {
-            float wv[8];
-            load8(w + c, wv);
+        auto add = [&](int c, const float (&wv)[8]) {
 #pragma unroll
             for (int b = 0; b < kBT; ++b) {
                 const float4 x = *reinterpret_cast<const float4*>(o + b * p.rank16 + c), y = *reinterpret_cast<const float4*>(o + b * p.rank16 + c + 4);
                 acc[b] = fmaf(wv[0], x.x, fmaf(wv[1], x.y, fmaf(wv[2], x.z, fmaf(wv[3], x.w, acc[b]))));
                 acc[b] = fmaf(wv[4], y.x, fmaf(wv[5], y.y, fmaf(wv[6], y.z, fmaf(wv[7], y.w, acc[b]))));
             }
+        };
+        float wv[8];
+#pragma unroll
+        for (int k = 0; k < kPieces; ++k) {
+            const int c = lane * 8 + 256 * k;
+            if (c < rank8) { ahead[r][k].get(wv); add(c, wv); }
         }
+        for (int c = lane * 8 + 256 * kPieces; c < rank8; c += 256) { load8(w_uv + (static_cast<long long>(h) * p.vdim + v) * p.ldu + c, wv); add(c, wv); }
 #pragma unroll
         for (int b = 0; b < kBT; ++b) {
-            const float r = warp_sum_f(acc[b]);
-            if (lane == 0 && b < nb) out[static_cast<long long>(b0 + b) * p.ldo + static_cast<long long>(h) * p.vdim + v] = Elem<T>::from_f(r);
+            const float x = warp_sum_f(acc[b]);
+            if (lane == 0 && b < nb) out[static_cast<long long>(b0 + b) * p.ldo + static_cast<long long>(h) * p.vdim + v] = Elem<T>::from_f(x);
         }
     }
 }

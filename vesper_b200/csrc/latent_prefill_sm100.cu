@@ -61,7 +61,7 @@ latent_prefill_sm100_kernel(const __grid_constant__ LatentMaps maps, LatentTileP
     extern __shared__ __align__(1024) uint8_t smem[];
     __shared__ LatentBars bar;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int r0 = blockIdx.x * kRows, h = blockIdx.y, b = blockIdx.z;
+    const int r0 = static_cast<int>(gridDim.z - 1 - blockIdx.z) * kRows, h = blockIdx.x, b = blockIdx.y;      // tiles with most keys first
     const int n_old = p.n_ctx - p.T;
     const int first_lo = max(0, n_old + r0 - p.window + 1);
     const int last_key = min(n_old + r0 + kRows - 1, p.n_ctx - 1);
@@ -258,7 +258,7 @@ latent_prefill_sm100_kernel(const __grid_constant__ LatentMaps maps, LatentTileP
 
 bool latent_sm100_supported(const vb200_latent_args& a) {
     return a.dtype == VB200_BF16 && a.dim % 8 == 0 && a.rot_dim % 8 == 0 && a.rot_dim > 0 && a.vdim % 8 == 0 && a.dim <= 128 && a.rot_dim <= 64 && a.vdim <= 128 &&
-           a.scale > 0.f && a.ldp % 8 == 0 && a.ldkv % 8 == 0 && a.ldo % 8 == 0 && reinterpret_cast<uintptr_t>(a.ctx_kv) % 16 == 0 &&
+           a.scale > 0.f && a.T <= 65535 * kRows && a.ldp % 8 == 0 && a.ldkv % 8 == 0 && a.ldo % 8 == 0 && reinterpret_cast<uintptr_t>(a.ctx_kv) % 16 == 0 &&
            reinterpret_cast<uintptr_t>(a.ctx_latent) % 16 == 0 && reinterpret_cast<uintptr_t>(a.out) % 16 == 0;
 }
 
@@ -291,7 +291,7 @@ int launch_latent_prefill_sm100(cudaStream_t s, const vb200_latent_args& a, int*
     size_t smem = static_cast<size_t>(nb_k) * kQBox + used();
     if (smem < 80 * 1024) smem = 80 * 1024;          // never a third CTA on an SM: it would find no TMEM
     if (int rc = allow_smem(latent_prefill_sm100_kernel, smem)) return rc;
-    return launch_pdl(latent_prefill_sm100_kernel, dim3(static_cast<unsigned>((a.T + kRows - 1) / kRows), static_cast<unsigned>(a.H), static_cast<unsigned>(a.B)), dim3(kThreads),
+    return launch_pdl(latent_prefill_sm100_kernel, dim3(static_cast<unsigned>(a.H), static_cast<unsigned>(a.B), static_cast<unsigned>((a.T + kRows - 1) / kRows)), dim3(kThreads),
                       smem, s, maps, p);
 }
 

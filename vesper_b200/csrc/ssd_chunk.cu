@@ -80,20 +80,29 @@ ssd_chunk_kernel(ChunkParams p) {
     const __nv_bfloat16* proj = p.proj + static_cast<long long>(b) * p.T * p.ldp;
 
     // ---- tile copies: 16-byte pieces, zero past the portion and past a matrix's width ----
+    // this thread's first piece and the step between its pieces, in (row, column) of a tile
     const int nv = p.N16 / 8;
+    const int nb_r0 = threadIdx.x / nv, nb_c0 = (threadIdx.x % nv) * 8, nb_dr = kThreads / nv, nb_dc = (kThreads % nv) * 8;
     auto copy_nb = [&](const __nv_bfloat16* dst, int ch, int col0) {
-        for (int i = threadIdx.x; i < kChunk * nv; i += kThreads) {
-            const int r = i / nv, c = (i - r * nv) * 8, t = ch * kChunk + r;
-            const bool ok = t < p.T && c < p.N;
-            cp_async16(dst + r * ldn + c, xbc + (ok ? static_cast<long long>(t) * p.channels + col0 + c : 0), ok);
+        const __nv_bfloat16* src = xbc + static_cast<long long>(ch) * kChunk * p.channels + col0;
+        const int rows = p.T - ch * kChunk;
+        int c = nb_c0;
+        for (int r = nb_r0; r < kChunk; r += nb_dr) {
+            const bool ok = r < rows && c < p.N;
+            cp_async16(dst + r * ldn + c, ok ? src + static_cast<long long>(r) * p.channels + c : xbc, ok);
+            c += nb_dc;
+            if (c >= p.N16) { c -= p.N16; ++r; }
         }
     };
+    constexpr int pv = kPw / 8;
+    const int x_r0 = threadIdx.x / pv, x_c = (threadIdx.x % pv) * 8;
     auto copy_x = [&](const __nv_bfloat16* dst, int ch) {
-        constexpr int pv = kPw / 8;
-        for (int i = threadIdx.x; i < kChunk * pv; i += kThreads) {
-            const int r = i / pv, c = (i % pv) * 8, t = ch * kChunk + r;
-            const bool ok = t < p.T && c < pn;
-            cp_async16(dst + r * ldp_s + c, xbc + (ok ? static_cast<long long>(t) * p.channels + h * p.P + p0 + c : 0), ok);
+        const __nv_bfloat16* src = xbc + static_cast<long long>(ch) * kChunk * p.channels + h * p.P + p0 + x_c;
+        const int rows = x_c < pn ? p.T - ch * kChunk : 0;
+#pragma unroll
+        for (int r = x_r0; r < kChunk; r += kThreads / pv) {
+            const bool ok = r < rows;
+            cp_async16(dst + r * ldp_s + x_c, ok ? src + static_cast<long long>(r) * p.channels : xbc, ok);
         }
     };
     const int col_b = inner + grp * p.N, col_c = col_b + p.G * p.N, col_dt = 2 * inner + 2 * p.G * p.N + h;

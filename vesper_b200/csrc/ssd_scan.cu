@@ -70,7 +70,7 @@ ssd_conv_kernel(SsdParams p, const T* __restrict__ proj, T* __restrict__ state, 
 #pragma unroll
     for (int j = 0; j < VEC; ++j) bias[j] = p.conv_b[c0 + j];
     if constexpr (TAPS > 0) {
-        float w[TAPS][VEC], x[TAPS][VEC];
+        float w[TAPS][VEC], x[TAPS - 1 + kAhead][VEC];           // a window of inputs: the taps before a block, then the block
 #pragma unroll
         for (int j = 0; j < VEC; ++j)
 #pragma unroll
@@ -78,24 +78,29 @@ ssd_conv_kernel(SsdParams p, const T* __restrict__ proj, T* __restrict__ state, 
 #pragma unroll
         for (int k = 0; k < TAPS - 1; ++k) fetch(t0 - (TAPS - 1) + k, x[k]);
         for (int tb = t0; tb < t1; tb += kAhead) {
-            float nx[kAhead][VEC];
-#pragma unroll
-            for (int u = 0; u < kAhead; ++u) fetch(min(tb + u, t1 - 1), nx[u]);
+            const int n = min(kAhead, t1 - tb);
+            const T* src = in + static_cast<long long>(tb) * p.ldp;
 #pragma unroll
             for (int u = 0; u < kAhead; ++u) {
-                if (tb + u >= t1) break;
+                const T* q = src + static_cast<long long>(min(u, n - 1)) * p.ldp;
+                if constexpr (VEC == 2) load2(q, x[TAPS - 1 + u]);
+                else x[TAPS - 1 + u][0] = Elem<T>::to_f(q[0]);
+            }
+#pragma unroll
+            for (int u = 0; u < kAhead; ++u) {
                 float a[VEC];
 #pragma unroll
                 for (int j = 0; j < VEC; ++j) {
-                    x[TAPS - 1][j] = nx[u][j];
                     a[j] = bias[j];
 #pragma unroll
-                    for (int k = 0; k < TAPS; ++k) a[j] = fmaf(w[k][j], x[k][j], a[j]);
-#pragma unroll
-                    for (int k = 0; k < TAPS - 1; ++k) x[k][j] = x[k + 1][j];
+                    for (int k = 0; k < TAPS; ++k) a[j] = fmaf(w[k][j], x[u + k][j], a[j]);
                 }
-                emit(tb + u, a);
+                if (u < n) emit(tb + u, a);
             }
+#pragma unroll
+            for (int k = 0; k < TAPS - 1; ++k)
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) x[k][j] = x[kAhead + k][j];
         }
     } else {
         for (int t = t0; t < t1; ++t) {

@@ -128,6 +128,33 @@ def bench_ssd(cx, K, W, B, T):
                 frac=gbs / cx.peaks["hbm"], tflops=flops / kern_us / 1e6, bound="hbm")
 
 
+def bench_like_prefill(cx, K, W, B, T):
+    """The Llama-style decoder's prompt attention (16 query / 4 KV heads of 128, RoPE and append fused) at the same batch and length."""
+    torch = cx.torch
+    g = torch.Generator(device=cx.dev).manual_seed(4)
+    r = lambda *n: torch.randn(*n, generator=g, device=cx.dev, dtype=torch.bfloat16)
+    q, k, v = r(B, 16, T, 128), r(B, 4, T, 128), r(B, 4, T, 128)
+    o, kc, vc = torch.empty_like(q), torch.zeros_like(k), torch.zeros_like(v)
+    call_us, kern_us = _timed(cx, lambda: capi.prefill(q, k, v, o, None, scale=128 ** -0.5, causal=True, theta=10000.0, k_cache=kc, v_cache=vc), K, W)
+    tf = 4.0 * B * 16 * 128 * T * (T + 1) / 2 / kern_us / 1e6
+    return dict(what=f"like kernel: GQA prompt attention B={B} H=16/4 T={T} D=128", kernel="prefill_sm100_kernel", kernel_us=kern_us, call_us=call_us, tflops=tf,
+                frac=tf / cx.peaks["tf"], bound="tensor")
+
+
+def bench_like_decode(cx, K, W, B, keys):
+    """The Llama-style decoder's decode attention (16 query / 4 KV heads of 128)."""
+    torch = cx.torch
+    g = torch.Generator(device=cx.dev).manual_seed(5)
+    r = lambda *n: torch.randn(*n, generator=g, device=cx.dev, dtype=torch.bfloat16)
+    q, k1, v1 = r(B, 16, 1, 128), r(B, 4, 1, 128), r(B, 4, 1, 128)
+    kc, vc, o = r(B, 4, keys, 128), r(B, 4, keys, 128), torch.empty_like(q)
+    seq = torch.full((B,), keys - 1, dtype=torch.int32, device=cx.dev)
+    call_us, kern_us = _timed(cx, lambda: capi.decode(q, o, kc, vc, scale=128 ** -0.5, k_new=k1, v_new=v1, theta=10000.0, seq_lens=seq, max_len=keys), K, W)
+    gbs = B * keys * 4 * 128 * 2 * 2.0 / kern_us / 1e3
+    return dict(what=f"like kernel: GQA decode B={B} H=16/4 keys={keys} D=128", kernel="decode_gqa_mma_kernel", kernel_us=kern_us, call_us=call_us, gbs=gbs,
+                frac=gbs / cx.peaks["hbm"], bound="hbm")
+
+
 def bench_projections(cx, K, W):
     """The layer's GEMMs at decode and prompt sizes, which both decoders share."""
     torch = cx.torch
@@ -199,9 +226,10 @@ def bench_hybrid(cx, K=20, W=3, layers=None, part="all"):
     out = {}
     if part in ("all", "kernels"):
         out["kernels"] = [
-            bench_latent_prefill(cx, K, W, 4, 2048, 1 << 20), bench_latent_prefill(cx, K, W, 4, 2048, 1024), bench_latent_prefill(cx, K, W, 8, 512, 1024),
+            bench_like_prefill(cx, K, W, 4, 2048), bench_like_prefill(cx, K, W, 8, 512), bench_latent_prefill(cx, K, W, 4, 2048, 1 << 20), bench_latent_prefill(cx, K, W, 4, 2048, 1024), bench_latent_prefill(cx, K, W, 8, 512, 1024),
             bench_latent_prefill(cx, K, W, 1, 8192, 1024), bench_latent_prefill(cx, K, W, 2, 2048, 1024, H=64),
-            bench_latent_decode(cx, K, W, 32, 4096), bench_latent_decode(cx, K, W, 128, 1024), bench_latent_decode(cx, K, W, 8, 1024), bench_latent_decode(cx, K, W, 32, 4096, H=64),
+            bench_like_decode(cx, K, W, 128, 2304), bench_like_decode(cx, K, W, 32, 2304), bench_like_decode(cx, K, W, 8, 576),       # bytes of the three below
+            bench_latent_decode(cx, K, W, 128, 4096), bench_latent_decode(cx, K, W, 32, 4096), bench_latent_decode(cx, K, W, 128, 1024), bench_latent_decode(cx, K, W, 8, 1024), bench_latent_decode(cx, K, W, 32, 4096, H=64),
             bench_ssd(cx, K, W, 8, 512), bench_ssd(cx, K, W, 1, 4096), bench_ssd(cx, K, W, 4, 2048), bench_ssd(cx, K, W, 8, 1), bench_ssd(cx, K, W, 64, 1)]
         out["projections"] = bench_projections(cx, K, W)
     if part in ("all", "models"):
