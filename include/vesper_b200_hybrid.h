@@ -144,7 +144,7 @@ typedef struct vb200_ssd_args {
     float* state;
     void* out; int64_t ldo;      /* [B*T, H * P] */
     void* workspace; size_t workspace_bytes;
-    int32_t form;                /* 0 = choose, 1 = token by token, 2 = chunked (bf16) */
+    int32_t form;                /* 0 = choose, 1 = token by token, 2 = chunked (bf16), 3 = chunked with warp-level products only */
 } vb200_ssd_args;
 size_t vb200_ssd_workspace_bytes(const vb200_ssd_args* a);
 int vb200_ssd_forward(const vb200_ssd_args* a);

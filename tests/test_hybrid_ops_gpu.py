@@ -350,13 +350,17 @@ def test_ssd_whole_portions_and_tokens(cuda, kind, name):
     want = c.want(seq)
     _close(c.run(seq, [L]), want, TOL[kind])
     chunked = kind == "bf16" and name != "odd"
-    assert c.core.last_kernel() == ("ssd_chunk_kernel" if chunked else "ssd_scan_kernel")
+    walk = chunked and SSD[name]["P"] <= 64 and SSD[name]["N"] <= 128
+    assert c.core.last_kernel() == ("ssd_walk_sm100_kernel" if walk else "ssd_chunk_kernel" if chunked else "ssd_scan_kernel")
     _close(c.run(seq, _cuts(L, [2, 64, 3, 1, 1, 63, 2, 65, 17])), want, TOL[kind])
     _close(c.run(seq, [L - 40] + [1] * 40), want, TOL[kind])
     _close(c.run(seq[:30], [1] * 30), want[:30], TOL[kind])
     if chunked:                                      # token by token and chunked forms agree, whatever the portion
         _close(c.run(seq, [L], form=1), want, TOL[kind])
         _close(c.run(seq, _cuts(L, [2, 5, 9, 70]), form=2), want, TOL[kind])
+        _close(c.run(seq, _cuts(L, [129, 98]), form=2), want, TOL[kind])
+        _close(c.run(seq, _cuts(L, [3, 200]), form=3), want, TOL[kind])
+        assert c.core.last_kernel() == "ssd_chunk_kernel"
 
 
 def test_ssd_state_is_fp32_class_over_a_long_prompt(cuda):
@@ -369,8 +373,11 @@ def test_ssd_state_is_fp32_class_over_a_long_prompt(cuda):
     c.core.w["conv_w"].fill_(1.0)
     c.core.w["conv_b"].zero_()
     seq = c.sequence(900)
-    for form, cuts in ((2, [900]), (2, [333, 567]), (1, [900])):
-        c.run(seq, cuts, form=form)
+    outs = None
+    for form, cuts in ((2, [900]), (2, [333, 567]), (3, [900]), (1, [900])):
+        out = c.run(seq, cuts, form=form)
+        outs = out if form == 2 and len(cuts) == 1 else outs
+        _close(out, _np(outs), TOL["bf16"])                  # segments, portions and tokens give the same outputs
         x = ref.silu(seq.astype(np.float64)[:, 128:384])
         x = bf16_round(x.astype(np.float32)).astype(np.float64)
         dt = ref.softplus(seq.astype(np.float64)[:, 384:] + c.w["dt_bias"])

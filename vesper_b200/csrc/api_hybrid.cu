@@ -189,7 +189,9 @@ int vb200_ssd_forward(const vb200_ssd_args* a) {
     if (!a->workspace || a->workspace_bytes < pl.total) return set_detail(VB200_ERR_WORKSPACE, "vb200_ssd_forward: workspace too small");
     DeviceGuard g;
     if (int rc = g.init(a->device)) return rc;
-    return launch_ssd(static_cast<cudaStream_t>(a->stream), *a, pl);
+    int* status = kernel_status_word();
+    if (!status) return VB200_ERR_CUDA;
+    return launch_ssd(static_cast<cudaStream_t>(a->stream), *a, pl, status);
 }
 
 const char* vb200_last_ssd_kernel(void) { return t_ssd_kernel; }

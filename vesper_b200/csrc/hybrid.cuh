@@ -75,8 +75,10 @@ struct SsdPlan {
 SsdPlan plan_ssd(const vb200_ssd_args& a);
 bool ssd_chunk_supported(const vb200_ssd_args& a);
 void plan_ssd_chunks(const vb200_ssd_args& a, int* slices, int* n_seg, int* seg_chunks);          // ssd_chunk.cu
-int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl);
-int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, const void* xbc, void* gated, float* states);   // ssd_chunk.cu
+int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, int* status);
+int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, const void* xbc, void* gated, float* states, int* status);   // ssd_chunk.cu
+bool ssd_walk_supported(const vb200_ssd_args& a);                                                     // ssd_walk_sm100.cu
+int launch_ssd_walk(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, const void* xbc, void* gated, const float* seg_state, int n_seg, int seg_chunks64, int* status);
 
 #ifdef __CUDACC__
 // Programmatic dependent launch: let the next kernel be scheduled, then wait for the previous one's results.

@@ -8,6 +8,8 @@
 // m16n8k16 products, fp32 accumulation.  C, B and x are bf16 values as they come from the convolution; everything the
 // decays touch (the weights of the second sum, the weighted B of the state update, S itself as a right operand) enters
 // as hi + lo bf16 halves, so the recurrence keeps fp32-class accuracy.
+// Heads of up to 64 columns and 128 state rows take the tcgen05 walk (ssd_walk_sm100.cu) instead; this file's kernel then
+// only computes what segments add.
 // When batch x heads does not fill the machine the portion is cut into segments: a first pass computes what each
 // segment adds to the state, a small kernel chains them, and the walk starts every segment from its own state.
 #include "hybrid.cuh"
@@ -351,14 +353,17 @@ void plan_ssd_chunks(const vb200_ssd_args& a, int* slices, int* n_seg, int* seg_
     const int pw = a.N <= 128 ? 64 : 32, chunks = (a.T + kChunk - 1) / kChunk;
     *slices = (a.P + pw - 1) / pw;
     const long long ctas = static_cast<long long>(a.B) * a.H * *slices;
-    long long want = (2LL * device_sm_count() + ctas - 1) / ctas;
-    if (want > chunks / 2) want = chunks / 2;
+    const bool walk = a.form != 3 && ssd_walk_supported(a);         // chunks of 128 tokens, one CTA per SM
+    long long want = walk ? device_sm_count() / ctas : (2LL * device_sm_count() + ctas - 1) / ctas;
+    const int unit = walk ? 4 : 2;                                   // fewest 64-token chunks of a segment
+    if (want > chunks / unit) want = chunks / unit;
     if (want < 1) want = 1;
     *seg_chunks = static_cast<int>((chunks + want - 1) / want);
+    if (walk) *seg_chunks = (*seg_chunks + 1) / 2 * 2;
     *n_seg = (chunks + *seg_chunks - 1) / *seg_chunks;
 }
 
-int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, const void* xbc, void* gated, float* states) {
+int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, const void* xbc, void* gated, float* states, int* status) {
     ChunkParams p{};
     p.T = a.T; p.H = a.H; p.P = a.P; p.N = a.N; p.G = a.G; p.channels = pl.channels; p.Pp = pl.Pp; p.N16 = pad_to(a.N, 16);
     plan_ssd_chunks(a, &p.slices, &p.n_seg, &p.seg_chunks);
@@ -379,7 +384,7 @@ int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl
             if (int rc = launch_pdl(ssd_segment_scan_kernel, dim3(static_cast<unsigned>((a.N * p.Pp + 255) / 256), static_cast<unsigned>(a.H), bs), dim3(256), 0, s, p)) return rc;
         }
         profile_mark_begin(s);
-        const int rc = launch_pdl(walk, dim3(static_cast<unsigned>(p.n_seg), hs, bs), dim3(kThreads), all, s, p);
+        const int rc = a.form != 3 && ssd_walk_supported(a) ? launch_ssd_walk(s, a, pl, xbc, gated, p.seg_state, p.n_seg, p.seg_chunks, status) : launch_pdl(walk, dim3(static_cast<unsigned>(p.n_seg), hs, bs), dim3(kThreads), all, s, p);
         profile_mark_end(s);
         return rc;
     };

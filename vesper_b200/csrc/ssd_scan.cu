@@ -258,7 +258,7 @@ SsdPlan plan_ssd(const vb200_ssd_args& a) {
     SsdPlan pl{};
     pl.channels = a.H * a.P + 2 * a.G * a.N;
     pl.Pp = pad_to(a.P, 4);
-    pl.chunked = a.T > 1 && a.form != 1 && ssd_chunk_supported(a) && (a.form == 2 || a.T >= 16);
+    pl.chunked = a.T > 1 && a.form != 1 && ssd_chunk_supported(a) && (a.form >= 2 || a.T >= 16);
     const size_t esz = a.dtype == VB200_F32 ? 4 : 2, M = static_cast<size_t>(a.B) * a.T;
     auto up = [](size_t x) { return (x + 255) / 256 * 256; };
     pl.conv_bytes = up(M * pl.channels * esz);
@@ -272,7 +272,7 @@ SsdPlan plan_ssd(const vb200_ssd_args& a) {
     return pl;
 }
 
-int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl) {
+int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, int* status) {
     SsdParams p{};
     p.B = a.B; p.T = a.T; p.H = a.H; p.P = a.P; p.N = a.N; p.G = a.G; p.taps = a.taps; p.channels = pl.channels; p.Pp = pl.Pp;
     p.ldp = a.ldp; p.conv_w = a.conv_w; p.conv_b = a.conv_b; p.dt_bias = a.dt_bias; p.A_log = a.A_log; p.D = a.D; p.slots = a.slots; p.pos = a.pos;
@@ -307,7 +307,7 @@ int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl) {
         }
         if constexpr (sizeof(T) == 2) {
             if (pl.chunked) {
-                if (int rc = launch_ssd_chunks(s, a, pl, xbc, gated, states)) return rc;
+                if (int rc = launch_ssd_chunks(s, a, pl, xbc, gated, states, status)) return rc;
                 return launch_group_norm<__nv_bfloat16, T>(s, a, gated);
             }
         }
