@@ -25,9 +25,10 @@ typedef enum vb200_epilogue {
     VB200_EPI_F32 = 1,      /* out_f32[m, n]   = acc            (logits)                        */
     VB200_EPI_ADD_F32 = 2,  /* out_f32[m, n]  += acc            (residual: h = h + proj(x))     */
     VB200_EPI_RELU2 = 4,    /* out_bf16[m, n]  = max(acc, 0)^2                                  */
-    VB200_EPI_SWIGLU = 3    /* out_bf16[m, n/2] = silu(acc[m, n]) * acc[m, n+1], n even:
+    VB200_EPI_SWIGLU = 3,   /* out_bf16[m, n/2] = silu(acc[m, n]) * acc[m, n+1], n even:
                                W holds gate and up rows interleaved (row 2j = gate_j,
                                row 2j+1 = up_j), see vb200_interleave_rows                      */
+    VB200_EPI_REGLU = 5     /* out_bf16[m, n/2] = max(acc[m, n], 0) * acc[m, n+1], rows as above */
 } vb200_epilogue;
 
 /* y = x W^T.  x [M, K] bf16 with row stride ldx, W [N, K] bf16 with row stride

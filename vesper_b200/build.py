@@ -24,7 +24,8 @@ LIB = os.path.join(LIBDIR, "libvesper_b200.so")
 
 SOURCES = ["api.cu", "rope_append.cu", "prefill_f32.cu", "prefill_sm100.cu", "prefill_pair_sm100.cu", "decode_splitkv.cu", "decode_generic.cu", "decode_static.cu",
            "linear_sm100.cu", "block_ops.cu", "decode_exchange.cu", "decode_gqa_mma.cu", "flash_bwd_f32.cu",
-           "api_hybrid.cu", "sequence_ops.cu", "latent_attention.cu", "latent_prefill_sm100.cu", "latent_decode_mma.cu", "ssd_scan.cu", "ssd_chunk.cu", "ssd_walk_sm100.cu"]
+           "api_hybrid.cu", "sequence_ops.cu", "latent_attention.cu", "latent_prefill_sm100.cu", "latent_decode_mma.cu", "ssd_scan.cu", "ssd_chunk.cu", "ssd_walk_sm100.cu",
+           "sigmoid_attention.cu", "sigmoid_prefill_sm100.cu", "sigmoid_decode_mma.cu", "selective_scan.cu", "moe.cu"]
 HEADERS = ["common.cuh", "kernels.h", "hybrid.cuh", os.path.join("..", "..", "include", "vesper_b200.h"),
            os.path.join("..", "..", "include", "vesper_b200_block.h"), os.path.join("..", "..", "include", "vesper_b200_hybrid.h")]
 
@@ -81,7 +82,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
 HOST_DIR = os.path.join(PKG, "host")
 HOST_LIB = os.path.join(LIBDIR, "libvesper_b200_host.so")
 HOST_SOURCES = ["tensor.cpp", "attention.cpp", "attention_modules.cpp", "transformer.cpp", "generator.cpp", "modules.cpp", "c_api.cpp",
-                "json.cpp", "checkpoint.cpp", "language_model.cpp", "sequence_mixer.cpp", "hybrid.cpp"]
+                "json.cpp", "checkpoint.cpp", "language_model.cpp", "sequence_mixer.cpp", "feed_forward.cpp", "hybrid.cpp"]
 
 
 def build_host(force: bool = False) -> str:

@@ -600,11 +600,12 @@ int vb200_linear_bias(int device, void* stream, const void* x, int64_t ldx, cons
                       const float* bias, void* out, int64_t ldo, int32_t M, int32_t N, int32_t K,
                       int32_t epilogue, int32_t splits) {
     if (!x || !w || !out || M <= 0 || N <= 0 || K <= 0) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: null pointer or non-positive size");
-    if (epilogue < VB200_EPI_BF16 || epilogue > VB200_EPI_RELU2) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: unknown epilogue");
+    if (epilogue < VB200_EPI_BF16 || epilogue > VB200_EPI_REGLU) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: unknown epilogue");
     if (ldx < K || ldw < K) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: ldx and ldw must be >= K");
-    const int64_t out_cols = epilogue == VB200_EPI_SWIGLU ? N / 2 : N;
+    const bool gated = epilogue == VB200_EPI_SWIGLU || epilogue == VB200_EPI_REGLU;
+    const int64_t out_cols = gated ? N / 2 : N;
     if (ldo < out_cols) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: ldo smaller than the output row");
-    if (epilogue == VB200_EPI_SWIGLU && N % 2 != 0) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: the SwiGLU epilogue needs an even N");
+    if (gated && N % 2 != 0) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear: a gated epilogue needs an even N");
     const int out_elem = (epilogue == VB200_EPI_F32 || epilogue == VB200_EPI_ADD_F32) ? 4 : 2;
     if (K % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0 || (ldo * out_elem) % 16 != 0 || !aligned16(x) || !aligned16(w) || !aligned16(out))
         return set_detail(VB200_ERR_ALIGNMENT, "vb200_linear: K % 8, and 16-byte aligned bases and row strides, are required");
@@ -636,11 +637,12 @@ int vb200_linear_f32(int device, void* stream, const float* x, int64_t ldx, cons
 int vb200_linear_ex(const vb200_linear_args* a) {
     if (!a || a->struct_size != sizeof(vb200_linear_args)) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_args: null or struct_size mismatch");
     if (!a->x || !a->w || !a->out || a->M <= 0 || a->N <= 0 || a->K <= 0) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: null pointer or non-positive size");
-    if (a->epilogue < VB200_EPI_BF16 || a->epilogue > VB200_EPI_RELU2) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: unknown epilogue");
+    if (a->epilogue < VB200_EPI_BF16 || a->epilogue > VB200_EPI_REGLU) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: unknown epilogue");
     if (a->ldx < a->K || a->ldw < a->K) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: ldx and ldw must be >= K");
-    const int64_t out_cols = a->epilogue == VB200_EPI_SWIGLU ? a->N / 2 : a->N;
+    const bool gated = a->epilogue == VB200_EPI_SWIGLU || a->epilogue == VB200_EPI_REGLU;
+    const int64_t out_cols = gated ? a->N / 2 : a->N;
     if (a->ldo < out_cols) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: ldo smaller than the output row");
-    if (a->epilogue == VB200_EPI_SWIGLU && a->N % 2 != 0) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: the SwiGLU epilogue needs an even N");
+    if (gated && a->N % 2 != 0) return set_detail(VB200_ERR_INVALID_ARG, "vb200_linear_ex: a gated epilogue needs an even N");
     const int out_elem = (a->epilogue == VB200_EPI_F32 || a->epilogue == VB200_EPI_ADD_F32) ? 4 : 2;
     if (a->K % 8 != 0 || a->ldx % 8 != 0 || a->ldw % 8 != 0 || (a->ldo * out_elem) % 16 != 0 || !aligned16(a->x) || !aligned16(a->w) || !aligned16(a->out))
         return set_detail(VB200_ERR_ALIGNMENT, "vb200_linear_ex: K % 8, and 16-byte aligned bases and row strides, are required");

@@ -253,6 +253,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
             ws[k][r] = (n0 + r < N && k0 + k < K) ? w[static_cast<long long>(n0 + r) * ldw + k0 + k] : 0.f;
         }
         __syncthreads();
+        float part[4][4] = {};                   // sums of 16 products, added to the total as one: shorter chains of roundings
 #pragma unroll
         for (int k = 0; k < 16; ++k) {
             float a[4], b[4];
@@ -261,8 +262,12 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
-                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+                for (int j = 0; j < 4; ++j) part[i][j] = fmaf(a[i], b[j], part[i][j]);
         }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) acc[i][j] += part[i][j];
         __syncthreads();
     }
 #pragma unroll
@@ -271,6 +276,12 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
         for (int j = 0; j < 4; ++j) {
             const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
             if (m >= M || n >= N) continue;
+            if (epilogue == VB200_EPI_SWIGLU || epilogue == VB200_EPI_REGLU) {          // this thread holds the gate (even n) and its up
+                if (j & 1) continue;
+                const float g = acc[i][j] + (bias ? bias[n] : 0.f), u = acc[i][j + 1] + (bias ? bias[n + 1] : 0.f);
+                out[static_cast<long long>(m) * ldo + (n >> 1)] = (epilogue == VB200_EPI_REGLU ? fmaxf(g, 0.f) : g / (1.0f + expf(-g))) * u;
+                continue;
+            }
             const long long idx = static_cast<long long>(m) * ldo + n;
             float v = acc[i][j] + (bias ? bias[n] : 0.f);
             if (addend) v += addend[idx];

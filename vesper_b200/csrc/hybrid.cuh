@@ -45,6 +45,7 @@ void note_ssd_kernel(const char* name);
 // ---- sequence_ops.cu ----
 int launch_embed_sequence(cudaStream_t s, const vb200_embed_args& a, int* status);
 int launch_residual_add(cudaStream_t s, float* h, const float* addend, const float* vec, int M, int dim, const float* scale, void* scaled_out);
+int launch_norm_add(cudaStream_t s, const vb200_norm_add_args& a);
 int launch_rms_norm_f32(cudaStream_t s, const float* x, const float* w, float* out, int M, int dim, int count, float eps);
 
 // ---- latent attention ----
@@ -66,6 +67,17 @@ int launch_latent_prefill_sm100(cudaStream_t s, const vb200_latent_args& a, int*
 int launch_latent_decode(cudaStream_t s, const vb200_latent_args& a, int* status);
 int launch_latent_split_mma(cudaStream_t s, const vb200_latent_args& a, const LatentPlan& pl, const float* q, float* part, int* status);   // latent_decode_mma.cu
 
+// ---- causal depthwise convolution + silu, shared by the state-space mixers (ssd_scan.cu) ----
+struct ConvLaunch {
+    int dtype, B, T, channels, taps;
+    const void* proj; long long ldp, col;        // the channels start at column `col` of a projection row
+    const float *w, *b;                          // [channels, taps], [channels]
+    const int *slots, *pos;
+    void* state;                                 // [slots, taps, channels], input of position p in row p mod taps
+    void* out;                                   // [B*T, channels]
+};
+int launch_causal_conv(cudaStream_t s, const ConvLaunch& c);
+
 // ---- Mamba-2 ----
 struct SsdPlan {
     int channels, Pp;
@@ -79,6 +91,41 @@ int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, int* 
 int launch_ssd_chunks(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, const void* xbc, void* gated, float* states, int* status);   // ssd_chunk.cu
 bool ssd_walk_supported(const vb200_ssd_args& a);                                                     // ssd_walk_sm100.cu
 int launch_ssd_walk(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, const void* xbc, void* gated, const float* seg_state, int n_seg, int seg_chunks64, int* status);
+
+// ---- sigmoid attention with mixed heads ----
+struct SigPlan {
+    bool mma;                    // tensor-core kernel for this step (q' in bf16), else CUDA cores (q' in fp32)
+    int splits;                  // of a decode step
+    int qld;                     // columns of a q' row: G * dim padded to 16
+    size_t q_bytes, part_bytes, total;
+};
+SigPlan plan_sigattn(const vb200_sigattn_args& a);
+int launch_sigattn(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& pl, int* status);
+bool sig_prefill_sm100_supported(const vb200_sigattn_args& a);                                                                  // sigmoid_prefill_sm100.cu
+int launch_sig_prefill_sm100(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& pl, const void* q, int* status);
+bool sig_decode_mma_supported(const vb200_sigattn_args& a);                                                                     // sigmoid_decode_mma.cu
+int launch_sig_decode_mma(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& pl, const void* q, float* part, int* status);
+void note_sigattn_kernel(const char* name);
+
+// ---- selective scan ----
+struct SelectivePlan {
+    bool dt_gemm;                // step sizes by a product of their own (prompts), else inside the scan kernel
+    size_t conv_bytes, xdbl_bytes, dt_bytes, total;
+};
+SelectivePlan plan_selective(const vb200_selective_args& a);
+int launch_selective(cudaStream_t s, const vb200_selective_args& a, const SelectivePlan& pl, int* status);
+void note_selective_kernel(const char* name);
+
+// ---- mixture of experts ----
+struct MoePlan {
+    bool grouped;                // sorted by expert, tcgen05 products; else token by token on CUDA cores
+    int max_tiles;               // 128-row tiles the sorted rows can need
+    size_t logits, ids, weights, act, sorted_x, sorted_act, sorted_y, gather, row_weight, tiles, shared_act, total;      // byte offsets
+};
+MoePlan plan_moe(const vb200_moe_args& a);
+int launch_moe(cudaStream_t s, const vb200_moe_args& a, const MoePlan& pl, int* status);
+int launch_moe_route(cudaStream_t s, const float* logits, int ld, const float* correction, int M, int E, int top, int groups, int keep, float scale, int* ids, float* weights);
+void note_moe_kernel(const char* name);
 
 #ifdef __CUDACC__
 // Programmatic dependent launch: let the next kernel be scheduled, then wait for the previous one's results.

@@ -185,7 +185,7 @@ int launch_row_inv_rms(cudaStream_t s, const float* h, long long ld, float* inv_
 int launch_interleave_rows(cudaStream_t s, const void* a, const void* b, void* out, long long rows, long long cols);
 int launch_rms_norm(cudaStream_t s, const float* x, const float* weight, void* out_bf16, int M, int dim, float eps);
 int launch_silu_mul(cudaStream_t s, const void* gate, const void* up, void* out, long long n);
-// epilogue: VB200_EPI_F32, VB200_EPI_ADD_F32 or VB200_EPI_RELU2 (all fp32 here); addend as in LinearParams
+// epilogue: VB200_EPI_F32, VB200_EPI_ADD_F32, VB200_EPI_RELU2, VB200_EPI_SWIGLU or VB200_EPI_REGLU (all fp32 here); addend as in LinearParams
 int launch_linear_f32(cudaStream_t s, const float* x, long long ldx, const float* w, long long ldw, const float* bias, float* out,
                       long long ldo, int M, int N, int K, int epilogue = VB200_EPI_F32, const float* addend = nullptr);
 // norm_w / norm_out (nullable): also out_norm[m,:] = rmsnorm(out[m,:]) * norm_w as bf16

@@ -13,7 +13,7 @@
 //                         memory in a fixed order (deterministic) before the leader's epilogue.
 // Epilogues (fused, per output element): store bf16 | store fp32 | fp32 accumulate into the residual
 // stream (optionally plus a second fp32 addend) | squared ReLU -> bf16 | SwiGLU over interleaved (gate, up) weight rows -> bf16 (src/nn/swiglu.cpp:36-48,
-// ops::silu_mul src/ops/elementwise.cpp:1297-1328).
+// ops::silu_mul src/ops/elementwise.cpp:1297-1328) | the same with max(gate, 0).
 #include "kernels.h"
 
 #include <cuda.h>
@@ -70,6 +70,9 @@ __device__ __forceinline__ void ld_global_v8(const void* ptr, uint32_t (&w)[8]) 
     }
 }
 __device__ __forceinline__ float silu_f(float g) { return g / (1.0f + __expf(-g)); }
+template <int EPI> constexpr bool kGated = EPI == VB200_EPI_SWIGLU || EPI == VB200_EPI_REGLU;
+// the gate's activation of a gated epilogue
+template <int EPI> __device__ __forceinline__ float gate_f(float g) { return EPI == VB200_EPI_REGLU ? fmaxf(g, 0.f) : silu_f(g); }
 
 // One output element group of the wide kernel: 32 consecutive columns of one row.
 template <int EPI>
@@ -84,15 +87,15 @@ __device__ __forceinline__ void store_row32(const LinearParams& p, int row, int 
         for (int j = 0; j < 32; ++j)
             if (col0 + j < p.N) acc[j] = __float_as_uint(__uint_as_float(acc[j]) + __ldg(p.bias + col0 + j));
     }
-    if (EPI == VB200_EPI_SWIGLU) {
+    if (kGated<EPI>) {
         // columns (2j, 2j+1) = (gate_j, up_j) -> out[row, col0/2 + j]
         __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + static_cast<long long>(row) * p.ldo + (col0 >> 1);
         const int n_out = min(16, (p.N - col0) >> 1);
         uint32_t packed[8];
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
-            float a0 = silu_f(__uint_as_float(acc[4 * j])) * __uint_as_float(acc[4 * j + 1]);
-            float a1 = silu_f(__uint_as_float(acc[4 * j + 2])) * __uint_as_float(acc[4 * j + 3]);
+            float a0 = gate_f<EPI>(__uint_as_float(acc[4 * j])) * __uint_as_float(acc[4 * j + 1]);
+            float a1 = gate_f<EPI>(__uint_as_float(acc[4 * j + 2])) * __uint_as_float(acc[4 * j + 3]);
             packed[j] = Elem<__nv_bfloat16>::pack2(a0, a1);
         }
         if (n_out == 16) {
@@ -495,13 +498,13 @@ linear_skinny_kernel(const __grid_constant__ LinearMaps maps, LinearParams p, in
 #pragma unroll
             for (int j = 0; j < MT; ++j) acc[j] += bv;
         }
-        if (EPI == VB200_EPI_SWIGLU) {
+        if (kGated<EPI>) {
             __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
 #pragma unroll
             for (int j = 0; j < MT; ++j) {
                 const float other = __shfl_xor_sync(0xFFFFFFFFu, acc[j], 1);     // odd lanes hold the `up` rows
                 if (j < m_count && !(lane & 1) && n + 1 < p.N)
-                    out[static_cast<long long>(j) * p.ldo + (n >> 1)] = __float2bfloat16_rn(silu_f(acc[j]) * other);
+                    out[static_cast<long long>(j) * p.ldo + (n >> 1)] = __float2bfloat16_rn(gate_f<EPI>(acc[j]) * other);
             }
         } else if (n < p.N) {
 #pragma unroll
@@ -685,6 +688,7 @@ int launch_linear(cudaStream_t s, const LinearParams& p) {
         }
         case VB200_EPI_SWIGLU: return launch_epi<VB200_EPI_SWIGLU>(s, p);
         case VB200_EPI_RELU2: return launch_epi<VB200_EPI_RELU2>(s, p);
+        case VB200_EPI_REGLU: return launch_epi<VB200_EPI_REGLU>(s, p);
         default: return set_detail(VB200_ERR_INVALID_ARG, "unknown linear epilogue");
     }
 }

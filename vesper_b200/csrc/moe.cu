@@ -1,0 +1,245 @@
+// Mixture of experts: the router's choice, and the experts' products in two forms.
+//   token by token (any sizes, fp32 or bf16; decode steps)   every (token, chosen expert) pair streams its expert's weights through
+//                                                            CUDA cores; the shared expert is one more pair per token
+//   grouped (bf16 prompts)                                   (token, expert) pairs are sorted by expert and the rows of one expert form
+//                                                            128-row tiles of the tcgen05 product in linear_sm100.cu
+#include "hybrid.cuh"
+
+namespace vb200 {
+namespace {
+
+// ---- the choice: one warp per token ----
+constexpr int kRouteWarps = 4;
+
+struct Pick { float v; int i; };
+__device__ __forceinline__ Pick warp_argmax(Pick a) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+        const float v = __shfl_xor_sync(0xFFFFFFFFu, a.v, o);
+        const int i = __shfl_xor_sync(0xFFFFFFFFu, a.i, o);
+        if (v > a.v || (v == a.v && i < a.i)) { a.v = v; a.i = i; }
+    }
+    return a;
+}
+
+// s, choice [E], group [groups]: this warp's shared memory; choice is consumed
+__device__ __forceinline__ void route_token(const float* __restrict__ logits, const float* __restrict__ correction, int E, int top, int groups, int keep, float scale,
+                                            float* s, float* choice, float* group, int* __restrict__ ids, float* __restrict__ weights) {
+    const int lane = threadIdx.x & 31;
+    for (int e = lane; e < E; e += 32) {
+        const float v = 1.0f / (1.0f + expf(-logits[e]));
+        s[e] = v;
+        choice[e] = v + (correction != nullptr ? correction[e] : 0.f);
+    }
+    __syncwarp();
+    if (groups > 0) {
+        const int per = E / groups;
+        for (int g = lane; g < groups; g += 32) {
+            float a = -INFINITY, b = -INFINITY;          // the two largest
+            for (int i = 0; i < per; ++i) {
+                const float v = choice[g * per + i];
+                if (v > a) { b = a; a = v; }
+                else if (v > b) b = v;
+            }
+            group[g] = per > 1 ? a + b : a;
+        }
+        __syncwarp();
+        // a kept group is marked by NaN
+        for (int k = 0; k < keep; ++k) {
+            Pick best{-INFINITY, 0x7FFFFFFF};
+            for (int g = lane; g < groups; g += 32)
+                if (group[g] > best.v || (group[g] == best.v && best.i == 0x7FFFFFFF)) best = Pick{group[g], g};
+            best = warp_argmax(best);
+            if (lane == 0 && best.i < groups) group[best.i] = NAN;
+            __syncwarp();
+        }
+        for (int e = lane; e < E; e += 32)
+            if (!isnan(group[e / per])) choice[e] = -INFINITY;
+        __syncwarp();
+    }
+    float sum = 0.f, mine = 0.f;
+    int my_id = 0;
+    for (int k = 0; k < top; ++k) {
+        Pick best{-INFINITY, 0x7FFFFFFF};
+        for (int e = lane; e < E; e += 32)
+            if (choice[e] > best.v) best = Pick{choice[e], e};
+        best = warp_argmax(best);
+        const int id = best.i < E ? best.i : 0;
+        const float v = s[id];
+        sum += v;
+        if (lane == (k & 31)) { mine = v; my_id = id; }
+        if (lane == 0) choice[id] = -INFINITY;
+        if ((k & 31) == 31 || k + 1 == top) {            // park up to 32 picks, scaled below
+            const int k0 = k & ~31;
+            if (k0 + lane <= k) { ids[k0 + lane] = my_id; weights[k0 + lane] = mine; }
+        }
+        __syncwarp();
+    }
+    const float f = scale / (sum + 1e-20f);
+    for (int k = lane; k < top; k += 32) weights[k] *= f;
+}
+
+__global__ void __launch_bounds__(kRouteWarps * 32)
+moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int M, int E, int top, int groups, int keep, float scale, int* __restrict__ ids,
+                 float* __restrict__ weights) {
+    pdl_begin();
+    extern __shared__ float sm[];
+    const int warp = threadIdx.x >> 5, m = blockIdx.x * kRouteWarps + warp;
+    if (m >= M) return;
+    float* s = sm + warp * (2 * E + groups);
+    route_token(logits + static_cast<long long>(m) * ld, correction, E, top, groups, keep, scale, s, s + E, s + 2 * E, ids + static_cast<long long>(m) * top,
+                weights + static_cast<long long>(m) * top);
+}
+
+// ---- token by token ----
+struct MoeParams {
+    int M, dim, ff, ff_shared, E, top;
+    long long ld_out, ld_shared;
+    int act_ld;                  // activations of one (token, expert) pair
+};
+
+// dot product of a weight row and x (shared memory), eight columns per lane at a time; n8 = columns / 8
+template <typename T>
+__device__ __forceinline__ float row_dot(const T* __restrict__ w, const float* x, int n8) {
+    const int lane = threadIdx.x & 31;
+    float a = 0.f;
+    for (int k = lane; k < n8; k += 32) {
+        float v[8];
+        load8(w + k * 8, v);
+        const float4 x0 = *reinterpret_cast<const float4*>(x + k * 8), x1 = *reinterpret_cast<const float4*>(x + k * 8 + 4);
+        a = fmaf(v[0], x0.x, fmaf(v[1], x0.y, fmaf(v[2], x0.z, fmaf(v[3], x0.w, a))));
+        a = fmaf(v[4], x1.x, fmaf(v[5], x1.y, fmaf(v[6], x1.z, fmaf(v[7], x1.w, a))));
+    }
+    return warp_sum_f(a);
+}
+
+constexpr int kPairRows = 16;    // hidden units per CTA: two per warp
+
+// grid (ceil(max(ff, ff_shared) / kPairRows), top + (shared ? 1 : 0), M), 256 threads
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_pair_in_kernel(MoeParams p, const T* __restrict__ x, const int* __restrict__ ids, const T* __restrict__ w_in, const T* __restrict__ w_shared, T* __restrict__ act) {
+    pdl_begin();
+    extern __shared__ __align__(16) float xs[];
+    const int k = blockIdx.y, m = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const bool shared = k == p.top;
+    const int ff = shared ? p.ff_shared : p.ff, j0 = blockIdx.x * kPairRows;
+    if (j0 >= ff) return;
+    const T* w = shared ? w_shared : w_in + static_cast<long long>(ids[m * p.top + k]) * 2 * p.ff * p.dim;
+    for (int i = threadIdx.x * 8; i < p.dim; i += 256 * 8) {
+        float v[8];
+        load8(x + static_cast<long long>(m) * p.dim + i, v);
+        store8(xs + i, v);
+    }
+    __syncthreads();
+    T* dst = act + (static_cast<long long>(m) * (p.top + 1) + k) * p.act_ld;
+    for (int j = j0 + warp; j < min(ff, j0 + kPairRows); j += 8) {
+        const T* r = w + static_cast<long long>(2 * j) * p.dim;
+        const float g = row_dot(r, xs, p.dim / 8), u = row_dot(r + p.dim, xs, p.dim / 8);
+        if (lane == 0) dst[j] = Elem<T>::from_f(silu_for<T>(g) * u);
+    }
+    // the padding up to a multiple of eight is multiplied with zero weights and must be finite
+    if (j0 + kPairRows >= ff && threadIdx.x < 8 && ff + threadIdx.x < (ff + 7) / 8 * 8) dst[ff + threadIdx.x] = Elem<T>::from_f(0.f);
+}
+
+constexpr int kOutRows = 16;
+
+// grid (ceil(dim / kOutRows), M), 256 threads
+template <typename T>
+__global__ void __launch_bounds__(256)
+moe_pair_out_kernel(MoeParams p, const int* __restrict__ ids, const float* __restrict__ weights, const T* __restrict__ w_out, const T* __restrict__ w_shared, const T* __restrict__ act,
+                    float* __restrict__ y) {
+    pdl_begin();
+    extern __shared__ __align__(16) float as[];
+    const int m = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, d0 = blockIdx.x * kOutRows;
+    const int f8 = (p.ff + 7) / 8, s8 = (p.ff_shared + 7) / 8;
+    const T* src = act + static_cast<long long>(m) * (p.top + 1) * p.act_ld;
+    for (int i = threadIdx.x; i < p.top * f8 + s8; i += 256) {
+        const int k = min(i / f8, p.top), c = i - k * f8;
+        float v[8];
+        load8(src + k * p.act_ld + c * 8, v);
+        store8(as + i * 8, v);
+    }
+    __syncthreads();
+    for (int d = d0 + warp; d < min(p.dim, d0 + kOutRows); d += 8) {
+        float t = 0.f;
+        for (int k = 0; k < p.top; ++k) {
+            const int e = ids[m * p.top + k];
+            t = fmaf(weights[m * p.top + k], row_dot(w_out + (static_cast<long long>(e) * p.dim + d) * p.ld_out, as + k * f8 * 8, f8), t);
+        }
+        if (p.ff_shared > 0) t += row_dot(w_shared + static_cast<long long>(d) * p.ld_shared, as + p.top * f8 * 8, s8);
+        if (lane == 0) y[static_cast<long long>(m) * p.dim + d] = t;
+    }
+}
+
+int router_logits(cudaStream_t s, const vb200_moe_args& a, float* logits, int* status) {
+    if (a.dtype == VB200_F32)
+        return launch_linear_f32(s, static_cast<const float*>(a.x), a.dim, static_cast<const float*>(a.w_router), a.dim, nullptr, logits, pad_to(a.experts, 4), a.M, a.experts, a.dim);
+    LinearParams p{};
+    p.x = a.x; p.ldx = a.dim; p.w = a.w_router; p.ldw = a.dim; p.out = logits; p.ldo = pad_to(a.experts, 4); p.M = a.M; p.N = a.experts; p.K = a.dim;
+    p.epilogue = VB200_EPI_F32;
+    p.status = status;
+    return launch_linear(s, p);
+}
+
+}  // namespace
+
+MoePlan plan_moe(const vb200_moe_args& a) {
+    MoePlan pl{};
+    auto up = [](size_t x) { return (x + 255) / 256 * 256; };
+    const size_t esz = a.dtype == VB200_F32 ? 4 : 2, M = static_cast<size_t>(a.M), pairs = M * a.top;
+    size_t at = 0;
+    auto take = [&](size_t bytes) { const size_t o = at; at += up(bytes); return o; };
+    pl.grouped = false;
+    pl.logits = take(M * pad_to(a.experts, 4) * 4);
+    pl.ids = take(pairs * 4);
+    pl.weights = take(pairs * 4);
+    const size_t act_ld = pad_to(a.ff > a.ff_shared ? a.ff : a.ff_shared, 8);
+    pl.act = take(M * (a.top + 1) * act_ld * esz);
+    pl.total = at;
+    return pl;
+}
+
+int launch_moe_route(cudaStream_t s, const float* logits, int ld, const float* correction, int M, int E, int top, int groups, int keep, float scale, int* ids, float* weights) {
+    const size_t smem = sizeof(float) * kRouteWarps * (2 * E + groups);
+    if (int rc = allow_smem(moe_route_kernel, smem)) return rc;
+    return launch_pdl(moe_route_kernel, dim3(static_cast<unsigned>((M + kRouteWarps - 1) / kRouteWarps)), dim3(kRouteWarps * 32), smem, s, logits, ld, correction, M, E, top, groups, keep,
+                      scale, ids, weights);
+}
+
+int launch_moe(cudaStream_t s, const vb200_moe_args& a, const MoePlan& pl, int* status) {
+    uint8_t* ws = static_cast<uint8_t*>(a.workspace);
+    float *logits = reinterpret_cast<float*>(ws + pl.logits), *weights = reinterpret_cast<float*>(ws + pl.weights);
+    int* ids = reinterpret_cast<int*>(ws + pl.ids);
+    if (int rc = router_logits(s, a, logits, status)) return rc;
+    if (int rc = launch_moe_route(s, logits, pad_to(a.experts, 4), a.correction, a.M, a.experts, a.top, a.groups, a.keep, a.scale, ids, weights)) return rc;
+    MoeParams p{};
+    p.M = a.M; p.dim = a.dim; p.ff = a.ff; p.ff_shared = a.ff_shared; p.E = a.experts; p.top = a.top; p.ld_out = a.ld_out; p.ld_shared = a.ld_shared;
+    p.act_ld = pad_to(a.ff > a.ff_shared ? a.ff : a.ff_shared, 8);
+    auto go = [&](auto tag) -> int {
+        using T = decltype(tag);
+        T* act = reinterpret_cast<T*>(ws + pl.act);
+        const int widest = a.ff > a.ff_shared ? a.ff : a.ff_shared;
+        const size_t smem_in = sizeof(float) * a.dim, smem_out = sizeof(float) * (static_cast<size_t>(a.top) * pad_to(a.ff, 8) + pad_to(a.ff_shared, 8));
+        if (int rc = allow_smem(moe_pair_in_kernel<T>, smem_in)) return rc;
+        if (int rc = allow_smem(moe_pair_out_kernel<T>, smem_out)) return rc;
+        profile_mark_begin(s);
+        // grid z is limited to 65535 tokens: longer prompts go in slices
+        for (int m0 = 0; m0 < a.M; m0 += 65535) {
+            const int n = a.M - m0 < 65535 ? a.M - m0 : 65535;
+            T* act0 = act + static_cast<size_t>(m0) * (a.top + 1) * p.act_ld;
+            if (int rc = launch_pdl(moe_pair_in_kernel<T>, dim3(static_cast<unsigned>((widest + kPairRows - 1) / kPairRows), static_cast<unsigned>(a.top + (a.ff_shared > 0)), static_cast<unsigned>(n)),
+                                    dim3(256), smem_in, s, p, static_cast<const T*>(a.x) + static_cast<size_t>(m0) * a.dim, ids + static_cast<size_t>(m0) * a.top,
+                                    static_cast<const T*>(a.w_in), static_cast<const T*>(a.w_shared_in), act0)) return rc;
+            if (int rc = launch_pdl(moe_pair_out_kernel<T>, dim3(static_cast<unsigned>((a.dim + kOutRows - 1) / kOutRows), static_cast<unsigned>(n)), dim3(256), smem_out, s, p,
+                                    ids + static_cast<size_t>(m0) * a.top, weights + static_cast<size_t>(m0) * a.top, static_cast<const T*>(a.w_out),
+                                    static_cast<const T*>(a.w_shared_out), act0, a.y + static_cast<size_t>(m0) * a.dim)) return rc;
+        }
+        profile_mark_end(s);
+        note_moe_kernel("moe_pair_in_kernel");
+        return VB200_OK;
+    };
+    return a.dtype == VB200_F32 ? go(float{}) : go(__nv_bfloat16{});
+}
+
+}  // namespace vb200

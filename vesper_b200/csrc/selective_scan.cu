@@ -1,0 +1,325 @@
+// The selective state-space mixer with a state of its own per channel (Mamba-1): convolution and projections of the recurrence's inputs,
+// and the recurrence
+//
+//   S[c, n] = exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,    y_c = sum_n S[c, n] C_n + D_c x_c,    out = y * silu(z).
+//
+// Every (channel, state) pair has its own decay, so a chunk of tokens is no matrix product: the work is one exponential and two
+// multiply-adds per pair and token.  LP lanes share a channel, each holding NI of its states in registers over the whole portion; the
+// tokens come in tiles of kTile through a two-stage shared-memory ring filled with cp.async while the tile before is walked.
+#include "hybrid.cuh"
+
+#include <type_traits>
+
+namespace vb200 {
+namespace {
+
+constexpr int kTile = 32;          // tokens per shared-memory tile
+constexpr int kThreads = 128;
+
+struct ScanParams {
+    int B, T, inner, N, rank;
+    long long ldp, ldx, ldo;       // rows of proj, of [dt | B | C], of out
+    const float *A, *D, *dt_bias;
+    const int *slots, *pos;
+};
+
+__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// exp(dt * a): accurate in the fp32 form; where activations are bf16 the base-2 instruction (2 ulp), dt then carries log2 e
+template <typename T> __device__ __forceinline__ float decay_of(float dt, float a) {
+    if constexpr (sizeof(T) == 4) return expf(dt * a);
+    else return fast_exp2(dt * a);
+}
+template <typename T> __device__ __forceinline__ float decay_dt(float dt) { return sizeof(T) == 4 ? dt : dt * kLog2e; }
+
+// log(1 + exp(x)).  bf16 form: log(1 + u) = 2 artanh(u / (2 + u)) with u = exp(-|x|) <= 1, the series up to the 13th power (its
+// remainder is below 1e-8 of the sum at u = 1).
+template <typename T> __device__ __forceinline__ float softplus_for(float x) {
+    if constexpr (sizeof(T) == 4) return softplus_f(x);
+    const float u = fast_exp2(-fabsf(x) * kLog2e), s = __fdividef(u, 2.0f + u), q = s * s;
+    float r = 2.0f / 13.0f;
+    r = fmaf(r, q, 2.0f / 11.0f); r = fmaf(r, q, 2.0f / 9.0f); r = fmaf(r, q, 2.0f / 7.0f);
+    r = fmaf(r, q, 2.0f / 5.0f); r = fmaf(r, q, 2.0f / 3.0f); r = fmaf(r, q, 2.0f);
+    return fmaxf(x, 0.f) + s * r;
+}
+
+template <typename T, int LP, int NI>
+struct ScanTile {
+    static constexpr int kCh = kThreads / LP;                  // channels per CTA
+    static constexpr int kStates = LP * NI;
+    struct Stage {
+        alignas(16) T x[kTile][kCh], z[kTile][kCh];
+        alignas(16) float dt[kTile][kCh];
+        alignas(16) T bc[2][kTile][kStates];                   // B, C
+    };
+    Stage st[2];
+    alignas(16) float y[kTile][kCh + 1];
+};
+
+// grid (ceil(inner / kCh), B).  dt holds the step sizes before bias and softplus.
+template <typename T, int LP, int NI>
+__global__ void __launch_bounds__(kThreads)
+selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restrict__ xc, const T* __restrict__ xdbl, const float* __restrict__ dt, float* __restrict__ state,
+                      T* __restrict__ out) {
+    using S = ScanTile<T, LP, NI>;
+    constexpr int CH = S::kCh, V = 16 / sizeof(T);
+    extern __shared__ __align__(16) uint8_t raw[];
+    S& sm = *reinterpret_cast<S*>(raw);
+    const int tid = threadIdx.x, lane = tid % LP, ch = tid / LP, b = blockIdx.y, c0 = blockIdx.x * CH, c = c0 + ch;
+    const bool live = c < p.inner;
+    // weights do not depend on the launch before
+    float a[NI], S_[NI];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        const int n = lane * NI + i;
+        a[i] = live && n < p.N ? __ldg(p.A + static_cast<long long>(c) * p.N + n) : 0.f;
+    }
+    const float Dc = live ? __ldg(p.D + c) : 0.f;
+    pdl_begin();
+    const int pos = p.pos[b], slot = p.slots ? p.slots[b] : b;
+    float* sp = state + (static_cast<long long>(slot) * p.inner + c) * p.N + lane * NI;
+#pragma unroll
+    for (int i = 0; i < NI; i += 4) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (live && pos > 0 && lane * NI + i < p.N) v = *reinterpret_cast<const float4*>(sp + i);
+        S_[i] = v.x; S_[i + 1] = v.y; S_[i + 2] = v.z; S_[i + 3] = v.w;
+    }
+    const long long m0 = static_cast<long long>(b) * p.T;
+    auto load_tile = [&](int t0, int s) {
+        typename S::Stage& st = sm.st[s];
+        for (int i = tid; i < kTile * (CH / V); i += kThreads) {
+            const int t = i / (CH / V), k = (i - t * (CH / V)) * V;
+            const bool ok = t0 + t < p.T && c0 + k < p.inner;
+            const long long m = ok ? m0 + t0 + t : m0;
+            const int col = ok ? c0 + k : 0;
+            cp_async16(&st.x[t][k], xc + m * p.inner + col, ok);
+            cp_async16(&st.z[t][k], proj + m * p.ldp + p.inner + col, ok);
+        }
+        for (int i = tid; i < kTile * (CH / 4); i += kThreads) {
+            const int t = i / (CH / 4), k = (i - t * (CH / 4)) * 4;
+            const bool ok = t0 + t < p.T && c0 + k < p.inner;
+            cp_async16(&st.dt[t][k], dt + (ok ? (m0 + t0 + t) * p.inner + c0 + k : 0), ok);
+        }
+        constexpr int kVs = (S::kStates + V - 1) / V;
+        for (int i = tid; i < 2 * kTile * kVs; i += kThreads) {
+            const int w = i / (kTile * kVs), j = i - w * (kTile * kVs), t = j / kVs, k = (j - t * kVs) * V;
+            const bool ok = t0 + t < p.T && k < p.N;
+            cp_async16(&st.bc[w][t][k], xdbl + (ok ? (m0 + t0 + t) * p.ldx + p.rank + w * p.N + k : 0), ok);
+        }
+        cp_async_commit();
+    };
+    const int n_tiles = (p.T + kTile - 1) / kTile;
+    load_tile(0, 0);
+    for (int it = 0; it < n_tiles; ++it) {
+        const int t0 = it * kTile, nt = min(kTile, p.T - t0);
+        if (it + 1 < n_tiles) { load_tile(t0 + kTile, (it + 1) & 1); cp_async_wait<1>(); }
+        else cp_async_wait<0>();
+        __syncthreads();
+        typename S::Stage& st = sm.st[it & 1];
+        // softplus of the step sizes once per (token, channel), in place
+        for (int i = tid; i < kTile * CH; i += kThreads) {
+            const int t = i / CH, k = i - t * CH;
+            const float bk = c0 + k < p.inner ? __ldg(p.dt_bias + c0 + k) : 0.f;
+            st.dt[t][k] = softplus_for<T>(st.dt[t][k] + bk);
+        }
+        __syncthreads();
+#pragma unroll 4
+        for (int t = 0; t < nt; ++t) {
+            const float d = st.dt[t][ch], x = Elem<T>::to_f(st.x[t][ch]), dx = d * x, dl = decay_dt<T>(d);
+            float y = 0.f;
+            const T *Bt = &st.bc[0][t][lane * NI], *Ct = &st.bc[1][t][lane * NI];
+#pragma unroll
+            for (int i = 0; i < NI; i += 4) {
+                float bn[4], cn[4];
+                if constexpr (sizeof(T) == 2) {
+                    const uint2 ub = *reinterpret_cast<const uint2*>(Bt + i), uc = *reinterpret_cast<const uint2*>(Ct + i);
+                    const float2 b0 = Elem<__nv_bfloat16>::unpack2(ub.x), b1 = Elem<__nv_bfloat16>::unpack2(ub.y);
+                    const float2 c0_ = Elem<__nv_bfloat16>::unpack2(uc.x), c1_ = Elem<__nv_bfloat16>::unpack2(uc.y);
+                    bn[0] = b0.x; bn[1] = b0.y; bn[2] = b1.x; bn[3] = b1.y;
+                    cn[0] = c0_.x; cn[1] = c0_.y; cn[2] = c1_.x; cn[3] = c1_.y;
+                } else {
+                    const float4 vb = *reinterpret_cast<const float4*>(Bt + i), vc = *reinterpret_cast<const float4*>(Ct + i);
+                    bn[0] = vb.x; bn[1] = vb.y; bn[2] = vb.z; bn[3] = vb.w;
+                    cn[0] = vc.x; cn[1] = vc.y; cn[2] = vc.z; cn[3] = vc.w;
+                }
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    S_[i + e] = fmaf(decay_of<T>(dl, a[i + e]), S_[i + e], dx * bn[e]);
+                    y = fmaf(S_[i + e], cn[e], y);
+                }
+            }
+#pragma unroll
+            for (int o = LP / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xFFFFFFFFu, y, o);
+            if (lane == 0) sm.y[t][ch] = fmaf(Dc, x, y);
+        }
+        __syncthreads();
+        // gate and store, two channels per thread
+        for (int i = tid; i < nt * (CH / 2); i += kThreads) {
+            const int t = i / (CH / 2), k = (i - t * (CH / 2)) * 2;
+            if (c0 + k >= p.inner) continue;
+            const float v0 = sm.y[t][k] * silu_for<T>(Elem<T>::to_f(st.z[t][k])), v1 = sm.y[t][k + 1] * silu_for<T>(Elem<T>::to_f(st.z[t][k + 1]));
+            T* dst = out + (m0 + t0 + t) * p.ldo + c0 + k;
+            if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = Elem<__nv_bfloat16>::pack2(v0, v1);
+            else *reinterpret_cast<float2*>(dst) = make_float2(v0, v1);
+        }
+        __syncthreads();           // the stage after next is refilled at the top
+    }
+#pragma unroll
+    for (int i = 0; i < NI; i += 4)
+        if (live && lane * NI + i < p.N) *reinterpret_cast<float4*>(sp + i) = make_float4(S_[i], S_[i + 1], S_[i + 2], S_[i + 3]);
+}
+
+// One token per sequence, step sizes included: grid (ceil(inner / kCh), B).  The LP lanes of a channel share its row of W_dt.
+template <typename T, int LP, int NI>
+__global__ void __launch_bounds__(kThreads)
+selective_step_kernel(ScanParams p, const T* __restrict__ proj, const T* __restrict__ xc, const T* __restrict__ xdbl, const T* __restrict__ w_dt, float* __restrict__ state,
+                      T* __restrict__ out) {
+    constexpr int CH = kThreads / LP;
+    extern __shared__ __align__(16) uint8_t raw[];
+    float* row = reinterpret_cast<float*>(raw);        // [rank | B | C] of this token
+    const int tid = threadIdx.x, lane = tid % LP, b = blockIdx.y, c = blockIdx.x * CH + tid / LP, cc = min(c, p.inner - 1);
+    const bool live = c < p.inner;
+    float a[NI];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        const int n = lane * NI + i;
+        a[i] = n < p.N ? __ldg(p.A + static_cast<long long>(cc) * p.N + n) : 0.f;
+    }
+    const float bias = __ldg(p.dt_bias + cc), Dc = __ldg(p.D + cc);
+    constexpr int kAhead = 4;                          // pieces of W_dt fetched before the wait
+    const int n8 = p.rank / 8;
+    const T* wr = w_dt + static_cast<long long>(cc) * p.rank;
+    Raw8<T> w[kAhead];
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i)
+        if (lane + i * LP < n8) w[i].load(wr + (lane + i * LP) * 8);
+    pdl_begin();
+    const int pos = p.pos[b], slot = p.slots ? p.slots[b] : b;
+    float* sp = state + (static_cast<long long>(slot) * p.inner + cc) * p.N + lane * NI;
+    float S_[NI];
+#pragma unroll
+    for (int i = 0; i < NI; i += 4) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (pos > 0 && lane * NI + i < p.N) v = *reinterpret_cast<const float4*>(sp + i);
+        S_[i] = v.x; S_[i + 1] = v.y; S_[i + 2] = v.z; S_[i + 3] = v.w;
+    }
+    const float x = Elem<T>::to_f(xc[static_cast<long long>(b) * p.inner + cc]), z = Elem<T>::to_f(proj[b * p.ldp + p.inner + cc]);
+    for (int i = tid; i < p.rank + 2 * p.N; i += kThreads) row[i] = Elem<T>::to_f(xdbl[b * p.ldx + i]);
+    __syncthreads();
+    float d = 0.f;
+    auto dot8 = [&](const float (&wv)[8], int k) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) d = fmaf(wv[e], row[k * 8 + e], d);
+    };
+#pragma unroll
+    for (int i = 0; i < kAhead; ++i)
+        if (lane + i * LP < n8) { float wv[8]; w[i].get(wv); dot8(wv, lane + i * LP); }
+    for (int k = lane + kAhead * LP; k < n8; k += LP) { float wv[8]; load8(wr + k * 8, wv); dot8(wv, k); }
+#pragma unroll
+    for (int o = LP / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xFFFFFFFFu, d, o);
+    d = softplus_for<T>(d + bias);
+    const float dx = d * x, dl = decay_dt<T>(d);
+    const float *Bn = row + p.rank + lane * NI, *Cn = Bn + p.N;
+    float y = 0.f;
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {
+        if (lane * NI + i < p.N) {
+            S_[i] = fmaf(decay_of<T>(dl, a[i]), S_[i], dx * Bn[i]);
+            y = fmaf(S_[i], Cn[i], y);
+        }
+    }
+#pragma unroll
+    for (int o = LP / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xFFFFFFFFu, y, o);
+    if (!live) return;
+#pragma unroll
+    for (int i = 0; i < NI; i += 4)
+        if (lane * NI + i < p.N) *reinterpret_cast<float4*>(sp + i) = make_float4(S_[i], S_[i + 1], S_[i + 2], S_[i + 3]);
+    if (lane == 0) out[b * p.ldo + c] = Elem<T>::from_f(fmaf(Dc, x, y) * silu_for<T>(z));
+}
+
+// Calls f(LP, NI) with compile-time sizes that hold N states; `wide`: few CTAs, so as many lanes per channel as make sense.
+template <typename F>
+int with_shape(int N, bool wide, F f) {
+    using std::integral_constant;
+    auto lanes = [&](auto ni) -> int {
+        const int need = (N + decltype(ni)::value - 1) / decltype(ni)::value;
+        if (need <= 2) return f(integral_constant<int, 2>{}, ni);
+        if (need <= 4) return f(integral_constant<int, 4>{}, ni);
+        if (need <= 8) return f(integral_constant<int, 8>{}, ni);
+        return f(integral_constant<int, 16>{}, ni);
+    };
+    if (N <= 64 && (wide || N == 8)) return lanes(integral_constant<int, 4>{});
+    if (N <= 128) return lanes(integral_constant<int, 8>{});
+    if (N <= 256) return f(integral_constant<int, 16>{}, integral_constant<int, 16>{});
+    return f(integral_constant<int, 16>{}, integral_constant<int, 32>{});
+}
+
+int product(cudaStream_t s, int dtype, const void* x, long long ldx, const void* w, long long ldw, void* out, long long ldo, int M, int N, int K, bool f32_out, int* status) {
+    if (dtype == VB200_F32)
+        return launch_linear_f32(s, static_cast<const float*>(x), ldx, static_cast<const float*>(w), ldw, nullptr, static_cast<float*>(out), ldo, M, N, K);
+    LinearParams p{};
+    p.x = x; p.ldx = ldx; p.w = w; p.ldw = ldw; p.out = out; p.ldo = ldo; p.M = M; p.N = N; p.K = K;
+    p.epilogue = f32_out ? VB200_EPI_F32 : VB200_EPI_BF16;
+    p.status = status;
+    return launch_linear(s, p);
+}
+
+}  // namespace
+
+SelectivePlan plan_selective(const vb200_selective_args& a) {
+    SelectivePlan pl{};
+    auto up = [](size_t x) { return (x + 255) / 256 * 256; };
+    const size_t esz = a.dtype == VB200_F32 ? 4 : 2, M = static_cast<size_t>(a.B) * a.T;
+    pl.dt_gemm = a.T > 1;
+    pl.conv_bytes = up(M * a.inner * esz);
+    pl.xdbl_bytes = up(M * (a.rank + 2 * a.N) * esz);
+    pl.dt_bytes = pl.dt_gemm ? up(M * a.inner * 4) : 0;
+    pl.total = pl.conv_bytes + pl.xdbl_bytes + pl.dt_bytes;
+    return pl;
+}
+
+int launch_selective(cudaStream_t s, const vb200_selective_args& a, const SelectivePlan& pl, int* status) {
+    uint8_t* ws = static_cast<uint8_t*>(a.workspace);
+    void *xc = ws, *xdbl = ws + pl.conv_bytes;
+    float* dt = reinterpret_cast<float*>(ws + pl.conv_bytes + pl.xdbl_bytes);
+    const int M = a.B * a.T, ldx = a.rank + 2 * a.N;
+    if (int rc = launch_causal_conv(s, ConvLaunch{a.dtype, a.B, a.T, a.inner, a.taps, a.proj, a.ldp, 0, a.conv_w, a.conv_b, a.slots, a.pos, a.conv_state, xc})) return rc;
+    if (int rc = product(s, a.dtype, xc, a.inner, a.w_x, a.inner, xdbl, ldx, M, ldx, a.inner, false, status)) return rc;
+    if (pl.dt_gemm)
+        if (int rc = product(s, a.dtype, xdbl, ldx, a.w_dt, a.rank, dt, a.inner, M, a.inner, a.rank, true, status)) return rc;
+    ScanParams p{};
+    p.B = a.B; p.T = a.T; p.inner = a.inner; p.N = a.N; p.rank = a.rank; p.ldp = a.ldp; p.ldx = ldx; p.ldo = a.ldo;
+    p.A = a.A; p.D = a.D; p.dt_bias = a.dt_bias; p.slots = a.slots; p.pos = a.pos;
+    const bool wide = static_cast<long long>(a.B) * a.inner * a.N < 4LL * 1024 * device_sm_count();
+    auto go = [&](auto tag) -> int {
+        using T = decltype(tag);
+        const T *proj = static_cast<const T*>(a.proj), *x = static_cast<const T*>(xc), *d = static_cast<const T*>(xdbl);
+        T* out = static_cast<T*>(a.out);
+        return with_shape(a.N, wide, [&](auto lp, auto ni) -> int {
+            constexpr int LP = decltype(lp)::value, NI = decltype(ni)::value, CH = kThreads / LP;
+            const dim3 grid(static_cast<unsigned>((a.inner + CH - 1) / CH), static_cast<unsigned>(a.B));
+            profile_mark_begin(s);
+            int rc;
+            if (a.T == 1) {
+                const size_t smem = sizeof(float) * ldx;
+                rc = allow_smem(selective_step_kernel<T, LP, NI>, smem);
+                if (rc == VB200_OK) rc = launch_pdl(selective_step_kernel<T, LP, NI>, grid, dim3(kThreads), smem, s, p, proj, x, d, static_cast<const T*>(a.w_dt), a.state, out);
+                note_selective_kernel("selective_step_kernel");
+            } else {
+                const size_t smem = sizeof(ScanTile<T, LP, NI>);
+                rc = allow_smem(selective_scan_kernel<T, LP, NI>, smem);
+                if (rc == VB200_OK) rc = launch_pdl(selective_scan_kernel<T, LP, NI>, grid, dim3(kThreads), smem, s, p, proj, x, d, dt, a.state, out);
+                note_selective_kernel("selective_scan_kernel");
+            }
+            profile_mark_end(s);
+            return rc;
+        });
+    };
+    return a.dtype == VB200_F32 ? go(float{}) : go(__nv_bfloat16{});
+}
+
+}  // namespace vb200

@@ -45,7 +45,7 @@ embed_sequence_kernel(const int* __restrict__ ids, int tokens, int dim, int voca
         if (embed_copy != nullptr) embed_copy[base + i] = v;
         if (add != nullptr) v += add[i];
         h[base + i] = v;
-        if (scaled_out != nullptr) scaled_out[base + i] = __float2bfloat16_rn(v * scale[i]);
+        if (scaled_out != nullptr) scaled_out[base + i] = __float2bfloat16_rn(scale != nullptr ? v * scale[i] : v);
     }
 }
 
@@ -75,7 +75,64 @@ rms_norm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, fl
     for (int i = threadIdx.x; i < dim; i += blockDim.x) o[i] = xr[i] * inv * w[i];
 }
 
+// One CTA per row.  The row to be normed stays in registers between the two passes (up to 256 * 4 * kNormVec columns; wider rows are
+// gathered twice).
+constexpr int kNormVec = 8;
+
+__global__ void __launch_bounds__(256)
+norm_add_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ w, int dim, int count, float eps, const __nv_bfloat16* __restrict__ rows,
+                const int* __restrict__ gather, int n_gather, const float* __restrict__ scale, __nv_bfloat16* __restrict__ copy_out) {
+    pdl_begin();
+    const long long m = blockIdx.x, base = m * dim;
+    const int nv = dim / 4;
+    __shared__ float part[8];
+    auto load = [&](int c) {
+        float4 v = y != nullptr ? *reinterpret_cast<const float4*>(y + base + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int k = 0; k < n_gather; ++k) {
+            const uint2 u = *reinterpret_cast<const uint2*>(rows + static_cast<long long>(gather[m * n_gather + k]) * dim + c * 4);
+            const float2 a = Elem<__nv_bfloat16>::unpack2(u.x), b = Elem<__nv_bfloat16>::unpack2(u.y);
+            v.x += a.x; v.y += a.y; v.z += b.x; v.w += b.y;
+        }
+        return v;
+    };
+    float4 v[kNormVec];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < kNormVec; ++i) {
+        const int c = threadIdx.x + i * 256;
+        if (c < nv) { v[i] = load(c); ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w; }
+    }
+    for (int c = threadIdx.x + kNormVec * 256; c < nv; c += 256) { const float4 t = load(c); ss += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w; }
+    const float inv = 1.0f / sqrtf(block_sum<8>(ss, part) / static_cast<float>(count) + eps);
+    auto finish = [&](int c, const float4& t) {
+        const float4 g = *reinterpret_cast<const float4*>(w + c * 4);
+        float4 h = *reinterpret_cast<const float4*>(x + base + c * 4);
+        h.x += t.x * inv * g.x; h.y += t.y * inv * g.y; h.z += t.z * inv * g.z; h.w += t.w * inv * g.w;
+        *reinterpret_cast<float4*>(x + base + c * 4) = h;
+        if (copy_out != nullptr) {
+            if (scale != nullptr) {
+                const float4 s4 = *reinterpret_cast<const float4*>(scale + c * 4);
+                h.x *= s4.x; h.y *= s4.y; h.z *= s4.z; h.w *= s4.w;
+            }
+            uint2 u;
+            u.x = Elem<__nv_bfloat16>::pack2(h.x, h.y); u.y = Elem<__nv_bfloat16>::pack2(h.z, h.w);
+            *reinterpret_cast<uint2*>(copy_out + base + c * 4) = u;
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < kNormVec; ++i) {
+        const int c = threadIdx.x + i * 256;
+        if (c < nv) finish(c, v[i]);
+    }
+    for (int c = threadIdx.x + kNormVec * 256; c < nv; c += 256) finish(c, load(c));
+}
+
 }  // namespace
+
+int launch_norm_add(cudaStream_t s, const vb200_norm_add_args& a) {
+    return launch_pdl(norm_add_kernel, dim3(static_cast<unsigned>(a.M)), dim3(256), 0, s, a.x, a.y, a.w, a.dim, a.count, a.eps, static_cast<const __nv_bfloat16*>(a.rows),
+                      a.gather, a.gather != nullptr ? a.n_gather : 0, a.scale, static_cast<__nv_bfloat16*>(a.copy_out));
+}
 
 int launch_embed_sequence(cudaStream_t s, const vb200_embed_args& a, int* status) {
     const dim3 grid(static_cast<unsigned>(a.B * a.T));

@@ -15,6 +15,14 @@ struct SsdParams {
     int slices, p4s, rows;      // scan kernel: slices of a head's columns, float4 columns per slice, state rows per pass
 };
 
+struct ConvTask {
+    int T, taps, channels;
+    long long ldp;
+    const float *conv_w, *conv_b;
+    const int *slots, *pos;
+    long long col;              // first convolved column of a projection row
+};
+
 constexpr int kConvTile = 32;   // tokens per CTA
 constexpr int kAhead = 8;       // tokens whose loads are in flight
 
@@ -33,14 +41,14 @@ __device__ __forceinline__ void store2(float* p, const float (&v)[2]) { *reinter
 // inputs ahead of the portion) and it alone writes it, after its own reads.
 template <typename T, int VEC, int TAPS>
 __global__ void __launch_bounds__(128)
-ssd_conv_kernel(SsdParams p, const T* __restrict__ proj, T* __restrict__ state, T* __restrict__ out) {
+ssd_conv_kernel(ConvTask p, const T* __restrict__ proj, T* __restrict__ state, T* __restrict__ out) {
     pdl_begin();
     const int c0 = (blockIdx.x * 128 + threadIdx.x) * VEC;
     if (c0 >= p.channels) return;
     const int b = blockIdx.z, t0 = blockIdx.y * kConvTile, t1 = min(p.T, t0 + kConvTile);
     const int taps = TAPS > 0 ? TAPS : p.taps;
     const int pos = p.pos[b], slot = p.slots ? p.slots[b] : b;
-    const T* in = proj + static_cast<long long>(b) * p.T * p.ldp + static_cast<long long>(p.H) * p.P + c0;
+    const T* in = proj + static_cast<long long>(b) * p.T * p.ldp + p.col + c0;
     T* st = state + static_cast<long long>(slot) * taps * p.channels + c0;
     T* o = out + static_cast<long long>(b) * p.T * p.channels + c0;
     auto fetch = [&](int t, float (&v)[VEC]) {           // the input of portion token t, which may lie ahead of the portion
@@ -272,6 +280,21 @@ SsdPlan plan_ssd(const vb200_ssd_args& a) {
     return pl;
 }
 
+int launch_causal_conv(cudaStream_t s, const ConvLaunch& c) {
+    const ConvTask p{c.T, c.taps, c.channels, c.ldp, c.w, c.b, c.slots, c.pos, c.col};
+    auto go = [&](auto tag) -> int {
+        using T = decltype(tag);
+        const bool vec = c.col % 2 == 0 && c.channels % 2 == 0 && c.ldp % 2 == 0;
+        auto conv = [&](auto kernel, int v) {
+            const dim3 grid(static_cast<unsigned>((c.channels + 128 * v - 1) / (128 * v)), static_cast<unsigned>((c.T + kConvTile - 1) / kConvTile), static_cast<unsigned>(c.B));
+            return launch_pdl(kernel, grid, dim3(128), 0, s, p, static_cast<const T*>(c.proj), static_cast<T*>(c.state), static_cast<T*>(c.out));
+        };
+        return vec ? (c.taps == 4 ? conv(ssd_conv_kernel<T, 2, 4>, 2) : conv(ssd_conv_kernel<T, 2, 0>, 2))
+                   : (c.taps == 4 ? conv(ssd_conv_kernel<T, 1, 4>, 1) : conv(ssd_conv_kernel<T, 1, 0>, 1));
+    };
+    return c.dtype == VB200_F32 ? go(float{}) : go(__nv_bfloat16{});
+}
+
 int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, int* status) {
     SsdParams p{};
     p.B = a.B; p.T = a.T; p.H = a.H; p.P = a.P; p.N = a.N; p.G = a.G; p.taps = a.taps; p.channels = pl.channels; p.Pp = pl.Pp;
@@ -295,16 +318,8 @@ int launch_ssd(cudaStream_t s, const vb200_ssd_args& a, const SsdPlan& pl, int* 
     auto go = [&](auto tag) -> int {
         using T = decltype(tag);
         const T* proj = static_cast<const T*>(a.proj);
-        {
-            const bool vec = (a.H * a.P) % 2 == 0 && p.channels % 2 == 0 && a.ldp % 2 == 0;
-            auto conv = [&](auto kernel, int v) {
-                const dim3 grid(static_cast<unsigned>((p.channels + 128 * v - 1) / (128 * v)), static_cast<unsigned>((a.T + kConvTile - 1) / kConvTile), static_cast<unsigned>(a.B));
-                return launch_pdl(kernel, grid, dim3(128), 0, s, p, proj, static_cast<T*>(a.conv_state), static_cast<T*>(xbc));
-            };
-            const int rc = vec ? (a.taps == 4 ? conv(ssd_conv_kernel<T, 2, 4>, 2) : conv(ssd_conv_kernel<T, 2, 0>, 2))
-                               : (a.taps == 4 ? conv(ssd_conv_kernel<T, 1, 4>, 1) : conv(ssd_conv_kernel<T, 1, 0>, 1));
-            if (rc) return rc;
-        }
+        if (int rc = launch_causal_conv(s, ConvLaunch{a.dtype, a.B, a.T, p.channels, a.taps, a.proj, a.ldp, static_cast<long long>(a.H) * a.P, a.conv_w, a.conv_b, a.slots,
+                                                      a.pos, a.conv_state, xbc})) return rc;
         if constexpr (sizeof(T) == 2) {
             if (pl.chunked) {
                 if (int rc = launch_ssd_chunks(s, a, pl, xbc, gated, states, status)) return rc;

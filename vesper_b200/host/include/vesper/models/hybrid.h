@@ -1,28 +1,39 @@
-// models::HybridLM -- decoders whose layers each name their sequence mixer and feed-forward in the configuration
-// (architecture "Nitenex"): token + bigram embedding, pre-norm layers (mixer, then dense squared-ReLU feed-forward),
-// a range of layers that may run several times with the same weights, RMSNorm and a tied output head.
+// models::HybridLM -- decoders whose layers each name their sequence mixer and feed-forward in the configuration.
+//   "Nitenex"  token + bigram embedding, pre-norm layers (latent attention or Mamba-2, then dense squared ReLU), a range of
+//              layers that may run several times with the same weights, RMSNorm and a tied output head
+//   "Zudisun"  layers that read the stream itself and norm their outputs (sigmoid attention with mixed heads or Mamba-1, then a
+//              ReLU-gated feed-forward with biases or a mixture of experts), RMSNorm and an output head of its own
 //
-// As in TransformerLM the residual stream is fp32, norms are deferred into the GEMMs around them, and decode steps
-// take positions from the device, so one step can be captured in a CUDA graph.  Each execution of a layer has a
+// As in TransformerLM the residual stream is fp32, norms ahead of a projection are deferred into the GEMMs around them, and
+// decode steps take positions from the device, so one step can be captured in a CUDA graph.  Each execution of a layer has a
 // cache or recurrent state of its own; sequences live in slots of those.
 #pragma once
 #include <vesper/models/language_model.h>
+#include <vesper/nn/feed_forward.h>
 #include <vesper/nn/sequence_mixer.h>
 
 namespace vesper::models {
 
+// What an architecture fixes about its blocks and its configuration does not say.
+struct HybridStyle {
+    bool norm_outputs = false;     // x += norm(sublayer(x)) instead of x += sublayer(norm(x))
+    bool tied_head = true;
+    nn::FeedForwardStyle feed_forward;
+};
+
 struct HybridConfig {
+    HybridStyle style;
     int64_t vocab = 0, width = 0;
     double eps = 1e-6;
     struct Layer {
         std::string type;          // mixer kind
         Json mixer;                // its sizes
-        int64_t ff = 0;            // feed-forward width, 0 = none
+        Json mlp;                  // its feed-forward, null = none
     };
     std::vector<Layer> layers;
     struct { int64_t start = 0, stop = 0, times = 0; } loop;               // times 0 = no loop
     struct { int64_t buckets = 0, mul_prev = 0, mul_cur = 0; } bigram;     // buckets 0 = none
-    static HybridConfig from_json(const Json& config);
+    static HybridConfig from_json(const Json& config, const HybridStyle& style);
 };
 
 class HybridLM : public LanguageModel {
@@ -72,6 +83,10 @@ private:
     void ensure_buffers(int64_t rows, const nn::MixerStep& step);
     // Runs the model on B x T ids with lengths in lens [B] (advanced); leaves the final residual stream, returns nothing.
     void run(const int32_t* ids, nn::MixerStep step, int32_t* lens);
+    void run_pre_norm(const nn::MixerStep& step);
+    void run_output_norm(const nn::MixerStep& step);
+    void copy_to_tap(size_t run, int64_t rows);
+    const float* step_vector(size_t run) const;         // of the loop pass that execution opens, or null
     void head(int64_t out_rows, int64_t first_row, int64_t row_stride);
     Tensor forward_rows(const Tensor& tokens, const std::vector<int64_t>& slots, int64_t start_pos, bool last_only);
 
@@ -80,7 +95,9 @@ private:
     int64_t max_len_, max_sequences_, dim_;        // dim_: width padded to a multiple of 8
     double norm_eps_;                               // eps and (via the norm weights) scale of norms over padded rows
     float norm_gain_ = 1.0f;
-    Tensor embed_, bigram_, final_norm_, loop_step_;
+    Tensor embed_, bigram_, final_norm_, loop_step_, head_;      // head_: undefined where tied
+    std::map<std::string, std::vector<int64_t>> shapes_;
+    int64_t shared_value_cols_ = 0;
     std::vector<std::unique_ptr<Layer>> layers_;
     std::vector<Run> runs_;
     std::vector<std::unique_ptr<nn::SequenceState>> states_;     // one per run

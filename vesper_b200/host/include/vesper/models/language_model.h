@@ -19,6 +19,7 @@ public:
 
     virtual int64_t vocab_size() const = 0;
     virtual int64_t max_seq_len() const = 0;
+    // -1: a size that the checkpoint's tensor gives.
     virtual std::map<std::string, std::vector<int64_t>> parameter_shapes() const = 0;
     // One parameter from host fp32 values.
     virtual void load_parameter(const std::string& name, const float* host_values, int64_t numel) = 0;

@@ -73,10 +73,15 @@ std::unique_ptr<LanguageModel> make_transformer(const Json& c, const LoadOptions
     return std::make_unique<TransformerLM>(t);
 }
 
+ModelFactory hybrid(const HybridStyle& style) {
+    return [style](const Json& c, const LoadOptions& o) -> std::unique_ptr<LanguageModel> { return std::make_unique<HybridLM>(HybridConfig::from_json(c, style), o); };
+}
+
 std::map<std::string, ModelFactory>& registry() {
     static std::map<std::string, ModelFactory> r = {
         {"TransformerLM", make_transformer},
-        {"Nitenex", [](const Json& c, const LoadOptions& o) -> std::unique_ptr<LanguageModel> { return std::make_unique<HybridLM>(HybridConfig::from_json(c), o); }},
+        {"Nitenex", hybrid(HybridStyle{})},
+        {"Zudisun", hybrid(HybridStyle{true, false, {nn::Activation::GatedRelu, true}})},
     };
     return r;
 }
@@ -104,7 +109,9 @@ std::unique_ptr<LanguageModel> load_model(const std::string& folder, const LoadO
     for (const auto& kv : model->parameter_shapes()) {
         auto it = ckpt.entries().find(kv.first);
         if (it == ckpt.entries().end()) throw std::runtime_error("checkpoint has no tensor named " + kv.first);
-        if (it->second.shape != kv.second) throw std::runtime_error("checkpoint tensor " + kv.first + " has another shape than the configuration gives");
+        bool same = it->second.shape.size() == kv.second.size();
+        for (size_t i = 0; same && i < kv.second.size(); ++i) same = kv.second[i] < 0 ? it->second.shape[i] > 0 : it->second.shape[i] == kv.second[i];
+        if (!same) throw std::runtime_error("checkpoint tensor " + kv.first + " has another shape than the configuration gives");
         const std::vector<float> v = ckpt.read(kv.first);
         model->load_parameter(kv.first, v.data(), static_cast<int64_t>(v.size()));
     }

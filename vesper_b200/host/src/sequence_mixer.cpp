@@ -1,7 +1,9 @@
-// nn::LatentAttention and nn::Mamba2 over the C ABI of vesper_b200_hybrid.h.
+// nn::LatentAttention, nn::SigmoidAttention, nn::Mamba2 and nn::Mamba1 over the C ABI of vesper_b200_hybrid.h.
 #include <vesper/nn/sequence_mixer.h>
 
 #include <vesper_b200_hybrid.h>
+
+#include <cuda_runtime.h>
 
 #include <algorithm>
 #include <cmath>
@@ -24,19 +26,34 @@ int64_t positive(const Json& m, const char* key) {
 
 }  // namespace
 
-void load_rows(Tensor& dst, int64_t row0, int64_t rows, int64_t cols, const float* host_values) {
-    const int64_t ld = dst.shape()[1];
-    Tensor part = dst.narrow(0, row0, rows);
-    if (dst.dtype() == DType::Float32) {
+namespace {
+// rows of `bytes` host bytes, to device rows `step` apart
+void copy_rows(char* dst, int64_t bytes, int64_t step, const void* src, int64_t rows) {
+    const size_t n = static_cast<size_t>(bytes);
+    const cudaError_t rc = cudaMemcpy2D(dst, n * static_cast<size_t>(step), src, n, n, static_cast<size_t>(rows), cudaMemcpyHostToDevice);
+    if (rc != cudaSuccess) throw std::runtime_error(std::string("loading a parameter: ") + cudaGetErrorString(rc));
+}
+}  // namespace
+
+void load_rows(Tensor& dst, int64_t row0, int64_t rows, int64_t cols, const float* host_values, int64_t step) {
+    const int64_t ld = dst.shape()[1], esz = dst.dtype() == DType::Float32 ? 4 : 2;
+    if (row0 < 0 || cols > ld || row0 + (rows - 1) * step >= dst.shape()[0]) throw std::runtime_error("load_rows: rows outside the matrix");
+    char* base = dst.data_ptr<char>() + row0 * ld * esz;
+    if (esz == 4) {
         std::vector<float> tmp(static_cast<size_t>(rows * ld), 0.0f);
         for (int64_t r = 0; r < rows; ++r) std::copy(host_values + r * cols, host_values + (r + 1) * cols, tmp.begin() + r * ld);
-        part.copy_from_host(tmp.data());
+        copy_rows(base, ld * esz, step, tmp.data(), rows);
     } else {
         std::vector<uint16_t> tmp(static_cast<size_t>(rows * ld), 0);
         for (int64_t r = 0; r < rows; ++r)
             for (int64_t c = 0; c < cols; ++c) tmp[static_cast<size_t>(r * ld + c)] = float_to_bf16(host_values[r * cols + c]);
-        part.copy_from_host(tmp.data());
+        copy_rows(base, ld * esz, step, tmp.data(), rows);
     }
+}
+
+void load_vector(Tensor& dst, int64_t first, int64_t n, const float* host_values, int64_t step) {
+    if (first < 0 || first + (n - 1) * step >= static_cast<int64_t>(dst.numel())) throw std::runtime_error("load_vector: outside the vector");
+    copy_rows(dst.data_ptr<char>() + first * 4, 4, step, host_values, n);
 }
 
 Tensor vector_from_host(const float* host_values, int64_t n) {
@@ -244,8 +261,231 @@ void Mamba2::forward(const MixerStep& st, SequenceState& state, Tensor& projecte
     check(vb200_ssd_forward(&x.a), "mamba2");
 }
 
+// ---- sigmoid attention with mixed heads ------------------------------------------------------------
+
+int64_t distance_bucket(int64_t n, int64_t rows, double reach) {
+    const int64_t half = rows / 2;
+    if (n < half) return n;
+    if (half == 0 || reach <= static_cast<double>(half)) return rows - 1;
+    // the quotient of two logarithms may round below an edge it lands on exactly
+    const double x = std::log(static_cast<double>(n) / static_cast<double>(half)) / std::log(reach / static_cast<double>(half)) * static_cast<double>(rows - half);
+    return std::min(rows - 1, half + static_cast<int64_t>(std::floor(x + 1e-9)));
+}
+
+SigmoidAttention::SigmoidAttention(const Json& m, int64_t width, int64_t width_ld, double eps, DType dtype) : SequenceMixer(width, width_ld, eps, dtype) {
+    heads_ = positive(m, "heads");
+    kv_heads_ = positive(m, "kv_heads");
+    dim_ = positive(m, "dim");
+    vdim_ = positive(m, "vdim");
+    if (heads_ % kv_heads_ != 0) throw std::runtime_error("configuration: heads must be divisible by kv_heads");
+    scale_ = m.at("scale").as_double();
+    reach_ = m.at("bias_max").as_double();
+    const Json& temp = m.get("q_temp");
+    if (!temp.is_null()) {
+        temp_coef_ = temp.at("coef").as_double();
+        temp_every_ = positive(temp, "every");
+    }
+    const Json& mix = m.get("v_mix");
+    value_mixing_ = !mix.is_null() && mix.as_bool();
+    proj_rows_ = heads_ * (dim_ + 1) + kv_heads_ * (dim_ + vdim_);
+    mixed_cols_ = heads_ * vdim_;
+    in_weight_ = zeros({proj_rows_, width_ld}, dtype, Device::CUDA);
+    out_weight_ = zeros({width_ld, mixed_ld()}, dtype, Device::CUDA);
+    talk_ = zeros({heads_, heads_}, DType::Float32, Device::CUDA);
+    bias_ = zeros({heads_, 1}, DType::Float32, Device::CUDA);
+}
+
+std::map<std::string, std::vector<int64_t>> SigmoidAttention::parameter_shapes() const {
+    std::map<std::string, std::vector<int64_t>> m = {{"q", {heads_ * dim_, width_}}, {"k", {kv_heads_ * dim_, width_}}, {"v", {kv_heads_ * vdim_, width_}}, {"g", {heads_, width_}},
+                                                     {"rel", {-1, heads_}}, {"talk", {heads_, heads_}}, {"pb", {heads_}}, {"o", {width_, heads_ * vdim_}}};
+    if (value_mixing_) m["vmix"] = {};
+    return m;
+}
+
+void SigmoidAttention::set_free_size(const std::string& name, int64_t numel) {
+    if (name == "rel") bias_rows_ = numel / heads_;
+}
+
+void SigmoidAttention::load_parameter(const std::string& name, const float* v) {
+    const int64_t q = heads_ * dim_, k = kv_heads_ * dim_, vv = kv_heads_ * vdim_;
+    if (name == "q") load_rows(in_weight_, 0, q, width_, v);
+    else if (name == "k") load_rows(in_weight_, q, k, width_, v);
+    else if (name == "v") load_rows(in_weight_, q + k, vv, width_, v);
+    else if (name == "g") load_rows(in_weight_, q + k + vv, heads_, width_, v);
+    else if (name == "o") load_rows(out_weight_, 0, width_, mixed_cols_, v);
+    else if (name == "vmix") lambda_ = v[0];
+    else if (name == "rel") { host_rel_.assign(v, v + bias_rows_ * heads_); fold_bias(); }
+    else if (name == "pb") { host_offset_.assign(v, v + heads_); fold_bias(); }
+    else if (name == "talk") { host_talk_.assign(v, v + heads_ * heads_); load_vector(talk_, 0, heads_ * heads_, v); fold_bias(); }
+    else throw std::runtime_error("SigmoidAttention: no parameter named " + name);
+}
+
+// What a score gets that depends on its head and distance only, [heads, distances]: the relative bias mixed like the scores, plus the
+// head's offset.  The last distance stands for all beyond it.
+void SigmoidAttention::fold_bias() {
+    if (host_rel_.empty() || host_talk_.empty() || host_offset_.empty()) return;
+    std::vector<int64_t> bucket;
+    for (int64_t n = 0;; ++n) {
+        bucket.push_back(distance_bucket(n, bias_rows_, reach_));
+        if (bucket.back() == bias_rows_ - 1) break;
+    }
+    const int64_t len = static_cast<int64_t>(bucket.size());
+    std::vector<float> folded(static_cast<size_t>(heads_ * len));
+    for (int64_t h = 0; h < heads_; ++h) {
+        std::vector<float> by_row(static_cast<size_t>(bias_rows_));
+        for (int64_t r = 0; r < bias_rows_; ++r) {
+            double x = host_offset_[static_cast<size_t>(h)];
+            for (int64_t g = 0; g < heads_; ++g) x += static_cast<double>(host_talk_[static_cast<size_t>(h * heads_ + g)]) * host_rel_[static_cast<size_t>(r * heads_ + g)];
+            by_row[static_cast<size_t>(r)] = static_cast<float>(x);
+        }
+        for (int64_t n = 0; n < len; ++n) folded[static_cast<size_t>(h * len + n)] = by_row[static_cast<size_t>(bucket[static_cast<size_t>(n)])];
+    }
+    bias_ = empty({heads_, len}, DType::Float32, Device::CUDA);
+    bias_.copy_from_host(folded.data());
+}
+
+std::unique_ptr<SequenceState> SigmoidAttention::make_state(int64_t slots, int64_t max_len) const {
+    auto st = std::make_unique<SequenceState>();
+    st->ring = zeros({slots, max_len, pad8(kv_heads_ * dim_)}, dtype_, Device::CUDA);
+    st->values = zeros({slots, max_len, pad8(kv_heads_ * vdim_)}, dtype_, Device::CUDA);
+    return st;
+}
+
+struct SigmoidAttention::Args {
+    vb200_sigattn_args a{};
+    Args(const SigmoidAttention& m, const MixerStep& st, int64_t cap) {
+        a.struct_size = sizeof(a);
+        a.device = m.in_weight_.device_index();
+        a.stream = current_stream();
+        a.dtype = m.dtype_ == DType::Float32 ? VB200_F32 : VB200_BF16;
+        a.B = static_cast<int>(st.B); a.T = static_cast<int>(st.T);
+        a.H = static_cast<int>(m.heads_); a.G = static_cast<int>(m.kv_heads_); a.dim = static_cast<int>(m.dim_); a.vdim = static_cast<int>(m.vdim_);
+        a.scale = static_cast<float>(m.scale_); a.eps = static_cast<float>(m.eps_);
+        a.temp_coef = static_cast<float>(m.temp_coef_); a.temp_every = static_cast<int>(std::min<int64_t>(m.temp_every_, INT32_MAX));
+        a.ldp = m.proj_ld(); a.ldo = m.mixed_ld();
+        a.ldk = pad8(m.kv_heads_ * m.dim_); a.ldv = pad8(m.kv_heads_ * m.vdim_);
+        a.talk = m.talk_.data_ptr<float>(); a.bias = m.bias_.data_ptr<float>(); a.n_bias = static_cast<int>(m.bias_.shape()[1]);
+        a.lambda = m.lambda_;
+        a.slots = st.slots; a.pos = st.pos;
+        a.cap = static_cast<int>(std::min<int64_t>(cap, INT32_MAX));
+        a.start_pos = static_cast<int>(st.start_pos);
+        a.max_len = static_cast<int>(std::min<int64_t>(st.max_len, INT32_MAX));
+    }
+};
+
+int64_t SigmoidAttention::workspace_bytes(const MixerStep& st) const {
+    const Args x(*this, st, INT32_MAX);
+    return static_cast<int64_t>(vb200_sigattn_workspace_bytes(&x.a));
+}
+
+void SigmoidAttention::forward(const MixerStep& st, SequenceState& state, Tensor& projected, Tensor& mixed) {
+    Args x(*this, st, state.ring.shape()[1]);
+    x.a.proj = projected.data_ptr<char>();
+    x.a.k_cache = state.ring.data_ptr<char>();
+    x.a.v_cache = state.values.data_ptr<char>();
+    x.a.out = mixed.data_ptr<char>();
+    x.a.workspace = st.workspace;
+    x.a.workspace_bytes = static_cast<size_t>(st.workspace_bytes);
+    if (value_mixing_) {
+        if (!st.values) throw std::runtime_error("SigmoidAttention: value mixing needs the step's shared values");
+        x.a.first_values = st.values->data;
+        x.a.value_role = st.values->filled ? 2 : 1;
+        st.values->filled = true;
+    }
+    check(vb200_sigattn_forward(&x.a), "sigmoid attention");
+}
+
+// ---- Mamba-1 -------------------------------------------------------------------------------------
+
+Mamba1::Mamba1(const Json& m, int64_t width, int64_t width_ld, double eps, DType dtype) : SequenceMixer(width, width_ld, eps, dtype) {
+    inner_ = positive(m, "inner");
+    state_ = positive(m, "state");
+    rank_ = positive(m, "dt_rank");
+    taps_ = positive(m, "conv");
+    inner8_ = pad8(inner_); state8_ = pad8(state_); rank8_ = pad8(rank_);
+    proj_rows_ = 2 * inner8_;
+    mixed_cols_ = inner_;
+    in_weight_ = zeros({proj_rows_, width_ld}, dtype, Device::CUDA);
+    out_weight_ = zeros({width_ld, mixed_ld()}, dtype, Device::CUDA);
+    w_x_ = zeros({rank8_ + 2 * state8_, inner8_}, dtype, Device::CUDA);
+    w_dt_ = zeros({inner8_, rank8_}, dtype, Device::CUDA);
+    conv_w_ = zeros({inner8_, taps_}, DType::Float32, Device::CUDA);
+    conv_b_ = zeros({inner8_}, DType::Float32, Device::CUDA);
+    dt_bias_ = zeros({inner8_}, DType::Float32, Device::CUDA);
+    a_ = zeros({inner8_, state8_}, DType::Float32, Device::CUDA);
+    d_ = zeros({inner8_}, DType::Float32, Device::CUDA);
+}
+
+std::map<std::string, std::vector<int64_t>> Mamba1::parameter_shapes() const {
+    return {{"in", {2 * inner_, width_}}, {"conv", {inner_, taps_}}, {"conv.b", {inner_}}, {"x", {rank_ + 2 * state_, inner_}}, {"dt", {inner_, rank_}}, {"dt.b", {inner_}},
+            {"A_log", {inner_, state_}}, {"D", {inner_}}, {"o", {width_, inner_}}};
+}
+
+void Mamba1::load_parameter(const std::string& name, const float* v) {
+    if (name == "in") {
+        load_rows(in_weight_, 0, inner_, width_, v);
+        load_rows(in_weight_, inner8_, inner_, width_, v + inner_ * width_);
+    } else if (name == "x") {
+        load_rows(w_x_, 0, rank_, inner_, v);
+        load_rows(w_x_, rank8_, state_, inner_, v + rank_ * inner_);
+        load_rows(w_x_, rank8_ + state8_, state_, inner_, v + (rank_ + state_) * inner_);
+    } else if (name == "A_log") {
+        std::vector<float> a(static_cast<size_t>(inner_ * state_));
+        for (size_t i = 0; i < a.size(); ++i) a[i] = static_cast<float>(-std::exp(static_cast<double>(v[i])));
+        load_rows(a_, 0, inner_, state_, a.data());
+    } else if (name == "conv") load_rows(conv_w_, 0, inner_, taps_, v);
+    else if (name == "conv.b") load_vector(conv_b_, 0, inner_, v);
+    else if (name == "dt") load_rows(w_dt_, 0, inner_, rank_, v);
+    else if (name == "dt.b") load_vector(dt_bias_, 0, inner_, v);
+    else if (name == "D") load_vector(d_, 0, inner_, v);
+    else if (name == "o") load_rows(out_weight_, 0, width_, inner_, v);
+    else throw std::runtime_error("Mamba1: no parameter named " + name);
+}
+
+std::unique_ptr<SequenceState> Mamba1::make_state(int64_t slots, int64_t) const {
+    auto st = std::make_unique<SequenceState>();
+    st->ring = zeros({slots, taps_, inner8_}, dtype_, Device::CUDA);
+    st->recurrent = zeros({slots, inner8_, state8_}, DType::Float32, Device::CUDA);
+    return st;
+}
+
+struct Mamba1::Args {
+    vb200_selective_args a{};
+    Args(const Mamba1& m, const MixerStep& st) {
+        a.struct_size = sizeof(a);
+        a.device = m.in_weight_.device_index();
+        a.stream = current_stream();
+        a.dtype = m.dtype_ == DType::Float32 ? VB200_F32 : VB200_BF16;
+        a.B = static_cast<int>(st.B); a.T = static_cast<int>(st.T); a.inner = static_cast<int>(m.inner8_); a.N = static_cast<int>(m.state8_);
+        a.rank = static_cast<int>(m.rank8_); a.taps = static_cast<int>(m.taps_);
+        a.ldp = m.proj_ld(); a.ldo = m.mixed_ld();
+        a.conv_w = m.conv_w_.data_ptr<float>(); a.conv_b = m.conv_b_.data_ptr<float>();
+        a.w_x = m.w_x_.data_ptr<char>(); a.w_dt = m.w_dt_.data_ptr<char>();
+        a.dt_bias = m.dt_bias_.data_ptr<float>(); a.A = m.a_.data_ptr<float>(); a.D = m.d_.data_ptr<float>();
+        a.slots = st.slots; a.pos = st.pos;
+    }
+};
+
+int64_t Mamba1::workspace_bytes(const MixerStep& st) const {
+    const Args x(*this, st);
+    return static_cast<int64_t>(vb200_selective_workspace_bytes(&x.a));
+}
+
+void Mamba1::forward(const MixerStep& st, SequenceState& state, Tensor& projected, Tensor& mixed) {
+    Args x(*this, st);
+    x.a.proj = projected.data_ptr<char>();
+    x.a.conv_state = state.ring.data_ptr<char>();
+    x.a.state = state.recurrent.data_ptr<float>();
+    x.a.out = mixed.data_ptr<char>();
+    x.a.workspace = st.workspace;
+    x.a.workspace_bytes = static_cast<size_t>(st.workspace_bytes);
+    check(vb200_selective_forward(&x.a), "mamba1");
+}
+
 std::unique_ptr<SequenceMixer> make_mixer(const std::string& type, const Json& mixer, int64_t width, int64_t width_ld, double eps, DType dtype) {
     if (type == "latent_attention") return std::make_unique<LatentAttention>(mixer, width, width_ld, eps, dtype);
+    if (type == "attention") return std::make_unique<SigmoidAttention>(mixer, width, width_ld, eps, dtype);
+    if (type == "mamba1") return std::make_unique<Mamba1>(mixer, width, width_ld, eps, dtype);
     if (type == "mamba2") return std::make_unique<Mamba2>(mixer, width, width_ld, eps, dtype);
     throw std::runtime_error("configuration: no sequence mixer of type '" + type + "'");
 }
