@@ -29,10 +29,11 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool vali
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// exp(dt * a): accurate in the fp32 form; where activations are bf16 the base-2 instruction (2 ulp), dt then carries log2 e
-template <typename T> __device__ __forceinline__ float decay_of(float dt, float a) {
-    if constexpr (sizeof(T) == 4) return expf(dt * a);
-    else return fast_exp2(dt * a);
+// exp(dt * a) * s + u.  fp32 form: s + (exp(dt * a) - 1) * s, because the rounding of a factor close to one would add up over a long
+// memory.  Where activations are bf16: the base-2 instruction (2 ulp), dt then carries log2 e.
+template <typename T> __device__ __forceinline__ float decayed(float s, float dt, float a, float u) {
+    if constexpr (sizeof(T) == 4) return s + fmaf(expm1f(dt * a), s, u);
+    else return fmaf(fast_exp2(dt * a), s, u);
 }
 template <typename T> __device__ __forceinline__ float decay_dt(float dt) { return sizeof(T) == 4 ? dt : dt * kLog2e; }
 
@@ -148,7 +149,7 @@ selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
                 }
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    S_[i + e] = fmaf(decay_of<T>(dl, a[i + e]), S_[i + e], dx * bn[e]);
+                    S_[i + e] = decayed<T>(S_[i + e], dl, a[i + e], dx * bn[e]);
                     y = fmaf(S_[i + e], cn[e], y);
                 }
             }
@@ -228,7 +229,7 @@ selective_step_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
 #pragma unroll
     for (int i = 0; i < NI; ++i) {
         if (lane * NI + i < p.N) {
-            S_[i] = fmaf(decay_of<T>(dl, a[i]), S_[i], dx * Bn[i]);
+            S_[i] = decayed<T>(S_[i], dl, a[i], dx * Bn[i]);
             y = fmaf(S_[i], Cn[i], y);
         }
     }

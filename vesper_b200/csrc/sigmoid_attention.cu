@@ -37,7 +37,7 @@ sig_append_kernel(SigParams p, const T* __restrict__ proj, T* __restrict__ kc, T
     const int kcols = p.G * p.dim, vcols = p.G * p.vdim;
     const bool fits = pos < p.cap;
     if (!fits && threadIdx.x == 0) atomicCAS(p.status, 0, (2 << 24) | b);
-    float temp = p.scale;
+    float temp = p.scale * (sizeof(QT) == 2 ? -kLog2e : 1.0f);       // the tensor-core kernels compute 2^(-score log2 e)
     if (p.temp_every > 0) temp *= 1.0f + p.temp_coef * logf(static_cast<float>((pos + 1) / p.temp_every) + 1.0f);
     for (int h = warp; h < p.H + p.G; h += 8) {
         const T* x = src + h * p.dim;     // the key heads follow the query heads

@@ -1,5 +1,266 @@
+// Prompt attention of sigmoid-attention layers on sm_100a.
+//
+//   O_i[h] = gate * sum_{j <= i} sigmoid(s_ij) v_j[group of h],   s_ij = q'_i[h] . k_j + bias[h, min(i - j, last)]
+//
+// q' holds the mixed queries of a head against the concatenated keys of all groups (kd = G * dim columns), already times -log2(e):
+// sigmoid(s) = 1 / (1 + 2^(s')).  Weights are not normalised, so there is no running maximum, no correction of O, and two warps
+// can share a row: nothing has to be reduced over keys.
+//
+// One CTA per 128 query rows of one (batch, head), one CTA per SM; keys in blocks of 128.
+//   warps 0-7  weights and epilogue: warps w and w + 4 own the same 32 rows (TMEM lanes), and 64 keys of a block each
+//   warp  8    TMA producer: Q once, then one ring of [128 rows x 64 columns] boxes that K and V share in the order of their use
+//   warp  9    tcgen05.mma issuer, TMEM owner
+// TMEM (512 columns): S0 [0, 128) S1 [128, 256) O [256, 256 + vdim).  QK of block j+1 is issued before PV of block j.  The weights stay
+// fp32-class in the second product: each half of a block is packed over its own 64 columns of S as bf16 hi (32 columns) and lo (32).
+// Two elements share one reciprocal: 1/a = b * (1/(ab)); 2^(s') is cut at 2^60, which leaves a weight below 1e-18.
 #include "hybrid.cuh"
+
 namespace vb200 {
-bool sig_prefill_sm100_supported(const vb200_sigattn_args&) { return false; }
-int launch_sig_prefill_sm100(cudaStream_t, const vb200_sigattn_args&, const SigPlan&, const void*, int*) { return VB200_ERR_UNSUPPORTED; }
+namespace {
+
+constexpr int kRows = 128, kKeys = 128;
+constexpr int kBox = 128 * 128;               // [128 rows x 64 columns]
+constexpr int kMaxSlots = 12;
+constexpr int kWeightThreads = 256;
+constexpr int kThreads = kWeightThreads + 64;
+constexpr float kCut = 60.0f;
+
+struct SigMaps { CUtensorMap q, k, v; };
+
+struct SigTileParams {
+    int T, start_pos, vdim, R, n_bias, gate_col;
+    int ks, nb_k, nb_v, slots_ring;           // 16-column steps of kd, 64-column boxes, ring slots
+    const float* bias;
+    const __nv_bfloat16* proj;
+    __nv_bfloat16* out;
+    long long ldp, ldo;
+    const int* slots;
+    int* status;
+};
+
+struct SigBars {
+    uint64_t q_full, full[kMaxSlots], empty[kMaxSlots], s_full[2], p_ready[2], o_done, drain;
+    uint32_t tmem;
+    int abort_flag;
+};
+
+__device__ __forceinline__ float rcp_approx(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
 }
+
+__global__ void __launch_bounds__(kThreads, 1)
+sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) {
+    extern __shared__ __align__(1024) uint8_t smem[];
+    __shared__ SigBars bar;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int r0 = static_cast<int>(gridDim.z - 1 - blockIdx.z) * kRows, h = blockIdx.x, b = blockIdx.y;      // tiles with most keys first
+    const int last_key = p.start_pos + min(r0 + kRows, p.T) - 1, n_blk = last_key / kKeys + 1;
+    uint8_t* q_smem = smem;
+    uint8_t* ring = q_smem + p.nb_k * kBox;
+    const WaitCtx ctx{&bar.abort_flag, p.status};
+
+    if (threadIdx.x == 0) {
+        bar.abort_flag = 0;
+        mbar_init(&bar.q_full, 1);
+        for (int i = 0; i < kMaxSlots; ++i) { mbar_init(&bar.full[i], 1); mbar_init(&bar.empty[i], 1); }
+        for (int i = 0; i < 2; ++i) { mbar_init(&bar.s_full[i], 1); mbar_init(&bar.p_ready[i], kWeightThreads); }
+        mbar_init(&bar.o_done, 1);
+        mbar_init(&bar.drain, 1);
+        mbar_fence_init();
+        if ((smem_u32(smem) & 1023) != 0) { bar.abort_flag = 1; atomicCAS(p.status, 0, (3 << 24) | 0x3); }      // the swizzle needs 1024-byte tiles
+    }
+    if (warp == 9) { tmem_alloc(&bar.tmem, 512); tmem_relinquish(); }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = bar.tmem;
+    const bool dead = *static_cast<volatile int*>(&bar.abort_flag) != 0;
+    pdl_begin();
+
+    if (dead) {
+    } else if (warp == 8) {
+        if (lane == 0) {
+            const int slot = p.slots ? p.slots[b] : b;
+            mbar_arrive_expect_tx(&bar.q_full, p.nb_k * kBox);
+            for (int i = 0; i < p.nb_k; ++i) tma_load_4d(q_smem + i * kBox, &maps.q, &bar.q_full, i * 64, h, r0, b);
+            bool ok = true;
+            int n = 0;
+            auto load = [&](const CUtensorMap* m, int col, int head, int key) {
+                const int s = n % p.slots_ring, round = n / p.slots_ring;
+                if (round > 0) ok = ok && mbar_wait(&bar.empty[s], (round - 1) & 1, ctx, 0xD1);
+                if (!ok) return;
+                mbar_arrive_expect_tx(&bar.full[s], kBox);
+                tma_load_4d(ring + s * kBox, m, &bar.full[s], col, head, key, slot);
+                ++n;
+            };
+            for (int i = 0; i < p.nb_k && ok; ++i) load(&maps.k, i * 64, 0, 0);
+            for (int j = 0; j < n_blk && ok; ++j) {
+                if (j + 1 < n_blk)
+                    for (int i = 0; i < p.nb_k && ok; ++i) load(&maps.k, i * 64, 0, (j + 1) * kKeys);
+                for (int i = 0; i < p.nb_v && ok; ++i) load(&maps.v, i * 64, h / p.R, j * kKeys);
+            }
+        }
+    } else if (warp == 9) {
+        if (lane == 0) {
+            const uint32_t idesc_qk = make_idesc_f16(1, 0, 0, kRows, kKeys);
+            const uint32_t q_addr = smem_u32(q_smem), ring_addr = smem_u32(ring);
+            bool ok = mbar_wait(&bar.q_full, 0, ctx, 0xD2);
+            int n = 0;
+            auto take = [&]() -> uint32_t {              // the next box of the ring
+                const int s = n % p.slots_ring;
+                ok = ok && mbar_wait(&bar.full[s], (n / p.slots_ring) & 1, ctx, 0xD3);
+                tc_fence_after();
+                return ring_addr + s * kBox;
+            };
+            auto give = [&]() { umma_commit(&bar.empty[n % p.slots_ring]); ++n; };
+            auto issue_qk = [&](int j) {
+                const uint32_t d = tmem + (j & 1) * kKeys;
+                for (int i = 0; i < p.nb_k; ++i) {
+                    const uint32_t kb = take();
+                    if (!ok) return;
+                    const int steps = min(4, p.ks - i * 4);
+                    for (int kk = 0; kk < steps; ++kk)
+                        umma_ss(d, make_smem_desc_sw128(q_addr + i * kBox + kk * 32, 16, 1024), make_smem_desc_sw128(kb + kk * 32, 16, 1024), idesc_qk, (i | kk) ? 1u : 0u);
+                    give();
+                }
+                umma_commit(&bar.s_full[j & 1]);
+            };
+            if (ok) issue_qk(0);
+            for (int j = 0; j < n_blk && ok; ++j) {
+                if (j + 1 < n_blk) issue_qk(j + 1);      // its S held the weights of block j-1, whose product was issued before
+                if (!ok) break;
+                ok = mbar_wait(&bar.p_ready[j & 1], (j >> 1) & 1, ctx, 0xD4);
+                if (!ok) break;
+                tc_fence_after();
+                const uint32_t a = tmem + (j & 1) * kKeys;
+                for (int i = 0; i < p.nb_v; ++i) {
+                    const uint32_t vb = take();
+                    if (!ok) break;
+                    const uint32_t idesc_pv = make_idesc_f16(1, 0, 1, kRows, min(64, (p.vdim - i * 64 + 15) / 16 * 16));
+                    for (int half = 0; half < 2; ++half)         // hi, lo
+                        for (int kk = 0; kk < kKeys / 16; ++kk)
+                            umma_ts(tmem + 2 * kKeys + i * 64, a + (kk >> 2) * 64 + half * 32 + (kk & 3) * 8, make_smem_desc_sw128(vb + kk * 2048, kBox, 1024), idesc_pv,
+                                    (j | half | kk) ? 1u : 0u);
+                    give();
+                }
+            }
+            if (ok) umma_commit(&bar.o_done);
+            umma_commit(&bar.drain);                     // nothing may be in flight when TMEM is freed
+            mbar_wait(&bar.drain, 0, ctx, 0xD5);
+        }
+    } else {
+        const int r = (warp & 3) * 32 + lane, half = warp >> 2;          // row of the tile = TMEM lane; half of a block's keys
+        const uint32_t lane_base = static_cast<uint32_t>((warp & 3) * 32) << 16;
+        const int me = p.start_pos + r0 + r;
+        const float* bias = p.bias + static_cast<long long>(h) * p.n_bias;
+        const float far = -kLog2e * __ldg(bias + p.n_bias - 1);
+        bool ok = true;
+        for (int j = 0; j < n_blk; ++j) {
+            ok = mbar_wait_warp(&bar.s_full[j & 1], (j >> 1) & 1, ctx, 0xD6);
+            if (!ok) break;
+            tc_fence_after();
+            const uint32_t s_addr = tmem + lane_base + (j & 1) * kKeys + half * 64;
+            const int k0 = j * kKeys + half * 64;
+            const int nearest = p.start_pos + r0 + (warp & 3) * 32 - (k0 + 63);         // smallest distance this warp meets in its half
+            uint32_t s[2][32];
+            tmem_ld32(s_addr, s[0]);
+            tmem_ld32(s_addr + 32, s[1]);
+            tmem_ld_wait();
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+                if (nearest >= p.n_bias - 1) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) s[c][i] = __float_as_uint(__uint_as_float(s[c][i]) + far);
+                } else {
+                    const int n0 = me - (k0 + c * 32);
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) {
+                        const int n = n0 - i;
+                        const float bv = __ldg(bias + min(max(n, 0), p.n_bias - 1));
+                        s[c][i] = __float_as_uint(fmaf(bv, -kLog2e, __uint_as_float(s[c][i])));
+                    }
+                }
+                uint32_t hi[16], lo[16];
+                const bool diagonal = nearest < 0;
+#pragma unroll
+                for (int i = 0; i < 16; ++i) {
+                    const float a = 1.0f + fast_exp2(fminf(__uint_as_float(s[c][2 * i]), kCut)), d = 1.0f + fast_exp2(fminf(__uint_as_float(s[c][2 * i + 1]), kCut));
+                    const float inv = rcp_approx(a * d);
+                    float w0 = inv * d, w1 = inv * a;
+                    if (diagonal) {
+                        const int n = me - (k0 + c * 32 + 2 * i);
+                        if (n < 0) w0 = 0.f;
+                        if (n < 1) w1 = 0.f;
+                    }
+                    split_hi_lo(w0, w1, hi[i], lo[i]);
+                }
+                tmem_st16(s_addr + c * 16, hi);
+                tmem_st16(s_addr + 32 + c * 16, lo);
+            }
+            tmem_st_wait();
+            tc_fence_before();
+            mbar_arrive(&bar.p_ready[j & 1]);
+        }
+        if (ok) ok = mbar_wait_warp(&bar.o_done, 0, ctx, 0xD7);
+        if (ok) {
+            tc_fence_after();
+            const bool live = r0 + r < p.T;
+            const long long m = static_cast<long long>(b) * p.T + r0 + r;
+            float gate = 0.f;
+            if (live) gate = 1.0f / (1.0f + __expf(-__bfloat162float(p.proj[m * p.ldp + p.gate_col + h])));
+            __nv_bfloat16* orow = p.out + m * p.ldo + static_cast<long long>(h) * p.vdim;
+            for (int c = half * 32; c < p.vdim; c += 64) {
+                uint32_t o[32];
+                tmem_ld32(tmem + lane_base + 2 * kKeys + c, o);
+                tmem_ld_wait();
+                if (live) {
+#pragma unroll
+                    for (int v = 0; v < 4; ++v) {
+                        if (c + v * 8 >= p.vdim) break;
+                        float f[8];
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(o[v * 8 + e]) * gate;
+                        store8(orow + c + v * 8, f);
+                    }
+                }
+            }
+        }
+        tc_fence_before();
+    }
+    __syncthreads();
+    if (warp == 9) tmem_dealloc(tmem, 512);
+    abort_linger(&bar.abort_flag);
+}
+
+}  // namespace
+
+bool sig_prefill_sm100_supported(const vb200_sigattn_args& a) {
+    return a.dtype == VB200_BF16 && a.G * a.dim <= 512 && a.vdim % 8 == 0 && a.vdim <= 256 && a.ldo % 8 == 0 && a.T <= 65535 * kRows &&
+           reinterpret_cast<uintptr_t>(a.out) % 16 == 0;
+}
+
+int launch_sig_prefill_sm100(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& pl, const void* q, int* status) {
+    const int kd = a.G * a.dim, n_ctx = a.start_pos + a.T, slots = a.slots ? 1 << 20 : a.B;      // a row's slot is the caller's promise
+    if (n_ctx > a.cap) return set_detail(VB200_ERR_INVALID_ARG, "vb200_sigattn_forward: the prompt does not fit the cache");
+    SigMaps maps;
+    if (int rc = make_map_4d(&maps.q, q, kd, a.H, a.T, a.B, pl.qld, static_cast<long long>(a.H) * pl.qld, static_cast<long long>(a.T) * a.H * pl.qld, kRows)) return rc;
+    if (int rc = make_map_4d(&maps.k, a.k_cache, kd, 1, n_ctx, slots, a.ldk, a.ldk, a.ldk * a.cap, kKeys)) return rc;
+    if (int rc = make_map_4d(&maps.v, a.v_cache, a.vdim, a.G, n_ctx, slots, a.vdim, a.ldv, a.ldv * a.cap, kKeys)) return rc;
+    SigTileParams p{};
+    p.T = a.T; p.start_pos = a.start_pos; p.vdim = a.vdim; p.R = a.H / a.G; p.n_bias = a.n_bias;
+    p.gate_col = a.H * a.dim + a.G * (a.dim + a.vdim);
+    p.ks = (kd + 15) / 16; p.nb_k = (kd + 63) / 64; p.nb_v = (a.vdim + 63) / 64;
+    p.bias = a.bias; p.proj = static_cast<const __nv_bfloat16*>(a.proj); p.out = static_cast<__nv_bfloat16*>(a.out);
+    p.ldp = a.ldp; p.ldo = a.ldo; p.slots = a.slots; p.status = status;
+    p.slots_ring = (208 * 1024 - p.nb_k * kBox) / kBox;
+    if (p.slots_ring > kMaxSlots) p.slots_ring = kMaxSlots;
+    size_t smem = static_cast<size_t>(p.nb_k + p.slots_ring) * kBox;
+    if (smem < 120 * 1024) smem = 120 * 1024;            // never a second CTA on an SM: it would find no TMEM
+    if (int rc = allow_smem(sig_prefill_sm100_kernel, smem)) return rc;
+    return launch_pdl(sig_prefill_sm100_kernel, dim3(static_cast<unsigned>(a.H), static_cast<unsigned>(a.B), static_cast<unsigned>((a.T + kRows - 1) / kRows)), dim3(kThreads), smem, s,
+                      maps, p);
+}
+
+}  // namespace vb200
