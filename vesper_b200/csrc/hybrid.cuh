@@ -104,6 +104,7 @@ int launch_sigattn(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& p
 bool sig_prefill_sm100_supported(const vb200_sigattn_args& a);                                                                  // sigmoid_prefill_sm100.cu
 int launch_sig_prefill_sm100(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& pl, const void* q, int* status);
 bool sig_decode_mma_supported(const vb200_sigattn_args& a);                                                                     // sigmoid_decode_mma.cu
+int sig_decode_ctas_per_sm(const vb200_sigattn_args& a);
 int launch_sig_decode_mma(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& pl, const void* q, float* part, int* status);
 void note_sigattn_kernel(const char* name);
 

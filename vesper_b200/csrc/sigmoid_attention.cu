@@ -178,9 +178,8 @@ SigPlan plan_sigattn(const vb200_sigattn_args& a) {
     pl.splits = 1;
     if (a.T == 1) {
         const int n_max = a.max_len > 0 && a.max_len < a.cap ? a.max_len : a.cap;
-        // tensor cores: one CTA per SM with 16 heads each; CUDA cores: one query of four warps per CTA
         const long long units = static_cast<long long>(a.B) * (pl.mma ? (a.H + 15) / 16 : a.H);
-        long long want = (pl.mma ? 1LL : 4LL) * device_sm_count() / units;
+        long long want = (pl.mma ? sig_decode_ctas_per_sm(a) : 4LL) * device_sm_count() / units;         // rounded down: a few CTAs more would be a second wave
         const long long most = (n_max + 63) / 64;
         if (want > most) want = most;
         if (want > 128) want = 128;
