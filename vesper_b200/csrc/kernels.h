@@ -176,8 +176,15 @@ struct LinearParams {
     float rms_eps;
     const float* row_scale;          // [M] or null
     const float* addend;             // += epilogue: a second fp32 matrix [M, N] (row stride ldo) added with it, or null
+    // Grouped product (launch_linear_grouped): the rows of x are sorted by group, group g has weights w + g * group_rows rows, and the device
+    // lists the 128-row tiles: {first row, end of the group's rows, group, 0}; group_rows rows of W per group, N <= group_rows
+    const int4* group_tiles;
+    const int* group_tile_count;     // device: tiles in the list
+    int group_tile_max;              // host: most tiles the list can hold
+    int groups, group_rows;
 };
 int launch_linear(cudaStream_t s, const LinearParams& p);
+int launch_linear_grouped(cudaStream_t s, const LinearParams& p);      // VB200_EPI_BF16 and VB200_EPI_SWIGLU
 // inv_rms[m] = 1 / sqrt(mean(h[m,:]^2) + eps)
 int launch_row_inv_rms(cudaStream_t s, const float* h, long long ld, float* inv_rms, int M, int dim, float eps);
 

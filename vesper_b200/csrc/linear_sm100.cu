@@ -196,7 +196,8 @@ struct WideCfg {
     static_assert(kTmemCols <= 512 && (kTmemCols & (kTmemCols - 1)) == 0, "TMEM allocation is a power of two <= 512");
 };
 
-template <int BN, int EPI>
+// GROUPED: rows sorted by group, each group with weights of its own; the row tiles come from a device list.
+template <int BN, int EPI, bool GROUPED = false>
 __global__ void __launch_bounds__(kThreads, 1)
 linear_wide_kernel(const __grid_constant__ LinearMaps maps, LinearParams p) {
     using C = WideCfg<BN>;
@@ -211,9 +212,8 @@ linear_wide_kernel(const __grid_constant__ LinearMaps maps, LinearParams p) {
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int m_tiles = (p.M + kTileA - 1) / kTileA;
+    int m_tiles = (p.M + kTileA - 1) / kTileA;
     const int n_tiles = (p.N + BN - 1) / BN;
-    const int tiles = m_tiles * n_tiles;
     const int k_blocks = (p.K + kBK - 1) / kBK;
     const WaitCtx ctx{abort_flag, p.status};
 
@@ -235,19 +235,23 @@ linear_wide_kernel(const __grid_constant__ LinearMaps maps, LinearParams p) {
     // anything); the activations may come from the kernel launched just before this one
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
     asm volatile("griddepcontrol.wait;" ::: "memory");
+    if (GROUPED) m_tiles = min(*p.group_tile_count, p.group_tile_max);
+    const int tiles = m_tiles * n_tiles;
 
     if (warp == 0) {
         if (lane == 0) {
             uint32_t it = 0;
             for (int t = blockIdx.x; t < tiles && !*abort_flag; t += gridDim.x) {
                 const int mt = t % m_tiles, nt = t / m_tiles;   // consecutive CTAs share a W tile through L2
+                int row0 = mt * kTileA, w0 = nt * BN;
+                if (GROUPED) { const int4 g = p.group_tiles[mt]; row0 = g.x; w0 += g.z * p.group_rows; }
                 for (int kb = 0; kb < k_blocks; ++kb, ++it) {
                     const int s = it % C::kStages;
                     if (it >= C::kStages && !mbar_wait(&empty[s], ((it / C::kStages) - 1) & 1, ctx, 0x41)) break;
                     uint8_t* st = smem + s * C::kStageBytes;
                     mbar_arrive_expect_tx(&full[s], C::kStageBytes);
-                    tma_load_2d(st, &maps.a, &full[s], kb * kBK, mt * kTileA);
-                    tma_load_2d(st + kABytes, &maps.b, &full[s], kb * kBK, nt * BN);
+                    tma_load_2d(st, &maps.a, &full[s], kb * kBK, row0);
+                    tma_load_2d(st + kABytes, &maps.b, &full[s], kb * kBK, w0);
                 }
             }
         }
@@ -287,14 +291,16 @@ linear_wide_kernel(const __grid_constant__ LinearMaps maps, LinearParams p) {
             const int buf = tile_no & 1;
             if (!mbar_wait_warp(&acc_full[buf], (tile_no >> 1) & 1, ctx, 0x45)) break;
             tc_fence_after();
-            const int row = mt * kTileA + quarter * 32 + lane;
+            int row = mt * kTileA, row_end = p.M;
+            if (GROUPED) { const int4 g = p.group_tiles[mt]; row = g.x; row_end = g.y; }
+            row += quarter * 32 + lane;
 #pragma unroll 1
             for (int c = 0; c < BN / 32; ++c) {
                 uint32_t acc[32];
                 tmem_ld32(tmem_base + (static_cast<uint32_t>(quarter * 32) << 16) + buf * BN + c * 32, acc);
                 tmem_ld_wait();
                 const int col0 = nt * BN + c * 32;
-                if (row < p.M && col0 < p.N) store_row32<EPI>(p, row, col0, acc);
+                if (row < row_end && col0 < p.N) store_row32<EPI>(p, row, col0, acc);
             }
             tc_fence_before();
             __syncwarp();
@@ -590,18 +596,18 @@ int sm_count(int* sms) {
     return VB200_OK;
 }
 
-template <int BN, int EPI>
+template <int BN, int EPI, bool GROUPED = false>
 int launch_wide(cudaStream_t s, const LinearParams& p) {
     using C = WideCfg<BN>;
     LinearMaps maps;
     if (int rc = make_map_2d(&maps.a, p.x, p.M, p.K, p.ldx, kTileA)) return rc;
-    if (int rc = make_map_2d(&maps.b, p.w, p.N, p.K, p.ldw, BN)) return rc;
-    auto kernel = linear_wide_kernel<BN, EPI>;
+    if (int rc = make_map_2d(&maps.b, p.w, GROUPED ? static_cast<long long>(p.groups) * p.group_rows : p.N, p.K, p.ldw, BN)) return rc;
+    auto kernel = linear_wide_kernel<BN, EPI, GROUPED>;
     static thread_local bool configured[64] = {};
     if (int rc = set_smem_once(kernel, C::kSmemBytes, configured)) return rc;
     int sms = 0;
     if (int rc = sm_count(&sms)) return rc;
-    const int tiles = ((p.M + kTileA - 1) / kTileA) * ((p.N + BN - 1) / BN);
+    const int tiles = (GROUPED ? p.group_tile_max : (p.M + kTileA - 1) / kTileA) * ((p.N + BN - 1) / BN);
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(static_cast<unsigned>(tiles < sms ? tiles : sms));
     cfg.blockDim = dim3(kThreads);
@@ -673,6 +679,14 @@ int launch_epi(cudaStream_t s, const LinearParams& p) {
 }
 
 }  // namespace
+
+int launch_linear_grouped(cudaStream_t s, const LinearParams& p) {
+    switch (p.epilogue) {
+        case VB200_EPI_BF16: return launch_wide<256, VB200_EPI_BF16, true>(s, p);
+        case VB200_EPI_SWIGLU: return launch_wide<256, VB200_EPI_SWIGLU, true>(s, p);
+        default: return set_detail(VB200_ERR_INVALID_ARG, "grouped linear: epilogue not available");
+    }
+}
 
 int launch_linear(cudaStream_t s, const LinearParams& p) {
     switch (p.epilogue) {

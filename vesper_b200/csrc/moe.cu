@@ -172,6 +172,73 @@ moe_pair_out_kernel(MoeParams p, const int* __restrict__ ids, const float* __res
     }
 }
 
+// ---- grouped by expert ----
+// grid E, 1024 threads: every CTA counts all pairs, then places its own expert's in their order.  gather[pair] = sorted row; token / weight of
+// every sorted row; the row tiles of the grouped products.
+constexpr int kSortThreads = 1024;
+
+__global__ void __launch_bounds__(kSortThreads)
+moe_sort_kernel(const int* __restrict__ ids, const float* __restrict__ weights, int pairs, int E, int* __restrict__ gather, float* __restrict__ row_weight, int4* __restrict__ tiles,
+                int* __restrict__ tile_count) {
+    pdl_begin();
+    extern __shared__ int count[];               // [E]
+    __shared__ int warp_sum[kSortThreads / 32], base[3];
+    const int e = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    for (int i = tid; i < E; i += kSortThreads) count[i] = 0;
+    __syncthreads();
+    const int per = (pairs + kSortThreads - 1) / kSortThreads, i0 = min(pairs, tid * per), i1 = min(pairs, i0 + per);
+    int mine = 0;
+    for (int i = i0; i < i1; ++i) {
+        const int id = ids[i];
+        atomicAdd(&count[id], 1);
+        mine += id == e;
+    }
+    int scan = mine;                             // inclusive over the warp
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) { const int v = __shfl_up_sync(0xFFFFFFFFu, scan, o); if (lane >= o) scan += v; }
+    if (lane == 31) warp_sum[warp] = scan;
+    __syncthreads();
+    if (warp == 0) {
+        int row = 0, tile = 0, all = 0;
+        for (int i = lane; i < E; i += 32) {
+            const int t = (count[i] + 127) / 128;
+            if (i < e) { row += count[i]; tile += t; }
+            all += t;
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            row += __shfl_xor_sync(0xFFFFFFFFu, row, o);
+            tile += __shfl_xor_sync(0xFFFFFFFFu, tile, o);
+            all += __shfl_xor_sync(0xFFFFFFFFu, all, o);
+        }
+        if (lane == 0) { base[0] = row; base[1] = tile; base[2] = all; }
+    } else if (warp == 1) {
+        const int v0 = warp_sum[lane];
+        int v = v0;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) { const int u = __shfl_up_sync(0xFFFFFFFFu, v, o); if (lane >= o) v += u; }
+        warp_sum[lane] = v - v0;
+    }
+    __syncthreads();
+    int at = base[0] + warp_sum[warp] + scan - mine;
+    for (int i = i0; i < i1; ++i)
+        if (ids[i] == e) { gather[i] = at; row_weight[at] = weights[i]; ++at; }
+    const int n = count[e], row_end = base[0] + n;
+    for (int t = tid; t < (n + 127) / 128; t += kSortThreads) tiles[base[1] + t] = make_int4(base[0] + t * 128, row_end, e, 0);
+    if (e == 0 && tid == 0) *tile_count = base[2];
+}
+
+// grid M, 128 threads: a token's row to its `top` places
+__global__ void __launch_bounds__(128)
+moe_scatter_rows_kernel(const uint4* __restrict__ x, const int* __restrict__ gather, int top, int n16, uint4* __restrict__ sorted) {
+    pdl_begin();
+    const long long m = blockIdx.x;
+    for (int c = threadIdx.x; c < n16; c += 128) {
+        const uint4 v = x[m * n16 + c];
+        for (int k = 0; k < top; ++k) sorted[static_cast<long long>(gather[m * top + k]) * n16 + c] = v;
+    }
+}
+
 int router_logits(cudaStream_t s, const vb200_moe_args& a, float* logits, int* status) {
     if (a.dtype == VB200_F32)
         return launch_linear_f32(s, static_cast<const float*>(a.x), a.dim, static_cast<const float*>(a.w_router), a.dim, nullptr, logits, pad_to(a.experts, 4), a.M, a.experts, a.dim);
@@ -182,6 +249,44 @@ int router_logits(cudaStream_t s, const vb200_moe_args& a, float* logits, int* s
     return launch_linear(s, p);
 }
 
+int launch_grouped(cudaStream_t s, const vb200_moe_args& a, const MoePlan& pl, const int* ids, const float* weights, int* status) {
+    uint8_t* ws = static_cast<uint8_t*>(a.workspace);
+    const int pairs = a.M * a.top;
+    int *gather = reinterpret_cast<int*>(ws + pl.gather), *tile_count = reinterpret_cast<int*>(ws + pl.tiles);
+    float* row_weight = reinterpret_cast<float*>(ws + pl.row_weight);
+    int4* tiles = reinterpret_cast<int4*>(ws + pl.tiles + 16);
+    if (int rc = launch_pdl(moe_sort_kernel, dim3(static_cast<unsigned>(a.experts)), dim3(kSortThreads), sizeof(int) * a.experts, s, ids, weights, pairs, a.experts, gather, row_weight,
+                            tiles, tile_count)) return rc;
+    if (int rc = launch_pdl(moe_scatter_rows_kernel, dim3(static_cast<unsigned>(a.M)), dim3(128), 0, s, static_cast<const uint4*>(a.x), static_cast<const int*>(gather), a.top, a.dim / 8,
+                            reinterpret_cast<uint4*>(ws + pl.sorted_x))) return rc;
+    LinearParams p{};
+    p.status = status;
+    p.group_tiles = tiles; p.group_tile_count = tile_count; p.group_tile_max = pl.max_tiles; p.groups = a.experts;
+    p.x = ws + pl.sorted_x; p.ldx = a.dim; p.w = a.w_in; p.ldw = a.dim; p.out = ws + pl.sorted_act; p.ldo = pad_to(a.ff, 8);
+    p.M = pairs; p.N = 2 * a.ff; p.K = a.dim; p.group_rows = 2 * a.ff;
+    p.epilogue = VB200_EPI_SWIGLU;
+    profile_mark_begin(s);
+    if (int rc = launch_linear_grouped(s, p)) return rc;
+    p.x = ws + pl.sorted_act; p.ldx = pad_to(a.ff, 8); p.w = a.w_out; p.ldw = a.ld_out; p.out = ws + pl.sorted_y; p.ldo = a.dim;
+    p.N = a.dim; p.K = a.ff; p.group_rows = a.dim; p.row_scale = row_weight;
+    p.epilogue = VB200_EPI_BF16;
+    if (int rc = launch_linear_grouped(s, p)) return rc;
+    profile_mark_end(s);
+    note_moe_kernel("linear_wide_kernel (grouped)");
+    if (a.ff_shared == 0) {
+        VB200_CUDA_TRY(cudaMemsetAsync(a.y, 0, static_cast<size_t>(a.M) * a.dim * sizeof(float), s));
+        return VB200_OK;
+    }
+    LinearParams q{};
+    q.status = status;
+    q.x = a.x; q.ldx = a.dim; q.w = a.w_shared_in; q.ldw = a.dim; q.out = ws + pl.shared_act; q.ldo = pad_to(a.ff_shared, 8);
+    q.M = a.M; q.N = 2 * a.ff_shared; q.K = a.dim; q.epilogue = VB200_EPI_SWIGLU;
+    if (int rc = launch_linear(s, q)) return rc;
+    q.x = ws + pl.shared_act; q.ldx = pad_to(a.ff_shared, 8); q.w = a.w_shared_out; q.ldw = a.ld_shared; q.out = a.y; q.ldo = a.dim;
+    q.N = a.dim; q.K = a.ff_shared; q.epilogue = VB200_EPI_F32;
+    return launch_linear(s, q);
+}
+
 }  // namespace
 
 MoePlan plan_moe(const vb200_moe_args& a) {
@@ -190,10 +295,23 @@ MoePlan plan_moe(const vb200_moe_args& a) {
     const size_t esz = a.dtype == VB200_F32 ? 4 : 2, M = static_cast<size_t>(a.M), pairs = M * a.top;
     size_t at = 0;
     auto take = [&](size_t bytes) { const size_t o = at; at += up(bytes); return o; };
-    pl.grouped = false;
+    // sorting pays when experts are shared: token by token every pair streams an expert of its own
+    pl.grouped = a.dtype == VB200_BF16 && a.form != 1 && pairs < (1u << 30) && (a.form == 2 || pairs >= 2 * static_cast<size_t>(a.experts));
+    pl.max_tiles = static_cast<int>((pairs + 127) / 128) + (a.experts < static_cast<int>(pairs) ? a.experts : static_cast<int>(pairs));
     pl.logits = take(M * pad_to(a.experts, 4) * 4);
     pl.ids = take(pairs * 4);
     pl.weights = take(pairs * 4);
+    if (pl.grouped) {
+        pl.gather = take(pairs * 4);
+        pl.row_weight = take(pairs * 4);
+        pl.tiles = take(16 + static_cast<size_t>(pl.max_tiles) * 16);
+        pl.sorted_x = take(pairs * a.dim * esz);
+        pl.sorted_act = take(pairs * pad_to(a.ff, 8) * esz);
+        pl.sorted_y = take(pairs * a.dim * esz);
+        pl.shared_act = take(M * pad_to(a.ff_shared, 8) * esz);
+        pl.total = at;
+        return pl;
+    }
     const size_t act_ld = pad_to(a.ff > a.ff_shared ? a.ff : a.ff_shared, 8);
     pl.act = take(M * (a.top + 1) * act_ld * esz);
     pl.total = at;
@@ -213,6 +331,7 @@ int launch_moe(cudaStream_t s, const vb200_moe_args& a, const MoePlan& pl, int* 
     int* ids = reinterpret_cast<int*>(ws + pl.ids);
     if (int rc = router_logits(s, a, logits, status)) return rc;
     if (int rc = launch_moe_route(s, logits, pad_to(a.experts, 4), a.correction, a.M, a.experts, a.top, a.groups, a.keep, a.scale, ids, weights)) return rc;
+    if (pl.grouped) return launch_grouped(s, a, pl, ids, weights, status);
     MoeParams p{};
     p.M = a.M; p.dim = a.dim; p.ff = a.ff; p.ff_shared = a.ff_shared; p.E = a.experts; p.top = a.top; p.ld_out = a.ld_out; p.ld_shared = a.ld_shared;
     p.act_ld = pad_to(a.ff > a.ff_shared ? a.ff : a.ff_shared, 8);
