@@ -93,10 +93,10 @@ def reference(c, w):
     return ReferenceHybrid(c, w)
 
 
-def build(c, w, dtype, **kw):
+def build(c, w, dtype, want_shapes=None, **kw):
     from vesper_b200.model import model_from_config
     m = model_from_config(c, dtype, **kw)
-    assert m.param_shapes() == shapes(c)
+    assert m.param_shapes() == (want_shapes or shapes(c))
     for k, v in w.items():
         m.set_param(k, v)
     return m

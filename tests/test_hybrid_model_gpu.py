@@ -1,9 +1,5 @@
-"""Hybrid decoders (models::HybridLM behind the registry) on the GPU against the plain model of hybrid_reference.py.
-
-The error at a position is the rms over the vocabulary of the logit difference, relative to the rms of all logits of
-the case.  Limit in fp32: 1e-4.  In bf16: three times what rounding alone does there, taken from runs of the plain model
-with every activation rounded to bf16 at a random place within half a step (random small models have ill-conditioned
-positions; a window, key, tap or state that is wrong costs far more)."""
+"""Hybrid decoders (models::HybridLM behind the registry) on the GPU against the plain model of hybrid_reference.py; limits as in
+sequence_check.py."""
 import json
 import os
 import subprocess
@@ -12,8 +8,9 @@ import sys
 import numpy as np
 import pytest
 
-from helpers import bf16_round
+import sequence_check
 from hybrid_cases import CASES, ReferenceHybrid, build, reference, save, weights
+from sequence_check import errors, run, status
 
 pytestmark = pytest.mark.gpu
 
@@ -21,30 +18,8 @@ ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 _cache = {}
 
 
-def errors(got, want):
-    d = got - want
-    return np.sqrt((d * d).mean(-1)) / np.sqrt((want * want).mean())
-
-
-class Sequence:
-    """Token ids with the plain model's logits and the error limit at every position."""
-
-    def __init__(self, c, w, ids, trials=5):
-        self.ids, self.want = ids, reference(c, w).forward(ids)
-        rng = np.random.default_rng(11)
-
-        def dither(a):
-            a = a.astype(np.float32)
-            return bf16_round(a * (1 + (rng.random(a.shape).astype(np.float32) - 0.5) * 2 ** -8)).astype(np.float64)
-        e = np.max([errors(ReferenceHybrid(c, w, round_act=dither).forward(ids), self.want) for _ in range(trials)], axis=0)
-        self.limits = {"float32": np.full(len(ids), 1e-4), "bfloat16": 3 * np.maximum(e, np.quantile(e, 0.9))}
-        self.rms = np.sqrt((self.want ** 2).mean())
-
-    def check(self, got, dtype, at=0, scale=1.0):
-        n = len(got)
-        d = got - self.want[at:at + n]
-        over = np.sqrt((d * d).mean(-1)) / self.rms / self.limits[dtype][at:at + n]
-        assert over.max() <= scale, (at + int(over.argmax()), over.max())
+def Sequence(c, w, ids, **kw):
+    return sequence_check.Sequence(ReferenceHybrid, c, w, ids, **kw)
 
 
 def case(name):
@@ -54,22 +29,6 @@ def case(name):
         w = weights(c, seed=len(name))
         _cache[name] = (c, w, Sequence(c, w, np.random.default_rng(1).integers(0, c["vocab"], 170)))
     return _cache[name]
-
-
-def status():
-    from vesper_b200 import capi
-    capi.check_kernel_status(0)
-
-
-def run(m, ids, cuts):
-    s = m.open_sequence()
-    out, at = [], 0
-    for n in cuts:
-        out.append(m.extend(s, ids[at:at + n]))
-        at += n
-    m.close_sequence(s)
-    status()
-    return np.concatenate(out)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])

@@ -54,6 +54,19 @@ def sigmoid_attention(q, k, v, q_pos, scale, rel, reach, talk, pb):
     return out
 
 
+def route_margin(logits, correction, top, groups, keep):
+    """How far the choice is from another one: the smallest gap between what is taken and what is not, groups and experts."""
+    choice, E, gap = sigmoid(logits) + correction, len(logits), np.inf
+    if groups:
+        score = np.sort(np.sort(choice.reshape(groups, E // groups), axis=1)[:, -2:].sum(axis=1))[::-1]
+        if keep < groups:
+            gap = score[keep - 1] - score[keep]
+    ids, _ = route(logits, correction, E if not groups else keep * (E // groups), groups, keep, 1.0)
+    if len(ids) > top:
+        gap = min(gap, choice[ids[top - 1]] - choice[ids[top]])
+    return gap
+
+
 def route(logits, correction, top, groups, keep, scale):
     """(expert ids, weights) of one token."""
     s = sigmoid(logits)
@@ -79,6 +92,7 @@ class ReferenceZudisun:
 
     def reset(self):
         self.pos, self.states = 0, {}
+        self.margins = {}                  # position -> smallest router margin of its layers
 
     def lin(self, x, name):
         y = self.rnd(x) @ self.w[name].T
@@ -112,7 +126,7 @@ class ReferenceZudisun:
                 self.v_first = v
             else:
                 lam = float(self.w[p + "vmix"].reshape(()))
-                v = self.rnd((1 - lam) * v + lam * self.v_first)
+                v = self.rnd((1 - lam) * v + lam * self.v_first.reshape(v.shape))
         k0, v0 = self.states.get(i, (np.zeros((0, G, d), self.real), np.zeros((0, G, dv), self.real)))
         k, v = np.concatenate([k0, k]), np.concatenate([v0, v])
         self.states[i] = (k, v)
@@ -131,7 +145,9 @@ class ReferenceZudisun:
         logits = self.rnd(x) @ self.w[p + ".router"].T
         g = r.get("groups") or {}
         for t in range(x.shape[0]):
-            ids, weights = route(logits[t], self.w[p + ".correction"], r["top"], g.get("count"), g.get("keep"), r["scale"])
+            choice = (logits[t], self.w[p + ".correction"], r["top"], g.get("count"), g.get("keep"))
+            ids, weights = route(*choice, r["scale"])
+            self.margins[self.pos + t] = min(self.margins.get(self.pos + t, np.inf), route_margin(*choice))
             for e, we in zip(ids, weights):
                 out[t] += we * self.gated(x[t:t + 1], f"{p}.e{e}", silu)[0]
         return out + self.gated(x, p + ".shared", silu) if m.get("shared") else out

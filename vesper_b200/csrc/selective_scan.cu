@@ -5,7 +5,7 @@
 //
 // Every (channel, state) pair has its own decay, so a chunk of tokens is no matrix product: the work is one exponential and two
 // multiply-adds per pair and token.  LP lanes share a channel, each holding NI of its states in registers over the whole portion; the
-// tokens come in tiles of kTile through a two-stage shared-memory ring filled with cp.async while the tile before is walked.
+// tokens come in tiles through a two-stage shared-memory ring filled with cp.async while the tile before is walked.
 #include "hybrid.cuh"
 
 #include <type_traits>
@@ -13,7 +13,6 @@
 namespace vb200 {
 namespace {
 
-constexpr int kTile = 32;          // tokens per shared-memory tile
 constexpr int kThreads = 128;
 
 struct ScanParams {
@@ -52,6 +51,7 @@ template <typename T, int LP, int NI>
 struct ScanTile {
     static constexpr int kCh = kThreads / LP;                  // channels per CTA
     static constexpr int kStates = LP * NI;
+    static constexpr int kTile = kStates * sizeof(T) > 1024 ? 8 : 32;      // tokens per shared-memory tile
     struct Stage {
         alignas(16) T x[kTile][kCh], z[kTile][kCh];
         alignas(16) float dt[kTile][kCh];
@@ -67,7 +67,7 @@ __global__ void __launch_bounds__(kThreads)
 selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restrict__ xc, const T* __restrict__ xdbl, const float* __restrict__ dt, float* __restrict__ state,
                       T* __restrict__ out) {
     using S = ScanTile<T, LP, NI>;
-    constexpr int CH = S::kCh, V = 16 / sizeof(T);
+    constexpr int CH = S::kCh, V = 16 / sizeof(T), kTile = S::kTile;
     extern __shared__ __align__(16) uint8_t raw[];
     S& sm = *reinterpret_cast<S*>(raw);
     const int tid = threadIdx.x, lane = tid % LP, ch = tid / LP, b = blockIdx.y, c0 = blockIdx.x * CH, c = c0 + ch;

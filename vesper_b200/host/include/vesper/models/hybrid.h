@@ -31,6 +31,7 @@ struct HybridConfig {
         Json mlp;                  // its feed-forward, null = none
     };
     std::vector<Layer> layers;
+    int64_t shared_value_cols = 0;                                          // of the layers that mix values, 0 = none
     struct { int64_t start = 0, stop = 0, times = 0; } loop;               // times 0 = no loop
     struct { int64_t buckets = 0, mul_prev = 0, mul_cur = 0; } bigram;     // buckets 0 = none
     static HybridConfig from_json(const Json& config, const HybridStyle& style);
@@ -97,7 +98,6 @@ private:
     float norm_gain_ = 1.0f;
     Tensor embed_, bigram_, final_norm_, loop_step_, head_;      // head_: undefined where tied
     std::map<std::string, std::vector<int64_t>> shapes_;
-    int64_t shared_value_cols_ = 0;
     std::vector<std::unique_ptr<Layer>> layers_;
     std::vector<Run> runs_;
     std::vector<std::unique_ptr<nn::SequenceState>> states_;     // one per run

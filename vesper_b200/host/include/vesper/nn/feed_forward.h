@@ -17,6 +17,7 @@ enum class Activation { SquaredRelu, GatedRelu, GatedSilu };
 struct FeedForwardStyle {
     Activation dense = Activation::SquaredRelu;
     bool dense_bias = false;
+    bool experts = false;              // mixtures of experts may take a dense layer's place
 };
 
 // One call: M rows of `width` padded to the weights' row length; x in the model's dtype, y fp32.
@@ -64,7 +65,6 @@ public:
     const Tensor& out_weight() const { return out_; }
     int64_t in_rows() const { return gated() ? 2 * ff_ : ff_; }
     int epilogue() const;
-    bool has_bias() const { return bias_; }
 
 private:
     bool gated() const { return activation_ != Activation::SquaredRelu; }
@@ -77,7 +77,12 @@ private:
 
 class MixtureOfExperts : public FeedForward {
 public:
-    // mlp: expert {ff}, router {experts, top, scale, groups {count, keep} (optional)}, shared {ff} (optional)
+    struct Sizes {
+        int64_t experts, top, groups = 0, keep = 0, ff, shared = 0;
+        double scale;
+        // expert {ff}, router {experts, top, scale, groups {count, keep} (optional)}, shared {ff} (optional)
+        explicit Sizes(const Json& mlp);
+    };
     MixtureOfExperts(const Json& mlp, int64_t width, int64_t width_ld, DType dtype);
     std::map<std::string, std::vector<int64_t>> parameter_shapes() const override;
     void load_parameter(const std::string& name, const float* host_values) override;
@@ -87,12 +92,14 @@ public:
 
 private:
     struct Args;
-    int64_t experts_, top_, groups_ = 0, keep_ = 0, ff_, shared_ = 0, width_, width_ld_;
-    double scale_;
+    Sizes z_;
+    int64_t width_, width_ld_;
     DType dtype_;
     Tensor router_, correction_, in_, out_, shared_in_, shared_out_;
 };
 
+// Throws where a layer entry's "mlp" is of an unknown kind or its sizes do not fit together.  Needs no device.
+void check_feed_forward(const Json& mlp, const FeedForwardStyle& style);
 // The feed-forward of a layer entry's "mlp".
 std::unique_ptr<FeedForward> make_feed_forward(const Json& mlp, const FeedForwardStyle& style, int64_t width, int64_t width_ld, DType dtype);
 

@@ -122,12 +122,19 @@ private:
 
 class SigmoidAttention : public SequenceMixer {
 public:
-    // mixer: heads, kv_heads, dim, vdim, scale, bias_max, q_temp {coef, every} (optional), v_mix (optional)
+    struct Sizes {
+        int64_t heads, kv_heads, dim, vdim, temp_every = 0;
+        double scale, reach, temp_coef = 0.0;
+        bool value_mixing = false;
+        // heads, kv_heads, dim, vdim, scale, bias_max, q_temp {coef, every} (optional), v_mix (optional)
+        explicit Sizes(const Json& mixer);
+        int64_t shared_value_cols() const { return value_mixing ? kv_heads * vdim : 0; }
+    };
     SigmoidAttention(const Json& mixer, int64_t width, int64_t width_ld, double eps, DType dtype);
     std::map<std::string, std::vector<int64_t>> parameter_shapes() const override;
     void load_parameter(const std::string& name, const float* host_values) override;
     void set_free_size(const std::string& name, int64_t numel) override;
-    int64_t shared_value_cols() const override { return value_mixing_ ? kv_heads_ * vdim_ : 0; }
+    int64_t shared_value_cols() const override { return z_.shared_value_cols(); }
     bool grows_with_length() const override { return true; }
     std::unique_ptr<SequenceState> make_state(int64_t slots, int64_t max_len) const override;
     int64_t workspace_bytes(const MixerStep& step) const override;
@@ -136,9 +143,8 @@ public:
 private:
     struct Args;
     void fold_bias();
-    int64_t heads_, kv_heads_, dim_, vdim_, bias_rows_ = 0, temp_every_ = 0;
-    double scale_, reach_, temp_coef_ = 0.0;
-    bool value_mixing_ = false;
+    Sizes z_;
+    int64_t bias_rows_ = 0;
     float lambda_ = 0.0f;
     std::vector<float> host_rel_, host_talk_, host_offset_;      // until all three are known: the folded table needs them together
     Tensor talk_, bias_;                                         // fp32 [heads, heads], [heads, distances]
@@ -146,7 +152,11 @@ private:
 
 class Mamba1 : public SequenceMixer {
 public:
-    // mixer: inner, state, dt_rank, conv
+    struct Sizes {
+        int64_t inner, state, rank, taps;
+        int64_t inner8, state8, rank8;           // padded to multiples of 8; the padding's weights are zero
+        explicit Sizes(const Json& mixer);       // inner, state, dt_rank, conv
+    };
     Mamba1(const Json& mixer, int64_t width, int64_t width_ld, double eps, DType dtype);
     std::map<std::string, std::vector<int64_t>> parameter_shapes() const override;
     void load_parameter(const std::string& name, const float* host_values) override;
@@ -156,8 +166,7 @@ public:
 
 private:
     struct Args;
-    int64_t inner_, state_, rank_, taps_;
-    int64_t inner8_, state8_, rank8_;                            // padded to multiples of 8; the padding's weights are zero
+    Sizes z_;
     Tensor w_x_, w_dt_;
     Tensor conv_w_, conv_b_, dt_bias_, a_, d_;                   // fp32; a = -exp(A_log)
 };
@@ -165,6 +174,8 @@ private:
 // Row of a relative-bias table of `rows` rows for distance n: a row each below rows / 2, then logarithmic up to `reach`.
 int64_t distance_bucket(int64_t n, int64_t rows, double reach);
 
+// Throws where a layer entry's mixer is unknown or its sizes do not fit together; returns its shared value columns.  Needs no device.
+int64_t check_mixer(const std::string& type, const Json& mixer);
 // The mixer a layer entry's "type" names.
 std::unique_ptr<SequenceMixer> make_mixer(const std::string& type, const Json& mixer, int64_t width, int64_t width_ld, double eps, DType dtype);
 

@@ -82,51 +82,54 @@ PendingRows DenseMlp::forward(const FeedForwardStep& s) {
 
 // ---- mixture of experts ----------------------------------------------------------------------------
 
-MixtureOfExperts::MixtureOfExperts(const Json& m, int64_t width, int64_t width_ld, DType dtype) : width_(width), width_ld_(width_ld), dtype_(dtype) {
+MixtureOfExperts::Sizes::Sizes(const Json& m) {
     const Json& r = m.at("router");
-    experts_ = positive(r, "experts");
-    top_ = positive(r, "top");
-    scale_ = r.at("scale").as_double();
-    ff_ = positive(m.at("expert"), "ff");
+    experts = positive(r, "experts");
+    top = positive(r, "top");
+    scale = r.at("scale").as_double();
+    ff = positive(m.at("expert"), "ff");
     const Json& g = r.get("groups");
     if (!g.is_null()) {
-        groups_ = positive(g, "count");
-        keep_ = positive(g, "keep");
-        if (experts_ % groups_ != 0 || keep_ > groups_ || top_ > keep_ * (experts_ / groups_))
+        groups = positive(g, "count");
+        keep = positive(g, "keep");
+        if (experts % groups != 0 || keep > groups || top > keep * (experts / groups))
             throw std::runtime_error("configuration: the experts must divide into the groups, and the kept groups hold 'top' experts");
     }
-    if (top_ > experts_) throw std::runtime_error("configuration: 'top' exceeds the number of experts");
+    if (top > experts) throw std::runtime_error("configuration: 'top' exceeds the number of experts");
     const Json& s = m.get("shared");
-    if (!s.is_null()) shared_ = positive(s, "ff");
-    router_ = zeros({experts_, width_ld}, dtype, Device::CUDA);
-    correction_ = zeros({experts_}, DType::Float32, Device::CUDA);
-    in_ = zeros({experts_ * 2 * ff_, width_ld}, dtype, Device::CUDA);
-    out_ = zeros({experts_ * width_ld, pad8(ff_)}, dtype, Device::CUDA);
-    if (shared_ > 0) {
-        shared_in_ = zeros({2 * shared_, width_ld}, dtype, Device::CUDA);
-        shared_out_ = zeros({width_ld, pad8(shared_)}, dtype, Device::CUDA);
+    if (!s.is_null()) shared = positive(s, "ff");
+}
+
+MixtureOfExperts::MixtureOfExperts(const Json& mlp, int64_t width, int64_t width_ld, DType dtype) : z_(mlp), width_(width), width_ld_(width_ld), dtype_(dtype) {
+    router_ = zeros({z_.experts, width_ld}, dtype, Device::CUDA);
+    correction_ = zeros({z_.experts}, DType::Float32, Device::CUDA);
+    in_ = zeros({z_.experts * 2 * z_.ff, width_ld}, dtype, Device::CUDA);
+    out_ = zeros({z_.experts * width_ld, pad8(z_.ff)}, dtype, Device::CUDA);
+    if (z_.shared > 0) {
+        shared_in_ = zeros({2 * z_.shared, width_ld}, dtype, Device::CUDA);
+        shared_out_ = zeros({width_ld, pad8(z_.shared)}, dtype, Device::CUDA);
     }
 }
 
 std::map<std::string, std::vector<int64_t>> MixtureOfExperts::parameter_shapes() const {
-    std::map<std::string, std::vector<int64_t>> m = {{"router", {experts_, width_}}, {"correction", {experts_}}};
+    std::map<std::string, std::vector<int64_t>> m = {{"router", {z_.experts, width_}}, {"correction", {z_.experts}}};
     auto expert = [&](const std::string& p, int64_t ff) {
         m[p + ".gate"] = {ff, width_};
         m[p + ".up"] = {ff, width_};
         m[p + ".down"] = {width_, ff};
     };
-    for (int64_t e = 0; e < experts_; ++e) expert("e" + std::to_string(e), ff_);
-    if (shared_ > 0) expert("shared", shared_);
+    for (int64_t e = 0; e < z_.experts; ++e) expert("e" + std::to_string(e), z_.ff);
+    if (z_.shared > 0) expert("shared", z_.shared);
     return m;
 }
 
 void MixtureOfExperts::load_parameter(const std::string& name, const float* v) {
-    if (name == "router") return load_rows(router_, 0, experts_, width_, v);
-    if (name == "correction") return load_vector(correction_, 0, experts_, v);
+    if (name == "router") return load_rows(router_, 0, z_.experts, width_, v);
+    if (name == "correction") return load_vector(correction_, 0, z_.experts, v);
     const size_t dot = name.find('.');
     const std::string who = name.substr(0, dot), what = dot == std::string::npos ? "" : name.substr(dot + 1);
     const bool shared = who == "shared";
-    const int64_t e = shared ? 0 : std::stoll(who.substr(1)), ff = shared ? shared_ : ff_;
+    const int64_t e = shared ? 0 : std::stoll(who.substr(1)), ff = shared ? z_.shared : z_.ff;
     Tensor &in = shared ? shared_in_ : in_, &out = shared ? shared_out_ : out_;
     if (what == "gate") load_rows(in, e * 2 * ff, ff, width_, v, 2);
     else if (what == "up") load_rows(in, e * 2 * ff + 1, ff, width_, v, 2);
@@ -141,15 +144,15 @@ struct MixtureOfExperts::Args {
         a.device = m.router_.device_index();
         a.stream = current_stream();
         a.dtype = m.dtype_ == DType::Float32 ? VB200_F32 : VB200_BF16;
-        a.M = static_cast<int>(M); a.dim = static_cast<int>(m.width_ld_); a.ff = static_cast<int>(m.ff_); a.ff_shared = static_cast<int>(m.shared_);
-        a.experts = static_cast<int>(m.experts_); a.top = static_cast<int>(m.top_); a.groups = static_cast<int>(m.groups_); a.keep = static_cast<int>(m.keep_);
-        a.scale = static_cast<float>(m.scale_);
+        a.M = static_cast<int>(M); a.dim = static_cast<int>(m.width_ld_); a.ff = static_cast<int>(m.z_.ff); a.ff_shared = static_cast<int>(m.z_.shared);
+        a.experts = static_cast<int>(m.z_.experts); a.top = static_cast<int>(m.z_.top); a.groups = static_cast<int>(m.z_.groups); a.keep = static_cast<int>(m.z_.keep);
+        a.scale = static_cast<float>(m.z_.scale);
         a.w_router = m.router_.data_ptr<char>();
         a.correction = m.correction_.data_ptr<float>();
         a.w_in = m.in_.data_ptr<char>();
         a.w_out = m.out_.data_ptr<char>();
         a.ld_out = m.out_.shape()[1];
-        if (m.shared_ > 0) {
+        if (m.z_.shared > 0) {
             a.w_shared_in = m.shared_in_.data_ptr<char>();
             a.w_shared_out = m.shared_out_.data_ptr<char>();
             a.ld_shared = m.shared_out_.shape()[1];
@@ -175,11 +178,17 @@ PendingRows MixtureOfExperts::forward(const FeedForwardStep& s) {
     return p;
 }
 
-std::unique_ptr<FeedForward> make_feed_forward(const Json& mlp, const FeedForwardStyle& style, int64_t width, int64_t width_ld, DType dtype) {
+void check_feed_forward(const Json& mlp, const FeedForwardStyle& style) {
     const std::string& kind = mlp.at("kind").as_string();
-    if (kind == "dense") return std::make_unique<DenseMlp>(positive(mlp, "ff"), style.dense, style.dense_bias, width, width_ld, dtype);
-    if (kind == "moe") return std::make_unique<MixtureOfExperts>(mlp, width, width_ld, dtype);
-    throw std::runtime_error("configuration: no feed-forward of kind '" + kind + "'");
+    if (kind == "dense") (void)positive(mlp, "ff");
+    else if (kind == "moe" && style.experts) (void)MixtureOfExperts::Sizes(mlp);
+    else throw std::runtime_error("configuration: no feed-forward of kind '" + kind + "'");
+}
+
+std::unique_ptr<FeedForward> make_feed_forward(const Json& mlp, const FeedForwardStyle& style, int64_t width, int64_t width_ld, DType dtype) {
+    check_feed_forward(mlp, style);
+    if (mlp.at("kind").as_string() == "dense") return std::make_unique<DenseMlp>(positive(mlp, "ff"), style.dense, style.dense_bias, width, width_ld, dtype);
+    return std::make_unique<MixtureOfExperts>(mlp, width, width_ld, dtype);
 }
 
 }  // namespace vesper::nn

@@ -32,6 +32,10 @@ HybridConfig HybridConfig::from_json(const Json& c, const HybridStyle& style) {
         x.type = l.at("type").as_string();
         x.mixer = l.at("mixer");
         x.mlp = l.get("mlp");
+        if (!x.mlp.is_null()) nn::check_feed_forward(x.mlp, style.feed_forward);
+        const int64_t cols = nn::check_mixer(x.type, x.mixer);
+        if (cols > 0 && h.shared_value_cols > 0 && cols != h.shared_value_cols) throw std::runtime_error("configuration: layers that mix values must have one number of value columns");
+        h.shared_value_cols = std::max(h.shared_value_cols, cols);
         h.layers.push_back(x);
     }
     const Json& loop = c.get("loop");
@@ -49,6 +53,7 @@ HybridConfig HybridConfig::from_json(const Json& c, const HybridStyle& style) {
         h.bigram.mul_cur = bigram.at("mul_cur").as_int();
         if (h.bigram.buckets <= 0) throw std::runtime_error("configuration: 'buckets' must be positive");
     }
+    if (style.norm_outputs && (h.loop.times > 0 || h.bigram.buckets > 0)) throw std::runtime_error("configuration: this architecture has no loop and no bigram embedding");
     if (h.vocab <= 0 || h.width <= 0) throw std::runtime_error("configuration: 'vocab' and 'width' must be positive");
     return h;
 }
@@ -97,17 +102,10 @@ HybridLM::HybridLM(const HybridConfig& config, const LoadOptions& options) : con
         if (!l.mlp.is_null()) {
             L->norm2 = zeros({dim_}, DType::Float32, Device::CUDA);
             L->ff = nn::make_feed_forward(l.mlp, config_.style.feed_forward, config_.width, dim_, dtype_);
-            if (!config_.style.norm_outputs && (!L->ff->dense() || L->ff->dense()->has_bias()))
-                throw std::runtime_error("configuration: this architecture has no feed-forward of kind '" + l.mlp.at("kind").as_string() + "'");
         }
-        const int64_t cols = L->mixer->shared_value_cols();
-        if (cols > 0 && shared_value_cols_ > 0 && cols != shared_value_cols_) throw std::runtime_error("configuration: layers that mix values must have one number of value columns");
-        shared_value_cols_ = std::max(shared_value_cols_, cols);
         grows = grows || L->mixer->grows_with_length();
         layers_.push_back(std::move(L));
     }
-    if (config_.style.norm_outputs && (config_.loop.times > 0 || config_.bigram.buckets > 0))
-        throw std::runtime_error("configuration: this architecture has no loop and no bigram embedding");
     max_len_ = options.max_seq_len > 0 ? options.max_seq_len : grows ? 32768 : int64_t{1} << 20;
     const int64_t n = static_cast<int64_t>(config_.layers.size());
     const auto& loop = config_.loop;
@@ -259,7 +257,7 @@ void HybridLM::ensure_buffers(int64_t rows, const nn::MixerStep& step) {
     if (keep_embedding_) b.embed = zeros({rows, dim_}, DType::Float32, Device::CUDA);
     b.xn = zeros({rows, dim_}, dtype_, Device::CUDA);
     if (config_.style.norm_outputs) b.y = zeros({rows, dim_}, DType::Float32, Device::CUDA);
-    if (shared_value_cols_ > 0) b.values = zeros({rows, shared_value_cols_}, dtype_, Device::CUDA);
+    if (config_.shared_value_cols > 0) b.values = zeros({rows, config_.shared_value_cols}, dtype_, Device::CUDA);
     b.inv = zeros({rows}, DType::Float32, Device::CUDA);
     b.proj = zeros({rows, proj}, dtype_, Device::CUDA);
     b.mixed = zeros({rows, mixed}, dtype_, Device::CUDA);
@@ -287,9 +285,9 @@ void HybridLM::run(const int32_t* ids, nn::MixerStep step, int32_t* lens) {
     step.workspace = b.workspace.data_ptr<char>();
     step.workspace_bytes = static_cast<int64_t>(b.workspace.numel()) * 4;
     nn::StepValues values;
-    if (shared_value_cols_ > 0) {
+    if (config_.shared_value_cols > 0) {
         values.data = b.values.data_ptr<char>();
-        values.cols = shared_value_cols_;
+        values.cols = config_.shared_value_cols;
         step.values = &values;
     }
 

@@ -81,7 +81,7 @@ std::map<std::string, ModelFactory>& registry() {
     static std::map<std::string, ModelFactory> r = {
         {"TransformerLM", make_transformer},
         {"Nitenex", hybrid(HybridStyle{})},
-        {"Zudisun", hybrid(HybridStyle{true, false, {nn::Activation::GatedRelu, true}})},
+        {"Zudisun", hybrid(HybridStyle{true, false, {nn::Activation::GatedRelu, true, true}})},
     };
     return r;
 }

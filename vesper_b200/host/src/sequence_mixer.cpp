@@ -272,51 +272,54 @@ int64_t distance_bucket(int64_t n, int64_t rows, double reach) {
     return std::min(rows - 1, half + static_cast<int64_t>(std::floor(x + 1e-9)));
 }
 
-SigmoidAttention::SigmoidAttention(const Json& m, int64_t width, int64_t width_ld, double eps, DType dtype) : SequenceMixer(width, width_ld, eps, dtype) {
-    heads_ = positive(m, "heads");
-    kv_heads_ = positive(m, "kv_heads");
-    dim_ = positive(m, "dim");
-    vdim_ = positive(m, "vdim");
-    if (heads_ % kv_heads_ != 0) throw std::runtime_error("configuration: heads must be divisible by kv_heads");
-    scale_ = m.at("scale").as_double();
-    reach_ = m.at("bias_max").as_double();
+SigmoidAttention::Sizes::Sizes(const Json& m) {
+    heads = positive(m, "heads");
+    kv_heads = positive(m, "kv_heads");
+    dim = positive(m, "dim");
+    vdim = positive(m, "vdim");
+    if (heads % kv_heads != 0) throw std::runtime_error("configuration: heads must be divisible by kv_heads");
+    scale = m.at("scale").as_double();
+    reach = m.at("bias_max").as_double();
     const Json& temp = m.get("q_temp");
     if (!temp.is_null()) {
-        temp_coef_ = temp.at("coef").as_double();
-        temp_every_ = positive(temp, "every");
+        temp_coef = temp.at("coef").as_double();
+        temp_every = positive(temp, "every");
     }
     const Json& mix = m.get("v_mix");
-    value_mixing_ = !mix.is_null() && mix.as_bool();
-    proj_rows_ = heads_ * (dim_ + 1) + kv_heads_ * (dim_ + vdim_);
-    mixed_cols_ = heads_ * vdim_;
+    value_mixing = !mix.is_null() && mix.as_bool();
+}
+
+SigmoidAttention::SigmoidAttention(const Json& m, int64_t width, int64_t width_ld, double eps, DType dtype) : SequenceMixer(width, width_ld, eps, dtype), z_(m) {
+    proj_rows_ = z_.heads * (z_.dim + 1) + z_.kv_heads * (z_.dim + z_.vdim);
+    mixed_cols_ = z_.heads * z_.vdim;
     in_weight_ = zeros({proj_rows_, width_ld}, dtype, Device::CUDA);
     out_weight_ = zeros({width_ld, mixed_ld()}, dtype, Device::CUDA);
-    talk_ = zeros({heads_, heads_}, DType::Float32, Device::CUDA);
-    bias_ = zeros({heads_, 1}, DType::Float32, Device::CUDA);
+    talk_ = zeros({z_.heads, z_.heads}, DType::Float32, Device::CUDA);
+    bias_ = zeros({z_.heads, 1}, DType::Float32, Device::CUDA);
 }
 
 std::map<std::string, std::vector<int64_t>> SigmoidAttention::parameter_shapes() const {
-    std::map<std::string, std::vector<int64_t>> m = {{"q", {heads_ * dim_, width_}}, {"k", {kv_heads_ * dim_, width_}}, {"v", {kv_heads_ * vdim_, width_}}, {"g", {heads_, width_}},
-                                                     {"rel", {-1, heads_}}, {"talk", {heads_, heads_}}, {"pb", {heads_}}, {"o", {width_, heads_ * vdim_}}};
-    if (value_mixing_) m["vmix"] = {};
+    std::map<std::string, std::vector<int64_t>> m = {{"q", {z_.heads * z_.dim, width_}}, {"k", {z_.kv_heads * z_.dim, width_}}, {"v", {z_.kv_heads * z_.vdim, width_}}, {"g", {z_.heads, width_}},
+                                                     {"rel", {-1, z_.heads}}, {"talk", {z_.heads, z_.heads}}, {"pb", {z_.heads}}, {"o", {width_, z_.heads * z_.vdim}}};
+    if (z_.value_mixing) m["vmix"] = {};
     return m;
 }
 
 void SigmoidAttention::set_free_size(const std::string& name, int64_t numel) {
-    if (name == "rel") bias_rows_ = numel / heads_;
+    if (name == "rel") bias_rows_ = numel / z_.heads;
 }
 
 void SigmoidAttention::load_parameter(const std::string& name, const float* v) {
-    const int64_t q = heads_ * dim_, k = kv_heads_ * dim_, vv = kv_heads_ * vdim_;
+    const int64_t q = z_.heads * z_.dim, k = z_.kv_heads * z_.dim, vv = z_.kv_heads * z_.vdim;
     if (name == "q") load_rows(in_weight_, 0, q, width_, v);
     else if (name == "k") load_rows(in_weight_, q, k, width_, v);
     else if (name == "v") load_rows(in_weight_, q + k, vv, width_, v);
-    else if (name == "g") load_rows(in_weight_, q + k + vv, heads_, width_, v);
+    else if (name == "g") load_rows(in_weight_, q + k + vv, z_.heads, width_, v);
     else if (name == "o") load_rows(out_weight_, 0, width_, mixed_cols_, v);
     else if (name == "vmix") lambda_ = v[0];
-    else if (name == "rel") { host_rel_.assign(v, v + bias_rows_ * heads_); fold_bias(); }
-    else if (name == "pb") { host_offset_.assign(v, v + heads_); fold_bias(); }
-    else if (name == "talk") { host_talk_.assign(v, v + heads_ * heads_); load_vector(talk_, 0, heads_ * heads_, v); fold_bias(); }
+    else if (name == "rel") { host_rel_.assign(v, v + bias_rows_ * z_.heads); fold_bias(); }
+    else if (name == "pb") { host_offset_.assign(v, v + z_.heads); fold_bias(); }
+    else if (name == "talk") { host_talk_.assign(v, v + z_.heads * z_.heads); load_vector(talk_, 0, z_.heads * z_.heads, v); fold_bias(); }
     else throw std::runtime_error("SigmoidAttention: no parameter named " + name);
 }
 
@@ -326,28 +329,28 @@ void SigmoidAttention::fold_bias() {
     if (host_rel_.empty() || host_talk_.empty() || host_offset_.empty()) return;
     std::vector<int64_t> bucket;
     for (int64_t n = 0;; ++n) {
-        bucket.push_back(distance_bucket(n, bias_rows_, reach_));
+        bucket.push_back(distance_bucket(n, bias_rows_, z_.reach));
         if (bucket.back() == bias_rows_ - 1) break;
     }
     const int64_t len = static_cast<int64_t>(bucket.size());
-    std::vector<float> folded(static_cast<size_t>(heads_ * len));
-    for (int64_t h = 0; h < heads_; ++h) {
+    std::vector<float> folded(static_cast<size_t>(z_.heads * len));
+    for (int64_t h = 0; h < z_.heads; ++h) {
         std::vector<float> by_row(static_cast<size_t>(bias_rows_));
         for (int64_t r = 0; r < bias_rows_; ++r) {
             double x = host_offset_[static_cast<size_t>(h)];
-            for (int64_t g = 0; g < heads_; ++g) x += static_cast<double>(host_talk_[static_cast<size_t>(h * heads_ + g)]) * host_rel_[static_cast<size_t>(r * heads_ + g)];
+            for (int64_t g = 0; g < z_.heads; ++g) x += static_cast<double>(host_talk_[static_cast<size_t>(h * z_.heads + g)]) * host_rel_[static_cast<size_t>(r * z_.heads + g)];
             by_row[static_cast<size_t>(r)] = static_cast<float>(x);
         }
         for (int64_t n = 0; n < len; ++n) folded[static_cast<size_t>(h * len + n)] = by_row[static_cast<size_t>(bucket[static_cast<size_t>(n)])];
     }
-    bias_ = empty({heads_, len}, DType::Float32, Device::CUDA);
+    bias_ = empty({z_.heads, len}, DType::Float32, Device::CUDA);
     bias_.copy_from_host(folded.data());
 }
 
 std::unique_ptr<SequenceState> SigmoidAttention::make_state(int64_t slots, int64_t max_len) const {
     auto st = std::make_unique<SequenceState>();
-    st->ring = zeros({slots, max_len, pad8(kv_heads_ * dim_)}, dtype_, Device::CUDA);
-    st->values = zeros({slots, max_len, pad8(kv_heads_ * vdim_)}, dtype_, Device::CUDA);
+    st->ring = zeros({slots, max_len, pad8(z_.kv_heads * z_.dim)}, dtype_, Device::CUDA);
+    st->values = zeros({slots, max_len, pad8(z_.kv_heads * z_.vdim)}, dtype_, Device::CUDA);
     return st;
 }
 
@@ -359,11 +362,11 @@ struct SigmoidAttention::Args {
         a.stream = current_stream();
         a.dtype = m.dtype_ == DType::Float32 ? VB200_F32 : VB200_BF16;
         a.B = static_cast<int>(st.B); a.T = static_cast<int>(st.T);
-        a.H = static_cast<int>(m.heads_); a.G = static_cast<int>(m.kv_heads_); a.dim = static_cast<int>(m.dim_); a.vdim = static_cast<int>(m.vdim_);
-        a.scale = static_cast<float>(m.scale_); a.eps = static_cast<float>(m.eps_);
-        a.temp_coef = static_cast<float>(m.temp_coef_); a.temp_every = static_cast<int>(std::min<int64_t>(m.temp_every_, INT32_MAX));
+        a.H = static_cast<int>(m.z_.heads); a.G = static_cast<int>(m.z_.kv_heads); a.dim = static_cast<int>(m.z_.dim); a.vdim = static_cast<int>(m.z_.vdim);
+        a.scale = static_cast<float>(m.z_.scale); a.eps = static_cast<float>(m.eps_);
+        a.temp_coef = static_cast<float>(m.z_.temp_coef); a.temp_every = static_cast<int>(std::min<int64_t>(m.z_.temp_every, INT32_MAX));
         a.ldp = m.proj_ld(); a.ldo = m.mixed_ld();
-        a.ldk = pad8(m.kv_heads_ * m.dim_); a.ldv = pad8(m.kv_heads_ * m.vdim_);
+        a.ldk = pad8(m.z_.kv_heads * m.z_.dim); a.ldv = pad8(m.z_.kv_heads * m.z_.vdim);
         a.talk = m.talk_.data_ptr<float>(); a.bias = m.bias_.data_ptr<float>(); a.n_bias = static_cast<int>(m.bias_.shape()[1]);
         a.lambda = m.lambda_;
         a.slots = st.slots; a.pos = st.pos;
@@ -386,7 +389,7 @@ void SigmoidAttention::forward(const MixerStep& st, SequenceState& state, Tensor
     x.a.out = mixed.data_ptr<char>();
     x.a.workspace = st.workspace;
     x.a.workspace_bytes = static_cast<size_t>(st.workspace_bytes);
-    if (value_mixing_) {
+    if (z_.value_mixing) {
         if (!st.values) throw std::runtime_error("SigmoidAttention: value mixing needs the step's shared values");
         x.a.first_values = st.values->data;
         x.a.value_role = st.values->filled ? 2 : 1;
@@ -397,55 +400,58 @@ void SigmoidAttention::forward(const MixerStep& st, SequenceState& state, Tensor
 
 // ---- Mamba-1 -------------------------------------------------------------------------------------
 
-Mamba1::Mamba1(const Json& m, int64_t width, int64_t width_ld, double eps, DType dtype) : SequenceMixer(width, width_ld, eps, dtype) {
-    inner_ = positive(m, "inner");
-    state_ = positive(m, "state");
-    rank_ = positive(m, "dt_rank");
-    taps_ = positive(m, "conv");
-    inner8_ = pad8(inner_); state8_ = pad8(state_); rank8_ = pad8(rank_);
-    proj_rows_ = 2 * inner8_;
-    mixed_cols_ = inner_;
+Mamba1::Sizes::Sizes(const Json& m) {
+    inner = positive(m, "inner");
+    state = positive(m, "state");
+    rank = positive(m, "dt_rank");
+    taps = positive(m, "conv");
+    inner8 = pad8(inner); state8 = pad8(state); rank8 = pad8(rank);
+}
+
+Mamba1::Mamba1(const Json& m, int64_t width, int64_t width_ld, double eps, DType dtype) : SequenceMixer(width, width_ld, eps, dtype), z_(m) {
+    proj_rows_ = 2 * z_.inner8;
+    mixed_cols_ = z_.inner;
     in_weight_ = zeros({proj_rows_, width_ld}, dtype, Device::CUDA);
     out_weight_ = zeros({width_ld, mixed_ld()}, dtype, Device::CUDA);
-    w_x_ = zeros({rank8_ + 2 * state8_, inner8_}, dtype, Device::CUDA);
-    w_dt_ = zeros({inner8_, rank8_}, dtype, Device::CUDA);
-    conv_w_ = zeros({inner8_, taps_}, DType::Float32, Device::CUDA);
-    conv_b_ = zeros({inner8_}, DType::Float32, Device::CUDA);
-    dt_bias_ = zeros({inner8_}, DType::Float32, Device::CUDA);
-    a_ = zeros({inner8_, state8_}, DType::Float32, Device::CUDA);
-    d_ = zeros({inner8_}, DType::Float32, Device::CUDA);
+    w_x_ = zeros({z_.rank8 + 2 * z_.state8, z_.inner8}, dtype, Device::CUDA);
+    w_dt_ = zeros({z_.inner8, z_.rank8}, dtype, Device::CUDA);
+    conv_w_ = zeros({z_.inner8, z_.taps}, DType::Float32, Device::CUDA);
+    conv_b_ = zeros({z_.inner8}, DType::Float32, Device::CUDA);
+    dt_bias_ = zeros({z_.inner8}, DType::Float32, Device::CUDA);
+    a_ = zeros({z_.inner8, z_.state8}, DType::Float32, Device::CUDA);
+    d_ = zeros({z_.inner8}, DType::Float32, Device::CUDA);
 }
 
 std::map<std::string, std::vector<int64_t>> Mamba1::parameter_shapes() const {
-    return {{"in", {2 * inner_, width_}}, {"conv", {inner_, taps_}}, {"conv.b", {inner_}}, {"x", {rank_ + 2 * state_, inner_}}, {"dt", {inner_, rank_}}, {"dt.b", {inner_}},
-            {"A_log", {inner_, state_}}, {"D", {inner_}}, {"o", {width_, inner_}}};
+    return {{"in", {2 * z_.inner, width_}}, {"conv", {z_.inner, z_.taps}}, {"conv.b", {z_.inner}}, {"x", {z_.rank + 2 * z_.state, z_.inner}}, {"dt", {z_.inner, z_.rank}}, {"dt.b", {z_.inner}},
+            {"A_log", {z_.inner, z_.state}}, {"D", {z_.inner}}, {"o", {width_, z_.inner}}};
 }
 
 void Mamba1::load_parameter(const std::string& name, const float* v) {
     if (name == "in") {
-        load_rows(in_weight_, 0, inner_, width_, v);
-        load_rows(in_weight_, inner8_, inner_, width_, v + inner_ * width_);
+        load_rows(in_weight_, 0, z_.inner, width_, v);
+        load_rows(in_weight_, z_.inner8, z_.inner, width_, v + z_.inner * width_);
     } else if (name == "x") {
-        load_rows(w_x_, 0, rank_, inner_, v);
-        load_rows(w_x_, rank8_, state_, inner_, v + rank_ * inner_);
-        load_rows(w_x_, rank8_ + state8_, state_, inner_, v + (rank_ + state_) * inner_);
+        load_rows(w_x_, 0, z_.rank, z_.inner, v);
+        load_rows(w_x_, z_.rank8, z_.state, z_.inner, v + z_.rank * z_.inner);
+        load_rows(w_x_, z_.rank8 + z_.state8, z_.state, z_.inner, v + (z_.rank + z_.state) * z_.inner);
     } else if (name == "A_log") {
-        std::vector<float> a(static_cast<size_t>(inner_ * state_));
+        std::vector<float> a(static_cast<size_t>(z_.inner * z_.state));
         for (size_t i = 0; i < a.size(); ++i) a[i] = static_cast<float>(-std::exp(static_cast<double>(v[i])));
-        load_rows(a_, 0, inner_, state_, a.data());
-    } else if (name == "conv") load_rows(conv_w_, 0, inner_, taps_, v);
-    else if (name == "conv.b") load_vector(conv_b_, 0, inner_, v);
-    else if (name == "dt") load_rows(w_dt_, 0, inner_, rank_, v);
-    else if (name == "dt.b") load_vector(dt_bias_, 0, inner_, v);
-    else if (name == "D") load_vector(d_, 0, inner_, v);
-    else if (name == "o") load_rows(out_weight_, 0, width_, inner_, v);
+        load_rows(a_, 0, z_.inner, z_.state, a.data());
+    } else if (name == "conv") load_rows(conv_w_, 0, z_.inner, z_.taps, v);
+    else if (name == "conv.b") load_vector(conv_b_, 0, z_.inner, v);
+    else if (name == "dt") load_rows(w_dt_, 0, z_.inner, z_.rank, v);
+    else if (name == "dt.b") load_vector(dt_bias_, 0, z_.inner, v);
+    else if (name == "D") load_vector(d_, 0, z_.inner, v);
+    else if (name == "o") load_rows(out_weight_, 0, width_, z_.inner, v);
     else throw std::runtime_error("Mamba1: no parameter named " + name);
 }
 
 std::unique_ptr<SequenceState> Mamba1::make_state(int64_t slots, int64_t) const {
     auto st = std::make_unique<SequenceState>();
-    st->ring = zeros({slots, taps_, inner8_}, dtype_, Device::CUDA);
-    st->recurrent = zeros({slots, inner8_, state8_}, DType::Float32, Device::CUDA);
+    st->ring = zeros({slots, z_.taps, z_.inner8}, dtype_, Device::CUDA);
+    st->recurrent = zeros({slots, z_.inner8, z_.state8}, DType::Float32, Device::CUDA);
     return st;
 }
 
@@ -456,8 +462,8 @@ struct Mamba1::Args {
         a.device = m.in_weight_.device_index();
         a.stream = current_stream();
         a.dtype = m.dtype_ == DType::Float32 ? VB200_F32 : VB200_BF16;
-        a.B = static_cast<int>(st.B); a.T = static_cast<int>(st.T); a.inner = static_cast<int>(m.inner8_); a.N = static_cast<int>(m.state8_);
-        a.rank = static_cast<int>(m.rank8_); a.taps = static_cast<int>(m.taps_);
+        a.B = static_cast<int>(st.B); a.T = static_cast<int>(st.T); a.inner = static_cast<int>(m.z_.inner8); a.N = static_cast<int>(m.z_.state8);
+        a.rank = static_cast<int>(m.z_.rank8); a.taps = static_cast<int>(m.z_.taps);
         a.ldp = m.proj_ld(); a.ldo = m.mixed_ld();
         a.conv_w = m.conv_w_.data_ptr<float>(); a.conv_b = m.conv_b_.data_ptr<float>();
         a.w_x = m.w_x_.data_ptr<char>(); a.w_dt = m.w_dt_.data_ptr<char>();
@@ -480,6 +486,13 @@ void Mamba1::forward(const MixerStep& st, SequenceState& state, Tensor& projecte
     x.a.workspace = st.workspace;
     x.a.workspace_bytes = static_cast<size_t>(st.workspace_bytes);
     check(vb200_selective_forward(&x.a), "mamba1");
+}
+
+int64_t check_mixer(const std::string& type, const Json& mixer) {
+    if (type == "attention") return SigmoidAttention::Sizes(mixer).shared_value_cols();
+    if (type == "mamba1") (void)Mamba1::Sizes(mixer);
+    else if (type != "latent_attention" && type != "mamba2") throw std::runtime_error("configuration: no sequence mixer of type '" + type + "'");
+    return 0;
 }
 
 std::unique_ptr<SequenceMixer> make_mixer(const std::string& type, const Json& mixer, int64_t width, int64_t width_ld, double eps, DType dtype) {
