@@ -778,6 +778,9 @@ def run_ours(args):
     if only == "hybrid":
         from vesper_b200.hybrid_bench import bench_hybrid
         hyb = bench_hybrid(cx, K, W, layers=args.model_layers, part=args.hybrid_part)
+    elif only == "zudisun":
+        from vesper_b200.zudisun_bench import bench_zudisun
+        hyb = bench_zudisun(cx, K, W, layers=args.model_layers, part=args.hybrid_part)
     cpu_baseline = None
     if cx.rank == 0 and cx.world == 1 and not args.no_cpu_baseline and only == "all":
         cpu_baseline, _ = cpu_prefill_sample(target_seconds=12.0)
@@ -800,7 +803,7 @@ def run_ours(args):
             "model": mdl,
         }
         if hyb is not None:
-            line["hybrid"] = hyb
+            line[only] = hyb
         if cpu_baseline is not None:
             line["cpu_baseline"] = cpu_baseline
         emit(line)
@@ -832,8 +835,8 @@ def main():
     ap.add_argument("--decode-steps", type=int, default=C3["steps"], help="consecutive decode steps (default: the workload's 256)")
     ap.add_argument("--model-layers", type=int, default=0, help="profiling runs: depth of the model section's decoder (default: the workload's 24)")
     ap.add_argument("--model-new", type=int, default=0, help="profiling runs: tokens to generate in the model section (default: 128)")
-    ap.add_argument("--only", default="all", choices=["all", "prefill", "decode", "sharded", "model", "hybrid"],
-                    help="run one section (profiling runs); hybrid: the hybrid decoder's mixers and model beside the Llama-style decoder (not part of the default run)")
+    ap.add_argument("--only", default="all", choices=["all", "prefill", "decode", "sharded", "model", "hybrid", "zudisun"],
+                    help="run one section (profiling runs); hybrid, zudisun: the mixers and models of the Nitenex and Zudisun decoders beside the Llama-style decoder (not part of the default run)")
     ap.add_argument("--hybrid-part", default="all", choices=["all", "kernels", "models"])
     args = ap.parse_args()
     if args.impl == "reference":

@@ -100,7 +100,7 @@ class GreedyArgs(C.Structure):
     ]
 
 
-EPI_BF16, EPI_F32, EPI_ADD_F32, EPI_SWIGLU, EPI_RELU2 = 0, 1, 2, 3, 4
+EPI_BF16, EPI_F32, EPI_ADD_F32, EPI_SWIGLU, EPI_RELU2, EPI_REGLU = 0, 1, 2, 3, 4, 5
 
 _lib = None
 

@@ -47,6 +47,22 @@ template <typename T> __device__ __forceinline__ float softplus_for(float x) {
     return fmaxf(x, 0.f) + s * r;
 }
 
+template <int N> __device__ __forceinline__ void load_states(const __nv_bfloat16* p, float (&v)[N]) {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+        const uint2 u = *reinterpret_cast<const uint2*>(p + i);
+        const float2 a = Elem<__nv_bfloat16>::unpack2(u.x), b = Elem<__nv_bfloat16>::unpack2(u.y);
+        v[i] = a.x; v[i + 1] = a.y; v[i + 2] = b.x; v[i + 3] = b.y;
+    }
+}
+template <int N> __device__ __forceinline__ void load_states(const float* p, float (&v)[N]) {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(p + i);
+        v[i] = a.x; v[i + 1] = a.y; v[i + 2] = a.z; v[i + 3] = a.w;
+    }
+}
+
 template <typename T, int LP, int NI>
 struct ScanTile {
     static constexpr int kCh = kThreads / LP;                  // channels per CTA
@@ -67,7 +83,7 @@ __global__ void __launch_bounds__(kThreads)
 selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restrict__ xc, const T* __restrict__ xdbl, const float* __restrict__ dt, float* __restrict__ state,
                       T* __restrict__ out) {
     using S = ScanTile<T, LP, NI>;
-    constexpr int CH = S::kCh, V = 16 / sizeof(T), kTile = S::kTile;
+    constexpr int CH = S::kCh, V = 16 / sizeof(T), kTile = S::kTile, U = NI <= 8 && sizeof(T) == 2 ? 4 : 1;
     extern __shared__ __align__(16) uint8_t raw[];
     S& sm = *reinterpret_cast<S*>(raw);
     const int tid = threadIdx.x, lane = tid % LP, ch = tid / LP, b = blockIdx.y, c0 = blockIdx.x * CH, c = c0 + ch;
@@ -128,34 +144,53 @@ selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
             st.dt[t][k] = softplus_for<T>(st.dt[t][k] + bk);
         }
         __syncthreads();
-#pragma unroll 4
-        for (int t = 0; t < nt; ++t) {
-            const float d = st.dt[t][ch], x = Elem<T>::to_f(st.x[t][ch]), dx = d * x, dl = decay_dt<T>(d);
-            float y = 0.f;
-            const T *Bt = &st.bc[0][t][lane * NI], *Ct = &st.bc[1][t][lane * NI];
+        // U tokens at a time: their loads, exponentials and sums are independent, only S += is a chain
+        for (int tb = 0; tb < nt; tb += U) {
+            float d[U], dx[U], y[U];
 #pragma unroll
-            for (int i = 0; i < NI; i += 4) {
-                float bn[4], cn[4];
-                if constexpr (sizeof(T) == 2) {
-                    const uint2 ub = *reinterpret_cast<const uint2*>(Bt + i), uc = *reinterpret_cast<const uint2*>(Ct + i);
-                    const float2 b0 = Elem<__nv_bfloat16>::unpack2(ub.x), b1 = Elem<__nv_bfloat16>::unpack2(ub.y);
-                    const float2 c0_ = Elem<__nv_bfloat16>::unpack2(uc.x), c1_ = Elem<__nv_bfloat16>::unpack2(uc.y);
-                    bn[0] = b0.x; bn[1] = b0.y; bn[2] = b1.x; bn[3] = b1.y;
-                    cn[0] = c0_.x; cn[1] = c0_.y; cn[2] = c1_.x; cn[3] = c1_.y;
-                } else {
-                    const float4 vb = *reinterpret_cast<const float4*>(Bt + i), vc = *reinterpret_cast<const float4*>(Ct + i);
-                    bn[0] = vb.x; bn[1] = vb.y; bn[2] = vb.z; bn[3] = vb.w;
-                    cn[0] = vc.x; cn[1] = vc.y; cn[2] = vc.z; cn[3] = vc.w;
-                }
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    S_[i + e] = decayed<T>(S_[i + e], dl, a[i + e], dx * bn[e]);
-                    y = fmaf(S_[i + e], cn[e], y);
-                }
+            for (int u = 0; u < U; ++u) {
+                const int t = tb + u;                    // past the portion: step size 0 keeps the state
+                d[u] = t < nt ? st.dt[t][ch] : 0.f;
+                const float x = Elem<T>::to_f(st.x[t][ch]);
+                dx[u] = d[u] * x;
+                d[u] = decay_dt<T>(d[u]);
+                y[u] = lane == 0 ? Dc * x : 0.f;
             }
 #pragma unroll
-            for (int o = LP / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xFFFFFFFFu, y, o);
-            if (lane == 0) sm.y[t][ch] = fmaf(Dc, x, y);
+            for (int u = 0; u < U; ++u) {
+                float bn[NI], cn[NI];
+                load_states(&st.bc[0][tb + u][lane * NI], bn);
+                load_states(&st.bc[1][tb + u][lane * NI], cn);
+#pragma unroll
+                for (int i = 0; i < NI; ++i) {
+                    S_[i] = decayed<T>(S_[i], d[u], a[i], dx[u] * bn[i]);
+                    y[u] = fmaf(S_[i], cn[i], y[u]);
+                }
+            }
+            // sums over the channel's lanes: halves of the tokens are exchanged until every lane holds U / LP of them (or all hold all)
+            if constexpr (U == 4 && LP >= 4) {
+                float z[2];
+                const bool odd = lane & 1;
+#pragma unroll
+                for (int k = 0; k < 2; ++k) {            // lanes l, l ^ 1: tokens 0, 1 stay with even lanes, 2, 3 with odd ones
+                    const float send = odd ? y[k] : y[k + 2], keep = odd ? y[k + 2] : y[k];
+                    z[k] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 1);
+                }
+                const bool high = lane & 2;
+                const float send = high ? z[0] : z[1], keep = high ? z[1] : z[0];
+                float v = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 2);
+#pragma unroll
+                for (int o = 4; o < LP; o <<= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
+                const int t = tb + (lane & 1) * 2 + ((lane >> 1) & 1);
+                if (lane < 4 && t < nt) sm.y[t][ch] = v;
+            } else {
+#pragma unroll
+                for (int u = 0; u < U; ++u) {
+#pragma unroll
+                    for (int o = LP / 2; o > 0; o >>= 1) y[u] += __shfl_xor_sync(0xFFFFFFFFu, y[u], o);
+                    if (lane == 0 && tb + u < nt) sm.y[tb + u][ch] = y[u];
+                }
+            }
         }
         __syncthreads();
         // gate and store, two channels per thread
@@ -313,7 +348,12 @@ int launch_selective(cudaStream_t s, const vb200_selective_args& a, const Select
             } else {
                 const size_t smem = sizeof(ScanTile<T, LP, NI>);
                 rc = allow_smem(selective_scan_kernel<T, LP, NI>, smem);
-                if (rc == VB200_OK) rc = launch_pdl(selective_scan_kernel<T, LP, NI>, grid, dim3(kThreads), smem, s, p, proj, x, d, dt, a.state, out);
+                // no programmatic launch: scheduled while the product before drains, the CTAs would pile up on the SMs that finish first
+                if (rc == VB200_OK) {
+                    selective_scan_kernel<T, LP, NI><<<grid, kThreads, smem, s>>>(p, proj, x, d, dt, a.state, out);
+                    note_launch();
+                    VB200_CUDA_TRY(cudaPeekAtLastError());
+                }
                 note_selective_kernel("selective_scan_kernel");
             }
             profile_mark_end(s);

@@ -8,7 +8,7 @@
 //
 // One CTA per 128 query rows of one (batch, head), one CTA per SM; keys in blocks of 128.
 //   warps 0-7  weights and epilogue: warps w and w + 4 own the same 32 rows (TMEM lanes), and 64 keys of a block each
-//   warp  8    TMA producer: Q once, then one ring of [128 rows x 64 columns] boxes that K and V share in the order of their use
+//   warp  8    TMA producer: Q once, then a ring of K stages (one or two [128 keys x 64 columns] boxes) and one of V blocks
 //   warp  9    tcgen05.mma issuer, TMEM owner
 // TMEM (512 columns): S0 [0, 128) S1 [128, 256) O [256, 256 + vdim).  QK of block j+1 is issued before PV of block j.  The weights stay
 // fp32-class in the second product: each half of a block is packed over its own 64 columns of S as bf16 hi (32 columns) and lo (32).
@@ -20,7 +20,8 @@ namespace {
 
 constexpr int kRows = 128, kKeys = 128;
 constexpr int kBox = 128 * 128;               // [128 rows x 64 columns]
-constexpr int kMaxSlots = 12;
+constexpr int kMaxStages = 6;
+constexpr int kBoxesPerSm = 14;               // of 16 KB: Q, K ring and V ring of the one CTA
 constexpr int kWeightThreads = 256;
 constexpr int kThreads = kWeightThreads + 64;
 constexpr float kCut = 60.0f;
@@ -29,7 +30,8 @@ struct SigMaps { CUtensorMap q, k, v; };
 
 struct SigTileParams {
     int T, start_pos, vdim, R, n_bias, gate_col;
-    int ks, nb_k, nb_v, slots_ring;           // 16-column steps of kd, 64-column boxes, ring slots
+    int ks, nb_k, nb_v, n_pv;                 // 16-column steps of kd, 64-column boxes, columns of the second product
+    int kbs, k_stages, v_stages;              // boxes per K stage, ring depths
     const float* bias;
     const __nv_bfloat16* proj;
     __nv_bfloat16* out;
@@ -39,7 +41,7 @@ struct SigTileParams {
 };
 
 struct SigBars {
-    uint64_t q_full, full[kMaxSlots], empty[kMaxSlots], s_full[2], p_ready[2], o_done, drain;
+    uint64_t q_full, k_full[kMaxStages], k_empty[kMaxStages], v_full[kMaxStages], v_empty[kMaxStages], s_full[2], p_ready[2], o_done, drain;
     uint32_t tmem;
     int abort_flag;
 };
@@ -58,13 +60,14 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
     const int r0 = static_cast<int>(gridDim.z - 1 - blockIdx.z) * kRows, h = blockIdx.x, b = blockIdx.y;      // tiles with most keys first
     const int last_key = p.start_pos + min(r0 + kRows, p.T) - 1, n_blk = last_key / kKeys + 1;
     uint8_t* q_smem = smem;
-    uint8_t* ring = q_smem + p.nb_k * kBox;
+    uint8_t* k_ring = q_smem + p.nb_k * kBox;
+    uint8_t* v_ring = k_ring + p.k_stages * p.kbs * kBox;
     const WaitCtx ctx{&bar.abort_flag, p.status};
 
     if (threadIdx.x == 0) {
         bar.abort_flag = 0;
         mbar_init(&bar.q_full, 1);
-        for (int i = 0; i < kMaxSlots; ++i) { mbar_init(&bar.full[i], 1); mbar_init(&bar.empty[i], 1); }
+        for (int i = 0; i < kMaxStages; ++i) { mbar_init(&bar.k_full[i], 1); mbar_init(&bar.k_empty[i], 1); mbar_init(&bar.v_full[i], 1); mbar_init(&bar.v_empty[i], 1); }
         for (int i = 0; i < 2; ++i) { mbar_init(&bar.s_full[i], 1); mbar_init(&bar.p_ready[i], kWeightThreads); }
         mbar_init(&bar.o_done, 1);
         mbar_init(&bar.drain, 1);
@@ -87,43 +90,47 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
             for (int i = 0; i < p.nb_k; ++i) tma_load_4d(q_smem + i * kBox, &maps.q, &bar.q_full, i * 64, h, r0, b);
             bool ok = true;
             int n = 0;
-            auto load = [&](const CUtensorMap* m, int col, int head, int key) {
-                const int s = n % p.slots_ring, round = n / p.slots_ring;
-                if (round > 0) ok = ok && mbar_wait(&bar.empty[s], (round - 1) & 1, ctx, 0xD1);
-                if (!ok) return;
-                mbar_arrive_expect_tx(&bar.full[s], kBox);
-                tma_load_4d(ring + s * kBox, m, &bar.full[s], col, head, key, slot);
-                ++n;
+            auto load_k = [&](int j) {
+                for (int i = 0; i < p.nb_k && ok; i += p.kbs, ++n) {
+                    const int st = n % p.k_stages, round = n / p.k_stages;
+                    if (round > 0) ok = mbar_wait(&bar.k_empty[st], (round - 1) & 1, ctx, 0xD1);
+                    if (!ok) return;
+                    mbar_arrive_expect_tx(&bar.k_full[st], p.kbs * kBox);
+                    for (int x = 0; x < p.kbs; ++x) tma_load_4d(k_ring + (st * p.kbs + x) * kBox, &maps.k, &bar.k_full[st], (i + x) * 64, 0, j * kKeys, slot);
+                }
             };
-            for (int i = 0; i < p.nb_k && ok; ++i) load(&maps.k, i * 64, 0, 0);
+            load_k(0);
             for (int j = 0; j < n_blk && ok; ++j) {
-                if (j + 1 < n_blk)
-                    for (int i = 0; i < p.nb_k && ok; ++i) load(&maps.k, i * 64, 0, (j + 1) * kKeys);
-                for (int i = 0; i < p.nb_v && ok; ++i) load(&maps.v, i * 64, h / p.R, j * kKeys);
+                if (j + 1 < n_blk) load_k(j + 1);
+                if (!ok) break;
+                const int st = j % p.v_stages, round = j / p.v_stages;
+                if (round > 0) ok = mbar_wait(&bar.v_empty[st], (round - 1) & 1, ctx, 0xD8);
+                if (!ok) break;
+                mbar_arrive_expect_tx(&bar.v_full[st], p.nb_v * kBox);
+                for (int i = 0; i < p.nb_v; ++i) tma_load_4d(v_ring + (st * p.nb_v + i) * kBox, &maps.v, &bar.v_full[st], i * 64, h / p.R, j * kKeys, slot);
             }
         }
     } else if (warp == 9) {
         if (lane == 0) {
             const uint32_t idesc_qk = make_idesc_f16(1, 0, 0, kRows, kKeys);
-            const uint32_t q_addr = smem_u32(q_smem), ring_addr = smem_u32(ring);
+            const uint32_t idesc_pv = make_idesc_f16(1, 0, 1, kRows, p.n_pv);
+            const uint32_t q_addr = smem_u32(q_smem), k_addr = smem_u32(k_ring), v_addr = smem_u32(v_ring);
             bool ok = mbar_wait(&bar.q_full, 0, ctx, 0xD2);
             int n = 0;
-            auto take = [&]() -> uint32_t {              // the next box of the ring
-                const int s = n % p.slots_ring;
-                ok = ok && mbar_wait(&bar.full[s], (n / p.slots_ring) & 1, ctx, 0xD3);
-                tc_fence_after();
-                return ring_addr + s * kBox;
-            };
-            auto give = [&]() { umma_commit(&bar.empty[n % p.slots_ring]); ++n; };
             auto issue_qk = [&](int j) {
                 const uint32_t d = tmem + (j & 1) * kKeys;
-                for (int i = 0; i < p.nb_k; ++i) {
-                    const uint32_t kb = take();
+                for (int i = 0; i < p.nb_k; i += p.kbs, ++n) {
+                    const int st = n % p.k_stages;
+                    ok = mbar_wait(&bar.k_full[st], (n / p.k_stages) & 1, ctx, 0xD3);
                     if (!ok) return;
-                    const int steps = min(4, p.ks - i * 4);
-                    for (int kk = 0; kk < steps; ++kk)
-                        umma_ss(d, make_smem_desc_sw128(q_addr + i * kBox + kk * 32, 16, 1024), make_smem_desc_sw128(kb + kk * 32, 16, 1024), idesc_qk, (i | kk) ? 1u : 0u);
-                    give();
+                    tc_fence_after();
+                    for (int x = 0; x < p.kbs; ++x) {
+                        const uint32_t kb = k_addr + (st * p.kbs + x) * kBox, qb = q_addr + (i + x) * kBox;
+                        const int steps = min(4, p.ks - (i + x) * 4);
+                        for (int kk = 0; kk < steps; ++kk)
+                            umma_ss(d, make_smem_desc_sw128(qb + kk * 32, 16, 1024), make_smem_desc_sw128(kb + kk * 32, 16, 1024), idesc_qk, (i | x | kk) ? 1u : 0u);
+                    }
+                    umma_commit(&bar.k_empty[st]);
                 }
                 umma_commit(&bar.s_full[j & 1]);
             };
@@ -131,20 +138,15 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
             for (int j = 0; j < n_blk && ok; ++j) {
                 if (j + 1 < n_blk) issue_qk(j + 1);      // its S held the weights of block j-1, whose product was issued before
                 if (!ok) break;
-                ok = mbar_wait(&bar.p_ready[j & 1], (j >> 1) & 1, ctx, 0xD4);
+                const int st = j % p.v_stages;
+                ok = mbar_wait(&bar.v_full[st], (j / p.v_stages) & 1, ctx, 0xD9) && mbar_wait(&bar.p_ready[j & 1], (j >> 1) & 1, ctx, 0xD4);
                 if (!ok) break;
                 tc_fence_after();
-                const uint32_t a = tmem + (j & 1) * kKeys;
-                for (int i = 0; i < p.nb_v; ++i) {
-                    const uint32_t vb = take();
-                    if (!ok) break;
-                    const uint32_t idesc_pv = make_idesc_f16(1, 0, 1, kRows, min(64, (p.vdim - i * 64 + 15) / 16 * 16));
-                    for (int half = 0; half < 2; ++half)         // hi, lo
-                        for (int kk = 0; kk < kKeys / 16; ++kk)
-                            umma_ts(tmem + 2 * kKeys + i * 64, a + (kk >> 2) * 64 + half * 32 + (kk & 3) * 8, make_smem_desc_sw128(vb + kk * 2048, kBox, 1024), idesc_pv,
-                                    (j | half | kk) ? 1u : 0u);
-                    give();
-                }
+                const uint32_t a = tmem + (j & 1) * kKeys, vb = v_addr + st * p.nb_v * kBox;
+                for (int half = 0; half < 2; ++half)     // hi, lo
+                    for (int kk = 0; kk < kKeys / 16; ++kk)
+                        umma_ts(tmem + 2 * kKeys, a + (kk >> 2) * 64 + half * 32 + (kk & 3) * 8, make_smem_desc_sw128(vb + kk * 2048, kBox, 1024), idesc_pv, (j | half | kk) ? 1u : 0u);
+                umma_commit(&bar.v_empty[st]);
             }
             if (ok) umma_commit(&bar.o_done);
             umma_commit(&bar.drain);                     // nothing may be in flight when TMEM is freed
@@ -254,9 +256,14 @@ int launch_sig_prefill_sm100(cudaStream_t s, const vb200_sigattn_args& a, const 
     p.ks = (kd + 15) / 16; p.nb_k = (kd + 63) / 64; p.nb_v = (a.vdim + 63) / 64;
     p.bias = a.bias; p.proj = static_cast<const __nv_bfloat16*>(a.proj); p.out = static_cast<__nv_bfloat16*>(a.out);
     p.ldp = a.ldp; p.ldo = a.ldo; p.slots = a.slots; p.status = status;
-    p.slots_ring = (208 * 1024 - p.nb_k * kBox) / kBox;
-    if (p.slots_ring > kMaxSlots) p.slots_ring = kMaxSlots;
-    size_t smem = static_cast<size_t>(p.nb_k + p.slots_ring) * kBox;
+    p.n_pv = pad_to(a.vdim, 16);
+    // rings: what Q leaves.  Two boxes per K stage halve the commits between products; V needs depth only where K is short
+    const int left = kBoxesPerSm - p.nb_k;
+    p.v_stages = left - 2 * p.nb_v >= 4 ? 2 : 1;
+    p.kbs = p.nb_k % 2 == 0 ? 2 : 1;
+    p.k_stages = (left - p.v_stages * p.nb_v) / p.kbs;
+    if (p.k_stages > kMaxStages) p.k_stages = kMaxStages;
+    size_t smem = static_cast<size_t>(p.nb_k + p.k_stages * p.kbs + p.v_stages * p.nb_v) * kBox;
     if (smem < 120 * 1024) smem = 120 * 1024;            // never a second CTA on an SM: it would find no TMEM
     if (int rc = allow_smem(sig_prefill_sm100_kernel, smem)) return rc;
     return launch_pdl(sig_prefill_sm100_kernel, dim3(static_cast<unsigned>(a.H), static_cast<unsigned>(a.B), static_cast<unsigned>((a.T + kRows - 1) / kRows)), dim3(kThreads), smem, s,
