@@ -48,6 +48,7 @@ template <typename T> __device__ __forceinline__ float softplus_for(float x) {
 }
 
 template <int N> __device__ __forceinline__ void load_states(const __nv_bfloat16* p, float (&v)[N]) {
+    static_assert(N % 4 == 0, "four at a time");
 #pragma unroll
     for (int i = 0; i < N; i += 4) {
         const uint2 u = *reinterpret_cast<const uint2*>(p + i);
@@ -56,6 +57,10 @@ template <int N> __device__ __forceinline__ void load_states(const __nv_bfloat16
     }
 }
 template <int N> __device__ __forceinline__ void load_states(const float* p, float (&v)[N]) {
+    if constexpr (N == 2) {
+        const float2 a = *reinterpret_cast<const float2*>(p);
+        v[0] = a.x; v[1] = a.y;
+    } else
 #pragma unroll
     for (int i = 0; i < N; i += 4) {
         const float4 a = *reinterpret_cast<const float4*>(p + i);
@@ -63,17 +68,44 @@ template <int N> __device__ __forceinline__ void load_states(const float* p, flo
     }
 }
 
+// a lane's states from / to memory; those from `count` on do not exist (zero, not stored)
+template <int N> __device__ __forceinline__ void load_state(const float* p, int count, float (&v)[N]) {
+    constexpr int W = N < 4 ? 2 : 4;
+#pragma unroll
+    for (int i = 0; i < N; i += W) {
+        if constexpr (W == 2) {
+            const float2 u = i < count ? *reinterpret_cast<const float2*>(p + i) : make_float2(0.f, 0.f);
+            v[i] = u.x; v[i + 1] = u.y;
+        } else {
+            const float4 u = i < count ? *reinterpret_cast<const float4*>(p + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            v[i] = u.x; v[i + 1] = u.y; v[i + 2] = u.z; v[i + 3] = u.w;
+        }
+    }
+}
+template <int N> __device__ __forceinline__ void store_state(float* p, int count, const float (&v)[N]) {
+    constexpr int W = N < 4 ? 2 : 4;
+#pragma unroll
+    for (int i = 0; i < N; i += W) {
+        if (i >= count) break;
+        if constexpr (W == 2) *reinterpret_cast<float2*>(p + i) = make_float2(v[i], v[i + 1]);
+        else *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
+    }
+}
+
 template <typename T, int LP, int NI>
 struct ScanTile {
     static constexpr int kCh = kThreads / LP;                  // channels per CTA
     static constexpr int kStates = LP * NI;
-    static constexpr int kTile = kStates * sizeof(T) > 1024 ? 8 : 32;      // tokens per shared-memory tile
+    static constexpr int kTile = kStates > 256 ? 8 : 32;      // tokens per shared-memory tile
     struct Stage {
         alignas(16) T x[kTile][kCh], z[kTile][kCh];
         alignas(16) float dt[kTile][kCh];
         alignas(16) T bc[2][kTile][kStates];                   // B, C
     };
     Stage st[2];
+    // of the tile being walked: step size (times log2 e in the bf16 form) and step size * input; B, C in fp32; y
+    alignas(16) float2 dd[kTile][kCh];
+    alignas(16) float bc[2][sizeof(T) == 2 ? kTile : 1][kStates];          // (fp32 inputs are read where they landed)
     alignas(16) float y[kTile][kCh + 1];
 };
 
@@ -95,16 +127,13 @@ selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
         const int n = lane * NI + i;
         a[i] = live && n < p.N ? __ldg(p.A + static_cast<long long>(c) * p.N + n) : 0.f;
     }
-    const float Dc = live ? __ldg(p.D + c) : 0.f;
+    // the gating pass gives a thread the same two channels in every tile: kThreads is a multiple of CH / 2
+    const int gk = (tid % (CH / 2)) * 2;
+    const float Ds[2] = {c0 + gk < p.inner ? __ldg(p.D + c0 + gk) : 0.f, c0 + gk + 1 < p.inner ? __ldg(p.D + c0 + gk + 1) : 0.f};
     pdl_begin();
     const int pos = p.pos[b], slot = p.slots ? p.slots[b] : b;
     float* sp = state + (static_cast<long long>(slot) * p.inner + c) * p.N + lane * NI;
-#pragma unroll
-    for (int i = 0; i < NI; i += 4) {
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (live && pos > 0 && lane * NI + i < p.N) v = *reinterpret_cast<const float4*>(sp + i);
-        S_[i] = v.x; S_[i + 1] = v.y; S_[i + 2] = v.z; S_[i + 3] = v.w;
-    }
+    load_state(sp, live && pos > 0 ? p.N - lane * NI : 0, S_);
     const long long m0 = static_cast<long long>(b) * p.T;
     auto load_tile = [&](int t0, int s) {
         typename S::Stage& st = sm.st[s];
@@ -137,76 +166,89 @@ selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
         else cp_async_wait<0>();
         __syncthreads();
         typename S::Stage& st = sm.st[it & 1];
-        // softplus of the step sizes once per (token, channel), in place
+        // once per (token, channel): the softplus of the step size and its products; past the portion a step size of 0 keeps the state
         for (int i = tid; i < kTile * CH; i += kThreads) {
             const int t = i / CH, k = i - t * CH;
             const float bk = c0 + k < p.inner ? __ldg(p.dt_bias + c0 + k) : 0.f;
-            st.dt[t][k] = softplus_for<T>(st.dt[t][k] + bk);
+            const float d = t < nt ? softplus_for<T>(st.dt[t][k] + bk) : 0.f;
+            sm.dd[t][k] = make_float2(decay_dt<T>(d), d * Elem<T>::to_f(st.x[t][k]));
+        }
+        if constexpr (sizeof(T) == 2) {
+            for (int i = tid; i < kTile * S::kStates / 2; i += kThreads) {       // four of B and C's 2 * kTile * kStates values at a time
+                float v[4];
+                load_states(&st.bc[0][0][0] + i * 4, v);
+                *reinterpret_cast<float4*>(&sm.bc[0][0][0] + i * 4) = make_float4(v[0], v[1], v[2], v[3]);
+            }
         }
         __syncthreads();
         // U tokens at a time: their loads, exponentials and sums are independent, only S += is a chain
         for (int tb = 0; tb < nt; tb += U) {
-            float d[U], dx[U], y[U];
+            float2 d[U];
+            float y[U];
 #pragma unroll
-            for (int u = 0; u < U; ++u) {
-                const int t = tb + u;                    // past the portion: step size 0 keeps the state
-                d[u] = t < nt ? st.dt[t][ch] : 0.f;
-                const float x = Elem<T>::to_f(st.x[t][ch]);
-                dx[u] = d[u] * x;
-                d[u] = decay_dt<T>(d[u]);
-                y[u] = lane == 0 ? Dc * x : 0.f;
-            }
+            for (int u = 0; u < U; ++u) d[u] = sm.dd[tb + u][ch];
 #pragma unroll
             for (int u = 0; u < U; ++u) {
                 float bn[NI], cn[NI];
-                load_states(&st.bc[0][tb + u][lane * NI], bn);
-                load_states(&st.bc[1][tb + u][lane * NI], cn);
+                if constexpr (sizeof(T) == 2) { load_states(&sm.bc[0][tb + u][lane * NI], bn); load_states(&sm.bc[1][tb + u][lane * NI], cn); }
+                else { load_states(&st.bc[0][tb + u][lane * NI], bn); load_states(&st.bc[1][tb + u][lane * NI], cn); }
+                if constexpr (sizeof(T) == 2) {
+                    const float2 dl2 = make_float2(d[u].x, d[u].x), dx2 = make_float2(d[u].y, d[u].y);
+                    float2 acc = make_float2(0.f, 0.f);
 #pragma unroll
-                for (int i = 0; i < NI; ++i) {
-                    S_[i] = decayed<T>(S_[i], d[u], a[i], dx[u] * bn[i]);
-                    y[u] = fmaf(S_[i], cn[i], y[u]);
+                    for (int i = 0; i < NI; i += 2) {
+                        const float2 e = __fmul2_rn(dl2, make_float2(a[i], a[i + 1]));
+                        const float2 n = __ffma2_rn(make_float2(fast_exp2(e.x), fast_exp2(e.y)), make_float2(S_[i], S_[i + 1]), __fmul2_rn(dx2, make_float2(bn[i], bn[i + 1])));
+                        S_[i] = n.x; S_[i + 1] = n.y;
+                        acc = __ffma2_rn(n, make_float2(cn[i], cn[i + 1]), acc);
+                    }
+                    y[u] = acc.x + acc.y;
+                } else {
+                    y[u] = 0.f;
+#pragma unroll
+                    for (int i = 0; i < NI; ++i) {
+                        S_[i] = decayed<T>(S_[i], d[u].x, a[i], d[u].y * bn[i]);
+                        y[u] = fmaf(S_[i], cn[i], y[u]);
+                    }
                 }
             }
-            // sums over the channel's lanes: halves of the tokens are exchanged until every lane holds U / LP of them (or all hold all)
+            // sums over the channel's lanes: halves of the tokens are exchanged until every lane holds one of them
             if constexpr (U == 4 && LP >= 4) {
                 float z[2];
-                const bool odd = lane & 1;
+                const bool odd = lane & 1, high = lane & 2;
 #pragma unroll
-                for (int k = 0; k < 2; ++k) {            // lanes l, l ^ 1: tokens 0, 1 stay with even lanes, 2, 3 with odd ones
+                for (int k = 0; k < 2; ++k) {            // tokens 0, 1 stay with even lanes, 2, 3 with odd ones
                     const float send = odd ? y[k] : y[k + 2], keep = odd ? y[k + 2] : y[k];
                     z[k] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 1);
                 }
-                const bool high = lane & 2;
                 const float send = high ? z[0] : z[1], keep = high ? z[1] : z[0];
                 float v = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 2);
 #pragma unroll
                 for (int o = 4; o < LP; o <<= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
-                const int t = tb + (lane & 1) * 2 + ((lane >> 1) & 1);
-                if (lane < 4 && t < nt) sm.y[t][ch] = v;
+                if (lane < 4) sm.y[tb + (lane & 1) * 2 + ((lane >> 1) & 1)][ch] = v;
             } else {
 #pragma unroll
                 for (int u = 0; u < U; ++u) {
 #pragma unroll
                     for (int o = LP / 2; o > 0; o >>= 1) y[u] += __shfl_xor_sync(0xFFFFFFFFu, y[u], o);
-                    if (lane == 0 && tb + u < nt) sm.y[tb + u][ch] = y[u];
+                    if (lane == 0) sm.y[tb + u][ch] = y[u];
                 }
             }
         }
         __syncthreads();
         // gate and store, two channels per thread
         for (int i = tid; i < nt * (CH / 2); i += kThreads) {
-            const int t = i / (CH / 2), k = (i - t * (CH / 2)) * 2;
+            const int t = i / (CH / 2), k = gk;
             if (c0 + k >= p.inner) continue;
-            const float v0 = sm.y[t][k] * silu_for<T>(Elem<T>::to_f(st.z[t][k])), v1 = sm.y[t][k + 1] * silu_for<T>(Elem<T>::to_f(st.z[t][k + 1]));
+            const float v0 = fmaf(Ds[0], Elem<T>::to_f(st.x[t][k]), sm.y[t][k]) * silu_for<T>(Elem<T>::to_f(st.z[t][k]));
+            const float v1 = fmaf(Ds[1], Elem<T>::to_f(st.x[t][k + 1]), sm.y[t][k + 1]) * silu_for<T>(Elem<T>::to_f(st.z[t][k + 1]));
             T* dst = out + (m0 + t0 + t) * p.ldo + c0 + k;
             if constexpr (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = Elem<__nv_bfloat16>::pack2(v0, v1);
             else *reinterpret_cast<float2*>(dst) = make_float2(v0, v1);
         }
         __syncthreads();           // the stage after next is refilled at the top
     }
-#pragma unroll
-    for (int i = 0; i < NI; i += 4)
-        if (live && lane * NI + i < p.N) *reinterpret_cast<float4*>(sp + i) = make_float4(S_[i], S_[i + 1], S_[i + 2], S_[i + 3]);
+    store_state(sp, live ? p.N - lane * NI : 0, S_);
 }
 
 // One token per sequence, step sizes included: grid (ceil(inner / kCh), B).  The LP lanes of a channel share its row of W_dt.
@@ -237,12 +279,7 @@ selective_step_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
     const int pos = p.pos[b], slot = p.slots ? p.slots[b] : b;
     float* sp = state + (static_cast<long long>(slot) * p.inner + cc) * p.N + lane * NI;
     float S_[NI];
-#pragma unroll
-    for (int i = 0; i < NI; i += 4) {
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (pos > 0 && lane * NI + i < p.N) v = *reinterpret_cast<const float4*>(sp + i);
-        S_[i] = v.x; S_[i + 1] = v.y; S_[i + 2] = v.z; S_[i + 3] = v.w;
-    }
+    load_state(sp, pos > 0 ? p.N - lane * NI : 0, S_);
     const float x = Elem<T>::to_f(xc[static_cast<long long>(b) * p.inner + cc]), z = Elem<T>::to_f(proj[b * p.ldp + p.inner + cc]);
     for (int i = tid; i < p.rank + 2 * p.N; i += kThreads) row[i] = Elem<T>::to_f(xdbl[b * p.ldx + i]);
     __syncthreads();
@@ -271,15 +308,15 @@ selective_step_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
 #pragma unroll
     for (int o = LP / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xFFFFFFFFu, y, o);
     if (!live) return;
-#pragma unroll
-    for (int i = 0; i < NI; i += 4)
-        if (lane * NI + i < p.N) *reinterpret_cast<float4*>(sp + i) = make_float4(S_[i], S_[i + 1], S_[i + 2], S_[i + 3]);
+    store_state(sp, p.N - lane * NI, S_);
     if (lane == 0) out[b * p.ldo + c] = Elem<T>::from_f(fmaf(Dc, x, y) * silu_for<T>(z));
 }
 
-// Calls f(LP, NI) with compile-time sizes that hold N states; `wide`: few CTAs, so as many lanes per channel as make sense.
+// Calls f(LP, NI) with compile-time sizes that hold N states; the fewer CTAs there would be, the fewer states per lane.
 template <typename F>
-int with_shape(int N, bool wide, F f) {
+int with_shape(int N, long long pairs, F f) {
+    const long long sms = device_sm_count();
+    const bool wide = pairs < 4 * 8 * kThreads * sms, widest = pairs < 2 * 4 * kThreads * sms;
     using std::integral_constant;
     auto lanes = [&](auto ni) -> int {
         const int need = (N + decltype(ni)::value - 1) / decltype(ni)::value;
@@ -288,6 +325,7 @@ int with_shape(int N, bool wide, F f) {
         if (need <= 8) return f(integral_constant<int, 8>{}, ni);
         return f(integral_constant<int, 16>{}, ni);
     };
+    if (N <= 32 && widest) return lanes(integral_constant<int, 2>{});
     if (N <= 64 && (wide || N == 8)) return lanes(integral_constant<int, 4>{});
     if (N <= 128) return lanes(integral_constant<int, 8>{});
     if (N <= 256) return f(integral_constant<int, 16>{}, integral_constant<int, 16>{});
@@ -330,12 +368,11 @@ int launch_selective(cudaStream_t s, const vb200_selective_args& a, const Select
     ScanParams p{};
     p.B = a.B; p.T = a.T; p.inner = a.inner; p.N = a.N; p.rank = a.rank; p.ldp = a.ldp; p.ldx = ldx; p.ldo = a.ldo;
     p.A = a.A; p.D = a.D; p.dt_bias = a.dt_bias; p.slots = a.slots; p.pos = a.pos;
-    const bool wide = static_cast<long long>(a.B) * a.inner * a.N < 4LL * 1024 * device_sm_count();
     auto go = [&](auto tag) -> int {
         using T = decltype(tag);
         const T *proj = static_cast<const T*>(a.proj), *x = static_cast<const T*>(xc), *d = static_cast<const T*>(xdbl);
         T* out = static_cast<T*>(a.out);
-        return with_shape(a.N, wide, [&](auto lp, auto ni) -> int {
+        return with_shape(a.N, static_cast<long long>(a.B) * a.inner * a.N, [&](auto lp, auto ni) -> int {
             constexpr int LP = decltype(lp)::value, NI = decltype(ni)::value, CH = kThreads / LP;
             const dim3 grid(static_cast<unsigned>((a.inner + CH - 1) / CH), static_cast<unsigned>(a.B));
             profile_mark_begin(s);
