@@ -257,7 +257,7 @@ int vb200_selective_forward(const vb200_selective_args* a) {
     if (!selective_sizes_ok(a)) return set_detail(VB200_ERR_INVALID_ARG, "vb200_selective_args: null, struct_size mismatch or non-positive size");
     if (!dtype_ok(a->dtype)) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_selective_forward: dtype must be bf16 or fp32");
     if (a->inner % 8 != 0 || a->N % 8 != 0 || a->rank % 8 != 0) return set_detail(VB200_ERR_ALIGNMENT, "vb200_selective_forward: inner, N and rank must be multiples of 8");
-    if (a->N > 512 || a->taps > 32 || a->rank + 2 * a->N > 48 * 1024) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_selective_forward: more than 512 states, 32 taps, or too large a rank");
+    if (a->N > 512 || a->taps > 32 || a->rank + 2 * a->N > 6 * 1024) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_selective_forward: more than 512 states, 32 taps, or too large a rank");
     if (a->B > 65535 || static_cast<int64_t>(a->T) > 65535LL * 32) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_selective_forward: batch too large");
     if (!a->proj || !a->conv_w || !a->conv_b || !a->w_x || !a->w_dt || !a->dt_bias || !a->A || !a->D || !a->pos || !a->conv_state || !a->state || !a->out)
         return set_detail(VB200_ERR_INVALID_ARG, "vb200_selective_forward: null pointer");

@@ -115,7 +115,7 @@ __global__ void __launch_bounds__(kThreads)
 selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restrict__ xc, const T* __restrict__ xdbl, const float* __restrict__ dt, float* __restrict__ state,
                       T* __restrict__ out) {
     using S = ScanTile<T, LP, NI>;
-    constexpr int CH = S::kCh, V = 16 / sizeof(T), kTile = S::kTile, U = NI <= 8 && sizeof(T) == 2 ? 4 : 1;
+    constexpr int CH = S::kCh, V = 16 / sizeof(T), kTile = S::kTile, U = NI <= 4 ? 4 : NI <= 8 ? 2 : 1;
     extern __shared__ __align__(16) uint8_t raw[];
     S& sm = *reinterpret_cast<S*>(raw);
     const int tid = threadIdx.x, lane = tid % LP, ch = tid / LP, b = blockIdx.y, c0 = blockIdx.x * CH, c = c0 + ch;
@@ -181,58 +181,96 @@ selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
             }
         }
         __syncthreads();
-        // U tokens at a time: their loads, exponentials and sums are independent, only S += is a chain
-        for (int tb = 0; tb < nt; tb += U) {
-            float2 d[U];
-            float y[U];
-#pragma unroll
-            for (int u = 0; u < U; ++u) d[u] = sm.dd[tb + u][ch];
-#pragma unroll
-            for (int u = 0; u < U; ++u) {
-                float bn[NI], cn[NI];
-                if constexpr (sizeof(T) == 2) { load_states(&sm.bc[0][tb + u][lane * NI], bn); load_states(&sm.bc[1][tb + u][lane * NI], cn); }
-                else { load_states(&st.bc[0][tb + u][lane * NI], bn); load_states(&st.bc[1][tb + u][lane * NI], cn); }
-                if constexpr (sizeof(T) == 2) {
-                    const float2 dl2 = make_float2(d[u].x, d[u].x), dx2 = make_float2(d[u].y, d[u].y);
-                    float2 acc = make_float2(0.f, 0.f);
-#pragma unroll
-                    for (int i = 0; i < NI; i += 2) {
-                        const float2 e = __fmul2_rn(dl2, make_float2(a[i], a[i + 1]));
-                        const float2 n = __ffma2_rn(make_float2(fast_exp2(e.x), fast_exp2(e.y)), make_float2(S_[i], S_[i + 1]), __fmul2_rn(dx2, make_float2(bn[i], bn[i + 1])));
-                        S_[i] = n.x; S_[i + 1] = n.y;
-                        acc = __ffma2_rn(n, make_float2(cn[i], cn[i + 1]), acc);
-                    }
-                    y[u] = acc.x + acc.y;
-                } else {
-                    y[u] = 0.f;
-#pragma unroll
-                    for (int i = 0; i < NI; ++i) {
-                        S_[i] = decayed<T>(S_[i], d[u].x, a[i], d[u].y * bn[i]);
-                        y[u] = fmaf(S_[i], cn[i], y[u]);
-                    }
-                }
-            }
-            // sums over the channel's lanes: halves of the tokens are exchanged until every lane holds one of them
-            if constexpr (U == 4 && LP >= 4) {
-                float z[2];
-                const bool odd = lane & 1, high = lane & 2;
-#pragma unroll
-                for (int k = 0; k < 2; ++k) {            // tokens 0, 1 stay with even lanes, 2, 3 with odd ones
-                    const float send = odd ? y[k] : y[k + 2], keep = odd ? y[k + 2] : y[k];
-                    z[k] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 1);
-                }
-                const float send = high ? z[0] : z[1], keep = high ? z[1] : z[0];
-                float v = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 2);
-#pragma unroll
-                for (int o = 4; o < LP; o <<= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
-                if (lane < 4) sm.y[tb + (lane & 1) * 2 + ((lane >> 1) & 1)][ch] = v;
-            } else {
+        if constexpr (sizeof(T) == 2) {
+            // U tokens at a time: their loads, exponentials and sums are independent, only S += is a chain.  In the smallest shape, which
+            // runs with few warps, the next tokens' loads and exponentials are under way while the sums of these are finished.
+            const float2* __restrict__ dd = &sm.dd[0][ch];
+            const float *__restrict__ Bs = &sm.bc[0][0][lane * NI], *__restrict__ Cs = &sm.bc[1][0][lane * NI];
+            float* __restrict__ ys = &sm.y[0][ch];
+            struct Batch { float2 e[U][NI / 2], bx[U][NI / 2], c[U][NI / 2]; };
+            auto prepare = [&](int tb, Batch& q) {
 #pragma unroll
                 for (int u = 0; u < U; ++u) {
+                    const float2 d = dd[(tb + u) * CH];
+                    float bn[NI], cn[NI];
+                    load_states(Bs + (tb + u) * S::kStates, bn);
+                    load_states(Cs + (tb + u) * S::kStates, cn);
+                    const float2 dl2 = make_float2(d.x, d.x), dx2 = make_float2(d.y, d.y);
 #pragma unroll
-                    for (int o = LP / 2; o > 0; o >>= 1) y[u] += __shfl_xor_sync(0xFFFFFFFFu, y[u], o);
-                    if (lane == 0) sm.y[tb + u][ch] = y[u];
+                    for (int i = 0; i < NI / 2; ++i) {
+                        const float2 m = __fmul2_rn(dl2, make_float2(a[2 * i], a[2 * i + 1]));
+                        q.e[u][i] = make_float2(fast_exp2(m.x), fast_exp2(m.y));
+                        q.bx[u][i] = __fmul2_rn(dx2, make_float2(bn[2 * i], bn[2 * i + 1]));
+                        q.c[u][i] = make_float2(cn[2 * i], cn[2 * i + 1]);
+                    }
                 }
+            };
+            auto finish = [&](int tb, const Batch& q) {
+                float y[U];
+#pragma unroll
+                for (int u = 0; u < U; ++u) {
+                    float2 acc = make_float2(0.f, 0.f);
+#pragma unroll
+                    for (int i = 0; i < NI / 2; ++i) {
+                        const float2 n = __ffma2_rn(q.e[u][i], make_float2(S_[2 * i], S_[2 * i + 1]), q.bx[u][i]);
+                        S_[2 * i] = n.x; S_[2 * i + 1] = n.y;
+                        acc = __ffma2_rn(n, q.c[u][i], acc);
+                    }
+                    y[u] = acc.x + acc.y;
+                }
+                // sums over the channel's lanes: halves of the tokens are exchanged until every lane holds one of them
+                if constexpr (U == 4 && LP >= 4) {
+                    float z[2];
+                    const bool odd = lane & 1, high = lane & 2;
+#pragma unroll
+                    for (int k = 0; k < 2; ++k) {        // tokens 0, 1 stay with even lanes, 2, 3 with odd ones
+                        const float send = odd ? y[k] : y[k + 2], keep = odd ? y[k + 2] : y[k];
+                        z[k] = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 1);
+                    }
+                    const float send = high ? z[0] : z[1], keep = high ? z[1] : z[0];
+                    float v = keep + __shfl_xor_sync(0xFFFFFFFFu, send, 2);
+#pragma unroll
+                    for (int o = 4; o < LP; o <<= 1) v += __shfl_xor_sync(0xFFFFFFFFu, v, o);
+                    if (lane < 4) ys[(tb + (lane & 1) * 2 + ((lane >> 1) & 1)) * (CH + 1)] = v;
+                } else {
+#pragma unroll
+                    for (int u = 0; u < U; ++u) {
+#pragma unroll
+                        for (int o = LP / 2; o > 0; o >>= 1) y[u] += __shfl_xor_sync(0xFFFFFFFFu, y[u], o);
+                        if (lane == 0) ys[(tb + u) * (CH + 1)] = y[u];
+                    }
+                }
+            };
+            if constexpr (NI == 2) {
+                Batch q[2];
+                prepare(0, q[0]);
+                for (int tb = 0; tb < nt; tb += 2 * U) { // kTile is a multiple of 2 U; tokens past the portion change nothing
+                    prepare(tb + U, q[1]);
+                    finish(tb, q[0]);
+                    if (tb + 2 * U < nt) prepare(tb + 2 * U, q[0]);
+                    finish(tb + U, q[1]);
+                }
+            } else {
+                for (int tb = 0; tb < nt; tb += U) {
+                    Batch q;
+                    prepare(tb, q);
+                    finish(tb, q);
+                }
+            }
+        } else {
+            for (int t = 0; t < nt; ++t) {
+                const float2 d = sm.dd[t][ch];
+                float bn[NI], cn[NI], y = 0.f;
+                load_states(&st.bc[0][t][lane * NI], bn);
+                load_states(&st.bc[1][t][lane * NI], cn);
+#pragma unroll
+                for (int i = 0; i < NI; ++i) {
+                    S_[i] = decayed<T>(S_[i], d.x, a[i], d.y * bn[i]);
+                    y = fmaf(S_[i], cn[i], y);
+                }
+#pragma unroll
+                for (int o = LP / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xFFFFFFFFu, y, o);
+                if (lane == 0) sm.y[t][ch] = y;
             }
         }
         __syncthreads();
@@ -251,15 +289,18 @@ selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
     store_state(sp, live ? p.N - lane * NI : 0, S_);
 }
 
-// One token per sequence, step sizes included: grid (ceil(inner / kCh), B).  The LP lanes of a channel share its row of W_dt.
+constexpr int kStepRows = 4;       // sequences that a CTA of the decode step takes in turn
+
+// One token per sequence, step sizes included: grid (ceil(inner / kCh), ceil(B / rows)).  The LP lanes of a channel share its row of W_dt,
+// which is fetched ahead of the wait and kept for all rows.
 template <typename T, int LP, int NI>
 __global__ void __launch_bounds__(kThreads)
-selective_step_kernel(ScanParams p, const T* __restrict__ proj, const T* __restrict__ xc, const T* __restrict__ xdbl, const T* __restrict__ w_dt, float* __restrict__ state,
+selective_step_kernel(ScanParams p, int rows, const T* __restrict__ proj, const T* __restrict__ xc, const T* __restrict__ xdbl, const T* __restrict__ w_dt, float* __restrict__ state,
                       T* __restrict__ out) {
     constexpr int CH = kThreads / LP;
     extern __shared__ __align__(16) uint8_t raw[];
-    float* row = reinterpret_cast<float*>(raw);        // [rank | B | C] of this token
-    const int tid = threadIdx.x, lane = tid % LP, b = blockIdx.y, c = blockIdx.x * CH + tid / LP, cc = min(c, p.inner - 1);
+    float* sm = reinterpret_cast<float*>(raw);         // [rows][dt | B | C]
+    const int tid = threadIdx.x, lane = tid % LP, b0 = blockIdx.y * rows, nb = min(rows, p.B - b0), c = blockIdx.x * CH + tid / LP, cc = min(c, p.inner - 1);
     const bool live = c < p.inner;
     float a[NI];
 #pragma unroll
@@ -268,55 +309,73 @@ selective_step_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
         a[i] = n < p.N ? __ldg(p.A + static_cast<long long>(cc) * p.N + n) : 0.f;
     }
     const float bias = __ldg(p.dt_bias + cc), Dc = __ldg(p.D + cc);
-    constexpr int kAhead = 4;                          // pieces of W_dt fetched before the wait
-    const int n8 = p.rank / 8;
+    constexpr int kAhead = 4;                          // pieces of W_dt kept in registers
+    const int n8 = p.rank / 8, ld = p.rank + 2 * p.N;
     const T* wr = w_dt + static_cast<long long>(cc) * p.rank;
     Raw8<T> w[kAhead];
 #pragma unroll
     for (int i = 0; i < kAhead; ++i)
         if (lane + i * LP < n8) w[i].load(wr + (lane + i * LP) * 8);
     pdl_begin();
-    const int pos = p.pos[b], slot = p.slots ? p.slots[b] : b;
-    float* sp = state + (static_cast<long long>(slot) * p.inner + cc) * p.N + lane * NI;
-    float S_[NI];
-    load_state(sp, pos > 0 ? p.N - lane * NI : 0, S_);
-    const float x = Elem<T>::to_f(xc[static_cast<long long>(b) * p.inner + cc]), z = Elem<T>::to_f(proj[b * p.ldp + p.inner + cc]);
-    for (int i = tid; i < p.rank + 2 * p.N; i += kThreads) row[i] = Elem<T>::to_f(xdbl[b * p.ldx + i]);
-    __syncthreads();
-    float d = 0.f;
-    auto dot8 = [&](const float (&wv)[8], int k) {
-#pragma unroll
-        for (int e = 0; e < 8; ++e) d = fmaf(wv[e], row[k * 8 + e], d);
+    float next[NI], xn, zn;
+    float* sp_next;
+    auto fetch = [&](int r) {
+        const int b = b0 + r, slot = p.slots ? p.slots[b] : b;
+        sp_next = state + (static_cast<long long>(slot) * p.inner + cc) * p.N + lane * NI;
+        load_state(sp_next, p.pos[b] > 0 ? p.N - lane * NI : 0, next);
+        xn = Elem<T>::to_f(xc[static_cast<long long>(b) * p.inner + cc]);
+        zn = Elem<T>::to_f(proj[b * p.ldp + p.inner + cc]);
     };
-#pragma unroll
-    for (int i = 0; i < kAhead; ++i)
-        if (lane + i * LP < n8) { float wv[8]; w[i].get(wv); dot8(wv, lane + i * LP); }
-    for (int k = lane + kAhead * LP; k < n8; k += LP) { float wv[8]; load8(wr + k * 8, wv); dot8(wv, k); }
-#pragma unroll
-    for (int o = LP / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xFFFFFFFFu, d, o);
-    d = softplus_for<T>(d + bias);
-    const float dx = d * x, dl = decay_dt<T>(d);
-    const float *Bn = row + p.rank + lane * NI, *Cn = Bn + p.N;
-    float y = 0.f;
-#pragma unroll
-    for (int i = 0; i < NI; ++i) {
-        if (lane * NI + i < p.N) {
-            S_[i] = decayed<T>(S_[i], dl, a[i], dx * Bn[i]);
-            y = fmaf(S_[i], Cn[i], y);
-        }
+    fetch(0);
+    for (int i = tid; i < nb * ld; i += kThreads) {
+        const int r = i / ld;
+        sm[i] = Elem<T>::to_f(xdbl[(b0 + r) * p.ldx + i - r * ld]);
     }
+    __syncthreads();
+    for (int r = 0; r < nb; ++r) {
+        float S_[NI];
 #pragma unroll
-    for (int o = LP / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xFFFFFFFFu, y, o);
-    if (!live) return;
-    store_state(sp, p.N - lane * NI, S_);
-    if (lane == 0) out[b * p.ldo + c] = Elem<T>::from_f(fmaf(Dc, x, y) * silu_for<T>(z));
+        for (int i = 0; i < NI; ++i) S_[i] = next[i];
+        const float x = xn, z = zn;
+        float* sp = sp_next;
+        if (r + 1 < nb) fetch(r + 1);                  // the next sequence's state is under way meanwhile
+        const float* row = sm + r * ld;
+        float d = 0.f;
+        auto dot8 = [&](const float (&wv)[8], int k) {
+            const float4 u = *reinterpret_cast<const float4*>(row + k * 8), v = *reinterpret_cast<const float4*>(row + k * 8 + 4);
+            d = fmaf(wv[0], u.x, fmaf(wv[1], u.y, fmaf(wv[2], u.z, fmaf(wv[3], u.w, d))));
+            d = fmaf(wv[4], v.x, fmaf(wv[5], v.y, fmaf(wv[6], v.z, fmaf(wv[7], v.w, d))));
+        };
+#pragma unroll
+        for (int i = 0; i < kAhead; ++i)
+            if (lane + i * LP < n8) { float wv[8]; w[i].get(wv); dot8(wv, lane + i * LP); }
+        for (int k = lane + kAhead * LP; k < n8; k += LP) { float wv[8]; load8(wr + k * 8, wv); dot8(wv, k); }
+#pragma unroll
+        for (int o = LP / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xFFFFFFFFu, d, o);
+        d = softplus_for<T>(d + bias);
+        const float dx = d * x, dl = decay_dt<T>(d);
+        const float *Bn = row + p.rank + lane * NI, *Cn = Bn + p.N;
+        float y = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            if (lane * NI + i < p.N) {
+                S_[i] = decayed<T>(S_[i], dl, a[i], dx * Bn[i]);
+                y = fmaf(S_[i], Cn[i], y);
+            }
+        }
+#pragma unroll
+        for (int o = LP / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xFFFFFFFFu, y, o);
+        if (!live) continue;
+        store_state(sp, p.N - lane * NI, S_);
+        if (lane == 0) out[(b0 + r) * p.ldo + c] = Elem<T>::from_f(fmaf(Dc, x, y) * silu_for<T>(z));
+    }
 }
 
-// Calls f(LP, NI) with compile-time sizes that hold N states; the fewer CTAs there would be, the fewer states per lane.
+// Calls f(LP, NI) with compile-time sizes that hold N states; the fewer CTAs there would be, the fewer states per lane (a decode step: four).
 template <typename F>
-int with_shape(int N, long long pairs, F f) {
+int with_shape(int N, long long pairs, bool step, F f) {
     const long long sms = device_sm_count();
-    const bool wide = pairs < 4 * 8 * kThreads * sms, widest = pairs < 2 * 4 * kThreads * sms;
+    const bool wide = step || pairs < 4 * 8 * kThreads * sms, widest = !step && pairs < 2 * 4 * kThreads * sms;
     using std::integral_constant;
     auto lanes = [&](auto ni) -> int {
         const int need = (N + decltype(ni)::value - 1) / decltype(ni)::value;
@@ -372,15 +431,19 @@ int launch_selective(cudaStream_t s, const vb200_selective_args& a, const Select
         using T = decltype(tag);
         const T *proj = static_cast<const T*>(a.proj), *x = static_cast<const T*>(xc), *d = static_cast<const T*>(xdbl);
         T* out = static_cast<T*>(a.out);
-        return with_shape(a.N, static_cast<long long>(a.B) * a.inner * a.N, [&](auto lp, auto ni) -> int {
+        return with_shape(a.N, static_cast<long long>(a.B) * a.inner * a.N, a.T == 1, [&](auto lp, auto ni) -> int {
             constexpr int LP = decltype(lp)::value, NI = decltype(ni)::value, CH = kThreads / LP;
             const dim3 grid(static_cast<unsigned>((a.inner + CH - 1) / CH), static_cast<unsigned>(a.B));
             profile_mark_begin(s);
             int rc;
             if (a.T == 1) {
-                const size_t smem = sizeof(float) * ldx;
+                // rows per CTA: W_dt and A are read once for them, as long as six CTAs per SM remain
+                int rows = 1;
+                while (rows < kStepRows && rows < a.B && static_cast<long long>(grid.x) * ((a.B + 2 * rows - 1) / (2 * rows)) >= 6 * device_sm_count()) rows *= 2;
+                const dim3 step_grid(grid.x, static_cast<unsigned>((a.B + rows - 1) / rows));
+                const size_t smem = sizeof(float) * ldx * rows;
                 rc = allow_smem(selective_step_kernel<T, LP, NI>, smem);
-                if (rc == VB200_OK) rc = launch_pdl(selective_step_kernel<T, LP, NI>, grid, dim3(kThreads), smem, s, p, proj, x, d, static_cast<const T*>(a.w_dt), a.state, out);
+                if (rc == VB200_OK) rc = launch_pdl(selective_step_kernel<T, LP, NI>, step_grid, dim3(kThreads), smem, s, p, rows, proj, x, d, static_cast<const T*>(a.w_dt), a.state, out);
                 note_selective_kernel("selective_step_kernel");
             } else {
                 const size_t smem = sizeof(ScanTile<T, LP, NI>);
