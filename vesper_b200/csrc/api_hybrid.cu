@@ -222,8 +222,8 @@ size_t vb200_sigattn_workspace_bytes(const vb200_sigattn_args* a) { return sigat
 int vb200_sigattn_forward(const vb200_sigattn_args* a) {
     if (!sigattn_sizes_ok(a)) return set_detail(VB200_ERR_INVALID_ARG, "vb200_sigattn_args: null, struct_size mismatch, non-positive size or heads not divisible by kv heads");
     if (!dtype_ok(a->dtype)) return set_detail(VB200_ERR_UNSUPPORTED, "vb200_sigattn_forward: dtype must be bf16 or fp32");
-    if (static_cast<int64_t>(a->H) * a->dim > 48 * 1024 || 4LL * (static_cast<int64_t>(a->G) * a->dim + a->vdim) > 48 * 1024)
-        return set_detail(VB200_ERR_UNSUPPORTED, "vb200_sigattn_forward: heads * dim above 48 K, or kv_heads * dim + vdim above 12 K");
+    if (static_cast<int64_t>(a->H) * (a->dim + a->H) > 48 * 1024 || 4LL * (static_cast<int64_t>(a->G) * a->dim + a->vdim) > 48 * 1024)
+        return set_detail(VB200_ERR_UNSUPPORTED, "vb200_sigattn_forward: heads * (dim + heads) above 48 K, or kv_heads * dim + vdim above 12 K");
     if (a->B > 65535 || (static_cast<int64_t>(a->T) + 3) / 4 * a->H > 65535) {
         if (a->B > 65535 || a->dtype == VB200_F32 || a->form == 1 || !plan_sigattn(*a).mma)
             return set_detail(VB200_ERR_UNSUPPORTED, "vb200_sigattn_forward: too many rows for one call");

@@ -98,19 +98,41 @@ struct MoeParams {
     int act_ld;                  // activations of one (token, expert) pair
 };
 
-// dot product of a weight row and x (shared memory), eight columns per lane at a time; n8 = columns / 8
-template <typename T>
-__device__ __forceinline__ float row_dot(const T* __restrict__ w, const float* x, int n8) {
+constexpr int kAhead = 4;        // 16-byte (fp32: 32-byte) pieces of a weight row that a lane has in flight
+
+__device__ __forceinline__ float dot8(const float (&v)[8], const float* x, float a) {
+    const float4 x0 = *reinterpret_cast<const float4*>(x), x1 = *reinterpret_cast<const float4*>(x + 4);
+    a = fmaf(v[0], x0.x, fmaf(v[1], x0.y, fmaf(v[2], x0.z, fmaf(v[3], x0.w, a))));
+    return fmaf(v[4], x1.x, fmaf(v[5], x1.y, fmaf(v[6], x1.z, fmaf(v[7], x1.w, a))));
+}
+
+// Warp-wide dot product of n8 pieces of eight columns with x in shared memory; row(i) is the address of piece i.
+template <typename T, int ROWS, typename F>
+__device__ __forceinline__ void piece_dots(int n8, const float* x, float (&sum)[ROWS], F row) {
     const int lane = threadIdx.x & 31;
-    float a = 0.f;
-    for (int k = lane; k < n8; k += 32) {
-        float v[8];
-        load8(w + k * 8, v);
-        const float4 x0 = *reinterpret_cast<const float4*>(x + k * 8), x1 = *reinterpret_cast<const float4*>(x + k * 8 + 4);
-        a = fmaf(v[0], x0.x, fmaf(v[1], x0.y, fmaf(v[2], x0.z, fmaf(v[3], x0.w, a))));
-        a = fmaf(v[4], x1.x, fmaf(v[5], x1.y, fmaf(v[6], x1.z, fmaf(v[7], x1.w, a))));
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) sum[r] = 0.f;
+    for (int i0 = lane; i0 < n8; i0 += 32 * kAhead) {
+        Raw8<T> w[kAhead][ROWS];
+#pragma unroll
+        for (int u = 0; u < kAhead; ++u)
+            if (i0 + 32 * u < n8) {
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r) w[u][r].load(row(i0 + 32 * u, r));
+            }
+#pragma unroll
+        for (int u = 0; u < kAhead; ++u)
+            if (i0 + 32 * u < n8) {
+#pragma unroll
+                for (int r = 0; r < ROWS; ++r) {
+                    float v[8];
+                    w[u][r].get(v);
+                    sum[r] = dot8(v, x + (i0 + 32 * u) * 8, sum[r]);
+                }
+            }
     }
-    return warp_sum_f(a);
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) sum[r] = warp_sum_f(sum[r]);
 }
 
 constexpr int kPairRows = 16;    // hidden units per CTA: two per warp
@@ -134,9 +156,10 @@ moe_pair_in_kernel(MoeParams p, const T* __restrict__ x, const int* __restrict__
     __syncthreads();
     T* dst = act + (static_cast<long long>(m) * (p.top + 1) + k) * p.act_ld;
     for (int j = j0 + warp; j < min(ff, j0 + kPairRows); j += 8) {
-        const T* r = w + static_cast<long long>(2 * j) * p.dim;
-        const float g = row_dot(r, xs, p.dim / 8), u = row_dot(r + p.dim, xs, p.dim / 8);
-        if (lane == 0) dst[j] = Elem<T>::from_f(silu_for<T>(g) * u);
+        const T* rows = w + static_cast<long long>(2 * j) * p.dim;
+        float gu[2];
+        piece_dots<T, 2>(p.dim / 8, xs, gu, [&](int i, int r) { return rows + r * p.dim + i * 8; });
+        if (lane == 0) dst[j] = Elem<T>::from_f(silu_for<T>(gu[0]) * gu[1]);
     }
     // the padding up to a multiple of eight is multiplied with zero weights and must be finite
     if (j0 + kPairRows >= ff && threadIdx.x < 8 && ff + threadIdx.x < (ff + 7) / 8 * 8) dst[ff + threadIdx.x] = Elem<T>::from_f(0.f);
@@ -144,7 +167,7 @@ moe_pair_in_kernel(MoeParams p, const T* __restrict__ x, const int* __restrict__
 
 constexpr int kOutRows = 16;
 
-// grid (ceil(dim / kOutRows), M), 256 threads
+// grid (ceil(dim / kOutRows), M), 256 threads: an output row is one dot product over the hidden units of all its token's experts, weighted ahead
 template <typename T>
 __global__ void __launch_bounds__(256)
 moe_pair_out_kernel(MoeParams p, const int* __restrict__ ids, const float* __restrict__ weights, const T* __restrict__ w_out, const T* __restrict__ w_shared, const T* __restrict__ act,
@@ -152,23 +175,25 @@ moe_pair_out_kernel(MoeParams p, const int* __restrict__ ids, const float* __res
     pdl_begin();
     extern __shared__ __align__(16) float as[];
     const int m = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, d0 = blockIdx.x * kOutRows;
-    const int f8 = (p.ff + 7) / 8, s8 = (p.ff_shared + 7) / 8;
+    const int f8 = (p.ff + 7) / 8, s8 = (p.ff_shared + 7) / 8, n8 = p.top * f8 + s8;
     const T* src = act + static_cast<long long>(m) * (p.top + 1) * p.act_ld;
-    for (int i = threadIdx.x; i < p.top * f8 + s8; i += 256) {
+    for (int i = threadIdx.x; i < n8; i += 256) {
         const int k = min(i / f8, p.top), c = i - k * f8;
+        const float w = k < p.top ? weights[m * p.top + k] : 1.0f;
         float v[8];
         load8(src + k * p.act_ld + c * 8, v);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] *= w;
         store8(as + i * 8, v);
     }
     __syncthreads();
-    for (int d = d0 + warp; d < min(p.dim, d0 + kOutRows); d += 8) {
-        float t = 0.f;
-        for (int k = 0; k < p.top; ++k) {
-            const int e = ids[m * p.top + k];
-            t = fmaf(weights[m * p.top + k], row_dot(w_out + (static_cast<long long>(e) * p.dim + d) * p.ld_out, as + k * f8 * 8, f8), t);
-        }
-        if (p.ff_shared > 0) t += row_dot(w_shared + static_cast<long long>(d) * p.ld_shared, as + p.top * f8 * 8, s8);
-        if (lane == 0) y[static_cast<long long>(m) * p.dim + d] = t;
+    for (int d = d0 + 2 * warp; d < min(p.dim, d0 + kOutRows); d += 16) {            // two rows at a time (dim is a multiple of 8)
+        float t[2];
+        piece_dots<T, 2>(n8, as, t, [&](int i, int r) {
+            const int k = min(i / f8, p.top), c = i - k * f8;
+            return k < p.top ? w_out + (static_cast<long long>(ids[m * p.top + k]) * p.dim + d + r) * p.ld_out + c * 8 : w_shared + static_cast<long long>(d + r) * p.ld_shared + c * 8;
+        });
+        if (lane == 0) *reinterpret_cast<float2*>(y + static_cast<long long>(m) * p.dim + d) = make_float2(t[0], t[1]);
     }
 }
 
@@ -296,7 +321,7 @@ MoePlan plan_moe(const vb200_moe_args& a) {
     size_t at = 0;
     auto take = [&](size_t bytes) { const size_t o = at; at += up(bytes); return o; };
     // sorting pays when experts are shared: token by token every pair streams an expert of its own
-    pl.grouped = a.dtype == VB200_BF16 && a.form != 1 && pairs < (1u << 30) && (a.form == 2 || pairs >= 2 * static_cast<size_t>(a.experts));
+    pl.grouped = a.dtype == VB200_BF16 && a.form != 1 && pairs < (1u << 30) && (a.form == 2 || 4 * pairs >= 5 * static_cast<size_t>(a.experts));
     pl.max_tiles = static_cast<int>((pairs + 127) / 128) + (a.experts < static_cast<int>(pairs) ? a.experts : static_cast<int>(pairs));
     pl.logits = take(M * pad_to(a.experts, 4) * 4);
     pl.ids = take(pairs * 4);

@@ -28,7 +28,9 @@ template <typename T, typename QT>
 __global__ void __launch_bounds__(256)
 sig_append_kernel(SigParams p, const T* __restrict__ proj, T* __restrict__ kc, T* __restrict__ vc, T* __restrict__ first, QT* __restrict__ qm) {
     pdl_begin();
-    extern __shared__ float qs[];         // [H * dim] scaled queries
+    extern __shared__ __align__(16) float qs[];         // [H * dim] scaled queries, then talk [H, H]
+    float* tk = qs + (p.H * p.dim + 3) / 4 * 4;
+    for (int i = threadIdx.x; i < p.H * p.H; i += 256) tk[i] = __ldg(p.talk + i);
     const int t = blockIdx.x, b = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long long m = static_cast<long long>(b) * p.T + t;
     const int pos = p.pos[b] + t;
@@ -59,6 +61,26 @@ sig_append_kernel(SigParams p, const T* __restrict__ proj, T* __restrict__ kc, T
         if (fits) vc[row * p.ldv + i] = Elem<T>::from_f(v);
     }
     __syncthreads();
+    if (p.dim % 2 == 0 && p.R <= 8) {                    // two columns of one group per thread
+        for (int c = threadIdx.x * 2; c < p.qld; c += 512) {
+            QT* dst = qm + m * p.H * p.qld + c;
+            const int g = min(c / p.dim, p.G - 1), d = c - g * p.dim;
+            const bool pad = c >= kcols;
+            float2 qr[8];
+#pragma unroll
+            for (int r = 0; r < 8; ++r) qr[r] = r < p.R && !pad ? *reinterpret_cast<const float2*>(qs + (g * p.R + r) * p.dim + d) : make_float2(0.f, 0.f);
+            for (int h = 0; h < p.H; ++h) {
+                const float* w = tk + h * p.H + g * p.R;
+                float2 a = make_float2(0.f, 0.f);
+#pragma unroll
+                for (int r = 0; r < 8; ++r)
+                    if (r < p.R) a = __ffma2_rn(make_float2(w[r], w[r]), qr[r], a);
+                if constexpr (sizeof(QT) == 2) *reinterpret_cast<uint32_t*>(dst + static_cast<long long>(h) * p.qld) = Elem<__nv_bfloat16>::pack2(a.x, a.y);
+                else *reinterpret_cast<float2*>(dst + static_cast<long long>(h) * p.qld) = a;
+            }
+        }
+        return;
+    }
     for (int c = threadIdx.x; c < p.qld; c += 256) {
         QT* dst = qm + m * p.H * p.qld + c;
         if (c >= kcols) {
@@ -67,25 +89,10 @@ sig_append_kernel(SigParams p, const T* __restrict__ proj, T* __restrict__ kc, T
         }
         const int g = c / p.dim, d = c - g * p.dim;
         const float* q = qs + g * p.R * p.dim + d;
-        if (p.R <= 8) {
-            float qr[8];
-#pragma unroll
-            for (int r = 0; r < 8; ++r) qr[r] = r < p.R ? q[r * p.dim] : 0.f;
-            for (int h = 0; h < p.H; ++h) {
-                const float* tk = p.talk + h * p.H + g * p.R;
-                float a = 0.f;
-#pragma unroll
-                for (int r = 0; r < 8; ++r)
-                    if (r < p.R) a = fmaf(__ldg(tk + r), qr[r], a);
-                dst[static_cast<long long>(h) * p.qld] = Elem<QT>::from_f(a);
-            }
-        } else {
-            for (int h = 0; h < p.H; ++h) {
-                const float* tk = p.talk + h * p.H + g * p.R;
-                float a = 0.f;
-                for (int r = 0; r < p.R; ++r) a = fmaf(__ldg(tk + r), q[r * p.dim], a);
-                dst[static_cast<long long>(h) * p.qld] = Elem<QT>::from_f(a);
-            }
+        for (int h = 0; h < p.H; ++h) {
+            float a = 0.f;
+            for (int r = 0; r < p.R; ++r) a = fmaf(tk[h * p.H + g * p.R + r], q[r * p.dim], a);
+            dst[static_cast<long long>(h) * p.qld] = Elem<QT>::from_f(a);
         }
     }
 }
@@ -205,7 +212,7 @@ int launch_sigattn(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& p
         T *kc = static_cast<T*>(a.k_cache), *vc = static_cast<T*>(a.v_cache), *first = static_cast<T*>(a.first_values), *out = static_cast<T*>(a.out);
         const T* proj = static_cast<const T*>(a.proj);
         const dim3 grid(static_cast<unsigned>(a.T), static_cast<unsigned>(a.B));
-        const size_t smem = sizeof(float) * a.H * a.dim;
+        const size_t smem = sizeof(float) * ((static_cast<size_t>(a.H) * a.dim + 3) / 4 * 4 + static_cast<size_t>(a.H) * a.H);
         auto append = [&](auto* qm) -> int {
             auto kernel = sig_append_kernel<T, std::remove_pointer_t<decltype(qm)>>;
             if (int rc = allow_smem(kernel, smem)) return rc;
