@@ -206,7 +206,7 @@ typedef struct vb200_sigattn_args {
     int32_t start_pos;               /* all rows' position when T > 1 */
     int32_t max_len;                 /* longest length a one-token step can meet (0 = cap): plans the key splits */
     void* workspace; size_t workspace_bytes;
-    int32_t form;                    /* 0 = choose, 1 = CUDA cores */
+    int32_t form;                    /* 0 = choose, 1 = CUDA cores, 2 = prompts on single SMs only */
 } vb200_sigattn_args;
 size_t vb200_sigattn_workspace_bytes(const vb200_sigattn_args* a);
 int vb200_sigattn_forward(const vb200_sigattn_args* a);

@@ -111,6 +111,8 @@ SIG = {  # H, G, dim, vdim, scale, temp (coef, every), distances
     "one head": (1, 1, 8, 8, 0.9, (0.5, 64), 1),
     "group of ten": (10, 1, 48, 200, 0.1, None, 33),
     "large rows": (12, 12, 64, 64, 0.1, (0.1, 9), 30),
+    "pairs of heads": (12, 6, 40, 64, 0.15, (0.3, 50), 140),
+    "pairs, wide values": (8, 2, 104, 128, 0.08, None, 300),
 }
 
 
@@ -199,7 +201,11 @@ def test_sigmoid_attention_prompts_portions_and_tokens(cuda, name, kind):
     close(c.run(core, cuda, p[:50], [1] * 50, slot=1), want[:50], "from the first token, in a used slot")
     if kind == "bf16":
         fits = c.G * c.dim <= 512 and c.vdim % 8 == 0
-        assert (tuned_prompt == "sig_prefill_sm100_kernel") == fits
+        pair = fits and (c.H // c.G) % 2 == 0 and c.vdim in (64, 128) and c.G * c.dim >= 192
+        assert tuned_prompt == ("sig_prefill_sm100_kernel (pair)" if pair else "sig_prefill_sm100_kernel" if fits else "sig_attend_generic_kernel")
+        if pair:
+            close(c.run(core, cuda, p, [L], form=2), want, "single SMs")
+            close(c.run(core, cuda, p, [129, L - 129], form=2), want, "single SMs, portions")
         assert (tuned_step == "sig_decode_mma_kernel") == (fits and c.G * c.vdim <= 512)
         close(c.run(core, cuda, p, [L - 3, 1, 1, 1], form=1), want, "CUDA cores")
 

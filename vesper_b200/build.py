@@ -26,7 +26,7 @@ SOURCES = ["api.cu", "rope_append.cu", "prefill_f32.cu", "prefill_sm100.cu", "pr
            "linear_sm100.cu", "block_ops.cu", "decode_exchange.cu", "decode_gqa_mma.cu", "flash_bwd_f32.cu",
            "api_hybrid.cu", "sequence_ops.cu", "latent_attention.cu", "latent_prefill_sm100.cu", "latent_decode_mma.cu", "ssd_scan.cu", "ssd_chunk.cu", "ssd_walk_sm100.cu",
            "sigmoid_attention.cu", "sigmoid_prefill_sm100.cu", "sigmoid_decode_mma.cu", "selective_scan.cu", "moe.cu"]
-HEADERS = ["common.cuh", "kernels.h", "hybrid.cuh", os.path.join("..", "..", "include", "vesper_b200.h"),
+HEADERS = ["common.cuh", "kernels.h", "hybrid.cuh", "cluster_pair.cuh", os.path.join("..", "..", "include", "vesper_b200.h"),
            os.path.join("..", "..", "include", "vesper_b200_block.h"), os.path.join("..", "..", "include", "vesper_b200_hybrid.h")]
 
 NVCC_FLAGS = [

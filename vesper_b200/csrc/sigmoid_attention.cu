@@ -223,7 +223,7 @@ int launch_sigattn(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& p
         profile_mark_begin(s);
         if (pl.mma) {
             rc = a.T > 1 ? launch_sig_prefill_sm100(s, a, pl, q, status) : launch_sig_decode_mma(s, a, pl, q, part, status);
-            note_sigattn_kernel(a.T > 1 ? "sig_prefill_sm100_kernel" : "sig_decode_mma_kernel");
+            if (a.T == 1) note_sigattn_kernel("sig_decode_mma_kernel");
         } else {
             const size_t sm = sizeof(float) * 4 * (a.G * a.dim + a.vdim);
             rc = allow_smem(sig_attend_generic_kernel<T>, sm);

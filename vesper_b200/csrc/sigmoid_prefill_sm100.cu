@@ -6,13 +6,18 @@
 // sigmoid(s) = 1 / (1 + 2^(s')).  Weights are not normalised, so there is no running maximum, no correction of O, and two warps
 // can share a row: nothing has to be reduced over keys.
 //
-// One CTA per 128 query rows of one (batch, head), one CTA per SM; keys in blocks of 128.
+// One CTA per 128 query rows of one (batch, head), one CTA per SM; keys in blocks of 128.  The key rows are as wide as all groups
+// together, so with one tile per CTA they come from L2 faster than it delivers; where two neighbouring heads share their values (PAIR), the
+// CTAs of the two heads form a cluster that runs every product as one tcgen05.mma.cta_group::2 of 256 rows, and each loads half of the keys
+// (64 of a block's 128) and half of the value columns.  The cluster's rank 0 issues the products; its barriers collect both CTAs' copies
+// and arrivals, its commits go to both.
 //   warps 0-7  weights and epilogue: warps w and w + 4 own the same 32 rows (TMEM lanes), and 64 keys of a block each
-//   warp  8    TMA producer: Q once, then a ring of K stages (one or two [128 keys x 64 columns] boxes) and one of V blocks
+//   warp  8    TMA producer: Q once, then a ring of K stages (a few boxes of 64 columns) and one of V blocks
 //   warp  9    tcgen05.mma issuer, TMEM owner
 // TMEM (512 columns): S0 [0, 128) S1 [128, 256) O [256, 256 + vdim).  QK of block j+1 is issued before PV of block j.  The weights stay
 // fp32-class in the second product: each half of a block is packed over its own 64 columns of S as bf16 hi (32 columns) and lo (32).
 // Two elements share one reciprocal: 1/a = b * (1/(ab)); 2^(s') is cut at 2^60, which leaves a weight below 1e-18.
+#include "cluster_pair.cuh"
 #include "hybrid.cuh"
 
 namespace vb200 {
@@ -20,7 +25,7 @@ namespace {
 
 constexpr int kRows = 128, kKeys = 128;
 constexpr int kBox = 128 * 128;               // [128 rows x 64 columns]
-constexpr int kMaxStages = 6;
+constexpr int kMaxStages = 8;
 constexpr int kBoxesPerSm = 14;               // of 16 KB: Q, K ring and V ring of the one CTA
 constexpr int kWeightThreads = 256;
 constexpr int kThreads = kWeightThreads + 64;
@@ -32,6 +37,7 @@ struct SigTileParams {
     int T, start_pos, vdim, R, n_bias, gate_col;
     int ks, nb_k, nb_v, n_pv;                 // 16-column steps of kd, 64-column boxes, columns of the second product
     int kbs, k_stages, v_stages;              // boxes per K stage, ring depths
+    int v_half;                               // PAIR: value columns of one CTA
     const float* bias;
     const __nv_bfloat16* proj;
     __nv_bfloat16* out;
@@ -52,31 +58,51 @@ __device__ __forceinline__ float rcp_approx(float x) {
     return y;
 }
 
+template <bool PAIR>
 __global__ void __launch_bounds__(kThreads, 1)
 sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) {
     extern __shared__ __align__(1024) uint8_t smem[];
     __shared__ SigBars bar;
+    constexpr int kKBox = PAIR ? kBox / 2 : kBox;         // this CTA's keys of a block x 64 columns
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int r0 = static_cast<int>(gridDim.z - 1 - blockIdx.z) * kRows, h = blockIdx.x, b = blockIdx.y;      // tiles with most keys first
+    const int cta = PAIR ? static_cast<int>(cluster_ctarank()) : 0;
     const int last_key = p.start_pos + min(r0 + kRows, p.T) - 1, n_blk = last_key / kKeys + 1;
     uint8_t* q_smem = smem;
     uint8_t* k_ring = q_smem + p.nb_k * kBox;
-    uint8_t* v_ring = k_ring + p.k_stages * p.kbs * kBox;
+    uint8_t* v_ring = k_ring + p.k_stages * p.kbs * kKBox;
     const WaitCtx ctx{&bar.abort_flag, p.status};
+    // copies credit the issuing CTA's barrier, commits go to both CTAs
+    auto load = [&](void* dst, const CUtensorMap* m, uint64_t* full, int c0, int c1, int c2, int c3) {
+        if constexpr (PAIR) tma_load_4d_pair(dst, m, map_to_cta(smem_u32(full), 0), c0, c1, c2, c3);
+        else tma_load_4d(dst, m, full, c0, c1, c2, c3);
+    };
+    auto expect = [&](uint64_t* full, int bytes) {
+        if (cta == 0) mbar_arrive_expect_tx(full, PAIR ? 2 * bytes : bytes);
+    };
+    auto commit = [&](uint64_t* to) {
+        if constexpr (PAIR) umma2_commit(to);
+        else umma_commit(to);
+    };
 
     if (threadIdx.x == 0) {
         bar.abort_flag = 0;
         mbar_init(&bar.q_full, 1);
         for (int i = 0; i < kMaxStages; ++i) { mbar_init(&bar.k_full[i], 1); mbar_init(&bar.k_empty[i], 1); mbar_init(&bar.v_full[i], 1); mbar_init(&bar.v_empty[i], 1); }
-        for (int i = 0; i < 2; ++i) { mbar_init(&bar.s_full[i], 1); mbar_init(&bar.p_ready[i], kWeightThreads); }
+        for (int i = 0; i < 2; ++i) { mbar_init(&bar.s_full[i], 1); mbar_init(&bar.p_ready[i], (PAIR ? 2 : 1) * kWeightThreads / 32); }
         mbar_init(&bar.o_done, 1);
         mbar_init(&bar.drain, 1);
         mbar_fence_init();
         if ((smem_u32(smem) & 1023) != 0) { bar.abort_flag = 1; atomicCAS(p.status, 0, (3 << 24) | 0x3); }      // the swizzle needs 1024-byte tiles
     }
-    if (warp == 9) { tmem_alloc(&bar.tmem, 512); tmem_relinquish(); }
+    if (warp == 9) {
+        __syncwarp();
+        if constexpr (PAIR) { tmem_alloc2(&bar.tmem, 512); tmem_relinquish2(); }
+        else { tmem_alloc(&bar.tmem, 512); tmem_relinquish(); }
+    }
     tc_fence_before();
     __syncthreads();
+    if constexpr (PAIR) { cluster_arrive(); cluster_wait(); }        // both CTAs' barriers exist before anything crosses the pair
     tc_fence_after();
     const uint32_t tmem = bar.tmem;
     const bool dead = *static_cast<volatile int*>(&bar.abort_flag) != 0;
@@ -86,8 +112,8 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
     } else if (warp == 8) {
         if (lane == 0) {
             const int slot = p.slots ? p.slots[b] : b;
-            mbar_arrive_expect_tx(&bar.q_full, p.nb_k * kBox);
-            for (int i = 0; i < p.nb_k; ++i) tma_load_4d(q_smem + i * kBox, &maps.q, &bar.q_full, i * 64, h, r0, b);
+            expect(&bar.q_full, p.nb_k * kBox);
+            for (int i = 0; i < p.nb_k; ++i) load(q_smem + i * kBox, &maps.q, &bar.q_full, i * 64, h, r0, b);
             bool ok = true;
             int n = 0;
             auto load_k = [&](int j) {
@@ -95,8 +121,8 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
                     const int st = n % p.k_stages, round = n / p.k_stages;
                     if (round > 0) ok = mbar_wait(&bar.k_empty[st], (round - 1) & 1, ctx, 0xD1);
                     if (!ok) return;
-                    mbar_arrive_expect_tx(&bar.k_full[st], p.kbs * kBox);
-                    for (int x = 0; x < p.kbs; ++x) tma_load_4d(k_ring + (st * p.kbs + x) * kBox, &maps.k, &bar.k_full[st], (i + x) * 64, 0, j * kKeys, slot);
+                    expect(&bar.k_full[st], p.kbs * kKBox);
+                    for (int x = 0; x < p.kbs; ++x) load(k_ring + (st * p.kbs + x) * kKBox, &maps.k, &bar.k_full[st], (i + x) * 64, 0, j * kKeys + 64 * cta, slot);
                 }
             };
             load_k(0);
@@ -106,14 +132,15 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
                 const int st = j % p.v_stages, round = j / p.v_stages;
                 if (round > 0) ok = mbar_wait(&bar.v_empty[st], (round - 1) & 1, ctx, 0xD8);
                 if (!ok) break;
-                mbar_arrive_expect_tx(&bar.v_full[st], p.nb_v * kBox);
-                for (int i = 0; i < p.nb_v; ++i) tma_load_4d(v_ring + (st * p.nb_v + i) * kBox, &maps.v, &bar.v_full[st], i * 64, h / p.R, j * kKeys, slot);
+                expect(&bar.v_full[st], p.nb_v * kBox);
+                for (int i = 0; i < p.nb_v; ++i) load(v_ring + (st * p.nb_v + i) * kBox, &maps.v, &bar.v_full[st], PAIR ? p.v_half * cta : i * 64, h / p.R, j * kKeys, slot);
             }
         }
     } else if (warp == 9) {
-        if (lane == 0) {
-            const uint32_t idesc_qk = make_idesc_f16(1, 0, 0, kRows, kKeys);
-            const uint32_t idesc_pv = make_idesc_f16(1, 0, 1, kRows, p.n_pv);
+        if (lane == 0 && cta == 0) {
+            constexpr int kM = PAIR ? 2 * kRows : kRows;
+            const uint32_t idesc_qk = make_idesc_f16(1, 0, 0, kM, kKeys);
+            const uint32_t idesc_pv = make_idesc_f16(1, 0, 1, kM, p.n_pv);
             const uint32_t q_addr = smem_u32(q_smem), k_addr = smem_u32(k_ring), v_addr = smem_u32(v_ring);
             bool ok = mbar_wait(&bar.q_full, 0, ctx, 0xD2);
             int n = 0;
@@ -125,14 +152,17 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
                     if (!ok) return;
                     tc_fence_after();
                     for (int x = 0; x < p.kbs; ++x) {
-                        const uint32_t kb = k_addr + (st * p.kbs + x) * kBox, qb = q_addr + (i + x) * kBox;
+                        const uint32_t kb = k_addr + (st * p.kbs + x) * kKBox, qb = q_addr + (i + x) * kBox;
                         const int steps = min(4, p.ks - (i + x) * 4);
-                        for (int kk = 0; kk < steps; ++kk)
-                            umma_ss(d, make_smem_desc_sw128(qb + kk * 32, 16, 1024), make_smem_desc_sw128(kb + kk * 32, 16, 1024), idesc_qk, (i | x | kk) ? 1u : 0u);
+                        for (int kk = 0; kk < steps; ++kk) {
+                            const uint64_t qd = make_smem_desc_sw128(qb + kk * 32, 16, 1024), kd = make_smem_desc_sw128(kb + kk * 32, 16, 1024);
+                            if constexpr (PAIR) umma2_ss(d, qd, kd, idesc_qk, (i | x | kk) ? 1u : 0u);
+                            else umma_ss(d, qd, kd, idesc_qk, (i | x | kk) ? 1u : 0u);
+                        }
                     }
-                    umma_commit(&bar.k_empty[st]);
+                    commit(&bar.k_empty[st]);
                 }
-                umma_commit(&bar.s_full[j & 1]);
+                commit(&bar.s_full[j & 1]);
             };
             if (ok) issue_qk(0);
             for (int j = 0; j < n_blk && ok; ++j) {
@@ -144,14 +174,19 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
                 tc_fence_after();
                 const uint32_t a = tmem + (j & 1) * kKeys, vb = v_addr + st * p.nb_v * kBox;
                 for (int half = 0; half < 2; ++half)     // hi, lo
-                    for (int kk = 0; kk < kKeys / 16; ++kk)
-                        umma_ts(tmem + 2 * kKeys, a + (kk >> 2) * 64 + half * 32 + (kk & 3) * 8, make_smem_desc_sw128(vb + kk * 2048, kBox, 1024), idesc_pv, (j | half | kk) ? 1u : 0u);
-                umma_commit(&bar.v_empty[st]);
+                    for (int kk = 0; kk < kKeys / 16; ++kk) {
+                        const uint32_t w = a + (kk >> 2) * 64 + half * 32 + (kk & 3) * 8;
+                        const uint64_t vd = make_smem_desc_sw128(vb + kk * 2048, kBox, 1024);
+                        if constexpr (PAIR) umma2_ts(tmem + 2 * kKeys, w, vd, idesc_pv, (j | half | kk) ? 1u : 0u);
+                        else umma_ts(tmem + 2 * kKeys, w, vd, idesc_pv, (j | half | kk) ? 1u : 0u);
+                    }
+                commit(&bar.v_empty[st]);
             }
-            if (ok) umma_commit(&bar.o_done);
-            umma_commit(&bar.drain);                     // nothing may be in flight when TMEM is freed
-            mbar_wait(&bar.drain, 0, ctx, 0xD5);
+            if (ok) commit(&bar.o_done);
+            commit(&bar.drain);                          // nothing may be in flight when TMEM is freed
         }
+        if (lane == 0) mbar_wait(&bar.drain, 0, ctx, 0xD5);
+        __syncwarp();
     } else {
         const int r = (warp & 3) * 32 + lane, half = warp >> 2;          // row of the tile = TMEM lane; half of a block's keys
         const uint32_t lane_base = static_cast<uint32_t>((warp & 3) * 32) << 16;
@@ -203,7 +238,11 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
             }
             tmem_st_wait();
             tc_fence_before();
-            mbar_arrive(&bar.p_ready[j & 1]);
+            __syncwarp();
+            if (lane == 0) {
+                if constexpr (PAIR) mbar_arrive_cluster(map_to_cta(smem_u32(&bar.p_ready[j & 1]), 0));
+                else mbar_arrive(&bar.p_ready[j & 1]);
+            }
         }
         if (ok) ok = mbar_wait_warp(&bar.o_done, 0, ctx, 0xD7);
         if (ok) {
@@ -232,7 +271,12 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
         tc_fence_before();
     }
     __syncthreads();
-    if (warp == 9) tmem_dealloc(tmem, 512);
+    if constexpr (PAIR) { cluster_arrive(); cluster_wait(); }        // nobody signals the peer any more
+    if (warp == 9) {
+        tc_fence_after();
+        if constexpr (PAIR) tmem_dealloc2(tmem, 512);
+        else tmem_dealloc(tmem, 512);
+    }
     abort_linger(&bar.abort_flag);
 }
 
@@ -246,28 +290,49 @@ bool sig_prefill_sm100_supported(const vb200_sigattn_args& a) {
 int launch_sig_prefill_sm100(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& pl, const void* q, int* status) {
     const int kd = a.G * a.dim, n_ctx = a.start_pos + a.T, slots = a.slots ? 1 << 20 : a.B;      // a row's slot is the caller's promise
     if (n_ctx > a.cap) return set_detail(VB200_ERR_INVALID_ARG, "vb200_sigattn_forward: the prompt does not fit the cache");
+    // two SMs per pair of heads that share their values; narrow keys are not what bounds the single form
+    const bool pair = (a.H / a.G) % 2 == 0 && (a.vdim == 64 || a.vdim == 128) && kd >= 192 && a.form != 2;
     SigMaps maps;
     if (int rc = make_map_4d(&maps.q, q, kd, a.H, a.T, a.B, pl.qld, static_cast<long long>(a.H) * pl.qld, static_cast<long long>(a.T) * a.H * pl.qld, kRows)) return rc;
-    if (int rc = make_map_4d(&maps.k, a.k_cache, kd, 1, n_ctx, slots, a.ldk, a.ldk, a.ldk * a.cap, kKeys)) return rc;
+    if (int rc = make_map_4d(&maps.k, a.k_cache, kd, 1, n_ctx, slots, a.ldk, a.ldk, a.ldk * a.cap, pair ? kKeys / 2 : kKeys)) return rc;
     if (int rc = make_map_4d(&maps.v, a.v_cache, a.vdim, a.G, n_ctx, slots, a.vdim, a.ldv, a.ldv * a.cap, kKeys)) return rc;
     SigTileParams p{};
     p.T = a.T; p.start_pos = a.start_pos; p.vdim = a.vdim; p.R = a.H / a.G; p.n_bias = a.n_bias;
     p.gate_col = a.H * a.dim + a.G * (a.dim + a.vdim);
-    p.ks = (kd + 15) / 16; p.nb_k = (kd + 63) / 64; p.nb_v = (a.vdim + 63) / 64;
+    p.ks = (kd + 15) / 16; p.nb_k = (kd + 63) / 64; p.nb_v = pair ? 1 : (a.vdim + 63) / 64; p.v_half = a.vdim / 2;
     p.bias = a.bias; p.proj = static_cast<const __nv_bfloat16*>(a.proj); p.out = static_cast<__nv_bfloat16*>(a.out);
     p.ldp = a.ldp; p.ldo = a.ldo; p.slots = a.slots; p.status = status;
     p.n_pv = pad_to(a.vdim, 16);
-    // rings: what Q leaves.  Two boxes per K stage halve the commits between products; V needs depth only where K is short
-    const int left = kBoxesPerSm - p.nb_k;
-    p.v_stages = left - 2 * p.nb_v >= 4 ? 2 : 1;
-    p.kbs = p.nb_k % 2 == 0 ? 2 : 1;
-    p.k_stages = (left - p.v_stages * p.nb_v) / p.kbs;
+    // rings: what Q leaves.  Several boxes per K stage: every commit between products costs; V needs depth only where K is short
+    const int k_box = pair ? kBox / 2 : kBox;
+    int left = (kBoxesPerSm - p.nb_k) * kBox;
+    p.v_stages = pair || left - 2 * p.nb_v * kBox >= 4 * kBox ? 2 : 1;
+    left -= p.v_stages * p.nb_v * kBox;
+    p.kbs = p.nb_k % 4 == 0 && left >= 8 * k_box ? 4 : p.nb_k % 2 == 0 ? 2 : 1;
+    p.k_stages = left / (p.kbs * k_box);
     if (p.k_stages > kMaxStages) p.k_stages = kMaxStages;
-    size_t smem = static_cast<size_t>(p.nb_k + p.k_stages * p.kbs + p.v_stages * p.nb_v) * kBox;
+    size_t smem = static_cast<size_t>(p.nb_k + p.v_stages * p.nb_v) * kBox + static_cast<size_t>(p.k_stages) * p.kbs * k_box;
     if (smem < 120 * 1024) smem = 120 * 1024;            // never a second CTA on an SM: it would find no TMEM
-    if (int rc = allow_smem(sig_prefill_sm100_kernel, smem)) return rc;
-    return launch_pdl(sig_prefill_sm100_kernel, dim3(static_cast<unsigned>(a.H), static_cast<unsigned>(a.B), static_cast<unsigned>((a.T + kRows - 1) / kRows)), dim3(kThreads), smem, s,
-                      maps, p);
+    auto kernel = pair ? sig_prefill_sm100_kernel<true> : sig_prefill_sm100_kernel<false>;
+    if (int rc = allow_smem(kernel, smem)) return rc;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(static_cast<unsigned>(a.H), static_cast<unsigned>(a.B), static_cast<unsigned>((a.T + kRows - 1) / kRows));
+    cfg.blockDim = dim3(kThreads);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = s;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = 2;
+    attr[1].val.clusterDim.y = 1;
+    attr[1].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pair ? 2 : 1;
+    VB200_CUDA_TRY(cudaLaunchKernelEx(&cfg, kernel, maps, p));
+    note_launch();
+    note_sigattn_kernel(pair ? "sig_prefill_sm100_kernel (pair)" : "sig_prefill_sm100_kernel");
+    return VB200_OK;
 }
 
 }  // namespace vb200
