@@ -35,7 +35,7 @@ struct SigMaps { CUtensorMap q, k, v; };
 
 struct SigTileParams {
     int T, start_pos, vdim, R, n_bias, gate_col;
-    int ks, nb_k, nb_v, n_pv;                 // 16-column steps of kd, 64-column boxes, columns of the second product
+    int nb_k, nb_v, n_pv;                     // 64-column boxes of a key and a value row, columns of the second product
     int kbs, k_stages, v_stages;              // boxes per K stage, ring depths
     int v_half;                               // PAIR: value columns of one CTA
     const float* bias;
@@ -47,7 +47,7 @@ struct SigTileParams {
 };
 
 struct SigBars {
-    uint64_t q_full, k_full[kMaxStages], k_empty[kMaxStages], v_full[kMaxStages], v_empty[kMaxStages], s_full[2], p_ready[2], o_done, drain;
+    uint64_t q_full[kMaxStages], k_full[kMaxStages], k_empty[kMaxStages], v_full[kMaxStages], v_empty[kMaxStages], s_full[2], p_ready[2], o_done, drain;
     uint32_t tmem;
     int abort_flag;
 };
@@ -87,8 +87,10 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
 
     if (threadIdx.x == 0) {
         bar.abort_flag = 0;
-        mbar_init(&bar.q_full, 1);
-        for (int i = 0; i < kMaxStages; ++i) { mbar_init(&bar.k_full[i], 1); mbar_init(&bar.k_empty[i], 1); mbar_init(&bar.v_full[i], 1); mbar_init(&bar.v_empty[i], 1); }
+        for (int i = 0; i < kMaxStages; ++i) {
+            mbar_init(&bar.q_full[i], 1);
+            mbar_init(&bar.k_full[i], 1); mbar_init(&bar.k_empty[i], 1); mbar_init(&bar.v_full[i], 1); mbar_init(&bar.v_empty[i], 1);
+        }
         for (int i = 0; i < 2; ++i) { mbar_init(&bar.s_full[i], 1); mbar_init(&bar.p_ready[i], (PAIR ? 2 : 1) * kWeightThreads / 32); }
         mbar_init(&bar.o_done, 1);
         mbar_init(&bar.drain, 1);
@@ -112,28 +114,32 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
     } else if (warp == 8) {
         if (lane == 0) {
             const int slot = p.slots ? p.slots[b] : b;
-            expect(&bar.q_full, p.nb_k * kBox);
-            for (int i = 0; i < p.nb_k; ++i) load(q_smem + i * kBox, &maps.q, &bar.q_full, i * 64, h, r0, b);
             bool ok = true;
-            int n = 0;
+            int ks = 0, vs = 0;
+            uint32_t k_phase = 1, v_phase = 1;           // parity 1: the first round finds every stage free
             auto load_k = [&](int j) {
-                for (int i = 0; i < p.nb_k && ok; i += p.kbs, ++n) {
-                    const int st = n % p.k_stages, round = n / p.k_stages;
-                    if (round > 0) ok = mbar_wait(&bar.k_empty[st], (round - 1) & 1, ctx, 0xD1);
+                for (int i = 0; i < p.nb_k; i += p.kbs) {
+                    if (j == 0) {                        // the queries come along with the first block's keys, stage by stage
+                        uint64_t* full = &bar.q_full[i / p.kbs];
+                        expect(full, p.kbs * kBox);
+                        for (int x = 0; x < p.kbs; ++x) load(q_smem + (i + x) * kBox, &maps.q, full, (i + x) * 64, h, r0, b);
+                    }
+                    ok = mbar_wait(&bar.k_empty[ks], k_phase, ctx, 0xD1);
                     if (!ok) return;
-                    expect(&bar.k_full[st], p.kbs * kKBox);
-                    for (int x = 0; x < p.kbs; ++x) load(k_ring + (st * p.kbs + x) * kKBox, &maps.k, &bar.k_full[st], (i + x) * 64, 0, j * kKeys + 64 * cta, slot);
+                    expect(&bar.k_full[ks], p.kbs * kKBox);
+                    for (int x = 0; x < p.kbs; ++x) load(k_ring + (ks * p.kbs + x) * kKBox, &maps.k, &bar.k_full[ks], (i + x) * 64, 0, j * kKeys + 64 * cta, slot);
+                    if (++ks == p.k_stages) { ks = 0; k_phase ^= 1; }
                 }
             };
             load_k(0);
             for (int j = 0; j < n_blk && ok; ++j) {
                 if (j + 1 < n_blk) load_k(j + 1);
                 if (!ok) break;
-                const int st = j % p.v_stages, round = j / p.v_stages;
-                if (round > 0) ok = mbar_wait(&bar.v_empty[st], (round - 1) & 1, ctx, 0xD8);
+                ok = mbar_wait(&bar.v_empty[vs], v_phase, ctx, 0xD8);
                 if (!ok) break;
-                expect(&bar.v_full[st], p.nb_v * kBox);
-                for (int i = 0; i < p.nb_v; ++i) load(v_ring + (st * p.nb_v + i) * kBox, &maps.v, &bar.v_full[st], PAIR ? p.v_half * cta : i * 64, h / p.R, j * kKeys, slot);
+                expect(&bar.v_full[vs], p.nb_v * kBox);
+                for (int i = 0; i < p.nb_v; ++i) load(v_ring + (vs * p.nb_v + i) * kBox, &maps.v, &bar.v_full[vs], PAIR ? p.v_half * cta : i * 64, h / p.R, j * kKeys, slot);
+                if (++vs == p.v_stages) { vs = 0; v_phase ^= 1; }
             }
         }
     } else if (warp == 9) {
@@ -141,26 +147,37 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
             constexpr int kM = PAIR ? 2 * kRows : kRows;
             const uint32_t idesc_qk = make_idesc_f16(1, 0, 0, kM, kKeys);
             const uint32_t idesc_pv = make_idesc_f16(1, 0, 1, kM, p.n_pv);
-            const uint32_t q_addr = smem_u32(q_smem), k_addr = smem_u32(k_ring), v_addr = smem_u32(v_ring);
-            bool ok = mbar_wait(&bar.q_full, 0, ctx, 0xD2);
-            int n = 0;
+            // what this one thread executes between two products is what holds the tensor pipe up: descriptors are built once (only the
+            // start address, in units of 16 bytes, moves), stages and parities are counted, the steps of a box are unrolled.  Columns
+            // past kd are zero in both operands, so every box takes its four steps.
+            const uint64_t q_desc = make_smem_desc_sw128(smem_u32(q_smem), 16, 1024), k_desc = make_smem_desc_sw128(smem_u32(k_ring), 16, 1024);
+            const uint64_t v_desc = make_smem_desc_sw128(smem_u32(v_ring), kBox, 1024);
+            const uint32_t k_stage16 = p.kbs * (kKBox >> 4), v_stage16 = p.nb_v * (kBox >> 4);
+            bool ok = true;
+            int ks = 0, vs = 0;
+            uint32_t k_phase = 0, v_phase = 0;
             auto issue_qk = [&](int j) {
                 const uint32_t d = tmem + (j & 1) * kKeys;
-                for (int i = 0; i < p.nb_k; i += p.kbs, ++n) {
-                    const int st = n % p.k_stages;
-                    ok = mbar_wait(&bar.k_full[st], (n / p.k_stages) & 1, ctx, 0xD3);
+                uint64_t qd = q_desc;
+                uint32_t acc = 0;
+                for (int i = 0; i < p.nb_k; i += p.kbs) {
+                    if (j == 0) ok = mbar_wait(&bar.q_full[i / p.kbs], 0, ctx, 0xD2);
+                    ok = ok && mbar_wait(&bar.k_full[ks], k_phase, ctx, 0xD3);
                     if (!ok) return;
                     tc_fence_after();
+                    uint64_t kd = k_desc + ks * k_stage16;
                     for (int x = 0; x < p.kbs; ++x) {
-                        const uint32_t kb = k_addr + (st * p.kbs + x) * kKBox, qb = q_addr + (i + x) * kBox;
-                        const int steps = min(4, p.ks - (i + x) * 4);
-                        for (int kk = 0; kk < steps; ++kk) {
-                            const uint64_t qd = make_smem_desc_sw128(qb + kk * 32, 16, 1024), kd = make_smem_desc_sw128(kb + kk * 32, 16, 1024);
-                            if constexpr (PAIR) umma2_ss(d, qd, kd, idesc_qk, (i | x | kk) ? 1u : 0u);
-                            else umma_ss(d, qd, kd, idesc_qk, (i | x | kk) ? 1u : 0u);
+#pragma unroll
+                        for (int kk = 0; kk < 4; ++kk) {
+                            if constexpr (PAIR) umma2_ss(d, qd + 2 * kk, kd + 2 * kk, idesc_qk, kk > 0 ? 1u : acc);
+                            else umma_ss(d, qd + 2 * kk, kd + 2 * kk, idesc_qk, kk > 0 ? 1u : acc);
                         }
+                        acc = 1;
+                        qd += kBox >> 4;
+                        kd += kKBox >> 4;
                     }
-                    commit(&bar.k_empty[st]);
+                    commit(&bar.k_empty[ks]);
+                    if (++ks == p.k_stages) { ks = 0; k_phase ^= 1; }
                 }
                 commit(&bar.s_full[j & 1]);
             };
@@ -168,19 +185,20 @@ sig_prefill_sm100_kernel(const __grid_constant__ SigMaps maps, SigTileParams p) 
             for (int j = 0; j < n_blk && ok; ++j) {
                 if (j + 1 < n_blk) issue_qk(j + 1);      // its S held the weights of block j-1, whose product was issued before
                 if (!ok) break;
-                const int st = j % p.v_stages;
-                ok = mbar_wait(&bar.v_full[st], (j / p.v_stages) & 1, ctx, 0xD9) && mbar_wait(&bar.p_ready[j & 1], (j >> 1) & 1, ctx, 0xD4);
+                ok = mbar_wait(&bar.v_full[vs], v_phase, ctx, 0xD9) && mbar_wait(&bar.p_ready[j & 1], (j >> 1) & 1, ctx, 0xD4);
                 if (!ok) break;
                 tc_fence_after();
-                const uint32_t a = tmem + (j & 1) * kKeys, vb = v_addr + st * p.nb_v * kBox;
-                for (int half = 0; half < 2; ++half)     // hi, lo
-                    for (int kk = 0; kk < kKeys / 16; ++kk) {
-                        const uint32_t w = a + (kk >> 2) * 64 + half * 32 + (kk & 3) * 8;
-                        const uint64_t vd = make_smem_desc_sw128(vb + kk * 2048, kBox, 1024);
-                        if constexpr (PAIR) umma2_ts(tmem + 2 * kKeys, w, vd, idesc_pv, (j | half | kk) ? 1u : 0u);
-                        else umma_ts(tmem + 2 * kKeys, w, vd, idesc_pv, (j | half | kk) ? 1u : 0u);
-                    }
-                commit(&bar.v_empty[st]);
+                const uint32_t w = tmem + (j & 1) * kKeys, o = tmem + 2 * kKeys, acc = j > 0 ? 1u : 0u;
+                const uint64_t vd = v_desc + vs * v_stage16;
+#pragma unroll
+                for (int i = 0; i < 2 * (kKeys / 16); ++i) {             // hi, then lo
+                    const int half = i / (kKeys / 16), kk = i % (kKeys / 16);
+                    const uint32_t at = w + (kk >> 2) * 64 + half * 32 + (kk & 3) * 8;
+                    if constexpr (PAIR) umma2_ts(o, at, vd + kk * (2048 >> 4), idesc_pv, i > 0 ? 1u : acc);
+                    else umma_ts(o, at, vd + kk * (2048 >> 4), idesc_pv, i > 0 ? 1u : acc);
+                }
+                commit(&bar.v_empty[vs]);
+                if (++vs == p.v_stages) { vs = 0; v_phase ^= 1; }
             }
             if (ok) commit(&bar.o_done);
             commit(&bar.drain);                          // nothing may be in flight when TMEM is freed
@@ -299,7 +317,7 @@ int launch_sig_prefill_sm100(cudaStream_t s, const vb200_sigattn_args& a, const 
     SigTileParams p{};
     p.T = a.T; p.start_pos = a.start_pos; p.vdim = a.vdim; p.R = a.H / a.G; p.n_bias = a.n_bias;
     p.gate_col = a.H * a.dim + a.G * (a.dim + a.vdim);
-    p.ks = (kd + 15) / 16; p.nb_k = (kd + 63) / 64; p.nb_v = pair ? 1 : (a.vdim + 63) / 64; p.v_half = a.vdim / 2;
+    p.nb_k = (kd + 63) / 64; p.nb_v = pair ? 1 : (a.vdim + 63) / 64; p.v_half = a.vdim / 2;
     p.bias = a.bias; p.proj = static_cast<const __nv_bfloat16*>(a.proj); p.out = static_cast<__nv_bfloat16*>(a.out);
     p.ldp = a.ldp; p.ldo = a.ldo; p.slots = a.slots; p.status = status;
     p.n_pv = pad_to(a.vdim, 16);
