@@ -381,6 +381,30 @@ def test_selective_scan_portions_and_slots(cuda, name, kind):
     _status()
 
 
+@pytest.mark.parametrize("kind", ["f32", "bf16"])
+def test_selective_steps_of_many_sequences(cuda, kind):
+    """Enough rows for the step sizes to become a product of their own; sequences at unequal lengths, one of them new."""
+    import torch
+    name, B = "small", 21
+    core, w, rng = _scan_case(name, kind, cuda, slots=B)
+    inner = SCAN[name][0]
+    lens = [int(n) for n in rng.integers(1, 30, B)]
+    lens[5] = 0
+    ps = [_rnd(kind)(rng.standard_normal((n + 3, 2 * inner))) for n in lens]
+    wants = [_scan_want(p, w, name, kind) for p in ps]
+    slots = rng.permutation(B).astype(np.int32)
+    core.state.fill_(50.0)
+    for b in range(B):
+        if lens[b]:
+            core.forward(_torch(ps[b][:lens[b]], cuda, core.dtype), 1, torch.zeros(1, dtype=torch.int32, device=cuda), slots=_torch(slots[b:b + 1], cuda))
+    for step in range(3):
+        proj = _torch(np.stack([ps[b][lens[b] + step] for b in range(B)]), cuda, core.dtype)
+        y = _np(core.forward(proj, B, _torch(np.array(lens, np.int32) + np.int32(step), cuda), slots=_torch(slots, cuda)))
+        for b in range(B):
+            assert np.abs(y[b] - wants[b][lens[b] + step]).max() <= (5e-5 if kind == "f32" else 2e-2) * np.abs(wants[b]).max(), (step, b)
+    _status()
+
+
 def test_selective_scan_keeps_a_long_memory(cuda):
     """A slow decay carries an early input over a thousand tokens, in one portion and over decoded tokens."""
     import torch

@@ -242,7 +242,8 @@ linear_wide_kernel(const __grid_constant__ LinearMaps maps, LinearParams p) {
         if (lane == 0) {
             uint32_t it = 0;
             for (int t = blockIdx.x; t < tiles && !*abort_flag; t += gridDim.x) {
-                const int mt = t % m_tiles, nt = t / m_tiles;   // consecutive CTAs share a W tile through L2
+                // consecutive CTAs share a W tile through L2; grouped: a row tile, and a group's W stays in L2 for its few row tiles
+                const int mt = GROUPED ? t / n_tiles : t % m_tiles, nt = GROUPED ? t % n_tiles : t / m_tiles;
                 int row0 = mt * kTileA, w0 = nt * BN;
                 if (GROUPED) { const int4 g = p.group_tiles[mt]; row0 = g.x; w0 += g.z * p.group_rows; }
                 for (int kb = 0; kb < k_blocks; ++kb, ++it) {
@@ -287,7 +288,7 @@ linear_wide_kernel(const __grid_constant__ LinearMaps maps, LinearParams p) {
         const int quarter = warp & 3;                 // TMEM lanes this warp may read
         uint32_t tile_no = 0;
         for (int t = blockIdx.x; t < tiles; t += gridDim.x, ++tile_no) {
-            const int mt = t % m_tiles, nt = t / m_tiles;
+            const int mt = GROUPED ? t / n_tiles : t % m_tiles, nt = GROUPED ? t % n_tiles : t / m_tiles;
             const int buf = tile_no & 1;
             if (!mbar_wait_warp(&acc_full[buf], (tile_no >> 1) & 1, ctx, 0x45)) break;
             tc_fence_after();

@@ -289,56 +289,43 @@ selective_scan_kernel(ScanParams p, const T* __restrict__ proj, const T* __restr
     store_state(sp, live ? p.N - lane * NI : 0, S_);
 }
 
-constexpr int kStepRows = 4;       // sequences that a CTA of the decode step takes in turn
+constexpr int kStepRows = 2;       // sequences that a CTA of the decode step takes in turn
 
-// One token per sequence, step sizes included: grid (ceil(inner / kCh), ceil(B / rows)).  The LP lanes of a channel share its row of W_dt,
-// which is fetched ahead of the wait and kept for all rows.
+// One token per sequence: grid (ceil(inner / kCh), ceil(B / rows)).  dt (nullable) holds the step sizes before bias and softplus; without it
+// they are computed here: the LP lanes of a channel share its row of W_dt, which is fetched ahead of the wait and kept for all rows.
 template <typename T, int LP, int NI>
 __global__ void __launch_bounds__(kThreads)
-selective_step_kernel(ScanParams p, int rows, const T* __restrict__ proj, const T* __restrict__ xc, const T* __restrict__ xdbl, const T* __restrict__ w_dt, float* __restrict__ state,
-                      T* __restrict__ out) {
+selective_step_kernel(ScanParams p, int rows, const T* __restrict__ proj, const T* __restrict__ xc, const T* __restrict__ xdbl, const T* __restrict__ w_dt,
+                      const float* __restrict__ dt, float* __restrict__ state, T* __restrict__ out) {
     constexpr int CH = kThreads / LP;
     extern __shared__ __align__(16) uint8_t raw[];
-    float* sm = reinterpret_cast<float*>(raw);         // [rows][dt | B | C]
+    float* sm = reinterpret_cast<float*>(raw);         // [rows][(dt |) B | C]
     const int tid = threadIdx.x, lane = tid % LP, b0 = blockIdx.y * rows, nb = min(rows, p.B - b0), c = blockIdx.x * CH + tid / LP, cc = min(c, p.inner - 1);
     const bool live = c < p.inner;
     float a[NI];
-#pragma unroll
-    for (int i = 0; i < NI; ++i) {
-        const int n = lane * NI + i;
-        a[i] = n < p.N ? __ldg(p.A + static_cast<long long>(cc) * p.N + n) : 0.f;
-    }
+    load_state(p.A + static_cast<long long>(cc) * p.N + lane * NI, p.N - lane * NI, a);
     const float bias = __ldg(p.dt_bias + cc), Dc = __ldg(p.D + cc);
     constexpr int kAhead = 4;                          // pieces of W_dt kept in registers
-    const int n8 = p.rank / 8, ld = p.rank + 2 * p.N;
+    const int n8 = dt != nullptr ? 0 : p.rank / 8, skip = dt != nullptr ? p.rank : 0, ld = p.rank + 2 * p.N - skip;      // staged columns
     const T* wr = w_dt + static_cast<long long>(cc) * p.rank;
     Raw8<T> w[kAhead];
 #pragma unroll
     for (int i = 0; i < kAhead; ++i)
         if (lane + i * LP < n8) w[i].load(wr + (lane + i * LP) * 8);
     pdl_begin();
-    float next[NI], xn, zn;
-    float* sp_next;
-    auto fetch = [&](int r) {
-        const int b = b0 + r, slot = p.slots ? p.slots[b] : b;
-        sp_next = state + (static_cast<long long>(slot) * p.inner + cc) * p.N + lane * NI;
-        load_state(sp_next, p.pos[b] > 0 ? p.N - lane * NI : 0, next);
-        xn = Elem<T>::to_f(xc[static_cast<long long>(b) * p.inner + cc]);
-        zn = Elem<T>::to_f(proj[b * p.ldp + p.inner + cc]);
-    };
-    fetch(0);
-    for (int i = tid; i < nb * ld; i += kThreads) {
-        const int r = i / ld;
-        sm[i] = Elem<T>::to_f(xdbl[(b0 + r) * p.ldx + i - r * ld]);
-    }
-    __syncthreads();
+    for (int r = 0; r < nb; ++r)
+        for (int i = tid; i < ld; i += kThreads) sm[r * ld + i] = Elem<T>::to_f(xdbl[(b0 + r) * p.ldx + skip + i]);
     for (int r = 0; r < nb; ++r) {
+        const int b = b0 + r, slot = p.slots ? p.slots[b] : b;
+        float* sp = state + (static_cast<long long>(slot) * p.inner + cc) * p.N + lane * NI;
         float S_[NI];
+        load_state(sp, p.N - lane * NI, S_);
+        if (p.pos[b] == 0) {                           // a new sequence ignores what its slot holds
 #pragma unroll
-        for (int i = 0; i < NI; ++i) S_[i] = next[i];
-        const float x = xn, z = zn;
-        float* sp = sp_next;
-        if (r + 1 < nb) fetch(r + 1);                  // the next sequence's state is under way meanwhile
+            for (int i = 0; i < NI; ++i) S_[i] = 0.f;
+        }
+        const float x = Elem<T>::to_f(xc[static_cast<long long>(b) * p.inner + cc]), z = Elem<T>::to_f(proj[b * p.ldp + p.inner + cc]);
+        if (r == 0) __syncthreads();
         const float* row = sm + r * ld;
         float d = 0.f;
         auto dot8 = [&](const float (&wv)[8], int k) {
@@ -349,12 +336,16 @@ selective_step_kernel(ScanParams p, int rows, const T* __restrict__ proj, const 
 #pragma unroll
         for (int i = 0; i < kAhead; ++i)
             if (lane + i * LP < n8) { float wv[8]; w[i].get(wv); dot8(wv, lane + i * LP); }
+#pragma unroll 1
         for (int k = lane + kAhead * LP; k < n8; k += LP) { float wv[8]; load8(wr + k * 8, wv); dot8(wv, k); }
+        if (dt != nullptr) d = dt[static_cast<long long>(b) * p.inner + cc];
+        else {
 #pragma unroll
-        for (int o = LP / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xFFFFFFFFu, d, o);
+            for (int o = LP / 2; o > 0; o >>= 1) d += __shfl_xor_sync(0xFFFFFFFFu, d, o);
+        }
         d = softplus_for<T>(d + bias);
         const float dx = d * x, dl = decay_dt<T>(d);
-        const float *Bn = row + p.rank + lane * NI, *Cn = Bn + p.N;
+        const float *Bn = row + ld - 2 * p.N + lane * NI, *Cn = Bn + p.N;
         float y = 0.f;
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
@@ -407,7 +398,7 @@ SelectivePlan plan_selective(const vb200_selective_args& a) {
     SelectivePlan pl{};
     auto up = [](size_t x) { return (x + 255) / 256 * 256; };
     const size_t esz = a.dtype == VB200_F32 ? 4 : 2, M = static_cast<size_t>(a.B) * a.T;
-    pl.dt_gemm = a.T > 1;
+    pl.dt_gemm = a.T > 1 || a.B >= 16;          // few rows: W_dt streams through the step kernel instead
     pl.conv_bytes = up(M * a.inner * esz);
     pl.xdbl_bytes = up(M * (a.rank + 2 * a.N) * esz);
     pl.dt_bytes = pl.dt_gemm ? up(M * a.inner * 4) : 0;
@@ -443,7 +434,7 @@ int launch_selective(cudaStream_t s, const vb200_selective_args& a, const Select
                 const dim3 step_grid(grid.x, static_cast<unsigned>((a.B + rows - 1) / rows));
                 const size_t smem = sizeof(float) * ldx * rows;
                 rc = allow_smem(selective_step_kernel<T, LP, NI>, smem);
-                if (rc == VB200_OK) rc = launch_pdl(selective_step_kernel<T, LP, NI>, step_grid, dim3(kThreads), smem, s, p, rows, proj, x, d, static_cast<const T*>(a.w_dt), a.state, out);
+                if (rc == VB200_OK) rc = launch_pdl(selective_step_kernel<T, LP, NI>, step_grid, dim3(kThreads), smem, s, p, rows, proj, x, d, static_cast<const T*>(a.w_dt), static_cast<const float*>(pl.dt_gemm ? dt : nullptr), a.state, out);
                 note_selective_kernel("selective_step_kernel");
             } else {
                 const size_t smem = sizeof(ScanTile<T, LP, NI>);
