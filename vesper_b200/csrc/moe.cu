@@ -132,7 +132,35 @@ __device__ __forceinline__ void piece_dots(int n8, const float* x, float (&sum)[
             }
     }
 #pragma unroll
-    for (int r = 0; r < ROWS; ++r) sum[r] = warp_sum_f(sum[r]);
+    for (int r = 0; r < ROWS; ++r) sum[r] = warp_sum_f(sum[r]);      // every lane has them
+}
+
+constexpr int kRouterThreads = 1024;
+
+// Router logits and choice of one token: grid M (few tokens; prompts take the product of linear_sm100.cu).
+template <typename T>
+__global__ void __launch_bounds__(kRouterThreads)
+moe_router_kernel(const T* __restrict__ x, const T* __restrict__ w, const float* __restrict__ correction, int dim, int E, int top, int groups, int keep, float scale,
+                  int* __restrict__ ids, float* __restrict__ weights) {
+    pdl_begin();
+    extern __shared__ __align__(16) float sm[];          // [dim] x | [E] logits | [2 E + groups] of the choice
+    float* logits = sm + dim;
+    const long long m = blockIdx.x;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    for (int i = threadIdx.x * 8; i < dim; i += kRouterThreads * 8) {
+        float v[8];
+        load8(x + m * dim + i, v);
+        store8(sm + i, v);
+    }
+    __syncthreads();
+    for (int e = 2 * warp; e < E; e += kRouterThreads / 16) {
+        const int second = min(e + 1, E - 1);
+        float z[2];
+        piece_dots<T, 2>(dim / 8, sm, z, [&](int i, int r) { return w + static_cast<long long>(r ? second : e) * dim + i * 8; });
+        if (lane < 2 && e + lane < E) logits[e + lane] = z[lane];
+    }
+    __syncthreads();
+    if (warp == 0) route_token(logits, correction, E, top, groups, keep, scale, logits + E, logits + 2 * E, logits + 3 * E, ids + m * top, weights + m * top);
 }
 
 constexpr int kPairRows = 16;    // hidden units per CTA: two per warp
@@ -354,8 +382,19 @@ int launch_moe(cudaStream_t s, const vb200_moe_args& a, const MoePlan& pl, int* 
     uint8_t* ws = static_cast<uint8_t*>(a.workspace);
     float *logits = reinterpret_cast<float*>(ws + pl.logits), *weights = reinterpret_cast<float*>(ws + pl.weights);
     int* ids = reinterpret_cast<int*>(ws + pl.ids);
-    if (int rc = router_logits(s, a, logits, status)) return rc;
-    if (int rc = launch_moe_route(s, logits, pad_to(a.experts, 4), a.correction, a.M, a.experts, a.top, a.groups, a.keep, a.scale, ids, weights)) return rc;
+    const size_t router_smem = sizeof(float) * (static_cast<size_t>(a.dim) + 3 * a.experts + a.groups);
+    if (a.M <= 32 && router_smem <= 100 * 1024) {
+        auto router = [&](auto tag) -> int {
+            using T = decltype(tag);
+            if (int rc = allow_smem(moe_router_kernel<T>, router_smem)) return rc;
+            return launch_pdl(moe_router_kernel<T>, dim3(static_cast<unsigned>(a.M)), dim3(kRouterThreads), router_smem, s, static_cast<const T*>(a.x), static_cast<const T*>(a.w_router), a.correction,
+                              a.dim, a.experts, a.top, a.groups, a.keep, a.scale, ids, weights);
+        };
+        if (int rc = a.dtype == VB200_F32 ? router(float{}) : router(__nv_bfloat16{})) return rc;
+    } else {
+        if (int rc = router_logits(s, a, logits, status)) return rc;
+        if (int rc = launch_moe_route(s, logits, pad_to(a.experts, 4), a.correction, a.M, a.experts, a.top, a.groups, a.keep, a.scale, ids, weights)) return rc;
+    }
     if (pl.grouped) return launch_grouped(s, a, pl, ids, weights, status);
     MoeParams p{};
     p.M = a.M; p.dim = a.dim; p.ff = a.ff; p.ff_shared = a.ff_shared; p.E = a.experts; p.top = a.top; p.ld_out = a.ld_out; p.ld_shared = a.ld_shared;

@@ -23,77 +23,81 @@ struct SigParams {
     int *status;
 };
 
-// grid (T, B), 256 threads, one token: norms, temperature, the new cache rows, and q'.
+constexpr int kAppendThreads = 128, kHeadSlice = 4;
+
+// grid (ceil(T / tokens), B, G), a few tokens and one key / value head with its query heads: norms, temperature, the new cache rows, and that
+// group's columns of q' for every head.
 template <typename T, typename QT>
-__global__ void __launch_bounds__(256)
-sig_append_kernel(SigParams p, const T* __restrict__ proj, T* __restrict__ kc, T* __restrict__ vc, T* __restrict__ first, QT* __restrict__ qm) {
+__global__ void __launch_bounds__(kAppendThreads)
+sig_append_kernel(SigParams p, int tokens, const T* __restrict__ proj, T* __restrict__ kc, T* __restrict__ vc, T* __restrict__ first, QT* __restrict__ qm) {
+    extern __shared__ __align__(16) float qs[];          // [tokens][R * dim] scaled queries, then this group's columns of talk [H, R]
+    const int q_ld = (p.R * p.dim + 3) / 4 * 4;
+    float* tk = qs + tokens * q_ld;
+    const int t0 = blockIdx.x * tokens, b = blockIdx.y, g = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nt = min(tokens, p.T - t0);
+    for (int i = tid; i < p.H * p.R; i += kAppendThreads) tk[i] = __ldg(p.talk + (i / p.R) * p.H + g * p.R + i % p.R);
     pdl_begin();
-    extern __shared__ __align__(16) float qs[];         // [H * dim] scaled queries, then talk [H, H]
-    float* tk = qs + (p.H * p.dim + 3) / 4 * 4;
-    for (int i = threadIdx.x; i < p.H * p.H; i += 256) tk[i] = __ldg(p.talk + i);
-    const int t = blockIdx.x, b = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const long long m = static_cast<long long>(b) * p.T + t;
-    const int pos = p.pos[b] + t;
-    const long long row = static_cast<long long>(p.slots ? p.slots[b] : b) * p.cap + pos;
-    const T* src = proj + m * p.ldp;
-    const int kcols = p.G * p.dim, vcols = p.G * p.vdim;
-    const bool fits = pos < p.cap;
-    if (!fits && threadIdx.x == 0) atomicCAS(p.status, 0, (2 << 24) | b);
-    float temp = p.scale * (sizeof(QT) == 2 ? -kLog2e : 1.0f);       // the tensor-core kernels compute 2^(-score log2 e)
-    if (p.temp_every > 0) temp *= 1.0f + p.temp_coef * logf(static_cast<float>((pos + 1) / p.temp_every) + 1.0f);
-    for (int h = warp; h < p.H + p.G; h += 8) {
-        const T* x = src + h * p.dim;     // the key heads follow the query heads
+    const long long m0 = static_cast<long long>(b) * p.T + t0;
+    const int pos0 = p.pos[b] + t0, fit = min(nt, p.cap - pos0);                     // tokens that the cache has room for
+    const long long row0 = static_cast<long long>(p.slots ? p.slots[b] : b) * p.cap + pos0;
+    const int vcols = p.G * p.vdim;
+    if (fit < nt && g == 0 && tid == 0) atomicCAS(p.status, 0, (2 << 24) | b);
+    const T* vsrc = proj + m0 * p.ldp + (p.H + p.G) * p.dim + g * p.vdim;
+    for (int u = 0; u < nt; ++u)
+        for (int i = tid; i < p.vdim; i += kAppendThreads) {
+            const T raw = vsrc[u * p.ldp + i];
+            const long long shared = (m0 + u) * vcols + g * p.vdim + i;
+            float v = Elem<T>::to_f(raw);
+            if (p.value_role == 1) first[shared] = raw;
+            else if (p.value_role == 2) v = (1.0f - p.lambda) * v + p.lambda * Elem<T>::to_f(first[shared]);
+            if (u < fit) vc[(row0 + u) * p.ldv + g * p.vdim + i] = Elem<T>::from_f(v);
+        }
+    for (int k = warp; k < nt * (p.R + 1); k += kAppendThreads / 32) {               // a token's query heads of the group, then its key head
+        const int u = k / (p.R + 1), h = k - u * (p.R + 1);
+        const T* x = proj + (m0 + u) * p.ldp + (h < p.R ? g * p.R + h : p.H + g) * p.dim;
         float ss = 0.f;
         for (int i = lane; i < p.dim; i += 32) { const float v = Elem<T>::to_f(x[i]); ss = fmaf(v, v, ss); }
         const float inv = 1.0f / sqrtf(warp_sum_f(ss) / static_cast<float>(p.dim) + p.eps);
-        if (h < p.H) {
-            for (int i = lane; i < p.dim; i += 32) qs[h * p.dim + i] = Elem<T>::to_f(x[i]) * inv * temp;
-        } else if (fits) {
-            T* dst = kc + row * p.ldk + (h - p.H) * p.dim;
+        if (h < p.R) {
+            float f = p.scale * (sizeof(QT) == 2 ? -kLog2e : 1.0f);                  // the tensor-core kernels compute 2^(-score log2 e)
+            if (p.temp_every > 0) f *= 1.0f + p.temp_coef * logf(static_cast<float>((pos0 + u + 1) / p.temp_every) + 1.0f);
+            for (int i = lane; i < p.dim; i += 32) qs[u * q_ld + h * p.dim + i] = Elem<T>::to_f(x[i]) * inv * f;
+        } else if (u < fit) {
+            T* dst = kc + (row0 + u) * p.ldk + g * p.dim;
             for (int i = lane; i < p.dim; i += 32) dst[i] = Elem<T>::from_f(Elem<T>::to_f(x[i]) * inv);
         }
     }
-    const T* vsrc = src + p.H * p.dim + kcols;
-    for (int i = threadIdx.x; i < vcols; i += 256) {
-        float v = Elem<T>::to_f(vsrc[i]);
-        if (p.value_role == 1) first[m * vcols + i] = vsrc[i];
-        else if (p.value_role == 2) v = (1.0f - p.lambda) * v + p.lambda * Elem<T>::to_f(first[m * vcols + i]);
-        if (fits) vc[row * p.ldv + i] = Elem<T>::from_f(v);
-    }
     __syncthreads();
-    if (p.dim % 2 == 0 && p.R <= 8) {                    // two columns of one group per thread
-        for (int c = threadIdx.x * 2; c < p.qld; c += 512) {
-            QT* dst = qm + m * p.H * p.qld + c;
-            const int g = min(c / p.dim, p.G - 1), d = c - g * p.dim;
-            const bool pad = c >= kcols;
-            float2 qr[8];
+    const int slices = (p.H + kHeadSlice - 1) / kHeadSlice, pad = p.qld - p.G * p.dim;
+    for (int u = 0; u < nt; ++u) {
+        QT* out = qm + (m0 + u) * p.H * p.qld + g * p.dim;
+        const float* q = qs + u * q_ld;
+        if (p.dim % 2 == 0 && p.R <= 8) {                // two columns and a slice of the heads per step
+            const int pairs = p.dim / 2;
+            for (int i = tid; i < pairs * slices; i += kAppendThreads) {
+                const int sl = i / pairs, d = (i - sl * pairs) * 2;
+                float2 qr[8];
 #pragma unroll
-            for (int r = 0; r < 8; ++r) qr[r] = r < p.R && !pad ? *reinterpret_cast<const float2*>(qs + (g * p.R + r) * p.dim + d) : make_float2(0.f, 0.f);
-            for (int h = 0; h < p.H; ++h) {
-                const float* w = tk + h * p.H + g * p.R;
-                float2 a = make_float2(0.f, 0.f);
+                for (int r = 0; r < 8; ++r) qr[r] = r < p.R ? *reinterpret_cast<const float2*>(q + r * p.dim + d) : make_float2(0.f, 0.f);
+                for (int h = sl * kHeadSlice; h < min(p.H, (sl + 1) * kHeadSlice); ++h) {
+                    float2 a = make_float2(0.f, 0.f);
 #pragma unroll
-                for (int r = 0; r < 8; ++r)
-                    if (r < p.R) a = __ffma2_rn(make_float2(w[r], w[r]), qr[r], a);
-                if constexpr (sizeof(QT) == 2) *reinterpret_cast<uint32_t*>(dst + static_cast<long long>(h) * p.qld) = Elem<__nv_bfloat16>::pack2(a.x, a.y);
-                else *reinterpret_cast<float2*>(dst + static_cast<long long>(h) * p.qld) = a;
+                    for (int r = 0; r < 8; ++r)
+                        if (r < p.R) { const float w = tk[h * p.R + r]; a = __ffma2_rn(make_float2(w, w), qr[r], a); }
+                    QT* dst = out + static_cast<long long>(h) * p.qld + d;
+                    if constexpr (sizeof(QT) == 2) *reinterpret_cast<uint32_t*>(dst) = Elem<__nv_bfloat16>::pack2(a.x, a.y);
+                    else *reinterpret_cast<float2*>(dst) = a;
+                }
+            }
+        } else {
+            for (int i = tid; i < p.dim * p.H; i += kAppendThreads) {
+                const int h = i / p.dim, d = i - h * p.dim;
+                float a = 0.f;
+                for (int r = 0; r < p.R; ++r) a = fmaf(tk[h * p.R + r], q[r * p.dim + d], a);
+                out[static_cast<long long>(h) * p.qld + d] = Elem<QT>::from_f(a);
             }
         }
-        return;
-    }
-    for (int c = threadIdx.x; c < p.qld; c += 256) {
-        QT* dst = qm + m * p.H * p.qld + c;
-        if (c >= kcols) {
-            for (int h = 0; h < p.H; ++h) dst[static_cast<long long>(h) * p.qld] = Elem<QT>::from_f(0.f);
-            continue;
-        }
-        const int g = c / p.dim, d = c - g * p.dim;
-        const float* q = qs + g * p.R * p.dim + d;
-        for (int h = 0; h < p.H; ++h) {
-            float a = 0.f;
-            for (int r = 0; r < p.R; ++r) a = fmaf(tk[h * p.H + g * p.R + r], q[r * p.dim], a);
-            dst[static_cast<long long>(h) * p.qld] = Elem<QT>::from_f(a);
-        }
+        if (g == p.G - 1)                                // columns past the last group
+            for (int i = tid; i < pad * p.H; i += kAppendThreads) out[static_cast<long long>(i / pad) * p.qld + p.dim + i % pad] = Elem<QT>::from_f(0.f);
     }
 }
 
@@ -211,12 +215,14 @@ int launch_sigattn(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& p
         using T = decltype(tag);
         T *kc = static_cast<T*>(a.k_cache), *vc = static_cast<T*>(a.v_cache), *first = static_cast<T*>(a.first_values), *out = static_cast<T*>(a.out);
         const T* proj = static_cast<const T*>(a.proj);
-        const dim3 grid(static_cast<unsigned>(a.T), static_cast<unsigned>(a.B));
-        const size_t smem = sizeof(float) * ((static_cast<size_t>(a.H) * a.dim + 3) / 4 * 4 + static_cast<size_t>(a.H) * a.H);
+        const size_t q_floats = (static_cast<size_t>(p.R) * a.dim + 3) / 4 * 4;
+        const int tokens = a.T >= 16 && q_floats <= 1024 ? 4 : 1;
+        const dim3 grid(static_cast<unsigned>((a.T + tokens - 1) / tokens), static_cast<unsigned>(a.B), static_cast<unsigned>(a.G));
+        const size_t smem = sizeof(float) * (tokens * q_floats + static_cast<size_t>(a.H) * p.R);
         auto append = [&](auto* qm) -> int {
             auto kernel = sig_append_kernel<T, std::remove_pointer_t<decltype(qm)>>;
             if (int rc = allow_smem(kernel, smem)) return rc;
-            return launch_pdl(kernel, grid, dim3(256), smem, s, p, proj, kc, vc, first, qm);
+            return launch_pdl(kernel, grid, dim3(kAppendThreads), smem, s, p, tokens, proj, kc, vc, first, qm);
         };
         if (int rc = pl.mma ? append(static_cast<__nv_bfloat16*>(q)) : append(static_cast<float*>(q))) return rc;
         int rc;
