@@ -26,15 +26,19 @@ struct SigParams {
 constexpr int kAppendThreads = 128, kHeadSlice = 4;
 
 // grid (ceil(T / tokens), B, G), a few tokens and one key / value head with its query heads: norms, temperature, the new cache rows, and that
-// group's columns of q' for every head.
-template <typename T, typename QT>
+// group's columns of q' for every head.  RM: query heads of a group, rounded up to a power of two (0: more than eight, or an odd head size).
+template <typename T, typename QT, int RM>
 __global__ void __launch_bounds__(kAppendThreads)
 sig_append_kernel(SigParams p, int tokens, const T* __restrict__ proj, T* __restrict__ kc, T* __restrict__ vc, T* __restrict__ first, QT* __restrict__ qm) {
-    extern __shared__ __align__(16) float qs[];          // [tokens][R * dim] scaled queries, then this group's columns of talk [H, R]
+    extern __shared__ __align__(16) float qs[];          // [tokens][R * dim] scaled queries, then this group's columns of talk [H, RM]
     const int q_ld = (p.R * p.dim + 3) / 4 * 4;
     float* tk = qs + tokens * q_ld;
     const int t0 = blockIdx.x * tokens, b = blockIdx.y, g = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nt = min(tokens, p.T - t0);
-    for (int i = tid; i < p.H * p.R; i += kAppendThreads) tk[i] = __ldg(p.talk + (i / p.R) * p.H + g * p.R + i % p.R);
+    const int t_ld = RM > 0 ? RM : p.R;
+    for (int i = tid; i < p.H * t_ld; i += kAppendThreads) {
+        const int h = i / t_ld, r = i - h * t_ld;
+        tk[i] = r < p.R ? __ldg(p.talk + h * p.H + g * p.R + r) : 0.f;
+    }
     pdl_begin();
     const long long m0 = static_cast<long long>(b) * p.T + t0;
     const int pos0 = p.pos[b] + t0, fit = min(nt, p.cap - pos0);                     // tokens that the cache has room for
@@ -71,18 +75,23 @@ sig_append_kernel(SigParams p, int tokens, const T* __restrict__ proj, T* __rest
     for (int u = 0; u < nt; ++u) {
         QT* out = qm + (m0 + u) * p.H * p.qld + g * p.dim;
         const float* q = qs + u * q_ld;
-        if (p.dim % 2 == 0 && p.R <= 8) {                // two columns and a slice of the heads per step
+        if constexpr (RM > 0) {                          // two columns and a slice of the heads per step
             const int pairs = p.dim / 2;
             for (int i = tid; i < pairs * slices; i += kAppendThreads) {
                 const int sl = i / pairs, d = (i - sl * pairs) * 2;
-                float2 qr[8];
+                float2 qr[RM];
 #pragma unroll
-                for (int r = 0; r < 8; ++r) qr[r] = r < p.R ? *reinterpret_cast<const float2*>(q + r * p.dim + d) : make_float2(0.f, 0.f);
-                for (int h = sl * kHeadSlice; h < min(p.H, (sl + 1) * kHeadSlice); ++h) {
+                for (int r = 0; r < RM; ++r) qr[r] = r < p.R ? *reinterpret_cast<const float2*>(q + r * p.dim + d) : make_float2(0.f, 0.f);
+#pragma unroll
+                for (int e = 0; e < kHeadSlice; ++e) {
+                    const int h = sl * kHeadSlice + e;
+                    if (h >= p.H) break;
                     float2 a = make_float2(0.f, 0.f);
 #pragma unroll
-                    for (int r = 0; r < 8; ++r)
-                        if (r < p.R) { const float w = tk[h * p.R + r]; a = __ffma2_rn(make_float2(w, w), qr[r], a); }
+                    for (int r = 0; r < RM; ++r) {       // talk is padded to RM columns with zeros
+                        const float w = tk[h * RM + r];
+                        a = __ffma2_rn(make_float2(w, w), qr[r], a);
+                    }
                     QT* dst = out + static_cast<long long>(h) * p.qld + d;
                     if constexpr (sizeof(QT) == 2) *reinterpret_cast<uint32_t*>(dst) = Elem<__nv_bfloat16>::pack2(a.x, a.y);
                     else *reinterpret_cast<float2*>(dst) = a;
@@ -218,9 +227,12 @@ int launch_sigattn(cudaStream_t s, const vb200_sigattn_args& a, const SigPlan& p
         const size_t q_floats = (static_cast<size_t>(p.R) * a.dim + 3) / 4 * 4;
         const int tokens = a.T >= 16 && q_floats <= 1024 ? 4 : 1;
         const dim3 grid(static_cast<unsigned>((a.T + tokens - 1) / tokens), static_cast<unsigned>(a.B), static_cast<unsigned>(a.G));
-        const size_t smem = sizeof(float) * (tokens * q_floats + static_cast<size_t>(a.H) * p.R);
+        const int rm = a.dim % 2 != 0 || p.R > 8 ? 0 : p.R <= 1 ? 1 : p.R <= 2 ? 2 : p.R <= 4 ? 4 : 8;
+        const size_t smem = sizeof(float) * (tokens * q_floats + static_cast<size_t>(a.H) * (rm > 0 ? rm : p.R));
         auto append = [&](auto* qm) -> int {
-            auto kernel = sig_append_kernel<T, std::remove_pointer_t<decltype(qm)>>;
+            using QT = std::remove_pointer_t<decltype(qm)>;
+            auto kernel = rm == 0 ? sig_append_kernel<T, QT, 0> : rm == 1 ? sig_append_kernel<T, QT, 1> : rm == 2 ? sig_append_kernel<T, QT, 2> : rm == 4 ? sig_append_kernel<T, QT, 4>
+                                                                                                                                  : sig_append_kernel<T, QT, 8>;
             if (int rc = allow_smem(kernel, smem)) return rc;
             return launch_pdl(kernel, grid, dim3(kAppendThreads), smem, s, p, tokens, proj, kc, vc, first, qm);
         };
