@@ -55,59 +55,77 @@ sig_append_kernel(SigParams p, int tokens, const T* __restrict__ proj, T* __rest
             else if (p.value_role == 2) v = (1.0f - p.lambda) * v + p.lambda * Elem<T>::to_f(first[shared]);
             if (u < fit) vc[(row0 + u) * p.ldv + g * p.vdim + i] = Elem<T>::from_f(v);
         }
+    const float scale = p.scale * (sizeof(QT) == 2 ? -kLog2e : 1.0f);                // the tensor-core kernels compute 2^(-score log2 e)
     for (int k = warp; k < nt * (p.R + 1); k += kAppendThreads / 32) {               // a token's query heads of the group, then its key head
         const int u = k / (p.R + 1), h = k - u * (p.R + 1);
         const T* x = proj + (m0 + u) * p.ldp + (h < p.R ? g * p.R + h : p.H + g) * p.dim;
-        float ss = 0.f;
-        for (int i = lane; i < p.dim; i += 32) { const float v = Elem<T>::to_f(x[i]); ss = fmaf(v, v, ss); }
-        const float inv = 1.0f / sqrtf(warp_sum_f(ss) / static_cast<float>(p.dim) + p.eps);
+        float keep[4], ss = 0.f;                         // the first 128 columns stay in registers
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int i = lane + 32 * j;
+            keep[j] = i < p.dim ? Elem<T>::to_f(x[i]) : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) ss = fmaf(keep[j], keep[j], ss);
+        for (int i = lane + 128; i < p.dim; i += 32) { const float v = Elem<T>::to_f(x[i]); ss = fmaf(v, v, ss); }
+        float f = 1.0f / sqrtf(warp_sum_f(ss) / static_cast<float>(p.dim) + p.eps);
         if (h < p.R) {
-            float f = p.scale * (sizeof(QT) == 2 ? -kLog2e : 1.0f);                  // the tensor-core kernels compute 2^(-score log2 e)
+            f *= scale;
             if (p.temp_every > 0) f *= 1.0f + p.temp_coef * logf(static_cast<float>((pos0 + u + 1) / p.temp_every) + 1.0f);
-            for (int i = lane; i < p.dim; i += 32) qs[u * q_ld + h * p.dim + i] = Elem<T>::to_f(x[i]) * inv * f;
+            float* dst = qs + u * q_ld + h * p.dim;
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (lane + 32 * j < p.dim) dst[lane + 32 * j] = keep[j] * f;
+            for (int i = lane + 128; i < p.dim; i += 32) dst[i] = Elem<T>::to_f(x[i]) * f;
         } else if (u < fit) {
             T* dst = kc + (row0 + u) * p.ldk + g * p.dim;
-            for (int i = lane; i < p.dim; i += 32) dst[i] = Elem<T>::from_f(Elem<T>::to_f(x[i]) * inv);
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (lane + 32 * j < p.dim) dst[lane + 32 * j] = Elem<T>::from_f(keep[j] * f);
+            for (int i = lane + 128; i < p.dim; i += 32) dst[i] = Elem<T>::from_f(Elem<T>::to_f(x[i]) * f);
         }
     }
     __syncthreads();
-    const int slices = (p.H + kHeadSlice - 1) / kHeadSlice, pad = p.qld - p.G * p.dim;
-    for (int u = 0; u < nt; ++u) {
-        QT* out = qm + (m0 + u) * p.H * p.qld + g * p.dim;
-        const float* q = qs + u * q_ld;
-        if constexpr (RM > 0) {                          // two columns and a slice of the heads per step
-            const int pairs = p.dim / 2;
-            for (int i = tid; i < pairs * slices; i += kAppendThreads) {
-                const int sl = i / pairs, d = (i - sl * pairs) * 2;
+    const long long token_ld = static_cast<long long>(p.H) * p.qld;
+    QT* out = qm + m0 * token_ld + g * p.dim;
+    if constexpr (RM > 0) {                              // two columns and a slice of the heads per step, whose mixing weights serve all tokens
+        const int slices = (p.H + kHeadSlice - 1) / kHeadSlice, pairs = p.dim / 2;
+        for (int i = tid; i < pairs * slices; i += kAppendThreads) {
+            const int sl = i / pairs, d = (i - sl * pairs) * 2, h0 = sl * kHeadSlice, nh = min(kHeadSlice, p.H - h0);
+            float w[kHeadSlice][RM];                     // talk is padded to RM columns with zeros
+#pragma unroll
+            for (int e = 0; e < kHeadSlice; ++e)
+#pragma unroll
+                for (int r = 0; r < RM; ++r) w[e][r] = e < nh ? tk[(h0 + e) * RM + r] : 0.f;
+            QT* dst = out + static_cast<long long>(h0) * p.qld + d;
+            for (int u = 0; u < nt; ++u, dst += token_ld) {
                 float2 qr[RM];
 #pragma unroll
-                for (int r = 0; r < RM; ++r) qr[r] = r < p.R ? *reinterpret_cast<const float2*>(q + r * p.dim + d) : make_float2(0.f, 0.f);
+                for (int r = 0; r < RM; ++r) qr[r] = r < p.R ? *reinterpret_cast<const float2*>(qs + u * q_ld + r * p.dim + d) : make_float2(0.f, 0.f);
 #pragma unroll
                 for (int e = 0; e < kHeadSlice; ++e) {
-                    const int h = sl * kHeadSlice + e;
-                    if (h >= p.H) break;
+                    if (e >= nh) break;
                     float2 a = make_float2(0.f, 0.f);
 #pragma unroll
-                    for (int r = 0; r < RM; ++r) {       // talk is padded to RM columns with zeros
-                        const float w = tk[h * RM + r];
-                        a = __ffma2_rn(make_float2(w, w), qr[r], a);
-                    }
-                    QT* dst = out + static_cast<long long>(h) * p.qld + d;
-                    if constexpr (sizeof(QT) == 2) *reinterpret_cast<uint32_t*>(dst) = Elem<__nv_bfloat16>::pack2(a.x, a.y);
-                    else *reinterpret_cast<float2*>(dst) = a;
+                    for (int r = 0; r < RM; ++r) a = __ffma2_rn(make_float2(w[e][r], w[e][r]), qr[r], a);
+                    if constexpr (sizeof(QT) == 2) *reinterpret_cast<uint32_t*>(dst + e * p.qld) = Elem<__nv_bfloat16>::pack2(a.x, a.y);
+                    else *reinterpret_cast<float2*>(dst + e * p.qld) = a;
                 }
             }
-        } else {
-            for (int i = tid; i < p.dim * p.H; i += kAppendThreads) {
-                const int h = i / p.dim, d = i - h * p.dim;
+        }
+    } else {
+        for (int i = tid; i < p.dim * p.H; i += kAppendThreads) {
+            const int h = i / p.dim, d = i - h * p.dim;
+            for (int u = 0; u < nt; ++u) {
                 float a = 0.f;
-                for (int r = 0; r < p.R; ++r) a = fmaf(tk[h * p.R + r], q[r * p.dim + d], a);
-                out[static_cast<long long>(h) * p.qld + d] = Elem<QT>::from_f(a);
+                for (int r = 0; r < p.R; ++r) a = fmaf(tk[h * p.R + r], qs[u * q_ld + r * p.dim + d], a);
+                out[u * token_ld + static_cast<long long>(h) * p.qld + d] = Elem<QT>::from_f(a);
             }
         }
-        if (g == p.G - 1)                                // columns past the last group
-            for (int i = tid; i < pad * p.H; i += kAppendThreads) out[static_cast<long long>(i / pad) * p.qld + p.dim + i % pad] = Elem<QT>::from_f(0.f);
     }
+    const int pad = p.qld - p.G * p.dim;                 // columns past the last group
+    if (g == p.G - 1)
+        for (int i = tid; i < nt * pad * p.H; i += kAppendThreads) out[static_cast<long long>(i / pad) * p.qld + p.dim + i % pad] = Elem<QT>::from_f(0.f);
 }
 
 __device__ __forceinline__ float sigmoid_exact(float x) { return 1.0f / (1.0f + expf(-x)); }
