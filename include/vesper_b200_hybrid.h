@@ -246,9 +246,9 @@ int vb200_selective_forward(const vb200_selective_args* a);
 const char* vb200_last_selective_kernel(void);
 
 /* ---- mixture of experts -------------------------------------------------------------------------------
- * Router logits z = W_router x (fp32), scores s = sigmoid(z), choice = s + correction.  With groups > 0 the experts form equal groups of
- * neighbours, a group's score is the sum of its two largest choices, and only experts of the `keep` best groups can be chosen.
- * The `top` largest choices are taken, with weights s / (sum of the chosen s + 1e-20) * scale.
+ * s = sigmoid(W_router x) in fp32; experts rank by s + correction.  groups > 0: consecutive experts are put together, as many to each of the
+ * groups; groups rank by their best two experts' ranks added up, and experts outside the first `keep` groups are out of the running.
+ * The first `top` experts get the weights s / (sum of their s + 1e-20) * scale.
  * y[m, :] = sum of weight * W_down_e (silu(W_gate_e x) * (W_up_e x)), plus the same of the shared expert (if any) with weight 1.
  * Gate and up rows are interleaved (row 2j = gate_j, row 2j + 1 = up_j).
  * Prompts (vb200_moe_rows(a) > 0): y receives the shared expert only, and the weighted outputs of the chosen experts stay as bf16 rows
